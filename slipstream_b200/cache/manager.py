@@ -96,7 +96,7 @@ class RequestPages:
     length: int = 0  # tokens whose keys and values are in the cache
     reserved: int = 0  # tokens covered by pages (>= length)
     tables: list[list[int]] = field(default_factory=list)  # per group: logical block -> page or -1
-    first_block: list[int] = field(default_factory=list)  # per group: first block still held
+    first_block: list[int] = field(default_factory=list)  # per group: first block a window has not passed
 
 
 def pool_sizes(groups: list[GroupLayout], page_sizes: list[int], tokens: int, max_num_seqs: int,
@@ -111,7 +111,8 @@ def pool_sizes(groups: list[GroupLayout], page_sizes: list[int], tokens: int, ma
         window = layout.spec.span  # the most keys a query of this group sees: a window's or a chunk's size
         if window is not None:
             span = min(max_model_len, window + max(1, max_step_tokens))
-            pages = min(pages, max_num_seqs * (-(-span // page) + 1))
+            kept = -(-layout.spec.keep_first // page)  # pages of first keys that never pass out of sight
+            pages = min(pages, max_num_seqs * (-(-span // page) + 1 + kept))
         sizes.append(pages)
     return sizes
 
@@ -210,6 +211,11 @@ class CacheManager:
         """First block that a query at position >= ``length`` can still see."""
         return self.groups[group].spec.first_visible(length) // self.page_sizes[group]
 
+    def kept_blocks(self, group: int) -> int:
+        """Leading blocks of a request that a window never passes (``CacheSpec.keep_first``)."""
+        keep = self.groups[group].spec.keep_first
+        return self.blocks_for(keep, group) if keep else 0
+
     def pages_needed(self, request_id: object, new_tokens: int) -> list[int]:
         """Pages each group must still hand out to cover ``new_tokens`` more tokens."""
         req = self.get(request_id)
@@ -225,7 +231,7 @@ class CacheManager:
         if window is None:
             return self.blocks_for(total_tokens, group)
         span = min(total_tokens, window + max(chunk, 1))
-        return min(self.blocks_for(total_tokens, group), self.blocks_for(span, group) + 1)
+        return min(self.blocks_for(total_tokens, group), self.blocks_for(span, group) + 1 + self.kept_blocks(group))
 
     def can_admit(self, total_tokens: int, first_tokens: int, chunk: int) -> AllocStatus:
         """Three-way answer of slipstream/memory/block_manager.py:108-128: NEVER when the request at
@@ -291,7 +297,7 @@ class CacheManager:
         for g in range(len(self.groups)):
             first = self._first_needed_block(g, req.length)
             table = req.tables[g]
-            for b in range(req.first_block[g], min(first, len(table))):
+            for b in range(max(req.first_block[g], self.kept_blocks(g)), min(first, len(table))):
                 if table[b] >= 0:
                     self.pools[g].give_back(table[b], request_id)
                     table[b] = -1
@@ -317,7 +323,8 @@ class CacheManager:
                 pages = sum(1 for p in table if p >= 0)
                 size = self.page_sizes[g]
                 held += pages * size
-                useful += min(req.length - req.first_block[g] * size, pages * size)
+                kept = min(self.kept_blocks(g), req.first_block[g])  # full blocks held in front of the window's
+                useful += min(req.length - (req.first_block[g] - kept) * size, pages * size)
         return 1.0 if held == 0 else useful / held
 
     def check_invariants(self) -> None:

@@ -62,6 +62,9 @@ struct DecodeTmaArgs {
     int* counters;
     int* err;
     const bf16* gate;  // optional sigmoid gate on the output, laid out like `out`, rows q_stride apart
+    const float* sinks;  // float32 [n_q] or null: one more term exp(sinks[h]) in the denominator of head h's softmax
+    int keep;  // with a sliding window: the request's first `keep` keys stay visible (common.cuh: key_tiles)
+    int out_f32;  // `out` is float32
 };
 
 template <int D, int NS = DT_STAGES>
@@ -88,8 +91,14 @@ __device__ __forceinline__ void st_cluster_f32x2(float* local, uint32_t rank, fl
     asm volatile("st.shared::cluster.v2.f32 [%0], {%1, %2};" ::"r"(remote), "f"(x), "f"(y) : "memory");
 }
 
+// two neighbouring elements of the output, in its type
+__device__ __forceinline__ void store_out2(const DecodeTmaArgs& a, int64_t at, float v0, float v1) {
+    if (a.out_f32) *reinterpret_cast<float2*>(reinterpret_cast<float*>(a.out) + at) = make_float2(v0, v1);
+    else *reinterpret_cast<__nv_bfloat162*>(a.out + at) = __floats2bfloat162_rn(v0, v1);
+}
+
 // (with three stages the registers are held to what lets two blocks share an SM, as the shared memory does)
-// FORM 1 is the usual decode step as a kernel of its own: rotation and page write inside, no window, the slices one
+// FORM 1 is the usual decode step as a kernel of its own: rotation and page write inside, no window, no sinks, the slices one
 // cluster, a rotary size in steps of 16.  What FORM 0 asks of its arguments FORM 1 knows, and its blocks, which run
 // every part of the kernel once from a cold instruction cache, branch over less.
 template <int D, int NS, int FORM>
@@ -121,6 +130,7 @@ attn_decode_tma(const __grid_constant__ CUtensorMap map_kv, const DecodeTmaArgs 
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int n_q = a.n_q, n_kv = a.n_kv, page_size = a.page_size, n_slices = a.n_slices;
     const int window = FORM == 0 ? a.window : 0;
+    const int keep = FORM == 0 ? a.keep : 0;
     const bool fused = FORM == 0 ? a.fused != 0 : true;
     const int G = n_q / n_kv, hblocks = (G + 15) / 16;
     const int r = blockIdx.x, kvh = blockIdx.y / hblocks, g0 = (blockIdx.y % hblocks) * 16;
@@ -131,13 +141,14 @@ attn_decode_tma(const __grid_constant__ CUtensorMap map_kv, const DecodeTmaArgs 
     const int row_q = a.q_start[r], seq_len = a.seq_lens[r];
     const int pos = seq_len - 1;
     const int lo = key_floor(pos, window);
-    const int kt_first = lo / MMA_BN, kt_last = pos / MMA_BN;
-    const int n_tiles = kt_last - kt_first + 1;
-    const int per = (n_tiles + n_slices - 1) / n_slices;
-    const int kt_lo = kt_first + slice * per, kt_hi = min(kt_last, kt_lo + per - 1);
-    const bool work = seq_len > 0 && kt_lo <= kt_hi;
+    const KeyTiles walk = key_tiles(lo, pos, keep, MMA_BN);  // this slice takes tiles j_lo .. j_hi of the walk
+    const int per = (walk.count + n_slices - 1) / n_slices;
+    const int j_last = walk.count - 1, j_lo = slice * per, j_hi = min(j_last, j_lo + per - 1);
+    const bool work = seq_len > 0 && j_lo <= j_hi;
+    const int tile_lo = work ? walk.at(j_lo) * MMA_BN : 0, tile_hi = work ? walk.at(j_hi) * MMA_BN + MMA_BN - 1 : 0;
+    const int first_key = tile_lo < keep ? tile_lo : max(lo, tile_lo);  // the first key of the slice that is seen
     const int half = a.rot_dim / 2;
-    const bool has_newest = fused && work && kt_hi == kt_last;
+    const bool has_newest = fused && work && j_hi == j_last;
 
     if (tid == 0) {
         for (int s = 0; s < NB; ++s) { fa::mbar_init(&full[s], 1); fa::mbar_init(&empty[s], 2); }  // a pair of warps per tile
@@ -147,8 +158,8 @@ attn_decode_tma(const __grid_constant__ CUtensorMap map_kv, const DecodeTmaArgs 
     TableRef table;
     table.p = a.block_tables; table.base = 0; table.shift = -1;
     if (work) {
-        table = stage_table(table_s, a.block_tables + (int64_t)r * a.max_blocks, max(lo, kt_lo * MMA_BN),
-                            min(pos, kt_hi * MMA_BN + MMA_BN - 1), page_size, DT_TABLE_MAX);
+        table = stage_table(table_s, a.block_tables + (int64_t)r * a.max_blocks, first_key, min(pos, tile_hi), page_size,
+                            DT_TABLE_MAX);
         if (fused) {
             for (int i = tid; i < half; i += DT_THREADS) {
                 const float angle = __fmul_rn((float)pos, a.inv_freq[i]);
@@ -159,6 +170,16 @@ attn_decode_tma(const __grid_constant__ CUtensorMap map_kv, const DecodeTmaArgs 
     __syncthreads();  // barriers, table, sines and cosines
 
     float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+    if (FORM == 0 && a.sinks && slice == 0 && warp == 0) {  // the sink's term, one time: in the first warp of the first slice
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+            const int row = (lane >> 2) + h * 8;
+            if (row < heads_here) {
+                m[h] = a.sinks[kvh * G + g0 + row] * 1.4426950408889634f;
+                l[h] = (lane & 3) == 0 ? 1.f : 0.f;
+            }
+        }
+    }
     float o[D / 8][4];
 #pragma unroll
     for (int d = 0; d < D / 8; ++d) o[d][0] = o[d][1] = o[d][2] = o[d][3] = 0.f;
@@ -170,7 +191,7 @@ attn_decode_tma(const __grid_constant__ CUtensorMap map_kv, const DecodeTmaArgs 
         if (work) {
             if (lane == 0) asm volatile("prefetch.tensormap [%0];" ::"l"(&map_kv) : "memory");
             const int ppt = MMA_BN / page_size;
-            const int b_first = max(lo, kt_lo * MMA_BN) / page_size, b_last = min(pos, kt_hi * MMA_BN + MMA_BN - 1) / page_size;
+            const int b_first = first_key / page_size, b_last = min(pos, tile_hi) / page_size;
             int64_t spare = table.p[b_first - table.base];  // a page of this request, for blocks that have none
             if (spare < 0 || spare >= a.num_pages) {
                 if (lane == 0) atomicOr(a.err, SS_ERR_PAGE_RANGE);
@@ -180,12 +201,12 @@ attn_decode_tma(const __grid_constant__ CUtensorMap map_kv, const DecodeTmaArgs 
             const bool mine = p < ppt;
             const uint64_t once = fa::l2_evict_first_policy();
             bool waited = false, ok = true;
-            for (int kt = kt_lo; kt <= kt_hi && ok; ++kt) {
-                const int i = kt - kt_lo, st = i % NS;
+            for (int j = j_lo; j <= j_hi && ok; ++j) {
+                const int kt = walk.at(j), i = j - j_lo, st = i % NS;
                 // the tile that lay in this stage before (i - NS) has been used up
                 if (i >= NS) ok = __all_sync(0xffffffffu, fa::mbar_wait(&empty[bar_of(i - NS)], phase_of(i - NS) & 1, gave_up));
                 if (!ok) break;
-                if (!fused && kt == kt_last && !waited) {
+                if (!fused && j == j_last && !waited) {
                     pdl_wait();  // the newest key and value are written by the kernel before this one
                     waited = true;
                 }
@@ -327,21 +348,21 @@ attn_decode_tma(const __grid_constant__ CUtensorMap map_kv, const DecodeTmaArgs 
             const float scale_log2 = a.scale * 1.4426950408889634f, cap_log2 = a.softcap * 1.4426950408889634f;
             const int p_lo = (lane >> 2) < heads_here ? pos : -1;
             const int p_hi = (lane >> 2) + 8 < heads_here ? pos : -1;
-            // pair (warp / 2) takes the tiles kt_lo + pair, + 2, ...; warp % 2 is the 32-key half.  Tile i lies in
+            // pair (warp / 2) takes the tiles j_lo + pair, + 2, ... of the walk; warp % 2 is the 32-key half.  Tile i lies in
             // stage i % NS: with two stages a pair has one of its own, and its next tile can only be fetched once
             // it is done with this one (a block that walks 16 tiles then moves one tile per pair in the time of a
             // product plus a trip to memory); with three, the third is being filled while both pairs work.
             const int pair = warp >> 1, key_off = (warp & 1) * 32;
-            for (int kt = kt_lo + pair; kt <= kt_hi; kt += 2) {
-                const int i = kt - kt_lo, st = NS == 2 ? pair : i % NS;
+            for (int j = j_lo + pair; j <= j_hi; j += 2) {
+                const int kt = walk.at(j), i = j - j_lo, st = NS == 2 ? pair : i % NS;
                 bf16* Ks = KV + st * STAGE;
                 bf16* Vs = Ks + MMA_BN * D;
                 // a wait that gives up makes every later wait give up at once
                 const bool ok = fa::mbar_wait(&full[bar_of(i)], phase_of(i) & 1, gave_up);
-                const int first_key = kt * MMA_BN + key_off;
-                if (fused && kt == kt_last && pos >= first_key && pos < first_key + 32) {
+                const int half_key = kt * MMA_BN + key_off;
+                if (fused && j == j_last && pos >= half_key && pos < half_key + 32) {
                     // the newest token's row of this half comes from the projection output, not from the page
-                    const int prow = pos - kt_last * MMA_BN;
+                    const int prow = pos % MMA_BN;
                     for (int c = lane; c < 2 * (D / 8); c += 32) {
                         const int col = (c % (D / 8)) * 8;
                         if (c < D / 8) *reinterpret_cast<uint4*>(const_cast<bf16*>(tile_at<D, true>(Ks, prow, col))) = *reinterpret_cast<const uint4*>(newest_k + col);
@@ -349,12 +370,12 @@ attn_decode_tma(const __grid_constant__ CUtensorMap map_kv, const DecodeTmaArgs 
                     }
                     __syncwarp();
                 }
-                if (ok && kt == kt_last && pos >= first_key && pos < first_key + 31) {
+                if (ok && j == j_last && pos >= half_key && pos < half_key + 31) {
                     // The rows behind the newest token hold whatever the page's last owner left there (and, for blocks
                     // without a page, a copy of the slice's first page, which may be that same page).  Their scores
                     // are masked, but their values still meet a weight of zero in P V, and 0 x inf is not 0:
                     // nothing of another request may reach this one, so those value rows are cleared.
-                    const int prow = pos - kt_last * MMA_BN;
+                    const int prow = pos % MMA_BN;
                     const int page_end = key_off + 31;  // the end of this warp's half of the tile
                     for (int c = lane; c < (page_end - prow) * (D / 8); c += 32) {
                         const int row = prow + 1 + c / (D / 8), col = (c % (D / 8)) * 8;
@@ -362,10 +383,10 @@ attn_decode_tma(const __grid_constant__ CUtensorMap map_kv, const DecodeTmaArgs 
                     }
                     __syncwarp();
                 }
-                if (ok && first_key <= pos) {
-                    const bool whole = heads_here == 16 && first_key + 31 <= pos && first_key >= lo;
-                    if (whole) warp_tile<D, 32, false, true>(qf, Ks, Vs, key_off, kt * MMA_BN, scale_log2, p_lo, p_hi, window, m, l, o, cap_log2);
-                    else warp_tile<D, 32, true, true>(qf, Ks, Vs, key_off, kt * MMA_BN, scale_log2, p_lo, p_hi, window, m, l, o, cap_log2);
+                if (ok && half_key <= pos) {
+                    const bool whole = heads_here == 16 && half_key + 31 <= pos && half_key >= lo;
+                    if (whole) warp_tile<D, 32, false, true>(qf, Ks, Vs, key_off, kt * MMA_BN, scale_log2, p_lo, p_hi, window, m, l, o, cap_log2, keep);
+                    else warp_tile<D, 32, true, true>(qf, Ks, Vs, key_off, kt * MMA_BN, scale_log2, p_lo, p_hi, window, m, l, o, cap_log2, keep);
                 }
                 __syncwarp();
                 if (lane == 0) {
@@ -437,8 +458,7 @@ attn_decode_tma(const __grid_constant__ CUtensorMap map_kv, const DecodeTmaArgs 
                     v0 = gated<true>(v0, __low2float(g2));
                     v1 = gated<true>(v1, __high2float(g2));
                 }
-                *reinterpret_cast<__nv_bfloat162*>(a.out + (int64_t)row_q * a.out_stride + (head0 + row) * D + d) =
-                    __floats2bfloat162_rn(v0, v1);
+                store_out2(a, (int64_t)row_q * a.out_stride + (head0 + row) * D + d, v0, v1);
             } else {
                 float* po = a.part_o + (((int64_t)r * n_q + head0 + row) * n_groups + group) * D + d;
                 po[0] = acc0 * inv;
@@ -478,8 +498,8 @@ attn_decode_tma(const __grid_constant__ CUtensorMap map_kv, const DecodeTmaArgs 
                     v0 = gated<true>(v0, __low2float(g2));
                     v1 = gated<true>(v1, __high2float(g2));
                 }
-                *reinterpret_cast<__nv_bfloat162*>(a.out + (int64_t)row_q * a.out_stride + (head0 + row) * D + d) =
-                    __floats2bfloat162_rn(v0, v1);
+                if (FORM == 0) store_out2(a, (int64_t)row_q * a.out_stride + (head0 + row) * D + d, v0, v1);
+                else *reinterpret_cast<__nv_bfloat162*>(a.out + (int64_t)row_q * a.out_stride + (head0 + row) * D + d) = __floats2bfloat162_rn(v0, v1);
             } else {  // several clusters share the keys of this head block: the cluster's result goes to scratch
                 float* po = a.part_o + (((int64_t)r * n_q + head0 + row) * n_groups + group) * D + d;
                 po[0] = acc0 * inv;
@@ -530,6 +550,8 @@ attn_decode_tma(const __grid_constant__ CUtensorMap map_kv, const DecodeTmaArgs 
 #pragma unroll 8
         for (int sl = 0; sl < n_groups; ++sl) acc += __ldcg(po + (int64_t)sl * D) * w[sl];
         if (FORM == 0 && a.gate) acc = gated<true>(acc, to_float(a.gate[(int64_t)row_q * a.q_stride + (head0 + row) * D + d]));
-        a.out[(int64_t)row_q * a.out_stride + (head0 + row) * D + d] = __float2bfloat16_rn(acc);
+        const int64_t at = (int64_t)row_q * a.out_stride + (head0 + row) * D + d;
+        if (FORM == 0 && a.out_f32) reinterpret_cast<float*>(a.out)[at] = acc;
+        else a.out[at] = __float2bfloat16_rn(acc);
     }
 }

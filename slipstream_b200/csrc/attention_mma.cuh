@@ -13,7 +13,9 @@
 //
 // Key tiles start at multiples of 64 counted from the request's first token.  Masking is
 // the packed-index causal rule of slipstream/models/layers/attention.py:46-51 plus an
-// optional window; softmax statistics are float32 (:64-88); probabilities are rounded to
+// optional window (which may keep the request's first `keep` keys in sight: common.cuh, key_tiles); softmax statistics
+// are float32 (:64-88); with out_f32 the heads' outputs are written as float32, with `diff` (prefill) the two maps of a
+// differential head are combined where they are written; probabilities are rounded to
 // bfloat16 for the second product as the reference's `.to(query.dtype)` does.
 // kv layout: [page][2][kv head][offset in page][D].
 #pragma once
@@ -85,12 +87,13 @@ __device__ __forceinline__ TableRef stage_table(int32_t* smem_table, const int32
 }
 
 // Stage keys [k0, k0 + 64) of one kv head: K rows to Ks, V rows to Vs (row stride D + 8).
-// Rows outside [lo, hi] or without a page are zero-filled; the row of key `skip` is left alone.
+// Rows outside [lo, hi] (keys below `keep` count as inside) or without a page are zero-filled; the row of key `skip`
+// is left alone.
 template <int D>
 __device__ __forceinline__ void load_kv_tile(bf16* Ks, bf16* Vs, const bf16* __restrict__ kv,
                                              const TableRef table, int k0, int lo, int hi,
                                              int kvh, int n_kv, int page_size, int64_t num_pages, int* err,
-                                             int skip = -1) {
+                                             int skip = -1, int keep = 0) {
     constexpr int CPR = D / 8;  // 16-byte chunks per row
     constexpr int KSTR = D + 8;
     const int64_t v_off = (int64_t)n_kv * page_size * D;
@@ -98,7 +101,7 @@ __device__ __forceinline__ void load_kv_tile(bf16* Ks, bf16* Vs, const bf16* __r
         const int row = c / CPR, col = (c - row * CPR) * 8;
         const int key = k0 + row;
         if (key == skip) continue;
-        bool ok = key >= lo && key <= hi;
+        bool ok = (key >= lo || key < keep) && key <= hi;
         int64_t base = 0;
         if (ok) {
             const int blk = table.shift >= 0 ? key >> table.shift : key / page_size;
@@ -130,7 +133,7 @@ __device__ __forceinline__ const bf16* tile_at(const bf16* base, int row, int co
 template <int D, int NK, bool MASK, bool SWZ = false>
 __device__ __forceinline__ void warp_tile(const uint32_t (&qf)[D / 16][4], const bf16* Ks, const bf16* Vs,
                                           int key_off, int key0_abs, float scale_log2, int pos_lo, int pos_hi,
-                                          int window, float (&m)[2], float (&l)[2], float (&o)[D / 8][4], float cap_log2 = 0.f) {
+                                          int window, float (&m)[2], float (&l)[2], float (&o)[D / 8][4], float cap_log2 = 0.f, int keep = 0) {
     constexpr int KSTR = D + 8;
     constexpr int NT = NK / 8;
     const int lane = threadIdx.x & 31;
@@ -160,7 +163,7 @@ __device__ __forceinline__ void warp_tile(const uint32_t (&qf)[D / 16][4], const
             if (MASK) {  // tiles that every row of the warp sees whole skip this
                 const int key = key0_abs + key_off + n * 8 + ((lane & 3) << 1) + (e & 1);
                 const int pos = (e < 2) ? pos_lo : pos_hi;  // < 0: the row does not exist
-                ok = key <= pos && key >= ((e < 2) ? floor_lo : floor_hi);
+                ok = key <= pos && (key >= ((e < 2) ? floor_lo : floor_hi) || key < keep);
             }
             float v = s[n][e] * scale_log2;
             // a soft cap c on the scaled score: c tanh(score / c), here with both in units of log2(e);
@@ -235,7 +238,7 @@ attn_prefill_mma(const bf16* __restrict__ q, int64_t q_stride, bf16* __restrict_
                  const int32_t* __restrict__ tile_req, const int32_t* __restrict__ tile_row0,
                  const int32_t* __restrict__ q_start, const int32_t* __restrict__ seq_lens, int n_q, int n_kv,
                  int page_size, int64_t num_pages, float scale, int window, int* err, const bf16* __restrict__ gate,
-                 float softcap, const float* __restrict__ sinks) {
+                 float softcap, const float* __restrict__ sinks, int keep, int out_f32, const DiffPair diff) {
     pdl_launch_dependents();  // the next kernel may be scheduled now; it waits for this one itself
     pdl_wait();               // nothing below runs before the kernels before this one are complete
     constexpr int KSTR = D + 8;
@@ -254,7 +257,8 @@ attn_prefill_mma(const bf16* __restrict__ q, int64_t q_stride, bf16* __restrict_
     const int last_pos = seq_len - q_len + (row0 + rows_here - 1) / G;
     const int lo = key_floor(first_pos, window);
     __shared__ int32_t table_s[MMA_TABLE_MAX];
-    const TableRef table = stage_table(table_s, block_tables + (int64_t)r * max_blocks, lo, last_pos, page_size);
+    const KeyTiles walk = key_tiles(lo, last_pos, keep, MMA_BN);
+    const TableRef table = stage_table(table_s, block_tables + (int64_t)r * max_blocks, keep > 0 ? 0 : lo, last_pos, page_size);
     __syncthreads();
 
     // Q tile: row -> (token, head of the group)
@@ -265,8 +269,7 @@ attn_prefill_mma(const bf16* __restrict__ q, int64_t q_stride, bf16* __restrict_
         const int tok = ok ? gr / G : 0, g = ok ? gr - tok * G : 0;
         cp_async16(Qs + row * KSTR + col, q + (int64_t)(qs + tok) * q_stride + (int64_t)(kvh * G + g) * D + col, ok);
     }
-    const int kt_lo = lo / MMA_BN, kt_hi = last_pos / MMA_BN;
-    load_kv_tile<D>(KV, KV + MMA_BN * KSTR, kv, table, kt_lo * MMA_BN, lo, last_pos, kvh, n_kv, page_size, num_pages, err);
+    load_kv_tile<D>(KV, KV + MMA_BN * KSTR, kv, table, walk.at(0) * MMA_BN, lo, last_pos, kvh, n_kv, page_size, num_pages, err, -1, keep);
     cp_async_commit();
 
     // this thread's two rows
@@ -293,20 +296,20 @@ attn_prefill_mma(const bf16* __restrict__ q, int64_t q_stride, bf16* __restrict_
     uint32_t qf[D / 16][4];
     const float scale_log2 = scale * 1.4426950408889634f, cap_log2 = softcap * 1.4426950408889634f;
 
-    for (int kt = kt_lo; kt <= kt_hi; ++kt) {
-        const int stage = (kt - kt_lo) & 1;
+    for (int jt = 0; jt < walk.count; ++jt) {
+        const int kt = walk.at(jt), stage = jt & 1;
         bf16* Ks = KV + stage * 2 * MMA_BN * KSTR;
         bf16* Vs = Ks + MMA_BN * KSTR;
-        if (kt < kt_hi) {
+        if (jt + 1 < walk.count) {
             bf16* Kn = KV + (stage ^ 1) * 2 * MMA_BN * KSTR;
-            load_kv_tile<D>(Kn, Kn + MMA_BN * KSTR, kv, table, (kt + 1) * MMA_BN, lo, last_pos, kvh, n_kv, page_size, num_pages, err);
+            load_kv_tile<D>(Kn, Kn + MMA_BN * KSTR, kv, table, walk.at(jt + 1) * MMA_BN, lo, last_pos, kvh, n_kv, page_size, num_pages, err, -1, keep);
             cp_async_commit();
             cp_async_wait<1>();
         } else {
             cp_async_wait<0>();
         }
         __syncthreads();
-        if (kt == kt_lo) {
+        if (jt == 0) {
 #pragma unroll
             for (int ks = 0; ks < D / 16; ++ks)
                 ldmatrix_x4(qf[ks], Qs + (warp * 16 + (lane & 15)) * KSTR + ks * 16 + ((lane >> 4) << 3));
@@ -320,8 +323,8 @@ attn_prefill_mma(const bf16* __restrict__ q, int64_t q_stride, bf16* __restrict_
         const bool whole = warp * 16 + 15 < rows_here && kt * MMA_BN + MMA_BN - 1 <= warp_first_pos &&
                            kt * MMA_BN >= key_floor(warp_last_pos, window);
         if (active) {
-            if (whole) warp_tile<D, MMA_BN, false>(qf, Ks, Vs, 0, kt * MMA_BN, scale_log2, pos2[0], pos2[1], window, m, l, o, cap_log2);
-            else warp_tile<D, MMA_BN, true>(qf, Ks, Vs, 0, kt * MMA_BN, scale_log2, pos2[0], pos2[1], window, m, l, o, cap_log2);
+            if (whole) warp_tile<D, MMA_BN, false>(qf, Ks, Vs, 0, kt * MMA_BN, scale_log2, pos2[0], pos2[1], window, m, l, o, cap_log2, keep);
+            else warp_tile<D, MMA_BN, true>(qf, Ks, Vs, 0, kt * MMA_BN, scale_log2, pos2[0], pos2[1], window, m, l, o, cap_log2, keep);
         }
         __syncthreads();
     }
@@ -331,9 +334,43 @@ attn_prefill_mma(const bf16* __restrict__ q, int64_t q_stride, bf16* __restrict_
         l[h] += __shfl_xor_sync(0xffffffffu, l[h], 1);
         l[h] += __shfl_xor_sync(0xffffffffu, l[h], 2);
         const int row = warp * 16 + (lane >> 2) + h * 8;
-        if (row >= rows_here) continue;
-        const int gr = row0 + row, tok = gr / G, g = gr - tok * G;
         const float inv = l[h] > 0.f ? 1.f / l[h] : 0.f;
+        const int gr = row0 + row, tok = gr / G, g = gr - tok * G;
+        if (diff.on) {
+            // a head's two maps are neighbouring rows (G is even and a block begins with an even row), held by lanes
+            // whose numbers differ by 4: both form the difference, the squares are summed over the four lanes of a
+            // row, and each of the two writes every other run of 8 columns
+            const bool first_map = (row & 1) == 0;
+            float ss = 0.f;
+#pragma unroll
+            for (int d = 0; d < D / 8; ++d) {
+#pragma unroll
+                for (int e = 0; e < 2; ++e) {
+                    const float mine = o[d][2 * h + e] * inv, other = __shfl_xor_sync(0xffffffffu, mine, 4);
+                    const float v = first_map ? mine - diff.lam * other : other - diff.lam * mine;
+                    o[d][2 * h + e] = v;
+                    ss = fmaf(v, v, ss);  // columns beyond the values hold zeros
+                }
+            }
+            ss += __shfl_xor_sync(0xffffffffu, ss, 1);
+            ss += __shfl_xor_sync(0xffffffffu, ss, 2);
+            if (row >= rows_here) continue;
+            const float f = diff.mult / sqrtf(ss / (float)diff.dim + diff.eps);
+            bf16* dst = out + (int64_t)(qs + tok) * out_stride + (int64_t)((kvh * G + g) >> 1) * diff.dim + ((lane & 3) << 1);
+#pragma unroll
+            for (int d = 0; d < D / 8; ++d)
+                if ((d & 1) == (row & 1) && d * 8 < diff.dim)
+                    *reinterpret_cast<__nv_bfloat162*>(dst + d * 8) = __floats2bfloat162_rn(o[d][2 * h] * f, o[d][2 * h + 1] * f);
+            continue;
+        }
+        if (row >= rows_here) continue;
+        if (out_f32) {
+            float* dst = reinterpret_cast<float*>(out) + (int64_t)(qs + tok) * out_stride + (int64_t)(kvh * G + g) * D + ((lane & 3) << 1);
+#pragma unroll
+            for (int d = 0; d < D / 8; ++d)
+                *reinterpret_cast<float2*>(dst + d * 8) = make_float2(o[d][2 * h] * inv, o[d][2 * h + 1] * inv);
+            continue;
+        }
         bf16* dst = out + (int64_t)(qs + tok) * out_stride + (int64_t)(kvh * G + g) * D + ((lane & 3) << 1);
         const bf16* gt = gate ? gate + (int64_t)(qs + tok) * q_stride + (int64_t)(kvh * G + g) * D + ((lane & 3) << 1) : nullptr;
 #pragma unroll
@@ -361,7 +398,7 @@ attn_decode_mma(const bf16* __restrict__ q, int64_t q_stride, bf16* __restrict__
                 int page_size, int64_t num_pages, float scale, int window, int n_slices, int cluster,
                 const float* __restrict__ inv_freq, int rot_dim, int fused,
                 float* __restrict__ part_o, float* __restrict__ part_lse, int* __restrict__ counters, int* err,
-                const bf16* __restrict__ gate, float softcap, const float* __restrict__ sinks) {
+                const bf16* __restrict__ gate, float softcap, const float* __restrict__ sinks, int keep, int out_f32) {
     pdl_launch_dependents();  // the next kernel may be scheduled now; it waits for this one itself
     // Until pdl_wait() below, only what no kernel of this step writes is touched: the lengths, the block
     // table, and keys and values at positions before the newest token (earlier steps wrote those).  The
@@ -380,10 +417,9 @@ attn_decode_mma(const bf16* __restrict__ q, int64_t q_stride, bf16* __restrict__
     const int pos = seq_len - 1;
     const int lo = key_floor(pos, window);
 
-    const int kt_first = lo / MMA_BN, kt_last = pos / MMA_BN;
-    const int n_tiles = kt_last - kt_first + 1;
-    const int per = (n_tiles + n_slices - 1) / n_slices;
-    const int kt_lo = kt_first + slice * per, kt_hi = min(kt_last, kt_lo + per - 1);
+    const KeyTiles walk = key_tiles(lo, pos, keep, MMA_BN);  // a slice takes tiles j_lo .. j_hi of the walk
+    const int per = (walk.count + n_slices - 1) / n_slices;
+    const int j_last = walk.count - 1, j_lo = slice * per, j_hi = min(j_last, j_lo + per - 1);
 
     float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
     if (sinks && slice == 0 && warp == 0) {  // the sink's term is added one time: by the first warp of the first slice
@@ -400,10 +436,11 @@ attn_decode_mma(const bf16* __restrict__ q, int64_t q_stride, bf16* __restrict__
 #pragma unroll
     for (int d = 0; d < D / 8; ++d) o[d][0] = o[d][1] = o[d][2] = o[d][3] = 0.f;
 
-    if (seq_len > 0 && kt_lo <= kt_hi) {
+    if (seq_len > 0 && j_lo <= j_hi) {
         __shared__ int32_t table_s[MMA_TABLE_MAX];
-        const TableRef table = stage_table(table_s, block_tables + (int64_t)r * max_blocks, max(lo, kt_lo * MMA_BN),
-                                           min(pos, kt_hi * MMA_BN + MMA_BN - 1), page_size);
+        const int tile0 = walk.at(j_lo) * MMA_BN, first_key = tile0 < keep ? tile0 : max(lo, tile0);
+        const TableRef table = stage_table(table_s, block_tables + (int64_t)r * max_blocks, first_key,
+                                           min(pos, walk.at(j_hi) * MMA_BN + MMA_BN - 1), page_size);
         // fused: q is the projection output [q heads | k heads | v heads] before rotation.  This kernel rotates
         // its query heads in shared memory, and the block whose slice ends at the newest token rotates that
         // token's key, puts key and value into its tile and (first head block only) into their page.
@@ -417,7 +454,7 @@ attn_decode_mma(const bf16* __restrict__ q, int64_t q_stride, bf16* __restrict__
             }
         }
         __shared__ __align__(16) bf16 newest_k[256], newest_v[256];
-        const bool has_newest = fused && kt_hi == kt_last;
+        const bool has_newest = fused && j_hi == j_last;
         // after the wait: rotate the newest key, keep it and the value for the tile, write both to their page
         auto make_newest = [&]() {
             const bf16* kn = q + (int64_t)row_q * q_stride + (int64_t)(n_q + kvh) * D;
@@ -456,7 +493,7 @@ attn_decode_mma(const bf16* __restrict__ q, int64_t q_stride, bf16* __restrict__
         };
         // its row of the tile that holds it (the tile's fetch leaves that row alone)
         auto put_newest = [&](bf16* Ks, bf16* Vs) {
-            const int prow = pos - kt_last * MMA_BN;
+            const int prow = pos % MMA_BN;
             for (int c = tid; c < 2 * (D / 8); c += MMA_THREADS) {
                 const int col = (c % (D / 8)) * 8;
                 if (c < D / 8) *reinterpret_cast<uint4*>(Ks + prow * KSTR + col) = *reinterpret_cast<const uint4*>(newest_k + col);
@@ -470,9 +507,9 @@ attn_decode_mma(const bf16* __restrict__ q, int64_t q_stride, bf16* __restrict__
         constexpr int NS = DECODE_STAGES;
 #pragma unroll
         for (int st = 0; st < NS - 1; ++st) {
-            if (kt_lo + st <= kt_hi && kt_lo + st < kt_last) {
+            if (j_lo + st <= j_hi && j_lo + st < j_last) {
                 bf16* Kn = KV + st * 2 * MMA_BN * KSTR;
-                load_kv_tile<D>(Kn, Kn + MMA_BN * KSTR, kv, table, (kt_lo + st) * MMA_BN, lo, pos, kvh, n_kv, page_size, num_pages, err);
+                load_kv_tile<D>(Kn, Kn + MMA_BN * KSTR, kv, table, walk.at(j_lo + st) * MMA_BN, lo, pos, kvh, n_kv, page_size, num_pages, err, -1, keep);
             }
         }
         pdl_wait();
@@ -487,9 +524,9 @@ attn_decode_mma(const bf16* __restrict__ q, int64_t q_stride, bf16* __restrict__
         }
 #pragma unroll
         for (int st = 0; st < NS - 1; ++st) {
-            if (kt_lo + st <= kt_hi && kt_lo + st == kt_last) {
+            if (j_lo + st <= j_hi && j_lo + st == j_last) {
                 bf16* Kn = KV + st * 2 * MMA_BN * KSTR;
-                load_kv_tile<D>(Kn, Kn + MMA_BN * KSTR, kv, table, (kt_lo + st) * MMA_BN, lo, pos, kvh, n_kv, page_size, num_pages, err, skip);
+                load_kv_tile<D>(Kn, Kn + MMA_BN * KSTR, kv, table, walk.at(j_last) * MMA_BN, lo, pos, kvh, n_kv, page_size, num_pages, err, skip, keep);
                 if (fused) put_newest(Kn, Kn + MMA_BN * KSTR);
             }
             cp_async_commit();
@@ -498,19 +535,19 @@ attn_decode_mma(const bf16* __restrict__ q, int64_t q_stride, bf16* __restrict__
         const float scale_log2 = scale * 1.4426950408889634f, cap_log2 = softcap * 1.4426950408889634f;
         const int p_lo = (lane >> 2) < heads_here ? pos : -1;
         const int p_hi = (lane >> 2) + 8 < heads_here ? pos : -1;
-        for (int kt = kt_lo; kt <= kt_hi; ++kt) {
-            const int stage = (kt - kt_lo) % NS;
+        for (int j = j_lo; j <= j_hi; ++j) {
+            const int kt = walk.at(j), stage = (j - j_lo) % NS;
             bf16* Ks = KV + stage * 2 * MMA_BN * KSTR;
             bf16* Vs = Ks + MMA_BN * KSTR;
-            if (kt + NS - 1 <= kt_hi) {
-                bf16* Kn = KV + ((kt - kt_lo + NS - 1) % NS) * 2 * MMA_BN * KSTR;
-                load_kv_tile<D>(Kn, Kn + MMA_BN * KSTR, kv, table, (kt + NS - 1) * MMA_BN, lo, pos, kvh, n_kv, page_size, num_pages, err, skip);
-                if (fused && kt + NS - 1 == kt_last) put_newest(Kn, Kn + MMA_BN * KSTR);
+            if (j + NS - 1 <= j_hi) {
+                bf16* Kn = KV + ((j - j_lo + NS - 1) % NS) * 2 * MMA_BN * KSTR;
+                load_kv_tile<D>(Kn, Kn + MMA_BN * KSTR, kv, table, walk.at(j + NS - 1) * MMA_BN, lo, pos, kvh, n_kv, page_size, num_pages, err, skip, keep);
+                if (fused && j + NS - 1 == j_last) put_newest(Kn, Kn + MMA_BN * KSTR);
             }
             cp_async_commit();
             cp_async_wait<NS - 1>();  // everything but the NS - 1 newest groups: tile kt has landed
             __syncthreads();
-            if (kt == kt_lo) {
+            if (j == j_lo) {
                 if (fused && half > 0) {
                     for (int idx = tid; idx < 16 * half; idx += MMA_THREADS) {
                         const int row = idx / half, i = idx - row * half;
@@ -529,8 +566,8 @@ attn_decode_mma(const bf16* __restrict__ q, int64_t q_stride, bf16* __restrict__
             if (kt * MMA_BN + warp * 16 <= pos) {
                 const bool whole = heads_here == 16 && kt * MMA_BN + warp * 16 + 15 <= pos &&
                                    kt * MMA_BN + warp * 16 >= key_floor(pos, window);
-                if (whole) warp_tile<D, 16, false>(qf, Ks, Vs, warp * 16, kt * MMA_BN, scale_log2, p_lo, p_hi, window, m, l, o, cap_log2);
-                else warp_tile<D, 16, true>(qf, Ks, Vs, warp * 16, kt * MMA_BN, scale_log2, p_lo, p_hi, window, m, l, o, cap_log2);
+                if (whole) warp_tile<D, 16, false>(qf, Ks, Vs, warp * 16, kt * MMA_BN, scale_log2, p_lo, p_hi, window, m, l, o, cap_log2, keep);
+                else warp_tile<D, 16, true>(qf, Ks, Vs, warp * 16, kt * MMA_BN, scale_log2, p_lo, p_hi, window, m, l, o, cap_log2, keep);
             }
             __syncthreads();  // the stage may be refilled by the next iteration's prefetch
         }
@@ -590,7 +627,8 @@ attn_decode_mma(const bf16* __restrict__ q, int64_t q_stride, bf16* __restrict__
         const float val = ll > 0.f ? acc / ll : 0.f;
         const int head = kvh * G + g0 + row;
         if (n_slices == 1) {
-            out[(int64_t)row_q * out_stride + (int64_t)head * D + d] = __float2bfloat16_rn(
+            if (out_f32) reinterpret_cast<float*>(out)[(int64_t)row_q * out_stride + (int64_t)head * D + d] = val;
+            else out[(int64_t)row_q * out_stride + (int64_t)head * D + d] = __float2bfloat16_rn(
                 gate ? gated<true>(val, to_float(gate[(int64_t)row_q * q_stride + (int64_t)head * D + d])) : val);
         } else if (cluster) {
             Pc[row * D + d] = val;
@@ -628,7 +666,9 @@ attn_decode_mma(const bf16* __restrict__ q, int64_t q_stride, bf16* __restrict__
 #pragma unroll
             for (int sl = 0; sl < 8; ++sl) acc += p[sl] * (lse[sl] * inv);
             if (gate) acc = gated<true>(acc, to_float(gate[(int64_t)row_q * q_stride + (int64_t)(kvh * G + g0 + row) * D + d]));
-            out[(int64_t)row_q * out_stride + (int64_t)(kvh * G + g0 + row) * D + d] = __float2bfloat16_rn(acc);
+            const int64_t at = (int64_t)row_q * out_stride + (int64_t)(kvh * G + g0 + row) * D + d;
+            if (out_f32) reinterpret_cast<float*>(out)[at] = acc;
+            else out[at] = __float2bfloat16_rn(acc);
         }
         cluster_sync_before_exit();  // nobody leaves while its shared memory is still being read
         return;
@@ -677,6 +717,8 @@ attn_decode_mma(const bf16* __restrict__ q, int64_t q_stride, bf16* __restrict__
 #pragma unroll 8
         for (int sl = 0; sl < n_slices; ++sl) acc += __ldcg(po + (int64_t)sl * D) * w[sl];  // slices in order
         if (gate) acc = gated<true>(acc, to_float(gate[(int64_t)row_q * q_stride + (int64_t)head * D + d]));
-        out[(int64_t)row_q * out_stride + (int64_t)head * D + d] = __float2bfloat16_rn(acc);
+        const int64_t at = (int64_t)row_q * out_stride + (int64_t)head * D + d;
+        if (out_f32) reinterpret_cast<float*>(out)[at] = acc;
+        else out[at] = __float2bfloat16_rn(acc);
     }
 }

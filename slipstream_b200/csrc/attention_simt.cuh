@@ -10,7 +10,8 @@
 // in the request; window 0 = all earlier keys), which is the packed-index causal
 // rule of slipstream/models/layers/attention.py:46-51; scores are scaled after the
 // dot product and softmax is float32 as in :64-88.  `sinks` (float32, one per query head, or null): the softmax's
-// denominator also holds exp(sinks[h]), a term of its own with neither key nor value, which the scale does not touch.  Replaces the gather + eager
+// denominator also holds exp(sinks[h]), a term of its own with neither key nor value, which the scale does not touch.
+// `keep` (with a window): the request's first `keep` keys stay visible for good (common.cuh: key_tiles).  Replaces the gather + eager
 // loop of slipstream/kernels/attention_ref.py:68-89 and the Triton decode kernel
 // slipstream/kernels/triton_paged.py:97-206.
 //
@@ -36,7 +37,7 @@ attn_simt_kernel(const T* __restrict__ q, int64_t q_stride, T* __restrict__ out,
                  const int32_t* __restrict__ tile_req, const int32_t* __restrict__ tile_q0,
                  const int32_t* __restrict__ q_start, const int32_t* __restrict__ seq_lens,
                  int n_q, int n_kv, int page_size, int64_t num_pages, float scale, int window,
-                 int* err, const T* __restrict__ gate, float softcap, const float* __restrict__ sinks) {
+                 int* err, const T* __restrict__ gate, float softcap, const float* __restrict__ sinks, int keep) {
     pdl_launch_dependents();  // the next kernel may be scheduled now; it waits for this one itself
     pdl_wait();               // nothing below runs before the kernels before this one are complete
     constexpr int DPL = (D + 31) / 32;
@@ -75,14 +76,15 @@ attn_simt_kernel(const T* __restrict__ q, int64_t q_stride, T* __restrict__ out,
         for (int c = 0; c < DPL; ++c) acc[i][c] = 0.f;
     }
 
-    const int kt_lo = lo_min / ATT_BN, kt_hi = p_max / ATT_BN;
-    for (int kt = kt_lo; kt <= kt_hi; ++kt) {
+    const KeyTiles walk = key_tiles(lo_min, p_max, keep, ATT_BN);
+    for (int jt = 0; jt < walk.count; ++jt) {
+        const int kt = walk.at(jt);
         __syncthreads();
-        // stage keys and values of this tile as float32; rows outside [lo_min, p_max] are zero
+        // stage keys and values of this tile as float32; rows outside [lo_min, p_max] that are not kept are zero
         for (int row = w; row < ATT_BN; row += ATT_WARPS) {
             const int key = kt * ATT_BN + row;
             int64_t page = -1;
-            if (key >= lo_min && key <= p_max) {
+            if ((key >= lo_min || key < keep) && key <= p_max) {
                 page = table[key / page_size];
                 if (page >= num_pages) {
                     if (lane == 0) atomicOr(err, SS_ERR_PAGE_RANGE);
@@ -127,7 +129,7 @@ attn_simt_kernel(const T* __restrict__ q, int64_t q_stride, T* __restrict__ out,
         for (int i = 0; i < ATT_RPW; ++i) {
             const int row = w * ATT_RPW + i;
             const int pos = pos0 + row;
-            const bool ok = row < rows_here && key <= pos && key >= lowest[i];
+            const bool ok = row < rows_here && key <= pos && (key >= lowest[i] || key < keep);
             // softcap > 0: the scaled score is squashed to softcap * tanh(score / softcap) before the softmax
             const float sc = ok ? (softcap > 0.f ? softcap * tanhf(s[i] * scale / softcap) : s[i] * scale) : -INFINITY;
             const float m_new = fmaxf(m[i], warp_max(sc));
@@ -184,7 +186,7 @@ int launch_attn_simt(const void* q, int64_t q_stride, void* out, int64_t out_str
                      const int32_t* tile_q0, int n_tiles, const int32_t* q_start,
                      const int32_t* seq_lens, int n_q, int n_kv, int page_size, int64_t num_pages,
                      float scale, int window, const void* gate, int* err, cudaStream_t stream, float softcap = 0.f,
-                     const float* sinks = nullptr) {
+                     const float* sinks = nullptr, int keep = 0) {
     static_assert(ATT_RPW == 4, "the kernel packs four rows per warp into a float4");
     constexpr int smem = att_simt_smem_bytes<D>();
     static SsPerDevice opted;
@@ -192,6 +194,6 @@ int launch_attn_simt(const void* q, int64_t q_stride, void* out, int64_t out_str
     dim3 grid(n_tiles, n_q);
     ss_launch(attn_simt_kernel<T, D>, dim3(grid), dim3(ATT_WARPS * 32), smem, stream, 
         (const T*)q, q_stride, (T*)out, out_stride, (const T*)kv, block_tables, max_blocks, tile_req,
-        tile_q0, q_start, seq_lens, n_q, n_kv, page_size, num_pages, scale, window, err, (const T*)gate, softcap, sinks);
+        tile_q0, q_start, seq_lens, n_q, n_kv, page_size, num_pages, scale, window, err, (const T*)gate, softcap, sinks, keep);
     return SS_LAUNCH_CHECK();
 }

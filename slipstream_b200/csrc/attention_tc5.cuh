@@ -22,7 +22,8 @@
 // Masking is the packed-index causal rule of slipstream/models/layers/attention.py:46-51; softmax is float32
 // (:64-88).  Besides the causal rule a row sees what `span` says (a sliding window, a chunk, or everything: the
 // tiles begin at the first one the query tile's first row can see, and each row masks the keys in front of its own
-// lowest one), and a soft cap may squash the scaled scores.  Other head sizes and page sizes that do not divide 64
+// lowest one; a window may keep the first keys in sight, whose tiles then stand in front of the window's), and a soft
+// cap may squash the scaled scores.  Other head sizes and page sizes that do not divide 64
 // run the mma.sync kernel of attention_mma.cuh.  Every mbarrier wait is bounded (see gemm_tc5.cu).
 #pragma once
 
@@ -152,6 +153,9 @@ struct Args {
     int span;  // what a query sees besides the causal rule (common.cuh: key_floor); 0: every earlier key
     float softcap;  // > 0: a scaled score s enters the softmax as softcap * tanh(s / softcap)
     const float* sinks;  // float32 [n_q] or null: one more term exp(sinks[h]) in the denominator of head h's softmax
+    int keep;  // with a sliding window: the request's first `keep` keys stay visible (common.cuh: key_tiles)
+    int out_f32;  // `out` is float32
+    DiffPair diff;  // one layer of blocks only (gridDim.z == 1), dim a multiple of 8
 };
 
 template <int D>
@@ -210,16 +214,15 @@ attn_prefill_tc5(const __grid_constant__ CUtensorMap map_q, const __grid_constan
     const int rows_valid = toks_here * G;
     const int pos0 = seq_len - q_len + tok0;           // position of the tile's first token
     const int last_pos = pos0 + toks_here - 1;
-    // The key tiles 0 .. last_pos / 64 of this query tile are shared by the blocks of a thread-block cluster along z
-    // (one block when the grid has one layer): block `part` takes tiles t_lo .. t_lo + n_tiles - 1, and the
+    // The key tiles of this query tile (0 .. last_pos / 64 without a span) are shared by the blocks of a thread-block cluster along z
+    // (one block when the grid has one layer): block `part` takes numbers rel_lo .. rel_lo + n_tiles - 1 of the walk, and the
     // blocks' results are combined through their shared memory at the end.
     const int splits = gridDim.z, part = blockIdx.z;
     // (with a span the tiles begin at the one that holds the lowest key the tile's first token sees)
-    const int t_first = key_floor(pos0, a.span) / FA_BN;
-    const int all_tiles = last_pos / FA_BN + 1 - t_first;
+    const KeyTiles walk = key_tiles(key_floor(pos0, a.span), last_pos, a.keep, FA_BN);
+    const int all_tiles = walk.count;
     const int per_part = (all_tiles + splits - 1) / splits;
     const int rel_lo = min(part * per_part, all_tiles);
-    const int t_lo = t_first + rel_lo;
     const int n_tiles = min(all_tiles, rel_lo + per_part) - rel_lo;  // may be 0
     const int32_t* table = a.block_tables + (int64_t)r * a.max_blocks;
 
@@ -263,7 +266,7 @@ attn_prefill_tc5(const __grid_constant__ CUtensorMap map_q, const __grid_constan
         int64_t spare = __ldg(table);  // keys past the request's end are masked; any finite page will do
         if (spare < 0 || spare >= a.num_pages) spare = 0;
         auto entry = [&](int j) -> int32_t {  // the raw entry: it is looked at one tile later, when it has arrived
-            const int blk = (t_lo + j) * pages_per_tile + p;
+            const int blk = walk.at(rel_lo + j) * pages_per_tile + p;
             return (mine && blk < live_blocks) ? __ldg(table + blk) : -1;
         };
         int32_t next_entry = entry(0);
@@ -340,12 +343,13 @@ attn_prefill_tc5(const __grid_constant__ CUtensorMap map_q, const __grid_constan
         for (int j = 0; j < n_tiles && ok; ++j) {
             const int st = j & 1;
             ok = mbar_wait(&v_full[st], (j >> 1) & 1, gave_up);
-            if (ok && (t_lo + j) * FA_BN + FA_BN > seq_len) {
+            const int tile0 = walk.at(rel_lo + j) * FA_BN;
+            if (ok && tile0 + FA_BN > seq_len) {
                 // The request ends inside this tile.  Rows behind its last token lie in a page that may still hold
                 // what the page's last owner left; their weights are zero, but 0 x inf is not 0, and nothing of
                 // another request may reach this one: clear those value rows (whole 128-byte rows, so the swizzle
                 // does not matter) and make the writes visible to the tensor core's reads.
-                const int first = seq_len - (t_lo + j) * FA_BN;  // 1..63
+                const int first = seq_len - tile0;  // 1..63
                 for (int c = lane; c < (FA_BN - first) * HALVES * 8; c += 32) {
                     const int row = first + c / (HALVES * 8), rest = c % (HALVES * 8);
                     *reinterpret_cast<uint4*>(Vs + st * KV_BYTES + (rest / 8) * HALF_KV + row * 128 + (rest % 8) * 16) = make_uint4(0u, 0u, 0u, 0u);
@@ -400,7 +404,7 @@ attn_prefill_tc5(const __grid_constant__ CUtensorMap map_q, const __grid_constan
                 }
             }
             // raw scores; the scale is folded into the exponent below.  Four running maxima keep the chain short.
-            const int key0 = (t_lo + j) * FA_BN;
+            const int key0 = walk.at(rel_lo + j) * FA_BN;
             if (key0 + FA_BN - 1 > pos) {  // the diagonal tile: keys after the row's own position are masked
 #pragma unroll
                 for (int c = 0; c < 64; ++c)
@@ -409,7 +413,7 @@ attn_prefill_tc5(const __grid_constant__ CUtensorMap map_q, const __grid_constan
             if (key0 < lowest) {  // a tile that begins before the row's span: the keys in front of it are masked
 #pragma unroll
                 for (int c = 0; c < 64; ++c)
-                    if (key0 + c < lowest) sr[c >> 5][c & 31] = 0xff800000u;
+                    if (key0 + c < lowest && key0 + c >= a.keep) sr[c >> 5][c & 31] = 0xff800000u;
             }
             float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
@@ -475,13 +479,60 @@ attn_prefill_tc5(const __grid_constant__ CUtensorMap map_q, const __grid_constan
                 if (a.sinks && valid)
                     l = m_ref == -INFINITY ? 1.f : l + ex2(a.sinks[kvh * G + g] * 1.4426950408889634f - m_ref);
                 const float inv = l > 0.f ? 1.f / l : 0.f;
+                float diff_scale = 0.f;
+                if (a.diff.on) {
+                    // A head's two maps are neighbouring rows (G is even), that is neighbouring lanes.  First pass over
+                    // the columns: the squares of the difference (both lanes form it); the second, below, forms it
+                    // again, and each of the two lanes writes half of the columns.  Columns beyond the values are zero.
+                    float ss = 0.f;
+#pragma unroll 1
+                    for (int c = 0; c < D; c += 32) {
+                        uint32_t o[32];
+                        tmem_ld32(tmem + lane_base + 128 + c, o);
+                        tmem_ld_wait();
+#pragma unroll
+                        for (int e = 0; e < 32; ++e) {
+                            const float mine = __uint_as_float(o[e]) * inv, other = __shfl_xor_sync(0xffffffffu, mine, 1);
+                            const float v = (lane & 1) == 0 ? mine - a.diff.lam * other : other - a.diff.lam * mine;
+                            ss = fmaf(v, v, ss);
+                        }
+                    }
+                    diff_scale = a.diff.mult / sqrtf(ss / (float)a.diff.dim + a.diff.eps);
+                }
                 bf16* dst = a.out + (int64_t)(qs + tok0 + tok) * a.out_stride + (int64_t)(kvh * G + g) * D;
 #pragma unroll 1
                 for (int c = 0; c < D; c += 32) {
                     uint32_t o[32];
                     tmem_ld32(tmem + lane_base + 128 + c, o);
                     tmem_ld_wait();
-                    if (valid) {
+                    if (a.diff.on) {
+                        bf16* pair = a.out + (int64_t)(qs + tok0 + tok) * a.out_stride + (int64_t)((kvh * G + g) >> 1) * a.diff.dim + c;
+#pragma unroll
+                        for (int e = 0; e < 32; e += 8) {
+                            uint32_t packed[4];
+#pragma unroll
+                            for (int k = 0; k < 4; ++k) {
+                                float v[2];
+#pragma unroll
+                                for (int b = 0; b < 2; ++b) {
+                                    const float mine = __uint_as_float(o[e + 2 * k + b]) * inv, other = __shfl_xor_sync(0xffffffffu, mine, 1);
+                                    v[b] = ((lane & 1) == 0 ? mine - a.diff.lam * other : other - a.diff.lam * mine) * diff_scale;
+                                }
+                                __nv_bfloat162 v2 = __floats2bfloat162_rn(v[0], v[1]);
+                                packed[k] = *reinterpret_cast<uint32_t*>(&v2);
+                            }
+                            if (valid && ((e >> 4) == (lane & 1)) && c + e < a.diff.dim)
+                                *reinterpret_cast<uint4*>(pair + e) = make_uint4(packed[0], packed[1], packed[2], packed[3]);
+                        }
+                    } else if (a.out_f32) {
+                        if (valid) {
+                            float* fdst = reinterpret_cast<float*>(a.out) + (int64_t)(qs + tok0 + tok) * a.out_stride + (int64_t)(kvh * G + g) * D + c;
+#pragma unroll
+                            for (int e = 0; e < 32; e += 4)
+                                *reinterpret_cast<float4*>(fdst + e) = make_float4(__uint_as_float(o[e]) * inv, __uint_as_float(o[e + 1]) * inv,
+                                                                                  __uint_as_float(o[e + 2]) * inv, __uint_as_float(o[e + 3]) * inv);
+                        }
+                    } else if (valid) {
 #pragma unroll
                         for (int e = 0; e < 32; e += 8) {
                             uint32_t packed[4];
@@ -556,7 +607,11 @@ attn_prefill_tc5(const __grid_constant__ CUtensorMap map_q, const __grid_constan
                         for (int e = 0; e < 8; ++e) acc[e] += w[sp] * ld_cluster_f32(Osm + (c0 + c + e) * 128 + row, (uint32_t)sp);
                     }
                 }
-                if (valid) {
+                if (valid && a.out_f32) {
+                    float* fdst = reinterpret_cast<float*>(a.out) + (int64_t)(qs + tok0 + tok) * a.out_stride + (int64_t)(kvh * G + g) * D + c0 + c;
+                    *reinterpret_cast<float4*>(fdst) = make_float4(acc[0] * inv, acc[1] * inv, acc[2] * inv, acc[3] * inv);
+                    *reinterpret_cast<float4*>(fdst + 4) = make_float4(acc[4] * inv, acc[5] * inv, acc[6] * inv, acc[7] * inv);
+                } else if (valid) {
                     uint32_t packed[4];
 #pragma unroll
                     for (int k = 0; k < 4; ++k) {

@@ -50,16 +50,41 @@ __device__ __forceinline__ int key_floor(int pos, int span) {
     return 0;
 }
 
-// The gated unit with three constants, of which silu_mul is the case alpha = 1, no limit, shift = 0 (and bit for bit
-// the same then): g = min(gate, limit), u = clamp(up, -limit, limit) (limit <= 0: unclamped);
-// g * sigmoid(alpha * g) * (u + shift).  FAST as in silu_mul.
+// A sliding window may keep the request's first `keep` keys in sight for good (keep 0: none; it comes with a window
+// only).  The tiles of `bn` keys that queries at `lo`'s row and later ones up to position `last` walk are then the
+// ones that hold the kept keys, and those from the first tile of the window on: tile number j of the walk is at(j).
+// Without kept keys, or where the two runs meet, the walk is first .. last / bn.
+struct KeyTiles {
+    int kept, first, count;
+    __device__ __forceinline__ int at(int j) const { return j < kept ? j : first + (j - kept); }
+};
+__device__ __forceinline__ KeyTiles key_tiles(int lo, int last, int keep, int bn) {
+    KeyTiles t;
+    t.first = lo / bn;
+    t.kept = keep > 0 ? min((keep - 1) / bn + 1, t.first) : 0;
+    t.count = t.kept + last / bn - t.first + 1;
+    return t;
+}
+
+// What the attention kernels do with the outputs of a head's two softmax maps (query heads 2h and 2h + 1, side by side
+// in a kv group).  on: o = a_2h - lam * a_2h+1 over the first `dim` elements, times mult / sqrt(mean(o^2) + eps), all in
+// float32, is written as one head of `dim` elements.
+struct DiffPair {
+    int on;
+    float lam, mult, eps;
+    int dim;
+};
+
+// The gated unit with four constants, of which silu_mul is the case alpha = 1, no limit, shift = cubic = 0 (and bit for
+// bit the same then): g = min(gate, limit), u = clamp(up, -limit, limit) (limit <= 0: unclamped);
+// g * sigmoid(alpha * g + cubic * g^3) * (u + shift).  FAST as in silu_mul.
 template <bool FAST>
-__device__ __forceinline__ float glu_mul(float g, float u, float alpha, float limit, float shift) {
+__device__ __forceinline__ float glu_mul(float g, float u, float alpha, float limit, float shift, float cubic = 0.f) {
     if (limit > 0.f) {
         g = fminf(g, limit);
         u = fminf(fmaxf(u, -limit), limit);
     }
-    const float a = alpha * g;
+    const float a = cubic != 0.f ? g * fmaf(cubic, g * g, alpha) : alpha * g;
     return (FAST ? __fdividef(g, 1.0f + __expf(-a)) : g / (1.0f + expf(-a))) * (u + shift);
 }
 

@@ -149,8 +149,8 @@ struct GemmArgs {
     const float* in_squares;
     int in_tiles;
     float in_eps;
-    // the constants of the fused gated unit (common.cuh: glu_mul); 1, 0, 0 is SwiGLU
-    float act_alpha, act_limit, act_shift;
+    // the constants of the fused gated unit (common.cuh: glu_mul); 1, 0, 0, 0 is SwiGLU
+    float act_alpha, act_limit, act_shift, act_cubic;
     // hc_streams S > 0 (with `residual`): the stream is S hyper-connected streams, residual [N][S][M].  The product y
     // (rounded to bfloat16) is WRITTEN into them, stream t <- sum_s hc_mix[s][t] * stream s + hc_out[t] * y, and the
     // norm behind it READS u = sum_t hc_in[t] * stream t: scaled and tile_squares are formed from u.  The arithmetic
@@ -168,7 +168,7 @@ __device__ __forceinline__ void store_swiglu(const GemmArgs& g, int m, int n, fl
     if (m + 64 >= g.M || n >= g.N) return;
     gate *= scale; up *= scale;
     if (g.bias) { gate += bias_at(g, m); up += bias_at(g, m + 64); }
-    const float v = glu_mul<true>(gate, up, g.act_alpha, g.act_limit, g.act_shift);
+    const float v = glu_mul<true>(gate, up, g.act_alpha, g.act_limit, g.act_shift, g.act_cubic);
     const int64_t at = (int64_t)n * g.ldc + (m / TC_BM) * 64 + (m % TC_BM);
     if (g.out_f32) ((float*)g.C)[at] = v;
     else ((bf16*)g.C)[at] = __float2bfloat16_rn(v);
@@ -609,7 +609,7 @@ struct ManyArgs {
     const float* in_squares;
     int in_tiles;
     float in_eps;
-    float act_alpha, act_limit, act_shift;  // as in GemmArgs
+    float act_alpha, act_limit, act_shift, act_cubic;  // as in GemmArgs
     // Grouped form (grp_expert given): the rows of A are sorted by expert, B stacks the experts' weights (grp_b_rows
     // rows each, N of them real), and a row tile is an entry of three lists of grp_tiles entries: the expert (-1: the
     // entry holds nothing), the first row and the number of rows (at most 256; the rows behind them in the tile belong
@@ -890,8 +890,8 @@ gemm_tc5_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_con
                             v0 += bias_many(g, n0 + gc + 2 * e); v1 += bias_many(g, n0 + gc + 2 * e + 1);
                             u0 += bias_many(g, n0 + gc + 64 + 2 * e); u1 += bias_many(g, n0 + gc + 64 + 2 * e + 1);
                         }
-                        __nv_bfloat162 v = __floats2bfloat162_rn(glu_mul<true>(v0, u0, g.act_alpha, g.act_limit, g.act_shift),
-                                                                 glu_mul<true>(v1, u1, g.act_alpha, g.act_limit, g.act_shift));
+                        __nv_bfloat162 v = __floats2bfloat162_rn(glu_mul<true>(v0, u0, g.act_alpha, g.act_limit, g.act_shift, g.act_cubic),
+                                                                 glu_mul<true>(v1, u1, g.act_alpha, g.act_limit, g.act_shift, g.act_cubic));
                         packed[e] = *reinterpret_cast<uint32_t*>(&v);
                     }
                     uint4* dst = reinterpret_cast<uint4*>((bf16*)g.C + (int64_t)m * g.ldc + f0);
@@ -1003,7 +1003,7 @@ struct NormEnds {  // see GemmArgs: the output added to the float32 stream, the 
     const float* in_squares = nullptr;
     int in_tiles = 0;
     float in_eps = 0.f;
-    float act_alpha = 1.f, act_limit = 0.f, act_shift = 0.f;  // the fused gated unit's constants (SwiGLU)
+    float act_alpha = 1.f, act_limit = 0.f, act_shift = 0.f, act_cubic = 0.f;  // the fused gated unit's constants (SwiGLU)
     int hc_streams = 0;             // see GemmArgs
     const float* hc_weights = nullptr;  // host memory: mix [S * S], out [S], in [S]
 };
@@ -1034,7 +1034,7 @@ static int gemm_tc5(const void* A, const void* B, const void* bias, int bias_f32
     g.residual = ends.residual; g.tile_squares = ends.tile_squares; g.scaled = (bf16*)ends.scaled;
     g.norm_weight = ends.norm_weight; g.norm_w_f32 = ends.norm_w_f32;
     g.in_squares = ends.in_squares; g.in_tiles = ends.in_tiles; g.in_eps = ends.in_eps;
-    g.act_alpha = ends.act_alpha; g.act_limit = ends.act_limit; g.act_shift = ends.act_shift;
+    g.act_alpha = ends.act_alpha; g.act_limit = ends.act_limit; g.act_shift = ends.act_shift; g.act_cubic = ends.act_cubic;
     g.hc_streams = 0;
     if (ends.hc_streams > 0) {
         const int S = ends.hc_streams;
@@ -1075,10 +1075,10 @@ extern "C" int ss_gemm_tc5(const void* A, const void* B, const void* bias, int b
 // The product with the fused gated unit of other constants than SwiGLU's (common.cuh: glu_mul).
 extern "C" int ss_gemm_tc5_glu(const void* A, const void* B, const void* bias, int bias_f32, void* C, int M, int N, int K,
                                int64_t lda, int64_t ldb, int64_t ldc, int bn, int swapped, int out_f32, int slices,
-                               float alpha, float limit, float shift, float* partial, int* counters, int* err,
+                               float alpha, float limit, float shift, float cubic, float* partial, int* counters, int* err,
                                cudaStream_t stream) {
     NormEnds ends;
-    ends.act_alpha = alpha; ends.act_limit = limit; ends.act_shift = shift;
+    ends.act_alpha = alpha; ends.act_limit = limit; ends.act_shift = shift; ends.act_cubic = cubic;
     return gemm_tc5(A, B, bias, bias_f32, C, M, N, K, lda, ldb, ldc, bn, swapped, out_f32, slices, 1, partial, counters,
                     ends, err, stream);
 }
@@ -1126,10 +1126,10 @@ extern "C" int ss_gemm_tc5_scaled(const void* A, const void* B, const float* in_
 extern "C" int ss_gemm_tc5_scaled_glu(const void* A, const void* B, const float* in_squares, int in_tiles, float eps,
                                       const void* bias, int bias_f32, void* C, int M, int N, int K, int64_t lda, int64_t ldb,
                                       int64_t ldc, int bn, int out_f32, int slices, float alpha, float limit, float shift,
-                                      float* partial, int* counters, int* err, cudaStream_t stream) {
+                                      float cubic, float* partial, int* counters, int* err, cudaStream_t stream) {
     NormEnds ends;
     ends.in_squares = in_squares; ends.in_tiles = in_tiles; ends.in_eps = eps;
-    ends.act_alpha = alpha; ends.act_limit = limit; ends.act_shift = shift;
+    ends.act_alpha = alpha; ends.act_limit = limit; ends.act_shift = shift; ends.act_cubic = cubic;
     return gemm_tc5(A, B, bias, bias_f32, C, M, N, K, lda, ldb, ldc, bn, 1, out_f32, slices, 1, partial, counters,
                     ends, err, stream);
 }
@@ -1197,7 +1197,7 @@ static int gemm_tc5_many(const void* A, const void* B, const void* bias, int bia
     g.residual = ends.residual; g.tile_squares = ends.tile_squares; g.scaled = (bf16*)ends.scaled;
     g.norm_weight = ends.norm_weight; g.norm_w_f32 = ends.norm_w_f32;
     g.in_squares = ends.in_squares; g.in_tiles = ends.in_tiles; g.in_eps = ends.in_eps;
-    g.act_alpha = ends.act_alpha; g.act_limit = ends.act_limit; g.act_shift = ends.act_shift;
+    g.act_alpha = ends.act_alpha; g.act_limit = ends.act_limit; g.act_shift = ends.act_shift; g.act_cubic = ends.act_cubic;
     g.grp_expert = g.grp_row0 = g.grp_rows = nullptr; g.grp_tiles = 0; g.grp_b_rows = 0;
     const int tiles2 = n_m * ((N + bn - 1) / bn);
     const int pairs = tiles2 < max_pairs ? tiles2 : max_pairs;
@@ -1236,7 +1236,7 @@ extern "C" int ss_gemm_tc5_grouped(const void* A, const void* B, void* C, int to
     g.bias_f32 = 0; g.swiglu = swiglu; g.tile_cols = bn;
     g.residual = nullptr; g.tile_squares = nullptr; g.scaled = nullptr; g.norm_weight = nullptr; g.norm_w_f32 = 0;
     g.in_squares = nullptr; g.in_tiles = 0; g.in_eps = 0.f;
-    g.act_alpha = 1.f; g.act_limit = 0.f; g.act_shift = 0.f;
+    g.act_alpha = 1.f; g.act_limit = 0.f; g.act_shift = 0.f; g.act_cubic = 0.f;
     g.grp_expert = tile_expert; g.grp_row0 = tile_row0; g.grp_rows = tile_rows; g.grp_tiles = n_tiles; g.grp_b_rows = b_rows;
     const int n_sms = ss_sm_count();
     const int max_pairs = n_sms / 2 > 0 ? n_sms / 2 : 1;
@@ -1247,9 +1247,9 @@ extern "C" int ss_gemm_tc5_grouped(const void* A, const void* B, void* C, int to
 // The same product with the fused gated unit of other constants than SwiGLU's.
 extern "C" int ss_gemm_tc5_many_glu(const void* A, const void* B, const void* bias, int bias_f32, void* C, int M, int N,
                                     int K, int64_t lda, int64_t ldb, int64_t ldc, float alpha, float limit, float shift,
-                                    int* err, cudaStream_t stream) {
+                                    float cubic, int* err, cudaStream_t stream) {
     NormEnds ends;
-    ends.act_alpha = alpha; ends.act_limit = limit; ends.act_shift = shift;
+    ends.act_alpha = alpha; ends.act_limit = limit; ends.act_shift = shift; ends.act_cubic = cubic;
     return gemm_tc5_many(A, B, bias, bias_f32, C, M, N, K, lda, ldb, ldc, 0, 1, 0, ends, err, stream);
 }
 

@@ -1,0 +1,387 @@
+// Kernels between a layer's products and its attention, and behind them:
+//  * heads_to_pages: projected queries, keys and values into the forms the paged attention kernels read;
+//  * diff_combine: the two maps of differential heads into one output;
+//  * branch_norm: a branch's normed output joins the stream, and the next norm of the stream.
+// All arithmetic is float32 and rounds once where it is written.
+#include "common.cuh"
+
+// Sum over the block with one barrier: every thread adds the warps' sums in the same order.  `scratch` (32 floats) may
+// not be written again before the next barrier of the block.
+__device__ __forceinline__ float block_sum_once(float v, float* scratch) {
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n_warps = (blockDim.x + 31) >> 5;
+    v = warp_sum(v);
+    if (lane == 0) scratch[warp] = v;
+    __syncthreads();
+    return warp_sum(lane < n_warps ? scratch[lane] : 0.f);
+}
+
+__device__ __forceinline__ void unpack8(const uint4& r, float (&v)[8]) {
+    const uint32_t w[4] = {r.x, r.y, r.z, r.w};
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+        v[2 * e] = __uint_as_float(w[e] << 16);
+        v[2 * e + 1] = __uint_as_float(w[e] & 0xffff0000u);
+    }
+}
+__device__ __forceinline__ uint4 pack8(const float (&v)[8]) {
+    uint32_t w[4];
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+        const __nv_bfloat162 p = __floats2bfloat162_rn(v[2 * e], v[2 * e + 1]);
+        w[e] = *reinterpret_cast<const uint32_t*>(&p);
+    }
+    return make_uint4(w[0], w[1], w[2], w[3]);
+}
+__device__ __forceinline__ void load8f(const float* p, float (&v)[8]) {
+    const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
+    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+}
+__device__ __forceinline__ void store8f(float* p, const float (&v)[8]) {
+    *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+    *reinterpret_cast<float4*>(p + 4) = make_float4(v[4], v[5], v[6], v[7]);
+}
+
+// ---------------------------------------------------------------- projected heads -> queries and pages
+//
+// A row holds n_q * M query parts and (from k_col) n_kv * M key parts of d elements, M the maps of a head (1, or 2 for
+// differential heads: [map 1 | map 2] head by head), and from v_col n_kv values of dv elements (v_col may be k_col: the
+// values are then the keys as projected).  Per token:
+//   norm      with q_weight / k_weight: x / sqrt(mean(x^2) + eps) * w over ALL queries of the token at once, and over all
+//             its keys at once (not the values);
+//   rotation  of the first rot_dim elements of every part by position * inv_freq, in pairs of neighbours (2i, 2i + 1) or,
+//             not interleaved, (i, i + rot_dim / 2);
+//   queries   to q_out [token][n_q * M][D]: the part of map m of a head lies at m * d of its D elements, zeros elsewhere;
+//   keys      to their page: all maps of a kv head side by side in one row of D elements, zeros behind them;
+//   values    to theirs: dv elements, zeros behind them.
+// The score of query (head, map m) with such a key row is that of map m alone, so the attention kernels run n_q * M
+// query heads over n_kv key/value heads of D >= max(M * d, dv) elements.  kv: [page][2][kv head][offset][D].
+// A block per token.  VEC 8: bfloat16, 16-byte accesses, pairs of neighbours; VEC 1: any type and size.
+struct HeadsArgs {
+    const void* rows;
+    int64_t row_stride;
+    const int32_t* positions;
+    const int32_t* slots;
+    const float* inv_freq;
+    const float* q_weight;
+    const float* k_weight;
+    void* q_out;
+    void* kv;
+    int n_q, n_kv, maps, d, dv, D, k_col, v_col, rot_dim, interleaved, page_size;
+    float eps;
+    int64_t pool_slots;
+    int* err;
+};
+
+template <typename T, int VEC>
+__global__ void __launch_bounds__(512) heads_to_pages_kernel(const HeadsArgs a) {
+    pdl_launch_dependents();
+    pdl_wait();
+    __shared__ float cos_s[128], sin_s[128], scratch[2][32];
+    const int t = blockIdx.x;
+    const T* row = reinterpret_cast<const T*>(a.rows) + (int64_t)t * a.row_stride;
+    const float pos = (float)a.positions[t];
+    for (int i = threadIdx.x; i < a.rot_dim / 2; i += blockDim.x) sincosf(__fmul_rn(pos, a.inv_freq[i]), &sin_s[i], &cos_s[i]);
+    int64_t slot = (a.slots && a.kv) ? (int64_t)a.slots[t] : -1;
+    if (slot >= a.pool_slots) {
+        if (threadIdx.x == 0) atomicOr(a.err, SS_ERR_SLOT_RANGE);
+        slot = -1;
+    }
+    const int md = a.maps * a.d, D = a.D;
+    const int q_len = a.n_q * md, k_len = a.n_kv * md;
+    float q_rstd = 1.f, k_rstd = 1.f;
+    if (a.q_weight) {
+        float sq = 0.f, sk = 0.f;
+        for (int c = threadIdx.x * VEC; c < q_len + k_len; c += blockDim.x * VEC) {
+            const bool is_q = c < q_len;  // VEC divides q_len
+            const T* p = is_q ? row + c : row + a.k_col + (c - q_len);
+            float s = 0.f;
+            if constexpr (VEC == 8) {
+                float v[8];
+                unpack8(*reinterpret_cast<const uint4*>(p), v);
+#pragma unroll
+                for (int e = 0; e < 8; ++e) s = fmaf(v[e], v[e], s);
+            } else {
+                const float v = to_float(*p);
+                s = v * v;
+            }
+            if (is_q) sq += s; else sk += s;
+        }
+        q_rstd = 1.0f / sqrtf(block_sum_once(sq, scratch[0]) / (float)q_len + a.eps);
+        k_rstd = 1.0f / sqrtf(block_sum_once(sk, scratch[1]) / (float)k_len + a.eps);
+    } else {
+        __syncthreads();
+    }
+    const int64_t page = slot >= 0 ? slot / a.page_size : 0;
+    const int off = slot >= 0 ? (int)(slot % a.page_size) : 0;
+    // outputs in runs of VEC: queries, then (with a slot) keys and values
+    const int per_head = D / VEC, q_runs = a.n_q * a.maps * per_head, kv_runs = slot >= 0 ? a.n_kv * per_head : 0;
+    T* const q_out = reinterpret_cast<T*>(a.q_out) + (int64_t)t * a.n_q * a.maps * D;
+    T* const kv = reinterpret_cast<T*>(a.kv);
+    for (int run = threadIdx.x; run < q_runs + 2 * kv_runs; run += blockDim.x) {
+        const bool is_q = run < q_runs, is_v = run >= q_runs + kv_runs;
+        const int r = is_q ? run : (is_v ? run - q_runs - kv_runs : run - q_runs);
+        const int head = r / per_head, o = (r - head * per_head) * VEC;
+        T* dst;
+        int from = -1;  // place of the run's first element among its projection's; -1: zeros
+        int in_part = 0;
+        if (is_q) {
+            dst = q_out + (int64_t)head * D + o;
+            const int m = a.maps == 1 ? 0 : head % a.maps, h = a.maps == 1 ? head : head / a.maps;
+            in_part = o - m * a.d;
+            if (in_part >= 0 && in_part < a.d) from = h * md + o;
+        } else {
+            dst = kv + ((((page * 2 + (is_v ? 1 : 0)) * a.n_kv + head) * a.page_size + off) * (int64_t)D) + o;
+            if (is_v) {
+                if (o < a.dv) from = head * a.dv + o;
+            } else if (o < md) {
+                in_part = a.maps == 1 ? o : o % a.d;
+                from = head * md + o;
+            }
+        }
+        const T* src = row + (is_q ? 0 : (is_v ? a.v_col : a.k_col)) + from;
+        const float* w = is_q ? a.q_weight : a.k_weight;
+        const float rstd = is_q ? q_rstd : k_rstd;
+        const bool normed = w != nullptr && !is_v, turned = !is_v && in_part < a.rot_dim;
+        if constexpr (VEC == 8) {
+            float v[8];
+            if (from < 0) {
+                *reinterpret_cast<uint4*>(dst) = make_uint4(0u, 0u, 0u, 0u);
+                continue;
+            }
+            unpack8(*reinterpret_cast<const uint4*>(src), v);
+            if (normed) {
+                float w8[8];
+                load8f(w + from, w8);
+#pragma unroll
+                for (int e = 0; e < 8; ++e) v[e] = v[e] * rstd * w8[e];
+            }
+            if (turned) {
+#pragma unroll
+                for (int e = 0; e < 8; e += 2) {
+                    const int i = (in_part + e) >> 1;
+                    if (in_part + e < a.rot_dim) {
+                        const float c = cos_s[i], s = sin_s[i], x = v[e], y = v[e + 1];
+                        v[e] = __fadd_rn(__fmul_rn(x, c), __fmul_rn(-y, s));
+                        v[e + 1] = __fadd_rn(__fmul_rn(y, c), __fmul_rn(x, s));
+                    }
+                }
+            }
+            *reinterpret_cast<uint4*>(dst) = pack8(v);
+        } else {
+            float v = 0.f;
+            if (from >= 0) {
+                v = to_float(*src);
+                if (normed) v = v * rstd * w[from];
+                if (turned) {
+                    const int half = a.rot_dim >> 1;
+                    const bool second = a.interleaved ? (in_part & 1) != 0 : in_part >= half;
+                    const int to = a.interleaved ? (second ? -1 : 1) : (second ? -half : half);
+                    const int i = a.interleaved ? in_part >> 1 : (second ? in_part - half : in_part);
+                    float other = to_float(src[to]);
+                    if (normed) other = other * rstd * w[from + to];
+                    // (u, v) -> (u c - v s, v c + u s)
+                    v = __fadd_rn(__fmul_rn(v, cos_s[i]), __fmul_rn(second ? other : -other, sin_s[i]));
+                }
+            }
+            *dst = from_float<T>(v);
+        }
+    }
+}
+
+extern "C" int ss_heads_to_pages(const void* rows, int64_t row_stride, const int32_t* positions, const int32_t* slots,
+                                 const float* inv_freq, const float* q_weight, const float* k_weight, void* q_out, void* kv,
+                                 int n_tokens, int n_q, int n_kv, int maps, int d, int dv, int D, int k_col, int v_col,
+                                 int rot_dim, int interleaved, float eps, int page_size, int64_t num_pages, int dtype, int* err,
+                                 cudaStream_t stream) {
+    if (n_tokens <= 0) return 0;
+    if (n_q < 1 || n_kv < 0 || (maps != 1 && maps != 2) || d < 1 || dv < 1 || D % 8 != 0 || maps * d > D || dv > D || rot_dim < 0 ||
+        rot_dim > d || rot_dim % 2 || rot_dim > 256 || (rot_dim > 0 && !inv_freq) || (!q_weight != !k_weight && n_kv > 0) || page_size < 1)
+        return (int)cudaErrorInvalidValue;
+    HeadsArgs a;
+    a.rows = rows; a.row_stride = row_stride; a.positions = positions; a.slots = slots; a.inv_freq = inv_freq;
+    a.q_weight = q_weight; a.k_weight = k_weight; a.q_out = q_out; a.kv = kv; a.n_q = n_q; a.n_kv = n_kv; a.maps = maps;
+    a.d = d; a.dv = dv; a.D = D; a.k_col = k_col; a.v_col = v_col; a.rot_dim = rot_dim; a.interleaved = interleaved;
+    a.page_size = page_size; a.eps = eps; a.pool_slots = num_pages * page_size; a.err = err;
+    const bool wide = dtype == SS_BF16 && (interleaved || rot_dim == 0) && d % 8 == 0 && dv % 8 == 0 && k_col % 8 == 0 &&
+                      v_col % 8 == 0 && row_stride % 8 == 0 && ((uintptr_t)rows & 15) == 0 && ((uintptr_t)q_out & 15) == 0 &&
+                      ((uintptr_t)kv & 15) == 0 && ((uintptr_t)q_weight & 15) == 0 && ((uintptr_t)k_weight & 15) == 0;
+    if (wide) {
+        const int runs = (n_q * maps + 2 * n_kv) * (D / 8);
+        const int threads = runs >= 1024 ? 512 : (runs >= 512 ? 256 : 128);
+        ss_launch(heads_to_pages_kernel<bf16, 8>, dim3(n_tokens), dim3(threads), 0, stream, a);
+    } else if (dtype == SS_BF16) {
+        ss_launch(heads_to_pages_kernel<bf16, 1>, dim3(n_tokens), dim3(256), 0, stream, a);
+    } else {
+        ss_launch(heads_to_pages_kernel<float, 1>, dim3(n_tokens), dim3(256), 0, stream, a);
+    }
+    return SS_LAUNCH_CHECK();
+}
+
+// ---------------------------------------------------------------- the two maps of differential heads
+//
+// x: float32 [token][2 * heads][D], maps 2h and 2h + 1 of head h.  out [token][heads * dv]: with o = x_2h - lam * x_2h+1
+// over the first dv elements, o * mult / sqrt(mean(o^2) + eps).  A warp per (token, head).
+template <typename T>
+__global__ void __launch_bounds__(256)
+diff_combine_kernel(const float* __restrict__ x, T* __restrict__ out, int64_t pairs, int D, int dv, float lam, float mult, float eps) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int lane = threadIdx.x & 31;
+    const int64_t p = (int64_t)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    if (p >= pairs) return;
+    const float* x1 = x + p * 2 * D;
+    constexpr int EPL = 8;  // dv is at most 256
+    float o[EPL];
+    float ss = 0.f;
+#pragma unroll
+    for (int c = 0; c < EPL; ++c) {
+        const int e = lane + 32 * c;
+        o[c] = e < dv ? x1[e] - lam * x1[D + e] : 0.f;
+        ss = fmaf(o[c], o[c], ss);
+    }
+    const float f = mult / sqrtf(warp_sum(ss) / (float)dv + eps);
+#pragma unroll
+    for (int c = 0; c < EPL; ++c) {
+        const int e = lane + 32 * c;
+        if (e < dv) out[p * dv + e] = from_float<T>(o[c] * f);
+    }
+}
+
+extern "C" int ss_diff_combine(const float* x, void* out, int64_t n_tokens, int heads, int D, int dv, float lam, float mult,
+                               float eps, int dtype, cudaStream_t stream) {
+    if (n_tokens <= 0) return 0;
+    if (heads < 1 || dv < 1 || dv > D || dv > 256) return (int)cudaErrorInvalidValue;
+    const int64_t pairs = n_tokens * heads;
+    const int warps = pairs >= 8 * ss_sm_count() ? 8 : 2;
+    const dim3 grid((unsigned)((pairs + warps - 1) / warps)), block(warps * 32);
+    if (dtype == SS_BF16) ss_launch(diff_combine_kernel<bf16>, grid, block, 0, stream, x, (bf16*)out, pairs, D, dv, lam, mult, eps);
+    else ss_launch(diff_combine_kernel<float>, grid, block, 0, stream, x, (float*)out, pairs, D, dv, lam, mult, eps);
+    return SS_LAUNCH_CHECK();
+}
+
+// ---------------------------------------------------------------- a branch's normed output, and the next norm
+//
+// residual += mult * (y / sqrt(mean(y^2) + eps_y) * w_y) [+ anchor], then out = residual / sqrt(mean(residual^2) + eps) * w.
+// y null: the second half only.  With `rows` only those rows are produced and the stream stays as it is.  Weights are
+// float32.  A block per row.  VEC 8: hidden a multiple of 8, at most 8 elements a thread, each row read once; VEC 1: any.
+struct BranchArgs {
+    float* residual;
+    const void* y;
+    const float* y_weight;
+    const float* anchor;
+    const float* weight;
+    void* out;
+    const int32_t* rows;
+    int hidden;
+    float mult, y_eps, eps;
+};
+
+template <typename T, int VEC>
+__global__ void __launch_bounds__(1024) branch_norm_kernel(const BranchArgs a) {
+    pdl_launch_dependents();
+    __shared__ float scratch[2][32];
+    const int hidden = a.hidden;
+    if constexpr (VEC == 8) {
+        const int j = threadIdx.x * 8;
+        const bool on = j < hidden;
+        float wy[8], w[8];
+        if (on) {  // weights do not depend on the kernels in front
+            load8f(a.weight + j, w);
+            if (a.y) load8f(a.y_weight + j, wy);
+        }
+        pdl_wait();
+        const int64_t src = a.rows ? a.rows[blockIdx.x] : blockIdx.x;
+        float v[8];
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[e] = 0.f;
+        if (on) load8f(a.residual + src * hidden + j, v);
+        if (a.y) {
+            float y[8];
+#pragma unroll
+            for (int e = 0; e < 8; ++e) y[e] = 0.f;
+            float ss = 0.f;
+            if (on) {
+                if constexpr (sizeof(T) == 2) unpack8(*reinterpret_cast<const uint4*>(reinterpret_cast<const T*>(a.y) + src * hidden + j), y);
+                else load8f(reinterpret_cast<const float*>(a.y) + src * hidden + j, y);
+#pragma unroll
+                for (int e = 0; e < 8; ++e) ss = fmaf(y[e], y[e], ss);
+            }
+            float anchor[8];
+            if (on && a.anchor) load8f(a.anchor + src * hidden + j, anchor);
+            const float f = 1.0f / sqrtf(block_sum_once(ss, scratch[0]) / (float)hidden + a.y_eps);
+            if (on) {
+#pragma unroll
+                for (int e = 0; e < 8; ++e) v[e] = fmaf(a.mult, y[e] * f * wy[e], v[e]);
+                if (a.anchor) {
+#pragma unroll
+                    for (int e = 0; e < 8; ++e) v[e] += anchor[e];
+                }
+                if (!a.rows) store8f(a.residual + src * hidden + j, v);
+            }
+        }
+        float ss = 0.f;
+#pragma unroll
+        for (int e = 0; e < 8; ++e) ss = fmaf(v[e], v[e], ss);
+        const float f = 1.0f / sqrtf(block_sum_once(ss, scratch[1]) / (float)hidden + a.eps);
+        if (on) {
+#pragma unroll
+            for (int e = 0; e < 8; ++e) v[e] = v[e] * f * w[e];
+            T* out = reinterpret_cast<T*>(a.out) + (int64_t)blockIdx.x * hidden + j;
+            if constexpr (sizeof(T) == 2) *reinterpret_cast<uint4*>(out) = pack8(v);
+            else store8f(reinterpret_cast<float*>(out), v);
+        }
+    } else {
+        pdl_wait();
+        const int64_t src = a.rows ? a.rows[blockIdx.x] : blockIdx.x;
+        float* res = a.residual + src * hidden;
+        const T* y = a.y ? reinterpret_cast<const T*>(a.y) + src * hidden : nullptr;
+        const float* anchor = a.anchor ? a.anchor + src * hidden : nullptr;
+        T* out = reinterpret_cast<T*>(a.out) + (int64_t)blockIdx.x * hidden;
+        float fy = 0.f;
+        if (y) {
+            float ss = 0.f;
+            for (int j = threadIdx.x; j < hidden; j += blockDim.x) ss = fmaf(to_float(y[j]), to_float(y[j]), ss);
+            fy = 1.0f / sqrtf(block_sum_once(ss, scratch[0]) / (float)hidden + a.y_eps);
+        }
+        auto joined = [&](int j) {
+            float v = res[j];
+            if (y) {
+                v = fmaf(a.mult, to_float(y[j]) * fy * a.y_weight[j], v);
+                if (anchor) v += anchor[j];
+            }
+            return v;
+        };
+        float ss = 0.f;
+        for (int j = threadIdx.x; j < hidden; j += blockDim.x) {
+            const float v = joined(j);
+            ss = fmaf(v, v, ss);
+        }
+        const float f = 1.0f / sqrtf(block_sum_once(ss, scratch[1]) / (float)hidden + a.eps);
+        for (int j = threadIdx.x; j < hidden; j += blockDim.x) {  // every thread meets its own elements again
+            const float v = joined(j);
+            if (y && !a.rows) res[j] = v;
+            out[j] = from_float<T>(v * f * a.weight[j]);
+        }
+    }
+}
+
+extern "C" int ss_branch_norm(float* residual, const void* y, const float* y_weight, float y_eps, float mult, const float* anchor,
+                              const float* weight, float eps, void* out, const int32_t* rows, int n_rows, int hidden, int dtype,
+                              cudaStream_t stream) {
+    if (n_rows <= 0) return 0;
+    if (hidden < 1 || (y && !y_weight) || (!y && anchor)) return (int)cudaErrorInvalidValue;
+    BranchArgs a;
+    a.residual = residual; a.y = y; a.y_weight = y_weight; a.anchor = anchor; a.weight = weight; a.out = out; a.rows = rows;
+    a.hidden = hidden; a.mult = mult; a.y_eps = y_eps; a.eps = eps;
+    const bool aligned = (((uintptr_t)residual | (uintptr_t)y | (uintptr_t)y_weight | (uintptr_t)anchor | (uintptr_t)weight | (uintptr_t)out) & 15) == 0;
+    if (hidden % 8 == 0 && hidden <= 8192 && aligned) {
+        const dim3 block((hidden / 8 + 31) / 32 * 32);
+        if (dtype == SS_BF16) ss_launch(branch_norm_kernel<bf16, 8>, dim3(n_rows), block, 0, stream, a);
+        else ss_launch(branch_norm_kernel<float, 8>, dim3(n_rows), block, 0, stream, a);
+    } else {
+        const dim3 block(hidden >= 2048 ? 512 : (hidden >= 512 ? 256 : 128));
+        if (dtype == SS_BF16) ss_launch(branch_norm_kernel<bf16, 1>, dim3(n_rows), block, 0, stream, a);
+        else ss_launch(branch_norm_kernel<float, 1>, dim3(n_rows), block, 0, stream, a);
+    }
+    return SS_LAUNCH_CHECK();
+}

@@ -504,7 +504,7 @@ extern "C" int ss_rope_norm_cache(void* rows, int64_t row_stride, const int32_t*
 // product's fused epilogue uses too: a value does not depend on which of them ran.
 template <typename T>
 __global__ void glu_limited_kernel(const T* __restrict__ in, T* __restrict__ out, int64_t n, int inter, int block,
-                                   float alpha, float limit, float shift) {
+                                   float alpha, float limit, float shift, float cubic) {
     pdl_wait();
     const int64_t total = n * inter;
     for (int64_t idx = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total;
@@ -512,13 +512,13 @@ __global__ void glu_limited_kernel(const T* __restrict__ in, T* __restrict__ out
         const int64_t r = idx / inter;
         const int c = (int)(idx - r * inter);
         const T* gp = in + r * 2 * inter + (int64_t)(c / block) * 2 * block + (c % block);
-        out[idx] = from_float<T>(glu_mul<sizeof(T) == 2>(to_float(gp[0]), to_float(gp[block]), alpha, limit, shift));
+        out[idx] = from_float<T>(glu_mul<sizeof(T) == 2>(to_float(gp[0]), to_float(gp[block]), alpha, limit, shift, cubic));
     }
 }
 
 // bfloat16, 8 gate and the 8 matching up features per thread (block % 8 == 0, 16-byte aligned rows).
 __global__ void glu_limited_bf16x8_kernel(const bf16* __restrict__ in, bf16* __restrict__ out, int64_t n, int inter,
-                                          int block, float alpha, float limit, float shift) {
+                                          int block, float alpha, float limit, float shift, float cubic) {
     pdl_wait();
     const int per_row = inter / 8;
     const int64_t total = n * per_row;
@@ -536,8 +536,8 @@ __global__ void glu_limited_bf16x8_kernel(const bf16* __restrict__ in, bf16* __r
             const __nv_bfloat162 g2 = *reinterpret_cast<const __nv_bfloat162*>(&gw[e]);
             const __nv_bfloat162 u2 = *reinterpret_cast<const __nv_bfloat162*>(&uw[e]);
             const __nv_bfloat162 o2 = __floats2bfloat162_rn(
-                glu_mul<true>(__low2float(g2), __low2float(u2), alpha, limit, shift),
-                glu_mul<true>(__high2float(g2), __high2float(u2), alpha, limit, shift));
+                glu_mul<true>(__low2float(g2), __low2float(u2), alpha, limit, shift, cubic),
+                glu_mul<true>(__high2float(g2), __high2float(u2), alpha, limit, shift, cubic));
             ow[e] = *reinterpret_cast<const uint32_t*>(&o2);
         }
         *reinterpret_cast<uint4*>(out + r * inter + c) = make_uint4(ow[0], ow[1], ow[2], ow[3]);
@@ -545,7 +545,7 @@ __global__ void glu_limited_bf16x8_kernel(const bf16* __restrict__ in, bf16* __r
 }
 
 extern "C" int ss_glu_limited(const void* in, void* out, int64_t n, int inter, int block, float alpha, float limit,
-                              float shift, int dtype, cudaStream_t stream) {
+                              float shift, float cubic, int dtype, cudaStream_t stream) {
     if (n <= 0) return 0;
     if (block <= 0 || inter % block != 0) return (int)cudaErrorInvalidValue;
     const int threads = 256;
@@ -553,17 +553,17 @@ extern "C" int ss_glu_limited(const void* in, void* out, int64_t n, int inter, i
         int64_t blocks = (n * (inter / 8) + threads - 1) / threads;
         if (blocks > ss_sm_count() * 16) blocks = ss_sm_count() * 16;
         ss_launch(glu_limited_bf16x8_kernel, dim3((int)blocks), dim3(threads), 0, stream, (const bf16*)in, (bf16*)out, n,
-                  inter, block, alpha, limit, shift);
+                  inter, block, alpha, limit, shift, cubic);
         return SS_LAUNCH_CHECK();
     }
     int64_t blocks = (n * inter + threads - 1) / threads;
     if (blocks > ss_sm_count() * 32) blocks = ss_sm_count() * 32;
     if (dtype == SS_BF16)
         ss_launch(glu_limited_kernel<bf16>, dim3((int)blocks), dim3(threads), 0, stream, (const bf16*)in, (bf16*)out, n, inter,
-                  block, alpha, limit, shift);
+                  block, alpha, limit, shift, cubic);
     else
         ss_launch(glu_limited_kernel<float>, dim3((int)blocks), dim3(threads), 0, stream, (const float*)in, (float*)out, n,
-                  inter, block, alpha, limit, shift);
+                  inter, block, alpha, limit, shift, cubic);
     return SS_LAUNCH_CHECK();
 }
 

@@ -80,6 +80,7 @@ class DecodeGraph:
         self.mirror_event: torch.cuda.Event | None = None  # a copy of the whole mirror that may still be running
         self.row_owner: list[object] = [None] * B  # the cache manager's record of the request whose table each row holds
         self.row_synced = [[0] * B for _ in range(G)]  # entries of the request's table that the row holds
+        self.kept_blocks = [cache.kept_blocks(g) for g in range(G)]  # blocks that no window passes
         self.row_first = [[0] * B for _ in range(G)]  # first block not yet given back, as the row knows it
         self.full_copies = 0
 
@@ -168,7 +169,7 @@ class DecodeGraph:
                 first_known = 0 if fresh else self.row_first[g][i]
                 first = req.first_block[g]
                 if first > first_known and not fresh:  # pages a window has passed
-                    for b in range(first_known, min(first, synced)):
+                    for b in range(max(first_known, self.kept_blocks[g]), min(first, synced)):
                         idx.append(base + b)
                         val.append(-1)
                         mirror[base + b] = -1
@@ -264,7 +265,7 @@ class MixedGraph:
         self.max_blocks = [max(1, (runner.max_model_len + ps - 1) // ps) for ps in cache.page_sizes]
         self.tile_capacity = 2 * N + R  # entries per list: the most tiles a step has while a tile holds 64 rows of a
         # group of up to 128 heads, or 16 tokens
-        self.max_tile_lists = 4
+        self.max_tile_lists = 8
         names = ["token_ids", "positions", "q_start", "seq_lens", "slots", "first", "logit_rows", "slot_maps"]
         sizes = [N, N, R + 1, R, R, R, L, G * N]
         names += [f"table{g}" for g in range(G)]
@@ -322,7 +323,7 @@ class MixedGraph:
     def _static_tiles(self, key: tuple) -> tuple[torch.Tensor, torch.Tensor]:
         if key not in self.tile_keys:
             if len(self.tile_keys) == self.max_tile_lists:
-                raise RuntimeError("a captured step has room for four lists of query tiles")
+                raise RuntimeError("a captured step has room for eight lists of query tiles")
             self.tile_keys.append(key)
         o = self.offsets["tiles"] + self.tile_keys.index(key) * 2 * self.tile_capacity
         _kind, rows, group = key

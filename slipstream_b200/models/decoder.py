@@ -16,6 +16,7 @@ from dataclasses import dataclass
 
 import torch
 
+from slipstream_b200 import ops
 from slipstream_b200.cache import GroupLayout
 from slipstream_b200.parts.base import (Block, CacheSpec, Embedding, Head, LayerBinding, Norm, Part,
                                         PositionEncoding, Runtime, StateSpec, WeightSpec, settle)
@@ -25,10 +26,12 @@ from slipstream_b200.parts.base import (Block, CacheSpec, Embedding, Head, Layer
 class ExecEntry:
     """One place in the execution order.  ``block``: index of the block whose weights run.
     ``cache_of``: index (into the order) of an earlier entry whose pages this one reads
-    instead of writing its own."""
+    instead of writing its own.  ``add_embedding``: the embedding output (the stream as it was in front of the first
+    entry) is added to the stream right before this entry runs."""
 
     block: int
     cache_of: int | None = None
+    add_embedding: bool = False
 
 
 def _walk(part: Part) -> list[Part]:
@@ -96,8 +99,8 @@ class DecoderLM:
                 continue
             own = self.blocks[self.order[src].block].mixer.cache_spec()
             spec = self.blocks[entry.block].mixer.cache_spec()
-            if own is not None and spec is not None and (spec.window, spec.chunk) != (own.window, own.chunk):
-                kept[src] = dataclasses.replace(own, window=None, chunk=None)
+            if own is not None and spec is not None and (spec.window, spec.chunk, spec.keep_first) != (own.window, own.chunk, own.keep_first):
+                kept[src] = dataclasses.replace(own, window=None, chunk=None, keep_first=0)
         for pos, entry in enumerate(self.order):
             if not 0 <= entry.block < len(self.blocks):
                 raise ValueError(f"order[{pos}] names block {entry.block}, which does not exist")
@@ -153,18 +156,35 @@ class DecoderLM:
         return sum(per_block[e.block] for e in self.order) + self.final_norm.weight_bytes() + self.lm_head.weight_bytes()
 
     # ------------------------------------------------------------------ forward
+    @staticmethod
+    def _add_anchor(residual: torch.Tensor, pending, anchor: torch.Tensor):
+        """Add ``anchor`` to the stream: inside the kernel that applies the pending branch output where that can
+        take it (``with_anchor``), else as a pass of its own."""
+        if hasattr(pending, "with_anchor"):
+            return pending.with_anchor(anchor)
+        residual.copy_(ops.scaled_sum(residual, 1.0, anchor, 1.0))
+        return pending
+
     def forward(self, ctx) -> torch.Tensor:
         """Run the step's tokens through the order; float32 logits [wanted rows, vocab]."""
         residual = self.embedding.forward_step(ctx.token_ids, ctx, self.embedding_state)
         if self.position_encoding is not None:
             self.position_encoding.on_embedding(residual, ctx)
+        # a copy: the stream changes in place from here on
+        anchor = residual.clone() if any(entry.add_embedding for entry in self.order) else None
         pending = normed = None
         observer = ctx.extras.get("layer_observer")  # a caller's tap: (place in the order, stream, pending output)
         # the last block may end in the final norm when that norm needs no selection of rows
         closing = self.final_norm if ctx.extras.get("every_row_wanted") and ctx.num_logits else None
         for pos, (entry, binding) in enumerate(zip(self.order, self.bindings)):
             # a block's last projection may end in the first norm of the block that runs next
-            following = self.blocks[self.order[pos + 1].block].first_norm() if pos + 1 < len(self.order) else closing
+            # (not across a place where the embedding joins the stream in between)
+            following = closing
+            if pos + 1 < len(self.order):
+                after = self.order[pos + 1]
+                following = None if after.add_embedding else self.blocks[after.block].first_norm()
+            if entry.add_embedding:
+                pending = self._add_anchor(residual, pending, anchor)
             residual, pending, normed = self.blocks[entry.block].forward_chained(residual, pending, normed, following,
                                                                                  ctx, binding)
             if observer is not None:

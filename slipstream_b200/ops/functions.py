@@ -57,7 +57,7 @@ _OPS_SIGNATURES = {
                    c_int, c_float, c_int, c_void_p, c_void_p],
     "ss_rope_norm_cache": [c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_int, c_int, c_int, c_int,
                            c_int, c_int, c_int, c_float, c_int, c_int64, c_int, c_int, c_void_p, c_void_p],
-    "ss_glu_limited": [c_void_p, c_void_p, c_int64, c_int, c_int, c_float, c_float, c_float, c_int, c_void_p],
+    "ss_glu_limited": [c_void_p, c_void_p, c_int64, c_int, c_int, c_float, c_float, c_float, c_float, c_int, c_void_p],
     "ss_sigmoid_gate": [c_void_p, c_int64, c_void_p, c_int64, c_int64, c_int, c_int, c_void_p],
     "ss_group_norm": [c_void_p, c_int, c_int64, c_int, c_void_p, c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_void_p,
                       c_int, c_int, c_int, c_float, c_int, c_void_p, c_void_p],
@@ -105,24 +105,33 @@ _OPS_SIGNATURES = {
                    c_int, c_int, c_int, c_int, c_void_p],
     "ss_head_product": [c_void_p, c_int64, c_int, c_void_p, c_void_p, c_int64, c_int, c_int, c_int, c_int, c_int, c_int,
                         c_int, c_void_p, c_void_p, c_float, c_void_p, c_int64, c_int, c_int, c_void_p],
+    "ss_heads_to_pages": [c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
+                          c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int64, c_int,
+                          c_void_p, c_void_p],
+    "ss_diff_combine": [c_void_p, c_void_p, c_int64, c_int, c_int, c_int, c_float, c_float, c_float, c_int, c_void_p],
+    "ss_branch_norm": [c_void_p, c_void_p, c_void_p, c_float, c_float, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_int,
+                       c_int, c_int, c_void_p],
 }
 
 _ATTN_SIGNATURES = {
     "ss_attn_simt": [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_void_p, c_int, c_void_p,
                      c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int64, c_float,
-                     c_int, c_int, c_void_p, c_void_p, c_void_p, c_float, c_void_p],
+                     c_int, c_int, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_int],
     "ss_attn_prefill_mma": [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_void_p, c_int, c_void_p,
                             c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int64, c_float,
-                            c_int, c_void_p, c_void_p, c_void_p, c_float, c_void_p],
+                            c_int, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_int, c_int, c_int, c_float, c_float,
+                            c_float, c_int],
     "ss_attn_prefill_tc5": [c_void_p, c_int64, c_int, c_void_p, c_int64, c_void_p, c_void_p, c_int, c_void_p,
                             c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int64, c_float, c_int, c_int,
-                            c_void_p, c_void_p, c_float, c_void_p],
+                            c_void_p, c_void_p, c_float, c_void_p, c_int, c_int, c_int, c_float, c_float, c_float, c_int],
     "ss_attn_decode_tma": [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_void_p, c_int, c_int,
                            c_void_p, c_void_p, c_int, c_int, c_int, c_int64, c_float, c_int, c_int,
-                           c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_float],
+                           c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_float,
+                           c_void_p, c_int, c_int],
     "ss_attn_decode_mma": [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_void_p, c_int, c_int,
                            c_void_p, c_void_p, c_int, c_int, c_int, c_int64, c_float, c_int, c_int,
-                           c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_void_p],
+                           c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_int,
+                           c_int],
 }
 
 _GEMM_SIGNATURES = {
@@ -136,16 +145,16 @@ _GEMM_SIGNATURES = {
     "ss_gemm_tc5": [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int64, c_int64, c_int64,
                     c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p],
     "ss_gemm_tc5_glu": [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int64, c_int64, c_int64,
-                        c_int, c_int, c_int, c_int, c_float, c_float, c_float, c_void_p, c_void_p, c_void_p, c_void_p],
+                        c_int, c_int, c_int, c_int, c_float, c_float, c_float, c_float, c_void_p, c_void_p, c_void_p, c_void_p],
     "ss_gemm_tc5_many_glu": [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int64, c_int64, c_int64,
-                             c_float, c_float, c_float, c_void_p, c_void_p],
+                             c_float, c_float, c_float, c_float, c_void_p, c_void_p],
     "ss_gemm_tc5_to_stream": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int64, c_int64, c_int, c_int,
                               c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p],
     "ss_gemm_tc5_to_streams": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int64, c_int64, c_int, c_int,
                                c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p],
     "ss_gemm_tc5_scaled_glu": [c_void_p, c_void_p, c_void_p, c_int, c_float, c_void_p, c_int, c_void_p, c_int, c_int, c_int,
-                               c_int64, c_int64, c_int64, c_int, c_int, c_int, c_float, c_float, c_float, c_void_p, c_void_p,
-                               c_void_p, c_void_p],
+                               c_int64, c_int64, c_int64, c_int, c_int, c_int, c_float, c_float, c_float, c_float, c_void_p,
+                               c_void_p, c_void_p, c_void_p],
     "ss_gemm_tc5_grouped": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int64, c_int64, c_int, c_void_p,
                             c_void_p, c_void_p, c_int, c_void_p, c_void_p],
     "ss_gemm_tc5_scaled": [c_void_p, c_void_p, c_void_p, c_int, c_float, c_void_p, c_int, c_void_p, c_int, c_int, c_int,
@@ -168,7 +177,7 @@ def ops_library() -> ctypes.CDLL:
     lib = _state.get("ops")
     if lib is None:
         require_cuda()
-        lib = load_library("slipstream_ops", ["ops.cu", "ops_streams.cu", "ops_mixers.cu", "ops_cells.cu", "ops_gated.cu", "sampling.cu"])
+        lib = load_library("slipstream_ops", ["ops.cu", "ops_streams.cu", "ops_mixers.cu", "ops_cells.cu", "ops_gated.cu", "ops_heads.cu", "sampling.cu"])
         _declare(lib, _OPS_SIGNATURES)
         _state["ops"] = lib
     return lib  # type: ignore[return-value]
@@ -444,8 +453,8 @@ def rope_norm_cache(rows: torch.Tensor, positions: torch.Tensor, slots: torch.Te
 
 
 def glu_limited(gate_up: torch.Tensor, block: int | None = None, alpha: float = 1.0, limit: float = 0.0,
-                shift: float = 0.0) -> torch.Tensor:
-    """``g * sigmoid(alpha * g) * (u + shift)`` with ``g = min(gate, limit)`` and ``u = clamp(up, -limit, limit)``
+                shift: float = 0.0, cubic: float = 0.0) -> torch.Tensor:
+    """``g * sigmoid(alpha * g + cubic * g^3) * (u + shift)`` with ``g = min(gate, limit)`` and ``u = clamp(up, -limit, limit)``
     (``limit`` 0: unclamped) for ``gate_up`` [N, 2 * I] laid out as for `swiglu`."""
     _need(gate_up, None, "gate_up")
     n, two_i = gate_up.shape
@@ -455,7 +464,7 @@ def glu_limited(gate_up: torch.Tensor, block: int | None = None, alpha: float = 
         raise KernelError(f"block {block} does not divide the {inter} features")
     out = torch.empty((n, inter), dtype=gate_up.dtype, device=gate_up.device)
     _check(ops_library().ss_glu_limited(gate_up.data_ptr(), out.data_ptr(), n, inter, block, float(alpha), float(limit),
-                                        float(shift), _code(gate_up.dtype), _stream()), "glu_limited")
+                                        float(shift), float(cubic), _code(gate_up.dtype), _stream()), "glu_limited")
     return out
 
 
@@ -569,12 +578,47 @@ def _gate_ptr(gate: torch.Tensor | None, q: torch.Tensor, q_stride: int) -> int 
     return gate.data_ptr()
 
 
+@dataclasses.dataclass(frozen=True)
+class DiffPair:
+    """How the two maps of a differential head are combined (`diff_combine`): with ``o = a_1 - lam * a_2`` over the
+    first ``dim`` elements, ``o * mult / sqrt(mean(o^2) + eps)``."""
+
+    lam: float
+    mult: float
+    eps: float
+    dim: int
+
+
+def _diff_args(diff: DiffPair | None) -> tuple:
+    return (0, 0.0, 0.0, 0.0, 0) if diff is None else (1, float(diff.lam), float(diff.mult), float(diff.eps), int(diff.dim))
+
+
+def _kept(keep: int, window: int) -> int:
+    if keep < 0 or (keep and not window):
+        raise KernelError("kept first keys come with a window")
+    return int(keep)
+
+
+def _attention_out(out: torch.Tensor, gate: torch.Tensor | None, diff: DiffPair | None) -> int:
+    """Checks the output of a bfloat16 attention call; 1 when it is float32 (heads that are combined afterwards)."""
+    f32 = out.dtype == torch.float32
+    _need(out, torch.float32 if f32 else torch.bfloat16, "attention output")
+    if f32 and (gate is not None or diff is not None):
+        raise KernelError("float32 attention outputs come without a gate and without the combination of two maps")
+    return int(f32)
+
+
+def diff_in_attention(diff: DiffPair, n_q: int, n_kv: int) -> bool:
+    """Whether the prefill attention kernels can combine the two maps as they write (values in runs of 8 elements)."""
+    return (n_q // n_kv) % 2 == 0 and diff.dim % 8 == 0
+
+
 def paged_attention_simt(q: torch.Tensor, q_stride: int, out: torch.Tensor, kv: torch.Tensor,
                          block_tables: torch.Tensor, tile_req: torch.Tensor, tile_q0: torch.Tensor,
                          q_start: torch.Tensor, seq_lens: torch.Tensor, n_q: int, n_kv: int,
                          head_dim: int, scale: float, window: int = 0, chunk: int = 0,
                          gate: torch.Tensor | None = None, softcap: float = 0.0,
-                         sinks: torch.Tensor | None = None) -> None:
+                         sinks: torch.Tensor | None = None, keep: int = 0) -> None:
     """Causal grouped-query attention of the step's query rows over the pages (``window`` / ``chunk``: `key_span`).
     ``softcap`` c > 0 (in every attention entry point but the tcgen05 one): a scaled score s enters the softmax as
     ``c * tanh(s / c)``.
@@ -584,7 +628,8 @@ def paged_attention_simt(q: torch.Tensor, q_stride: int, out: torch.Tensor, kv: 
     ``q`` points at the first query head of row 0; rows are ``q_stride`` elements apart.
     ``out`` is [N, n_q * D].  ``tile_req`` / ``tile_q0`` list tiles of 16 consecutive query tokens
     of one request (request index, first token within the request's rows of this step).
-    ``sinks`` (in this entry point and the two mma.sync ones; float32 [n_q]): the softmax's denominator of head h also
+    ``keep`` (in every attention entry point; with ``window``): the request's first ``keep`` keys stay visible.
+    ``sinks`` (in every attention entry point; float32 [n_q]): the softmax's denominator of head h also
     holds ``exp(sinks[h])``, a term of its own with neither key nor value, which the scale does not touch."""
     _need(out, q.dtype, "attention output")
     _check_sinks(sinks, n_q)
@@ -598,7 +643,7 @@ def paged_attention_simt(q: torch.Tensor, q_stride: int, out: torch.Tensor, kv: 
                             tile_q0.data_ptr(), tile_req.numel(), q_start.data_ptr(), seq_lens.data_ptr(),
                             n_q, n_kv, kv.shape[3], kv.shape[0], float(scale), key_span(window, chunk),
                             _code(q.dtype), _gate_ptr(gate, q, q_stride), error_word(q.device).data_ptr(), _stream(),
-                            float(softcap or 0.0), _ptr(sinks)),
+                            float(softcap or 0.0), _ptr(sinks), _kept(keep, window)),
            "paged_attention_simt")
 
 
@@ -606,11 +651,14 @@ def paged_attention_prefill(q: torch.Tensor, q_stride: int, out: torch.Tensor, k
                             block_tables: torch.Tensor, tile_req: torch.Tensor, tile_row0: torch.Tensor,
                             q_start: torch.Tensor, seq_lens: torch.Tensor, n_q: int, n_kv: int, head_dim: int,
                             scale: float, window: int = 0, chunk: int = 0, gate: torch.Tensor | None = None,
-                            softcap: float = 0.0, sinks: torch.Tensor | None = None) -> None:
+                            softcap: float = 0.0, sinks: torch.Tensor | None = None, keep: int = 0,
+                            diff: DiffPair | None = None) -> None:
     """bfloat16 tensor-core attention for prompt portions and mixed batches.  A tile is 64 consecutive
     rows of one request, a row being a (query token, head of the kv group) pair in token-major order:
-    ``tile_req`` / ``tile_row0`` list (request index, first row)."""
-    _need(out, torch.bfloat16, "attention output")
+    ``tile_req`` / ``tile_row0`` list (request index, first row).  ``out`` bfloat16, or float32 without ``gate`` and
+    ``diff``.  ``diff`` (here and in the tcgen05 entry point, where `diff_in_attention`): ``out`` is
+    [N, n_q / 2 * diff.dim] and holds the combined heads of `diff_combine`."""
+    out_f32 = _attention_out(out, gate, diff)
     _need(kv, torch.bfloat16, "kv pages")
     _check_sinks(sinks, n_q)
     if q.dtype != torch.bfloat16:
@@ -624,7 +672,7 @@ def paged_attention_prefill(q: torch.Tensor, q_stride: int, out: torch.Tensor, k
                                    tile_row0.data_ptr(), tile_req.numel(), q_start.data_ptr(), seq_lens.data_ptr(),
                                    n_q, n_kv, kv.shape[3], kv.shape[0], float(scale), key_span(window, chunk),
                                    _gate_ptr(gate, q, q_stride), error_word(q.device).data_ptr(), _stream(),
-                                   float(softcap or 0.0), _ptr(sinks)),
+                                   float(softcap or 0.0), _ptr(sinks), _kept(keep, window), out_f32, *_diff_args(diff)),
            "paged_attention_prefill")
 
 
@@ -646,7 +694,8 @@ def paged_attention_prefill_tcgen05(q: torch.Tensor, q_stride: int, out: torch.T
                                     block_tables: torch.Tensor, tile_req: torch.Tensor, tile_tok0: torch.Tensor,
                                     q_start: torch.Tensor, seq_lens: torch.Tensor, n_q: int, n_kv: int,
                                     head_dim: int, scale: float, key_parts: int = 1, chunk: int = 0, window: int = 0,
-                                    softcap: float = 0.0, sinks: torch.Tensor | None = None) -> None:
+                                    softcap: float = 0.0, sinks: torch.Tensor | None = None, keep: int = 0,
+                                    diff: DiffPair | None = None) -> None:
     """bfloat16 causal attention for prompt portions and mixed batches on the tcgen05 tensor cores (Q, K, V
     tiles by TMA, S and O in tensor memory).  A tile is ``128 // (n_q // n_kv)`` consecutive query tokens of
     one request: ``tile_req`` / ``tile_tok0`` list (request index, first token within the request's rows); blocks
@@ -656,7 +705,7 @@ def paged_attention_prefill_tcgen05(q: torch.Tensor, q_stride: int, out: torch.T
     only the earlier keys of its own chunk of C positions; the key tiles in front of a query tile's first chunk are
     never fetched.  ``sinks`` (float32 [n_q]): one more term ``exp(sinks[h])`` in the denominator of head h, added where
     a row's sum is complete (by the block that writes the row, or once where a cluster combines its parts)."""
-    _need(out, torch.bfloat16, "attention output")
+    out_f32 = _attention_out(out, None, diff)
     _check_sinks(sinks, n_q)
     _need(kv, torch.bfloat16, "kv pages")
     if q.dtype != torch.bfloat16:
@@ -672,7 +721,7 @@ def paged_attention_prefill_tcgen05(q: torch.Tensor, q_stride: int, out: torch.T
                                    tile_tok0.data_ptr(), tile_req.numel(), q_start.data_ptr(), seq_lens.data_ptr(),
                                    n_q, n_kv, kv.shape[3], kv.shape[0], float(scale), int(key_parts),
                                    key_span(window, chunk), error_word(q.device).data_ptr(), _stream(),
-                                   float(softcap or 0.0), _ptr(sinks)),
+                                   float(softcap or 0.0), _ptr(sinks), _kept(keep, window), out_f32, *_diff_args(diff)),
            "paged_attention_prefill_tcgen05")
 
 
@@ -727,7 +776,7 @@ def paged_attention_decode(q: torch.Tensor, q_stride: int, out: torch.Tensor, kv
                            n_slices: int = 1, scratch: tuple[torch.Tensor, torch.Tensor] | None = None,
                            rope: tuple[torch.Tensor | None, int] | None = None, tma: bool | None = None,
                            stages: int = 2, chunk: int = 0, gate: torch.Tensor | None = None,
-                           softcap: float = 0.0, sinks: torch.Tensor | None = None) -> None:
+                           softcap: float = 0.0, sinks: torch.Tensor | None = None, keep: int = 0) -> None:
     """bfloat16 attention for requests that bring ONE token each, the keys of every request cut into
     ``n_slices`` slices that run in parallel.  Up to 8 slices form a thread-block cluster and are combined
     through shared memory; with more, the partial results (of every cluster of 8 in the TMA-fed kernel when the
@@ -742,13 +791,13 @@ def paged_attention_decode(q: torch.Tensor, q_stride: int, out: torch.Tensor, kv
     ``tma``: the kernel whose tiles are moved by TMA (head size 64 or 128, pages of 8, 16, 32 or 64 tokens;
     the default where it fits), or the one that moves them with cp.async (every head and page size).
     ``stages``: 2 or 3 tiles in the ring of the TMA-fed kernel."""
-    fits = tcgen05_attention_fits(head_dim, n_q, n_kv, kv.shape[3], 0) and sinks is None
+    fits = tcgen05_attention_fits(head_dim, n_q, n_kv, kv.shape[3], 0)
     _check_sinks(sinks, n_q)
     if tma is None:
         tma = fits
     elif tma and not fits:
         raise KernelError("the TMA decode kernel takes head size 64 or 128 and pages of 8, 16, 32 or 64 tokens")
-    _need(out, torch.bfloat16, "attention output")
+    out_f32 = _attention_out(out, gate, None)
     _need(kv, torch.bfloat16, "kv pages")
     if q.dtype != torch.bfloat16:
         raise KernelError("the tensor-core attention kernels take bfloat16")
@@ -783,9 +832,10 @@ def paged_attention_decode(q: torch.Tensor, q_stride: int, out: torch.Tensor, kv
         raise KernelError("a gated layer does not rotate inside the decode kernel")
     tail = (_gate_ptr(gate, q, q_stride), error_word(q.device).data_ptr(), _stream(), float(softcap or 0.0))
     if tma:
-        _check(lib.ss_attn_decode_tma(*args, int(stages), *tail), "paged_attention_decode")
+        _check(lib.ss_attn_decode_tma(*args, int(stages), *tail, _ptr(sinks), _kept(keep, window), out_f32),
+               "paged_attention_decode")
     else:
-        _check(lib.ss_attn_decode_mma(*args, *tail, _ptr(sinks)), "paged_attention_decode")
+        _check(lib.ss_attn_decode_mma(*args, *tail, _ptr(sinks), _kept(keep, window), out_f32), "paged_attention_decode")
 
 
 WIDE_CONTEXT = 8192  # from this many cached tokens a decode step of few requests may use more than 8 slices
@@ -840,7 +890,8 @@ def fuses_rope(qkv: torch.Tensor, ctx, head_dim: int, n_q: int, n_kv: int, page_
 def paged_attention(qkv: torch.Tensor, out: torch.Tensor, kv: torch.Tensor, block_tables: torch.Tensor,
                     ctx, n_q: int, n_kv: int, head_dim: int, scale: float, window: int = 0,
                     rope: tuple[torch.Tensor | None, int] | None = None, chunk: int = 0,
-                    gate: torch.Tensor | None = None, softcap: float = 0.0, sinks: torch.Tensor | None = None) -> None:
+                    gate: torch.Tensor | None = None, softcap: float = 0.0, sinks: torch.Tensor | None = None,
+                    keep: int = 0, diff: DiffPair | None = None) -> None:
     """Attention of the step's rows over the pages, choosing the kernel for the batch.
 
     ``qkv`` is the stacked projection output [N, (n_q + 2 n_kv) * D] whose first n_q heads are the
@@ -855,43 +906,162 @@ def paged_attention(qkv: torch.Tensor, out: torch.Tensor, kv: torch.Tensor, bloc
     ``gate``: a view of ``qkv`` [N, n_q * D]; the output is multiplied by its sigmoid, inside the attention kernel
     except behind the tcgen05 prefill kernel, where `sigmoid_gate` follows.
 
-    ``sinks`` (float32 [n_q]): one more term ``exp(sinks[h])`` in the softmax's denominator of head h; decode steps of
-    such layers run the cp.async kernel."""
+    ``sinks`` (float32 [n_q]): one more term ``exp(sinks[h])`` in the softmax's denominator of head h.  ``keep`` (with
+    ``window``): the request's first ``keep`` keys stay visible.
+
+    ``diff``: query heads 2h and 2h + 1 are the two maps of a differential head and ``out`` [N, n_q / 2 * diff.dim] takes
+    the combined heads.  The prefill kernels combine them as they write; where they cannot (decode steps, keys cut into
+    parts, float32), the heads are written in float32 and `diff_combine` follows, so the difference is formed from
+    unrounded outputs either way."""
+    if diff is not None and gate is not None:
+        raise KernelError("a gate on differential heads is not built")
     if rope is not None and not (qkv.dtype == torch.bfloat16 and ctx.is_decode_only):
         raise KernelError("only bfloat16 decode steps rotate inside the attention kernel")
     if qkv.dtype == torch.float32:
         tile_req, tile_q0 = ctx.query_tiles(16)
-        paged_attention_simt(qkv, qkv.shape[1], out, kv, block_tables, tile_req, tile_q0, ctx.q_start,
-                             ctx.seq_lens, n_q, n_kv, head_dim, scale, window, chunk, gate, softcap, sinks)
+        heads = out if diff is None else _heads_f32(out, n_q, head_dim)
+        paged_attention_simt(qkv, qkv.shape[1], heads, kv, block_tables, tile_req, tile_q0, ctx.q_start,
+                             ctx.seq_lens, n_q, n_kv, head_dim, scale, window, chunk, gate, softcap, sinks, keep)
+        if diff is not None:
+            diff_combine(heads, diff, n_q // 2, out)
         return
     group = n_q // n_kv
     if ctx.is_decode_only:
         static = ctx.extras.get("static_max_seq_len")  # fixed when the step is captured
         longest = static or ctx.max_seq_len
         wide = ctx.extras.get("decode_wide", False) if static else is_long_context(ctx.max_seq_len)
-        wide = bool(wide) and tcgen05_attention_fits(head_dim, n_q, n_kv, kv.shape[3], 0) and sinks is None
-        slices = decode_slices(ctx.num_requests, n_kv, group, min(longest, window or chunk or longest), wide,
+        wide = bool(wide) and tcgen05_attention_fits(head_dim, n_q, n_kv, kv.shape[3], 0)
+        slices = decode_slices(ctx.num_requests, n_kv, group, min(longest, (window or chunk or longest) + keep), wide,
                                sm_count(qkv.device))
         scratch = ctx.extras.get(("decode_scratch", n_q, head_dim))
-        paged_attention_decode(qkv, qkv.shape[1], out, kv, block_tables, ctx.q_start, ctx.seq_lens,
+        heads = out if diff is None else _heads_f32(out, n_q, head_dim)
+        paged_attention_decode(qkv, qkv.shape[1], heads, kv, block_tables, ctx.q_start, ctx.seq_lens,
                                ctx.num_requests, n_q, n_kv, head_dim, scale, window, slices, scratch, rope,
-                               stages=DECODE_RING_STAGES, chunk=chunk, gate=gate, softcap=softcap, sinks=sinks)
+                               stages=DECODE_RING_STAGES, chunk=chunk, gate=gate, softcap=softcap, sinks=sinks, keep=keep)
+        if diff is not None:
+            diff_combine(heads, diff, n_q // 2, out)
         return
+    fused = diff is None or diff_in_attention(diff, n_q, n_kv)
     if tcgen05_prefill_fits(head_dim, n_q, n_kv, kv.shape[3]):
         tile_req, tile_tok0 = ctx.query_tiles_longest_first(128 // group)
-        key = ("prefill_key_parts", 128 // group, n_kv, window or chunk)
+        key = ("prefill_key_parts", 128 // group, n_kv, (window or chunk) + keep)
         parts = ctx.extras.get(key)
         if parts is None:  # the same for every layer of the step that sees as far
             parts = ctx.extras[key] = prefill_key_parts(ctx.q_lens_host, ctx.seq_lens_host, 128 // group, n_kv,
-                                                        sm_count(qkv.device), window or chunk)
-        paged_attention_prefill_tcgen05(qkv, qkv.shape[1], out, kv, block_tables, tile_req, tile_tok0, ctx.q_start,
-                                        ctx.seq_lens, n_q, n_kv, head_dim, scale, parts, chunk, window, softcap, sinks)
+                                                        sm_count(qkv.device), (window or chunk) + keep)
+        fused = fused and (diff is None or parts == 1)
+        heads = out if fused else _heads_f32(out, n_q, head_dim)
+        paged_attention_prefill_tcgen05(qkv, qkv.shape[1], heads, kv, block_tables, tile_req, tile_tok0, ctx.q_start,
+                                        ctx.seq_lens, n_q, n_kv, head_dim, scale, parts, chunk, window, softcap, sinks, keep,
+                                        diff if fused else None)
+        if not fused:
+            diff_combine(heads, diff, n_q // 2, out)
         if gate is not None:
             sigmoid_gate(out, gate)
         return
     tile_req, tile_row0 = ctx.query_tiles(64, group)
-    paged_attention_prefill(qkv, qkv.shape[1], out, kv, block_tables, tile_req, tile_row0, ctx.q_start,
-                            ctx.seq_lens, n_q, n_kv, head_dim, scale, window, chunk, gate, softcap, sinks)
+    heads = out if fused else _heads_f32(out, n_q, head_dim)
+    paged_attention_prefill(qkv, qkv.shape[1], heads, kv, block_tables, tile_req, tile_row0, ctx.q_start,
+                            ctx.seq_lens, n_q, n_kv, head_dim, scale, window, chunk, gate, softcap, sinks, keep,
+                            diff if fused else None)
+    if not fused:
+        diff_combine(heads, diff, n_q // 2, out)
+
+
+def _heads_f32(out: torch.Tensor, n_q: int, head_dim: int) -> torch.Tensor:
+    return torch.empty((out.shape[0], n_q * head_dim), dtype=torch.float32, device=out.device)
+
+
+def diff_combine(heads: torch.Tensor, diff: DiffPair, n_heads: int, out: torch.Tensor) -> None:
+    """``heads`` (float32 [N, 2 * n_heads * D], maps 2h and 2h + 1 of head h) into ``out`` [N, n_heads * diff.dim]:
+    with ``o = map_1 - lam * map_2`` over the first ``dim`` elements, ``o * mult / sqrt(mean(o^2) + eps)`` in float32."""
+    _need(heads, torch.float32, "heads")
+    _need(out, None, "combined heads")
+    n = heads.shape[0]
+    d = heads.shape[1] // (2 * n_heads)
+    if heads.shape[1] != 2 * n_heads * d or tuple(out.shape) != (n, n_heads * diff.dim) or diff.dim > d:
+        raise KernelError("diff_combine: sizes do not match")
+    _check(ops_library().ss_diff_combine(heads.data_ptr(), out.data_ptr(), n, n_heads, d, diff.dim, float(diff.lam),
+                                         float(diff.mult), float(diff.eps), _code(out.dtype), _stream()), "diff_combine")
+
+
+def heads_to_pages(rows: torch.Tensor, positions: torch.Tensor, slots: torch.Tensor | None, kv: torch.Tensor | None,
+                   n_q: int, n_kv: int, dim: int, value_dim: int, head_dim: int, k_col: int, v_col: int, *, maps: int = 1,
+                   inv_freq: torch.Tensor | None = None, rotary_dim: int = 0, interleaved: bool = True,
+                   q_weight: torch.Tensor | None = None, k_weight: torch.Tensor | None = None, eps: float = 0.0) -> torch.Tensor:
+    """Projected heads into what the attention kernels read.  A row of ``rows`` holds ``n_q * maps`` query parts of
+    ``dim`` elements at column 0, ``n_kv * maps`` key parts at ``k_col`` and ``n_kv`` values of ``value_dim`` elements at
+    ``v_col`` (``v_col`` = ``k_col``: the values are the keys as projected).  ``q_weight`` / ``k_weight`` (float32, the size
+    of all queries or keys of a token): an RMS norm over all of them at once, before the rotation of the first
+    ``rotary_dim`` elements of every part.  Keys and values go to their pages ``kv`` [pages, 2, n_kv, page_size,
+    head_dim] at ``slots``, the maps of a key head side by side, zeros behind; the queries come back as
+    [N, n_q * maps * head_dim], map m of a head at ``m * dim`` of its elements and zeros elsewhere, so that its score with
+    such a key row is that of map m alone."""
+    if rows.dim() != 2 or rows.stride(1) != 1 or not rows.is_cuda:
+        raise KernelError("heads_to_pages takes CUDA rows with unit inner stride")
+    _need(positions, torch.int32, "positions")
+    n, part = rows.shape[0], maps * dim
+    values = part if v_col == k_col else value_dim
+    if head_dim < max(part, value_dim) or head_dim % 8 or max(n_q * part, k_col + n_kv * part, v_col + n_kv * value_dim) > rows.shape[1]:
+        raise KernelError("heads_to_pages: the rows are narrower than their heads, or head_dim is too small")
+    if v_col == k_col and value_dim != values:
+        raise KernelError("values that are the keys have the keys' size")
+    if rotary_dim:
+        _need(inv_freq, torch.float32, "inv_freq")
+        if inv_freq.numel() != rotary_dim // 2 or rotary_dim > dim:
+            raise KernelError("inv_freq must hold rotary_dim / 2 values, rotary_dim at most dim")
+    if (q_weight is None) != (k_weight is None):
+        raise KernelError("queries and keys are normed alike")
+    if q_weight is not None:
+        _need(q_weight, torch.float32, "q norm weight")
+        _need(k_weight, torch.float32, "k norm weight")
+        if q_weight.numel() != n_q * part or k_weight.numel() != n_kv * part:
+            raise KernelError("the norm's weights cover all queries and all keys of a token")
+    write = kv is not None and slots is not None
+    pages, page_size = 0, 1
+    if write:
+        _need(kv, rows.dtype, "kv pages")
+        _need(slots, torch.int32, "slots")
+        if kv.dim() != 5 or kv.shape[1] != 2 or kv.shape[2] != n_kv or kv.shape[4] != head_dim:
+            raise KernelError(f"kv pages have shape {tuple(kv.shape)}, expected [pages, 2, {n_kv}, page, {head_dim}]")
+        pages, page_size = kv.shape[0], kv.shape[3]
+    q = torch.empty((n, n_q * maps * head_dim), dtype=rows.dtype, device=rows.device)
+    _check(ops_library().ss_heads_to_pages(rows.data_ptr(), rows.stride(0), positions.data_ptr(), _ptr(slots) if write else None,
+                                           _ptr(inv_freq) if rotary_dim else None, _ptr(q_weight), _ptr(k_weight), q.data_ptr(),
+                                           _ptr(kv) if write else None, n, n_q, n_kv, maps, dim, value_dim, head_dim, k_col,
+                                           v_col, rotary_dim, int(interleaved), float(eps), page_size, pages,
+                                           _code(rows.dtype), error_word(rows.device).data_ptr(), _stream()), "heads_to_pages")
+    return q
+
+
+def branch_norm(residual: torch.Tensor, y: torch.Tensor | None, y_weight: torch.Tensor | None, y_eps: float, mult: float,
+                weight: torch.Tensor, eps: float, out_dtype: torch.dtype, *, anchor: torch.Tensor | None = None,
+                rows: torch.Tensor | None = None) -> torch.Tensor:
+    """``residual`` (float32 [N, H]) += ``mult * rmsnorm(y) * y_weight`` (+ ``anchor``, float32 [N, H]) in place, then
+    the RMS norm of the new stream times ``weight`` in ``out_dtype``.  Weights are float32, the arithmetic too, and the
+    result is rounded once.  With ``rows`` (int32 [M]) only those rows are produced and the stream stays as it is."""
+    _need(residual, torch.float32, "residual")
+    hidden = residual.shape[-1]
+    _need(weight, torch.float32, "norm weight")
+    if weight.numel() != hidden:
+        raise KernelError("norm weight has the wrong size")
+    if y is not None:
+        _need(y, out_dtype, "branch output")
+        _need(y_weight, torch.float32, "branch norm weight")
+        if y.shape != residual.shape or y_weight.numel() != hidden:
+            raise KernelError("branch output or its norm's weight does not match the stream")
+    if anchor is not None:
+        _need(anchor, torch.float32, "anchor")
+        if y is None or anchor.shape != residual.shape:
+            raise KernelError("an anchor comes with a branch output and has the stream's shape")
+    if rows is not None:
+        _need(rows, torch.int32, "rows")
+    n_out = residual.shape[0] if rows is None else rows.numel()
+    out = torch.empty((n_out, hidden), dtype=out_dtype, device=residual.device)
+    _check(ops_library().ss_branch_norm(residual.data_ptr(), _ptr(y), _ptr(y_weight) if y is not None else None, float(y_eps),
+                                        float(mult), _ptr(anchor), weight.data_ptr(), float(eps), out.data_ptr(), _ptr(rows),
+                                        n_out, hidden, _code(out_dtype), _stream()), "branch_norm")
+    return out
 
 
 # --------------------------------------------------------------------------- sampling
@@ -1042,14 +1212,14 @@ def _gemm_plan(tokens: int, features: int, k: int, sms: int) -> tuple[bool, int,
 def gemm_tcgen05(x: "torch.Tensor | PendingNorm", weight: torch.Tensor, bias: torch.Tensor | None = None,
                  out_dtype: torch.dtype | None = None, plan: tuple[bool, int, int] | None = None,
                  swiglu: bool = False, to_stream: tuple[torch.Tensor, torch.Tensor] | None = None,
-                 glu: tuple[float, float, float] | None = None, hc: "np.ndarray | None" = None):
+                 glu: tuple[float, float, float, float] | None = None, hc: "np.ndarray | None" = None):
     """``x @ weight.T + bias`` for bfloat16 ``x`` [tokens, K] and ``weight`` [features, K] on the tcgen05 tensor
     cores (TMA-fed, accumulator in tensor memory); output bfloat16 or float32.  K must be a multiple of 8.
 
     ``swiglu`` (at most 64 tokens, features a multiple of 128): the weight's rows alternate 64 gate and 64 up
     features; the result is ``silu(gate) * up`` with features / 2 columns, formed in the product's epilogue.
 
-    ``glu`` = (alpha, limit, shift) with ``swiglu``: the fused unit is `glu_limited`'s instead of SwiGLU.
+    ``glu`` = (alpha, limit, shift, cubic) with ``swiglu``: the fused unit is `glu_limited`'s instead of SwiGLU.
     ``hc`` with ``to_stream``: the stream is [tokens, S, features], S hyper-connected streams (at most 4), and ``hc`` a
     float32 host array of S * S + 2 S values, mix [from, to], out, in: the product is written into the streams as
     `hc_norm` writes a branch output, and what comes back describes ``sum_t in[t] * stream t``.
@@ -1136,7 +1306,7 @@ def gemm_tcgen05(x: "torch.Tensor | PendingNorm", weight: torch.Tensor, bias: to
                                                        pending.squares.shape[1], float(pending.eps), _ptr(bias), bias_f32,
                                                        out.data_ptr(), a.shape[0], tokens, k, k, k, out.shape[1], bn,
                                                        int(out_dtype == torch.float32), slices, float(glu[0]),
-                                                       float(glu[1]), float(glu[2]), _ptr(partial), _ptr(counters),
+                                                       float(glu[1]), float(glu[2]), float(glu[3]), _ptr(partial), _ptr(counters),
                                                        error_word(x.device).data_ptr(), _stream())
             _check(rc, "gemm_tcgen05 with a gated unit behind a pending norm")
             return out
@@ -1153,7 +1323,7 @@ def gemm_tcgen05(x: "torch.Tensor | PendingNorm", weight: torch.Tensor, bias: to
         rc = gemm_library().ss_gemm_tc5_glu(a.data_ptr(), b.data_ptr(), _ptr(bias), bias_f32, out.data_ptr(), a.shape[0],
                                             b.shape[0], k, k, k, out.shape[1], bn, int(swapped),
                                             int(out_dtype == torch.float32), slices, float(glu[0]), float(glu[1]),
-                                            float(glu[2]), _ptr(partial), _ptr(counters),
+                                            float(glu[2]), float(glu[3]), _ptr(partial), _ptr(counters),
                                             error_word(x.device).data_ptr(), _stream())
         _check(rc, "gemm_tcgen05 with a gated unit")
         return out
@@ -1168,7 +1338,7 @@ def gemm_tcgen05(x: "torch.Tensor | PendingNorm", weight: torch.Tensor, bias: to
 def gemm_tcgen05_many(x: "torch.Tensor | PendingNorm", weight: torch.Tensor, bias: torch.Tensor | None = None,
                       out_dtype: torch.dtype | None = None, swiglu: bool = False, tile_cols: int = 0,
                       to_stream: tuple[torch.Tensor, torch.Tensor] | None = None,
-                      glu: tuple[float, float, float] | None = None):
+                      glu: tuple[float, float, float, float] | None = None):
     """``x @ weight.T + bias`` for many rows of ``x`` (prompt portions) on the tcgen05 tensor cores: a persistent
     kernel, one block per SM, the blocks in pairs (``tcgen05.mma.cta_group::2``: each block of a pair loads half
     of A and half of B) that compute tiles of 256 rows with the accumulator double-buffered in tensor memory, so
@@ -1234,7 +1404,7 @@ def gemm_tcgen05_many(x: "torch.Tensor | PendingNorm", weight: torch.Tensor, bia
             raise KernelError("the constants of a gated unit come with the fused gate/up epilogue")
         rc = gemm_library().ss_gemm_tc5_many_glu(x.data_ptr(), weight.data_ptr(), _ptr(bias), bias_f32, out.data_ptr(),
                                                  tokens, features, k, k, k, out.shape[1], float(glu[0]), float(glu[1]),
-                                                 float(glu[2]), error_word(x.device).data_ptr(), _stream())
+                                                 float(glu[2]), float(glu[3]), error_word(x.device).data_ptr(), _stream())
         _check(rc, "gemm_tcgen05_many with a gated unit")
         return out
     rc = gemm_library().ss_gemm_tc5_many(x.data_ptr(), weight.data_ptr(), _ptr(bias), bias_f32, out.data_ptr(), tokens,
@@ -1407,23 +1577,23 @@ def gate_up_swiglu(x: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor | N
 
 
 def gate_up_glu(x: "torch.Tensor | PendingNorm", weight: torch.Tensor, bias: torch.Tensor | None, block: int,
-                alpha: float, limit: float, shift: float) -> torch.Tensor:
+                alpha: float, limit: float, shift: float, cubic: float = 0.0) -> torch.Tensor:
     """`gate_up_swiglu` with the gated unit of `glu_limited` (a steeper sigmoid, clamped inputs, a shifted up
-    branch).  Where `gate_up_swiglu` forms SwiGLU in the product's epilogue (small bfloat16 batches, long prompt
+    branch, a cubic term inside the sigmoid).  Where `gate_up_swiglu` forms SwiGLU in the product's epilogue (small bfloat16 batches, long prompt
     portions; runs of 64) this does the same with the unit's constants; everything else is the stacked product
     followed by the activation kernel."""
     if isinstance(x, PendingNorm):
         if (block == 64 and weight.shape[0] % 128 == 0 and x.shape[0] <= CLUSTER_BATCH
                 and takes_pending_norm(x, weight.shape[0], swiglu=True)):
-            return gemm_tcgen05(x, weight, bias, swiglu=True, glu=(alpha, limit, shift))
+            return gemm_tcgen05(x, weight, bias, swiglu=True, glu=(alpha, limit, shift, cubic))
         x = x.materialize()
     if x.dtype == torch.bfloat16 and block == 64 and weight.shape[0] % 128 == 0 and x.shape[1] % 8 == 0:
         sms = sm_count(x.device)
         if streams_weights(x.shape[0], weight.shape[0], x.shape[1], sms):
-            return gemm_tcgen05(x, weight, bias, swiglu=True, glu=(alpha, limit, shift))
+            return gemm_tcgen05(x, weight, bias, swiglu=True, glu=(alpha, limit, shift, cubic))
         if many_tokens_swiglu_fits(x.shape[0], weight.shape[0], sms):
-            return gemm_tcgen05_many(x, weight, bias, swiglu=True, glu=(alpha, limit, shift))
-    return glu_limited(linear(x, weight, bias), block, alpha, limit, shift)
+            return gemm_tcgen05_many(x, weight, bias, swiglu=True, glu=(alpha, limit, shift, cubic))
+    return glu_limited(linear(x, weight, bias), block, alpha, limit, shift, cubic)
 
 
 # --------------------------------------------------------------------------- grouped norm, state-space mixer, routed experts
@@ -2185,5 +2355,6 @@ __all__ = ["KernelError", "KernelBuildError", "embedding", "add_rmsnorm", "hc_no
            "gemm_simt", "paged_attention_simt", "paged_attention", "fuses_rope", "paged_attention_prefill", "paged_attention_prefill_tcgen05", "prefill_key_parts", "tcgen05_attention_fits", "tcgen05_prefill_fits", "paged_attention_decode", "decode_scratch", "decode_slices", "is_long_context", "require_cuda", "argmax", "sample", "mark_seen", "gather_tokens", "prepare_decode", "gemm_tcgen05", "gemm_tcgen05_many", "many_tokens_fits", "many_tokens_swiglu_fits", "gemm_plan", "gemm_library", "gate_up_swiglu", "set_programmatic_launch", "launch_count", "count_launches", "sm_count", "linear", "linear_add_rmsnorm", "adds_to_stream", "takes_pending_norm", "PendingNorm", "set_norm_fusion", "check_errors", "raise_for_status", "error_word", "ops_library",
            "attention_library", "group_norm", "round_stream", "conv_silu", "ssm_scan", "router", "moe_experts", "moe_combine",
            "norm_rope_cache", "turn_heads", "soft_cap", "embed_sum", "matrix_cell", "cell_output", "gated_recurrence", "xielu",
+           "DiffPair", "diff_in_attention", "diff_combine", "heads_to_pages", "branch_norm",
            "latent_rows", "head_product", "decay_attention", "gated_rmsnorm", "block_gates", "gated_linear_recurrence", "head_gate",
            "scaled_sum", "relu_square", "moe_experts_single", "moe_mix"]

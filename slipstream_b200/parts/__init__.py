@@ -4,16 +4,17 @@ from .base import (BLOCKS, EMBEDDINGS, FEED_FORWARDS, HEADS, MIXERS, NORMS, POSI
                    Embedding, FeedForward, Head, IntoNorm, LayerBinding, Mixer, Norm, Part, PositionEncoding, Registry, Runtime,
                    StateSpec, WeightSpec)
 from .attention import PagedAttention
-from .block import BranchNormBlock, ParallelBlock, PreNormBlock
+from .block import BranchNormBlock, ParallelBlock, PreNormBlock, SandwichBlock
+from .differential import DifferentialAttention
 from .embedding import LMHead, SummedEmbedding, TokenEmbedding
-from .mlp import ActivatedFeedForward, GatedFeedForward, SwiGLUFeedForward
+from .mlp import GELU_TANH, ActivatedFeedForward, GatedFeedForward, SwiGLUFeedForward
 from .experts import RoutedExperts
-from .norm import GroupRMSNorm, RMSNorm, StreamRounding
+from .norm import GroupRMSNorm, JoiningNorm, NormedBranch, RMSNorm, StreamRounding
 from .state_space import StateSpaceMixer
 from .recurrent import (ConvolvedInput, DecayedLinearAttention, GatedLinearRecurrenceMixer, GatedRecurrenceMixer,
                         MatrixMemoryMixer, ParallelMixers)
 from .latent_attention import LatentAttention
-from .rotary import NoPositionEncoding, RotaryEncoding, YarnRotaryEncoding
+from .rotary import BandedRotaryEncoding, NoPositionEncoding, RotaryEncoding, YarnRotaryEncoding
 from .streams import ConnectedNorm, HyperConnectionBlock, StreamWrite
 
 __all__ = ["BLOCKS", "EMBEDDINGS", "HEADS", "Embedding", "Head", "FEED_FORWARDS", "MIXERS", "NORMS", "POSITION_ENCODINGS", "Block", "CacheSpec",
@@ -23,4 +24,5 @@ __all__ = ["BLOCKS", "EMBEDDINGS", "HEADS", "Embedding", "Head", "FEED_FORWARDS"
            "HyperConnectionBlock", "StreamWrite", "BranchNormBlock", "GroupRMSNorm", "StreamRounding", "RoutedExperts",
            "StateSpaceMixer", "SummedEmbedding", "ActivatedFeedForward", "ConvolvedInput", "GatedRecurrenceMixer",
            "MatrixMemoryMixer", "LatentAttention", "ParallelBlock", "DecayedLinearAttention", "GatedLinearRecurrenceMixer",
-           "ParallelMixers"]
+           "ParallelMixers", "SandwichBlock", "DifferentialAttention", "GELU_TANH", "JoiningNorm", "NormedBranch",
+           "BandedRotaryEncoding"]

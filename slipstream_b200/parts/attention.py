@@ -22,8 +22,13 @@ frequencies ``theta^(-2m / value_dim)``, and cached so; a head's output at posit
 values) is turned back by -i before any gate, so that what is summed depends on i - j only.  ``softcap`` c: a scaled
 score s enters the softmax as ``c tanh(s / c)``.  ``head_gate``: head h's output is multiplied by
 ``sigmoid(w_g,h . x)``, one number per head and token (``W_g`` [heads, hidden] rides in the stacked product).
-``unit_sink``: the softmax's denominator holds one more 1 (a key whose score is 0 and which has no value).  ``names``: the checkpoint's tensor names by role (q, k, v, o, g,
-q_bias, k_bias, v_bias, o_bias, q_norm, k_norm).
+``unit_sink``: the softmax's denominator holds one more 1 (a key whose score is 0 and which has no value).
+``learned_sinks``: it holds ``exp(s_h)``, a learned number per head (tensor ``sink``) with neither key nor value, which
+the scale does not touch.  ``keep_first`` K (with ``window``): a query also sees the request's first K keys, at their true
+positions.  ``joint_norm_eps``: before the rotation ONE RMS norm over all query heads of a token together, and one over
+all its key heads, with weights of the whole projections' sizes (tensors ``q_norm`` / ``k_norm``).  ``tied_values``: the
+values are the keys as projected, before norm and rotation; there is no v.  ``names``: the checkpoint's tensor names by
+role (q, k, v, o, g, q_bias, k_bias, v_bias, o_bias, q_norm, k_norm, sink).
 
 Heads of a size the kernels do not take (they take multiples of 16), or values of another size than keys, are
 padded with zeros where the weights are bound: q/k/v/g rows and o columns of the padding are zero, so the
@@ -51,7 +56,8 @@ class PagedAttention(Mixer):
                  chunk: int | None = None, value_dim: int | None = None, unit_norm_eps: float | None = None,
                  gate: bool = False, has_kv: bool = True, names: dict[str, str] | None = None,
                  qk_norm_eps: float | None = None, rotate_values: bool = False, softcap: float | None = None,
-                 head_gate: bool = False, unit_sink: bool = False) -> None:
+                 head_gate: bool = False, unit_sink: bool = False, learned_sinks: bool = False, keep_first: int = 0,
+                 joint_norm_eps: float | None = None, tied_values: bool = False) -> None:
         if num_heads % num_kv_heads != 0:
             raise ValueError(f"num_heads ({num_heads}) must be divisible by num_kv_heads ({num_kv_heads})")
         value_dim = head_dim if value_dim is None else int(value_dim)
@@ -87,7 +93,18 @@ class PagedAttention(Mixer):
             raise ValueError("a gate on rotated values is not built")
         if gate and head_gate:
             raise ValueError("a layer gates its heads element by element or head by head, not both")
-        self.head_gate, self.unit_sink = bool(head_gate), bool(unit_sink)
+        if keep_first < 0 or (keep_first and window is None):
+            raise ValueError("kept first keys come with a window")
+        if unit_sink and learned_sinks:
+            raise ValueError("a layer has a unit sink or learned ones, not both")
+        self.head_gate, self.unit_sink, self.learned_sinks = bool(head_gate), bool(unit_sink), bool(learned_sinks)
+        self.keep_first = int(keep_first)
+        self.joint_norm_eps = None if joint_norm_eps is None else float(joint_norm_eps)
+        self.tied_values = bool(tied_values)
+        if self.spread and (gate or head_gate or rotate_values or not has_kv or qk_norm_eps is not None or unit_norm_eps is not None):
+            raise ValueError("joint norms and tied values come without gates, other norms, rotated or borrowed values")
+        if self.tied_values and value_dim != head_dim:
+            raise ValueError("values that are the keys have the keys' size")
         if self.qk_norm_eps is not None and unit_norm_eps is not None:
             raise ValueError("a layer norms its heads before the rotation or after it, not both")
         self.has_kv = bool(has_kv)
@@ -97,8 +114,19 @@ class PagedAttention(Mixer):
         self.names = {"q": f"{n}.q_proj.weight", "k": f"{n}.k_proj.weight", "v": f"{n}.v_proj.weight",
                       "o": f"{n}.o_proj.weight", "g": f"{n}.g_proj.weight", "q_bias": f"{n}.q_proj.bias",
                       "k_bias": f"{n}.k_proj.bias", "v_bias": f"{n}.v_proj.bias", "o_bias": f"{n}.o_proj.bias",
-                      "q_norm": f"{n}.q_norm.weight", "k_norm": f"{n}.k_norm.weight"}
+                      "q_norm": f"{n}.q_norm.weight", "k_norm": f"{n}.k_norm.weight", "sink": f"{n}.sink"}
         self.names.update(names or {})
+
+    @property
+    def spread(self) -> bool:
+        """Heads go from the projection to the attention kernels' forms by `ops.heads_to_pages`: the projection is
+        stacked without padding, and queries get rows of their own."""
+        return self.joint_norm_eps is not None or self.tied_values
+
+    @property
+    def sees(self) -> int:
+        """Keys a query sees at most under the mask (0: every earlier one)."""
+        return (self.window or self.chunk or 0) + self.keep_first
 
     @property
     def plain(self) -> bool:
@@ -106,7 +134,8 @@ class PagedAttention(Mixer):
         rotation (half-split pairs, unscaled sines, no unit norm, no gate, keys and values of its own)."""
         rotary_plain = getattr(self.position_encoding, "plain", True)
         return (rotary_plain and self.unit_norm_eps is None and not self.gate and self.has_kv
-                and not self.head_gate and not self.unit_sink
+                and not self.head_gate and not self.unit_sink and not self.learned_sinks and not self.keep_first
+                and not self.spread
                 and self.qk_norm_eps is None and not self.rotate_values and self.softcap is None
                 and self.key_dim == self.value_dim == self.head_dim)
 
@@ -114,7 +143,9 @@ class PagedAttention(Mixer):
         h, d, dv, names = self.hidden_size, self.key_dim, self.value_dim, self.names
         specs = [WeightSpec(names["q"], (self.num_heads * d, h)), WeightSpec(names["o"], (h, self.num_heads * dv))]
         if self.has_kv:
-            specs += [WeightSpec(names["k"], (self.num_kv_heads * d, h)), WeightSpec(names["v"], (self.num_kv_heads * dv, h))]
+            specs.append(WeightSpec(names["k"], (self.num_kv_heads * d, h)))
+            if not self.tied_values:
+                specs.append(WeightSpec(names["v"], (self.num_kv_heads * dv, h)))
         if self.gate:
             specs.append(WeightSpec(names["g"], (self.num_heads * dv, h)))
         if self.head_gate:
@@ -122,18 +153,24 @@ class PagedAttention(Mixer):
         if self.qkv_bias:
             specs.append(WeightSpec(names["q_bias"], (self.num_heads * d,), kind="vector"))
             if self.has_kv:
-                specs += [WeightSpec(names["k_bias"], (self.num_kv_heads * d,), kind="vector"),
-                          WeightSpec(names["v_bias"], (self.num_kv_heads * dv,), kind="vector")]
+                specs.append(WeightSpec(names["k_bias"], (self.num_kv_heads * d,), kind="vector"))
+                if not self.tied_values:
+                    specs.append(WeightSpec(names["v_bias"], (self.num_kv_heads * dv,), kind="vector"))
         if self.out_bias:
             specs.append(WeightSpec(names["o_bias"], (h,), kind="vector"))
         if self.qk_norm_eps is not None:
             specs.append(WeightSpec(names["q_norm"], (d,), kind="vector", init=("one_plus_normal", 0.1)))
             if self.has_kv:
                 specs.append(WeightSpec(names["k_norm"], (d,), kind="vector", init=("one_plus_normal", 0.1)))
+        if self.joint_norm_eps is not None:
+            specs += [WeightSpec(names["q_norm"], (self.num_heads * d,), kind="vector", init=("one_plus_normal", 0.1)),
+                      WeightSpec(names["k_norm"], (self.num_kv_heads * d,), kind="vector", init=("one_plus_normal", 0.1))]
+        if self.learned_sinks:
+            specs.append(WeightSpec(names["sink"], (self.num_heads,), kind="vector", init=("normal", 1.0)))
         return specs
 
     def cache_spec(self) -> CacheSpec:
-        return CacheSpec(self.num_kv_heads, self.head_dim, self.window, self.page_size, self.chunk)
+        return CacheSpec(self.num_kv_heads, self.head_dim, self.window, self.page_size, self.chunk, self.keep_first)
 
     def _pad_heads(self, t: torch.Tensor, heads: int, size: int) -> torch.Tensor:
         """[heads * size, ...] -> [heads * head_dim, ...] with zeros behind each head's ``size`` rows."""
@@ -149,12 +186,21 @@ class PagedAttention(Mixer):
         # one stacked product: [q | k | v | g]; k and v only if the layer has them, g only with a gate
         roles = [("q", nq, self.key_dim)]
         if self.has_kv:
-            roles += [("k", nkv, self.key_dim), ("v", nkv, self.value_dim)]
+            roles.append(("k", nkv, self.key_dim))
+            if not self.tied_values:
+                roles.append(("v", nkv, self.value_dim))
         if self.gate:
             roles.append(("g", nq, self.value_dim))
-        stacked = [self._pad_heads(weights[names[r]], heads, size) for r, heads, size in roles]
+        pad = (lambda t, heads, size: t) if self.spread else self._pad_heads
+        stacked = [pad(weights[names[r]], heads, size) for r, heads, size in roles]
         self.head_gate_col = sum(t.shape[0] for t in stacked)
         extra_rows = 0
+        if self.spread:  # rows of 16-byte multiples
+            self.k_col = nq * self.key_dim
+            self.v_col = self.k_col if self.tied_values else self.k_col + nkv * self.key_dim
+            extra_rows = -self.head_gate_col % 8
+            if extra_rows:
+                stacked.append(stacked[0].new_zeros((extra_rows, stacked[0].shape[1])))
         if self.head_gate:  # one row per head behind the heads themselves, then zeros up to a row of 16-byte multiples
             extra_rows = -(-nq // 8) * 8
             g = weights[names["g"]]
@@ -162,7 +208,7 @@ class PagedAttention(Mixer):
         self.qkv_weight = torch.cat(stacked, dim=0).contiguous()
         self.qkv_b = None
         if self.qkv_bias:
-            biases = [self._pad_heads(weights[names[f"{r}_bias"]], heads, size) if r != "g"
+            biases = [pad(weights[names[f"{r}_bias"]], heads, size) if r != "g"
                       else weights[names["q"]].new_zeros(heads * self.head_dim) for r, heads, size in roles]
             if extra_rows:
                 biases.append(weights[names["q"]].new_zeros(extra_rows))
@@ -178,10 +224,15 @@ class PagedAttention(Mixer):
             self.q_norm_weight = weights[names["q_norm"]].to(torch.float32).contiguous()
             if self.has_kv:
                 self.k_norm_weight = weights[names["k_norm"]].to(torch.float32).contiguous()
+        if self.joint_norm_eps is not None:
+            self.q_norm_weight = weights[names["q_norm"]].to(torch.float32).contiguous()
+            self.k_norm_weight = weights[names["k_norm"]].to(torch.float32).contiguous()
         if self.rotate_values:  # formed in double precision, rounded once
             pairs = torch.arange(0, self.value_dim, 2, dtype=torch.float64)
             self.value_inv_freq = (float(self.position_encoding.theta) ** (-pairs / self.value_dim)).to(torch.float32).to(runtime.device)
         self.sinks = torch.zeros(nq, dtype=torch.float32, device=runtime.device) if self.unit_sink else None
+        if self.learned_sinks:
+            self.sinks = weights[names["sink"]].to(torch.float32).contiguous()
         ops.attention_library(self.head_dim)  # compile now, not inside the first step
 
     # ------------------------------------------------------------------ decode steps replayed from a graph
@@ -196,18 +247,18 @@ class PagedAttention(Mixer):
         if not bf16 or not ops.tcgen05_prefill_fits(self.head_dim, self.num_heads, self.num_kv_heads, self.page_size or 16):
             return None
         return int(ops.prefill_key_parts(plan.q_lens, plan.seq_lens, 128 // group, self.num_kv_heads,
-                                         ops.sm_count(self.runtime.device), self.window or self.chunk or 0))
+                                         ops.sm_count(self.runtime.device), self.sees))
 
     def capture_group(self) -> object:
         # layers that see equally far answer `capture_variant` alike
-        return ("paged_attention", self.window or self.chunk or 0)
+        return ("paged_attention", self.sees)
 
     def prepare_capture(self, ctx, variant: object, max_model_len: int) -> None:
         if not ctx.is_decode_only:
             # a captured step with prompt portions: the number of key parts is the variant's (the choice follows the
             # lengths of the step, which a replay does not know on the host)
             ctx.extras[("prefill_key_parts", 128 // (self.num_heads // self.num_kv_heads), self.num_kv_heads,
-                        self.window or self.chunk or 0)] = int(variant or 1)
+                        self.sees)] = int(variant or 1)
             return
         # the number of slices must not follow the lengths of the step that happens to be captured
         ctx.extras["static_max_seq_len"] = max_model_len
@@ -227,6 +278,12 @@ class PagedAttention(Mixer):
         write into the decode kernel is off for it, since that kernel takes the projection output as it is."""
         return None
 
+    def _check_spread(self, layer: LayerBinding) -> None:
+        if not layer.writes_cache:
+            raise ValueError(f"{self.name}: a layer with keys and values of its own writes its pages")
+        if getattr(self.position_encoding, "mscale", 1.0) != 1.0:
+            raise ValueError(f"{self.name}: scaled sines are not built for this layer")
+
     def forward(self, x: torch.Tensor, ctx, layer: LayerBinding, into: IntoNorm | None = None) -> torch.Tensor:
         meta = ctx.groups[layer.group]
         qkv = ops.linear(x, self.qkv_weight, self.qkv_b)
@@ -234,11 +291,18 @@ class PagedAttention(Mixer):
         if not plain_projection:
             self.after_projection(qkv, ctx)
         inv_freq, rotary_dim = self.position_encoding.rotary_table()
+        q = qkv
         # a decode step's attention kernel rotates and writes the newest key and value itself
         fused = (plain_projection and self.plain and layer.writes_cache
                  and ops.fuses_rope(qkv, ctx, self.head_dim, self.num_heads, self.num_kv_heads, layer.kv.shape[3]))
         early_norm = self.qk_norm_eps is not None or self.rotate_values
-        if early_norm:
+        if self.spread:
+            self._check_spread(layer)
+            q = ops.heads_to_pages(qkv, ctx.positions, meta.slot_mapping, layer.kv, self.num_heads, self.num_kv_heads, self.key_dim,
+                                   self.value_dim, self.head_dim, self.k_col, self.v_col, inv_freq=inv_freq, rotary_dim=rotary_dim,
+                                   interleaved=getattr(self.position_encoding, "interleaved", False),
+                                   q_weight=self.q_norm_weight, k_weight=self.k_norm_weight, eps=self.joint_norm_eps or 0.0)
+        elif early_norm:
             if getattr(self.position_encoding, "mscale", 1.0) != 1.0:
                 raise ValueError(f"{self.name}: scaled sines are not built for layers that norm before the rotation")
             if self.has_kv != layer.writes_cache:
@@ -267,11 +331,11 @@ class PagedAttention(Mixer):
             ops.rope_and_cache(qkv, ctx.positions, meta.slot_mapping, inv_freq, layer.kv, self.num_heads,
                                self.num_kv_heads, self.head_dim, rotary_dim, write_cache=layer.writes_cache)
         out = torch.empty((x.shape[0], self.num_heads * self.head_dim), dtype=x.dtype, device=x.device)
-        ops.paged_attention(qkv, out, layer.kv, meta.block_tables, ctx, self.num_heads, self.num_kv_heads,
+        ops.paged_attention(q, out, layer.kv, meta.block_tables, ctx, self.num_heads, self.num_kv_heads,
                             self.head_dim, self.scale, self.window or 0,
                             rope=(inv_freq, rotary_dim) if fused else None, chunk=self.chunk or 0,
                             gate=qkv[:, qkv.shape[1] - out.shape[1]:] if self.gate else None, softcap=self.softcap or 0.0,
-                            sinks=self.sinks)
+                            sinks=self.sinks, keep=self.keep_first)
         if self.head_gate:
             ops.head_gate(out, qkv[:, self.head_gate_col: self.head_gate_col + self.num_heads], self.num_heads, self.head_dim)
         if self.rotate_values:

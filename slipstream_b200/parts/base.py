@@ -50,7 +50,8 @@ class CacheSpec:
     every earlier key stays visible; an integer W means only the last W keys are,
     so pages wholly before the window are given back.  ``chunk`` C: a query sees only the keys of its own chunk
     of C positions (chunks counted from the request's first token), so pages wholly before the chunk of the
-    request's next token are given back.  ``page_size``: tokens per page this mixer's kernels
+    request's next token are given back.  ``keep_first`` K (with a window): the request's first K keys stay visible for
+    good, so the pages that hold them are kept as long as the request lives.  ``page_size``: tokens per page this mixer's kernels
     want; None takes the engine's default.  Mixers whose specs are equal share a cache group (one page pool, one
     block table per request); a group has its own page size and its own number of pages."""
 
@@ -59,9 +60,10 @@ class CacheSpec:
     window: int | None = None
     page_size: int | None = None
     chunk: int | None = None
+    keep_first: int = 0
 
     def first_visible(self, position: int) -> int:
-        """The lowest key a query at ``position`` (or any later one) can see."""
+        """The lowest key a query at ``position`` (or any later one) can see, besides those ``keep_first`` keeps."""
         first = 0
         if self.window is not None:
             first = max(first, position - self.window + 1)
@@ -71,7 +73,7 @@ class CacheSpec:
 
     @property
     def span(self) -> int | None:
-        """The most keys a query can see (None: all earlier ones)."""
+        """The most keys a query can see (None: all earlier ones), besides those ``keep_first`` keeps."""
         bounds = [b for b in (self.window, self.chunk) if b is not None]
         return min(bounds) if bounds else None
 

@@ -124,3 +124,34 @@ class ParallelBlock(Block):
         mixed = self.mixer.forward(x, ctx, layer)
         fed = self.feed_forward.forward(x, ctx) if self.feed_forward is not None else None
         return residual, self.norm.write_of(mixed, fed), None
+
+
+@BLOCKS.register("sandwich_norm")
+class SandwichBlock(Block):
+    """``x + m * norm1b(mixer(norm1(x)))`` then ``x + m * norm2b(ffn(norm2(x)))``: a norm on both sides of each branch
+    and a multiplier on what joins the stream.  ``feed_forward`` may be None.  All norms are `JoiningNorm`: a branch's
+    output stays pending, and the kernel of the next norm, of this block or of the next one, norms it, adds it and norms
+    the new stream in one pass."""
+
+    cuda_graph_safe = True
+
+    def __init__(self, mixer: Mixer, feed_forward: FeedForward | None, mixer_norm: Norm, mixer_out_norm: Norm,
+                 ffn_norm: Norm | None, ffn_out_norm: Norm | None, residual_mult: float = 1.0) -> None:
+        if len({feed_forward is None, ffn_norm is None, ffn_out_norm is None}) != 1:
+            raise ValueError("a feed-forward and its two norms come together")
+        self.mixer, self.feed_forward = mixer, feed_forward
+        self.mixer_norm, self.mixer_out_norm = mixer_norm, mixer_out_norm
+        self.ffn_norm, self.ffn_out_norm = ffn_norm, ffn_out_norm
+        self.residual_mult = float(residual_mult)
+
+    def children(self) -> list[Part]:
+        return [p for p in (self.mixer_norm, self.mixer, self.mixer_out_norm, self.ffn_norm, self.feed_forward, self.ffn_out_norm)
+                if p is not None]
+
+    def forward(self, residual: torch.Tensor, pending, ctx, layer: LayerBinding):
+        x = self.mixer_norm.add_norm(residual, pending)
+        pending = self.mixer_out_norm.branch(self.mixer.forward(x, ctx, layer), self.residual_mult)
+        if self.feed_forward is not None:
+            x = self.ffn_norm.add_norm(residual, pending)
+            pending = self.ffn_out_norm.branch(self.feed_forward.forward(x, ctx), self.residual_mult)
+        return residual, pending

@@ -2,17 +2,24 @@
 (slipstream/models/layers/mlp.py:33-40).  The gate and up matrices are stacked at
 load so that one product feeds the activation kernel.
 
-The activation has three constants, so that relatives of SwiGLU are the same part: with ``g = min(gate, limit)``
+The activation has four constants, so that relatives of SwiGLU are the same part: with ``g = min(gate, limit)``
 and ``u = clamp(up, -limit, limit)`` (no ``limit``: unclamped) the hidden vector is
-``g * sigmoid(alpha * g) * (u + up_shift)``; alpha = 1, no limit and up_shift = 0 is SwiGLU."""
+``g * sigmoid(alpha * g + cubic * g^3) * (u + up_shift)``; alpha = 1, no limit and up_shift = cubic = 0 is SwiGLU.
+The tanh form of GELU is ``z * sigmoid(2 sqrt(2 / pi) (z + 0.044715 z^3))``, because (1 + tanh(a)) / 2 = sigmoid(2a):
+``GELU_TANH`` holds its two constants."""
 
 from __future__ import annotations
+
+import math
 
 import torch
 
 from slipstream_b200 import ops
 
 from .base import FEED_FORWARDS, FeedForward, IntoNorm, Runtime, WeightSpec
+
+
+GELU_TANH = {"alpha": 2.0 * math.sqrt(2.0 / math.pi), "cubic": 2.0 * math.sqrt(2.0 / math.pi) * 0.044715}
 
 
 @FEED_FORWARDS.register("swiglu")
@@ -22,7 +29,7 @@ class SwiGLUFeedForward(FeedForward):
     takes_pending_norm = True
 
     def __init__(self, name: str, hidden_size: int, intermediate_size: int, bias: bool = False, *,
-                 alpha: float = 1.0, limit: float | None = None, up_shift: float = 0.0,
+                 alpha: float = 1.0, limit: float | None = None, up_shift: float = 0.0, cubic: float = 0.0,
                  names: dict[str, str] | None = None) -> None:
         """``names``: the checkpoint's tensor names by role (gate, up, down, gate_bias, up_bias, down_bias)."""
         self.name = name
@@ -32,6 +39,7 @@ class SwiGLUFeedForward(FeedForward):
         self.alpha = float(alpha)
         self.limit = None if limit is None else float(limit)
         self.up_shift = float(up_shift)
+        self.cubic = float(cubic)
         if self.limit is not None and not self.limit > 0.0:
             raise ValueError("limit must be positive")
         n = name
@@ -42,7 +50,7 @@ class SwiGLUFeedForward(FeedForward):
 
     @property
     def is_swiglu(self) -> bool:
-        return self.alpha == 1.0 and self.limit is None and self.up_shift == 0.0
+        return self.alpha == 1.0 and self.limit is None and self.up_shift == 0.0 and self.cubic == 0.0
 
     def weight_specs(self) -> list[WeightSpec]:
         h, i, names = self.hidden_size, self.intermediate_size, self.names
@@ -84,7 +92,7 @@ class SwiGLUFeedForward(FeedForward):
             hidden = ops.gate_up_swiglu(x, self.gate_up, self.gate_up_bias, self.block)
         else:
             hidden = ops.gate_up_glu(x, self.gate_up, self.gate_up_bias, self.block, self.alpha, self.limit or 0.0,
-                                     self.up_shift)
+                                     self.up_shift, self.cubic)
         if into is not None:
             return into.close(hidden, self.down, self.down_bias)
         return ops.linear(hidden, self.down, self.down_bias)
@@ -95,7 +103,6 @@ GatedFeedForward = FEED_FORWARDS.register("gated_linear_unit")(SwiGLUFeedForward
 
 
 def _softplus(z: float) -> float:
-    import math
     return z if z > 30.0 else math.log1p(math.exp(z))
 
 

@@ -7,6 +7,8 @@ in float32; the branch output that has not been added yet comes in as ``delta``.
 
 from __future__ import annotations
 
+from dataclasses import dataclass, replace
+
 import torch
 
 from slipstream_b200 import ops
@@ -99,6 +101,56 @@ class GroupRMSNorm(Norm):
     def forward(self, x: torch.Tensor, gate: torch.Tensor | None = None) -> torch.Tensor:
         """``norm(x)`` (``x`` in the compute dtype or float32), or ``norm(x * silu(gate))``."""
         return ops.group_norm(x, self.weight, self.groups, self.eps, self.runtime.dtype, gate=gate)
+
+
+@dataclass
+class NormedBranch:
+    """A branch output that has not joined the stream yet: the next norm's kernel adds ``mult * norm(y)`` (and
+    ``anchor``, float32, if there is one) where it reads the stream."""
+
+    y: torch.Tensor
+    norm: "JoiningNorm"
+    mult: float
+    anchor: torch.Tensor | None = None
+
+    def with_anchor(self, anchor: torch.Tensor) -> "NormedBranch":
+        return replace(self, anchor=anchor)
+
+
+@NORMS.register("joining_rmsnorm")
+class JoiningNorm(Norm):
+    """RMS norm ``x / sqrt(mean(x^2) + eps) * weight``, formed in float32 and rounded once, for blocks that norm a branch
+    on both sides (`SandwichBlock`).  In front of a branch (and as the model's last norm) it is ``add_norm``, whose kernel
+    first lets the pending branch output join the stream, under that output's own norm; behind a branch it is
+    ``branch(y, mult)``, which leaves its work to the next ``add_norm``."""
+
+    cuda_graph_safe = True
+
+    def __init__(self, tensor: str, size: int, eps: float) -> None:
+        self.tensor, self.size, self.eps = tensor, size, float(eps)
+
+    def weight_specs(self) -> list[WeightSpec]:
+        return [WeightSpec(self.tensor, (self.size,), kind="vector", init=("one_plus_normal", 0.1))]
+
+    def bind(self, weights: dict[str, torch.Tensor], runtime: Runtime) -> None:
+        super().bind(weights, runtime)
+        self.weight = weights[self.tensor].to(torch.float32).contiguous()
+
+    def weight_bytes(self) -> int:
+        return self.weight.numel() * self.weight.element_size()
+
+    def branch(self, y: torch.Tensor, mult: float = 1.0) -> NormedBranch:
+        return NormedBranch(y, self, mult)
+
+    def add_norm(self, residual: torch.Tensor, delta: "NormedBranch | None",
+                 rows: torch.Tensor | None = None) -> torch.Tensor:
+        if delta is None:
+            return ops.branch_norm(residual, None, None, 0.0, 0.0, self.weight, self.eps, self.runtime.dtype, rows=rows)
+        return ops.branch_norm(residual, delta.y, delta.norm.weight, delta.norm.eps, delta.mult, self.weight, self.eps,
+                               self.runtime.dtype, anchor=delta.anchor, rows=rows)
+
+    def forward(self, x: torch.Tensor) -> torch.Tensor:
+        return self.add_norm(x, None)
 
 
 @NORMS.register("stream_rounding")

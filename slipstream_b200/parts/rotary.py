@@ -93,6 +93,35 @@ class YarnRotaryEncoding(RotaryEncoding):
         return (f / self.factor * ramp + f * (1.0 - ramp)).to(torch.float32)
 
 
+@POSITION_ENCODINGS.register("banded_rotary")
+class BandedRotaryEncoding(RotaryEncoding):
+    """Rotary frequencies for a context ``factor`` times longer than the trained one of ``original`` positions, by the
+    number of turns t = original * f / (2 pi) that the wave of a frequency f = theta^(-2i/d) makes within it: more than
+    ``high`` turns keep f, fewer than ``low`` turn ``factor`` times slower, and between the two the frequency is
+    ``f (1 - s) / factor + f s`` with s = (t - low) / (high - low).  (The scaling of Llama 3.1.)  The table is formed in
+    double precision on the host and rounded to float32 once."""
+
+    def __init__(self, head_dim: int, theta: float, rotary_dim: int | None = None, interleaved: bool = False, *,
+                 factor: float, original: float, low: float, high: float) -> None:
+        super().__init__(head_dim, theta, rotary_dim, interleaved)
+        self.factor, self.original, self.low, self.high = float(factor), float(original), float(low), float(high)
+        if min(self.factor, self.original, self.low) <= 0.0 or self.high < self.low:
+            raise ValueError("factor, original and low must be positive, high at least low")
+
+    def inverse_frequencies(self) -> torch.Tensor:
+        out = []
+        for i in range(self.rotary_dim // 2):
+            f = self.theta ** (-2.0 * i / self.rotary_dim)
+            turns = self.original * f / (2.0 * math.pi)
+            if turns < self.low:
+                f = f / self.factor
+            elif turns <= self.high and self.high > self.low:
+                s = (turns - self.low) / (self.high - self.low)
+                f = (1.0 - s) * f / self.factor + s * f
+            out.append(f)
+        return torch.tensor(out, dtype=torch.float64).to(torch.float32)
+
+
 @POSITION_ENCODINGS.register("none")
 class NoPositionEncoding(PositionEncoding):
     """Queries and keys are used as projected."""
