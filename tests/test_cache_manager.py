@@ -190,3 +190,33 @@ def test_pool_sizes_give_a_windowed_group_only_what_its_windows_can_hold():
     assert cost(tokens) <= budget < cost(tokens + 64)
     # everything fits: no more than the requests can ever hold
     assert tokens_that_fit(layouts, [16, 64], per_token, 1 << 50, 4, 4096, 512) == 4 * (4096 + 64)
+
+
+def test_a_window_that_keeps_the_first_keys_keeps_their_pages():
+    """With 5 kept tokens on pages of 4, the first two pages of a request stay while the window's pages come and go; they
+    return when the request ends."""
+    m = manager(pages=12, page=4, groups=[GroupLayout(CacheSpec(2, 16, window=6, keep_first=5), 1)])
+    assert m.kept_blocks(0) == 2
+    m.admit("a")
+    held = []
+    for n in [3, 1, 9, 2, 1, 1, 1, 7, 5, 1, 1, 10]:
+        m.reserve("a", n)
+        m.commit("a", n)
+        table, length = m.get("a").tables[0], m.length("a")
+        held.append([b for b, p in enumerate(table) if p >= 0])
+        first = max(0, length - 6 + 1) // 4
+        assert held[-1] == sorted(set(range(min(2, len(table)))) | set(range(first, len(table))))
+        assert m.get("a").tables[0][:2] == [0, 1][: len(table)]
+        assert 0.0 < m.utilization() <= 1.0
+        m.check_invariants()
+    # at most: the window with a step's tokens, one page for its place, and the kept pages
+    assert max(len(h) for h in held) <= m.peak_pages(0, 42, 10)
+    m.release("a")
+    assert m.all_pages_free()
+    m.check_invariants()
+
+
+def test_pools_of_windowed_groups_have_room_for_kept_pages():
+    from slipstream_b200.cache import pool_sizes
+    plain, keeping = (GroupLayout(CacheSpec(2, 16, window=8, keep_first=k), 1) for k in (0, 9))
+    assert pool_sizes([plain, keeping], [4, 4], 4000, 3, 1000, 4) == [3 * (3 + 1), 3 * (3 + 1 + 3)]
