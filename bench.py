@@ -27,6 +27,10 @@ summed from three tables, hyper-connected streams, a feed-forward without a gate
 windowed attention with a unit sink beside a gated linear recurrence, un-gated routed experts with groups, pass-through
 experts and a gated shared expert, one norm for both branches of a layer).
 
+``--compare fusipel`` does the same for the Fusipel decoder (differential attention under a window that keeps the first
+tokens, attention whose values are the keys with a joint norm and learned sinks, norms on both sides of every branch, a
+feed-forward with the tanh form of GELU, layers that run twice with the embedding joining in between).
+
 ``--only decode|prefill`` runs one part and prints a short line (profiling, and measurements beside the
 headline): ``--only decode --batch 1 --prompt-len 32000 --context-len 32768`` is a decode step behind a long
 context, ``--only prefill --chunk 512 --prefix 8192 --context-len 32768`` a prompt portion behind cached tokens.
@@ -1288,6 +1292,220 @@ def run_compare_lakadra(args) -> int:
     return 0
 
 
+def fusipel_config(z: dict, window: int) -> dict:
+    """config.json of a Fusipel decoder at the layer sizes ``z``: differential heads (two maps of half the head size over
+    values of the whole, so that the projections have the dense model's sizes; a window that keeps 4 tokens) and heads
+    whose values are the keys (a joint norm, sinks) in turn.  A quarter of the layers runs twice in a row, so that a step
+    runs as many layers as the dense model does."""
+    def rot(dims):
+        return dict(base=1000000.0, dims=dims, scaling=dict(factor=8.0, low=1.0, high=4.0, original=8192))
+
+    runs, d = z["layers"], z["dim"]
+    twice = runs // 4
+    layers = []
+    for i in range(runs - twice):
+        if i % 2:
+            kind, mixer = "attention_2", dict(heads=z["heads"], kv_heads=z["kv_heads"], dim=d, vdim=d, scale=d ** -0.5, rot=rot(d // 4))
+        else:
+            kind, mixer = "attention", dict(heads=z["heads"], kv_heads=z["kv_heads"], dim=d // 2, vdim=d, scale=(d // 2) ** -0.5,
+                                            diff=0.6, rot=rot(d // 8), mask=dict(size=window, keep_first=4))
+        layers.append(dict(type=kind, mixer=mixer, mlp=dict(kind="dense", ff=z["ff"])))
+    return dict(architecture="Fusipel", vocab=z["vocab"], width=z["width"], norm=dict(eps=1e-6), residual_mult=0.5, layers=layers,
+                loop=dict(start=2, stop=2 + twice, times=2), max_position_embeddings=8192)
+
+
+def run_compare_fusipel(args) -> int:
+    """The Fusipel decoder beside the Qwen2.5 decoder at equal layer sizes (whole steps), then every kernel the design
+    adds or runs in a form of its own, alone at the 7B layer sizes, beside the like kernel of the Qwen2.5 path or its
+    nearest relative among the other decoders'."""
+    import numpy as np
+    import torch
+
+    from slipstream_b200 import ops
+    from slipstream_b200.engine.context import query_tiles_host, query_tiles_longest_first_host
+    from slipstream_b200.parts import GELU_TANH
+
+    pk, pk_kind = peaks()
+    rng = np.random.default_rng(0)
+    dev = torch.device("cuda:0")
+    batch, ctx_tokens, T, page = args.batch, args.prompt_len, args.chunk, 16
+    result: dict = {"compare": "fusipel", "peaks": pk_kind, "batch": batch, "context": ctx_tokens, "prefill_tokens": T,
+                    "window": args.window, "sizes": {}}
+    for name in (args.sizes.split(",") if args.sizes else COMPARE_SIZES):
+        qwen, _ = compare_configs(COMPARE_SIZES[name], 8192, 1, False)
+        result["sizes"][name] = {}
+        for which, config in (("qwen2", qwen), ("fusipel", fusipel_config(COMPARE_SIZES[name], args.window))):
+            if which == "qwen2" and args.skip_qwen2:
+                continue
+            print(f"[bench] {name} {which} ...", file=sys.stderr, flush=True)
+            result["sizes"][name][which] = measure_model(config, args, pk, rng)
+            print(f"[bench] {name} {which}: {result['sizes'][name][which]}", file=sys.stderr, flush=True)
+    if args.no_kernels:
+        print(json.dumps(result))
+        return 0
+
+    print("[bench] single kernels ...", file=sys.stderr, flush=True)
+    z = COMPARE_SIZES["7b"]
+    h, n_q, n_kv, d, inter = z["width"], z["heads"], z["kv_heads"], z["dim"], z["ff"]
+    half = d // 2  # a map's size
+    gen = torch.Generator(device=dev).manual_seed(1)
+    kernels: dict = {}
+
+    def rand(*shape, dtype=torch.bfloat16, std=0.5):
+        return (torch.randn(*shape, generator=gen, device=dev) * std).to(dtype)
+
+    def sweep(run, copies: int = 6) -> float:
+        """Microseconds a launch, the operands rotating through ``copies`` sets; replayed from a graph, as an engine's
+        steps are, so that launches of a few microseconds are not timed at the speed of the host."""
+        for i in range(copies):
+            run(i)
+        torch.cuda.synchronize()  # the operands are complete before another stream captures launches that read them
+        graph = torch.cuda.CUDAGraph()
+        with torch.cuda.graph(graph):
+            for i in range(copies * 2):
+                run(i % copies)
+        times = []
+        for _ in range(8):
+            torch.cuda.synchronize()
+            start, stop = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            start.record()
+            graph.replay()
+            stop.record()
+            torch.cuda.synchronize()
+            times.append(start.elapsed_time(stop) * 1e3 / (2 * copies))
+        return sorted(times[3:])[2]
+
+    def hbm(name: str, us: float, nbytes: float) -> None:
+        gbs = nbytes / us / 1e3
+        kernels[name] = {"us": round(us, 2), "gbs": round(gbs, 1), "hbm_frac": round(gbs / pk["hbm_gbs"], 3)}
+
+    def tensor(name: str, us: float, flops: float) -> None:
+        tf = flops / us / 1e6
+        kernels[name] = {"us": round(us, 2), "tflops": round(tf, 1), "bf16_frac": round(tf / pk["bf16_tflops"], 3)}
+
+    eps, glu = 1e-6, (GELU_TANH["alpha"], 0.0, 0.0, GELU_TANH["cubic"])
+    diff = ops.DiffPair(0.7, 0.4, eps, d)
+    sinks = rand(n_q, dtype=torch.float32)
+    for tokens, tag in ((T, "prefill"), (batch, "decode")):
+        streams = [rand(tokens, h, dtype=torch.float32) for _ in range(6)]
+        anchor = rand(tokens, h, dtype=torch.float32)
+        ys = [rand(tokens, h) for _ in range(6)]
+        w, wb = rand(h, dtype=torch.float32), rand(h, dtype=torch.float32)
+        us = sweep(lambda i: ops.add_rmsnorm(streams[i], ys[i], w, eps, torch.bfloat16))
+        hbm(f"{tag}_add_rmsnorm (qwen2)", us, tokens * h * 12.0)
+        us = sweep(lambda i: ops.branch_norm(streams[i], ys[i], wb, eps, 0.5, w, eps, torch.bfloat16))
+        hbm(f"{tag}_branch_norm (norm behind the branch, join, next norm)", us, tokens * h * 12.0)
+        us = sweep(lambda i: ops.branch_norm(streams[i], ys[i], wb, eps, 0.5, w, eps, torch.bfloat16, anchor=anchor))
+        hbm(f"{tag}_branch_norm with the embedding joining", us, tokens * h * 16.0)
+        del streams, ys, anchor
+        positions = torch.arange(tokens, dtype=torch.int32, device=dev)
+        rows = [rand(tokens, (n_q + 2 * n_kv) * d) for _ in range(6)]
+        kvs = [torch.zeros(max(tokens // page, 1), 2, n_kv, page, d, dtype=torch.bfloat16, device=dev) for _ in range(6)]
+        inv = torch.rand(d // 2, device=dev)
+        us = sweep(lambda i: ops.rope_and_cache(rows[i], positions, positions, inv, kvs[i], n_q, n_kv, d, d))
+        hbm(f"{tag}_rope_and_cache (qwen2)", us, tokens * d * 2.0 * (2 * n_q + 4 * n_kv))
+        wq, wk = rand(d, dtype=torch.float32), rand(d, dtype=torch.float32)
+        us = sweep(lambda i: ops.norm_rope_cache(rows[i], positions, positions, kvs[i], n_q, n_kv, d, inv_freq=inv, rotary_dim=d,
+                                                 q_weight=wq, k_weight=wk, norm_dim=d, eps=eps))
+        hbm(f"{tag}_norm_rope_cache (sarudra: a norm per head)", us, tokens * d * 2.0 * (2 * n_q + 4 * n_kv))
+        wq, wk = rand(n_q * d, dtype=torch.float32), rand(n_kv * d, dtype=torch.float32)
+        inv4, inv8 = inv[: d // 8].contiguous(), inv[: d // 16].contiguous()
+        us = sweep(lambda i: ops.heads_to_pages(rows[i], positions, positions, kvs[i], n_q, n_kv, d, d, d, n_q * d, n_q * d, inv_freq=inv4,
+                                                rotary_dim=d // 4, q_weight=wq, k_weight=wk, eps=eps))
+        hbm(f"{tag}_heads_to_pages (joint norm, values are the keys)", us, tokens * d * 2.0 * (2 * n_q + 3 * n_kv))
+        us = sweep(lambda i: ops.heads_to_pages(rows[i], positions, positions, kvs[i], n_q, n_kv, half, d, d, n_q * d, (n_q + n_kv) * d, maps=2,
+                                                inv_freq=inv8, rotary_dim=d // 8))
+        hbm(f"{tag}_heads_to_pages (two maps: queries leave twice as wide)", us, tokens * d * 2.0 * (3 * n_q + 4 * n_kv))
+        heads = [rand(tokens, 2 * n_q * d, dtype=torch.float32) for _ in range(3)]
+        out = torch.empty(tokens, n_q * d, dtype=torch.bfloat16, device=dev)
+        us = sweep(lambda i: ops.diff_combine(heads[i], diff, n_q, out), 3)
+        hbm(f"{tag}_diff_combine (alone; inside the attention kernel in prompt steps)", us, tokens * n_q * d * 10.0)
+        del rows, kvs, heads, out
+        x = rand(tokens, h)
+        gate_up = [rand(2 * inter, h, std=0.02) for _ in range(4)]
+        if tag == "prefill":
+            us = sweep(lambda i: ops.gate_up_swiglu(x, gate_up[i], None, 64), 4)
+            tensor("prefill_gate_up_swiglu (qwen2)", us, 4.0 * tokens * h * inter)
+            us = sweep(lambda i: ops.gate_up_glu(x, gate_up[i], None, 64, *glu), 4)
+            tensor("prefill_gate_up with the tanh form of GELU", us, 4.0 * tokens * h * inter)
+        else:
+            us = sweep(lambda i: ops.gate_up_swiglu(x, gate_up[i], None, 64), 4)
+            hbm("decode_gate_up_swiglu (qwen2)", us, 4.0 * h * inter)
+            us = sweep(lambda i: ops.gate_up_glu(x, gate_up[i], None, 64, *glu), 4)
+            hbm("decode_gate_up with the tanh form of GELU", us, 4.0 * h * inter)
+        del gate_up
+
+    # attention: a prompt in one step, then decode steps.  Differential heads: 2 n_q query heads of the kernel; the
+    # operations counted are those of the design (a map's scores over half the head size)
+    def pages_for(n_req: int, tokens: int):
+        per = (tokens + page - 1) // page
+        return torch.arange(n_req * per, dtype=torch.int32, device=dev).view(n_req, per)
+
+    one_q = torch.tensor([0, T], dtype=torch.int32, device=dev)
+    one_len = torch.tensor([T], dtype=torch.int32, device=dev)
+    table = pages_for(1, T)
+    kv_pages = [rand(T // page + 1, 2, n_kv, page, d) for _ in range(6)]
+    qs, q2s = rand(T, n_q * d), rand(T, 2 * n_q * d)
+    out, out2 = torch.empty(T, n_q * d, dtype=torch.bfloat16, device=dev), torch.empty(T, 2 * n_q * d, dtype=torch.float32, device=dev)
+
+    def prefill(name: str, q, heads: int, window: int, flops_per_key: float, into=out, **more) -> None:
+        group = heads // n_kv
+        req, tok0 = (torch.from_numpy(a).to(dev) for a in query_tiles_longest_first_host(
+            np.asarray([T], dtype=np.int32), np.asarray([T], dtype=np.int32), 128 // group))
+        us = sweep(lambda i: ops.paged_attention_prefill_tcgen05(q, q.shape[1], into, kv_pages[i], table, req, tok0, one_q, one_len,
+                                                                 heads, n_kv, d, d ** -0.5, 1, 0, window, **more))
+        pos = np.arange(T)
+        keys = float(np.minimum(pos + 1, window + min(more.get("keep", 0), T)).sum() if window else (pos + 1).sum())
+        tensor(name, us, keys * flops_per_key)
+
+    per_head, per_diff = 4.0 * n_q * d, 2.0 * n_q * (2.0 * half + 2.0 * d)
+    prefill("prefill_attention (qwen2)", qs, n_q, 0, per_head)
+    prefill("prefill_attention with learned sinks", qs, n_q, 0, per_head, sinks=sinks)
+    prefill("prefill_attention, two maps combined inside", q2s, 2 * n_q, 0, per_diff, diff=diff)
+    prefill("prefill_attention, two maps, float32 outputs", q2s, 2 * n_q, 0, per_diff, into=out2)
+    prefill("prefill_attention, window of 512 (qwen2's kernel)", qs, n_q, 512, per_head)
+    prefill("prefill_attention, two maps combined inside, window of 512 that keeps 4", q2s, 2 * n_q, 512, per_diff, diff=diff, keep=4)
+    group = n_q // n_kv
+    req, row0 = (torch.from_numpy(a).to(dev) for a in query_tiles_host(np.asarray([T * 2 * group], dtype=np.int32), 64))
+    us = sweep(lambda i: ops.paged_attention_prefill(q2s, q2s.shape[1], out, kv_pages[i], table, req, row0, one_q, one_len, 2 * n_q, n_kv, d,
+                                                     d ** -0.5, 0, diff=diff))
+    tensor("prefill_attention mma.sync, two maps combined inside", us, T * (T + 1) / 2 * per_diff)
+    req, row0 = (torch.from_numpy(a).to(dev) for a in query_tiles_host(np.asarray([T * group], dtype=np.int32), 64))
+    us = sweep(lambda i: ops.paged_attention_prefill(qs, qs.shape[1], out, kv_pages[i], table, req, row0, one_q, one_len, n_q, n_kv, d,
+                                                     d ** -0.5, 0))
+    tensor("prefill_attention mma.sync (qwen2's heads)", us, T * (T + 1) / 2 * per_head)
+    del kv_pages, qs, q2s, out, out2
+
+    for n_req, tokens in ((batch, ctx_tokens), (batch, 8000), (64, 4000)):
+        copies = 6 if n_req * tokens < 20000 else 3
+        kv_pages = [rand(n_req * ((tokens + page - 1) // page), 2, n_kv, page, d) for _ in range(copies)]
+        table = pages_for(n_req, tokens)
+        starts = torch.arange(n_req + 1, dtype=torch.int32, device=dev)
+        lens = torch.full((n_req,), tokens, dtype=torch.int32, device=dev)
+        q, q2 = rand(n_req, n_q * d), rand(n_req, 2 * n_q * d)
+        out, out2 = torch.empty_like(q), torch.empty(n_req, 2 * n_q * d, dtype=torch.float32, device=dev)
+
+        def decode(name: str, q, heads: int, window: int, into, **more) -> None:
+            seen = min(tokens, window + more.get("keep", 0)) if window else tokens
+            slices = ops.decode_slices(n_req, n_kv, heads // n_kv, seen, False, ops.sm_count(dev))
+            us = sweep(lambda i: ops.paged_attention_decode(q, q.shape[1], into, kv_pages[i], table, starts, lens, n_req, heads, n_kv, d,
+                                                            d ** -0.5, window, slices, stages=ops.functions.DECODE_RING_STAGES, **more), copies)
+            hbm(f"decode_attention {n_req} x {tokens}: {name}", us, n_req * seen * 4.0 * n_kv * d + n_req * (q.shape[1] * 2.0 + into.numel() / n_req * into.element_size()))
+
+        decode("qwen2's heads, rotation outside", q, n_q, 0, out)
+        decode("learned sinks", q, n_q, 0, out, sinks=sinks)
+        decode("learned sinks, cp.async", q, n_q, 0, out, sinks=sinks, tma=False)
+        decode("two maps, float32 outputs", q2, 2 * n_q, 0, out2)
+        if tokens > 1024:
+            decode("window of 1024 (qwen2's heads)", q, n_q, 1024, out)
+            decode("two maps, window of 1024 that keeps 4", q2, 2 * n_q, 1024, out2, keep=4)
+        del kv_pages
+    ops.check_errors(dev)
+    result["kernels_7b"] = kernels
+    print(json.dumps(result))
+    return 0
+
+
 def main() -> int:
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -1307,7 +1525,7 @@ def main() -> int:
     ap.add_argument("--workload", choices=sorted(WORKLOADS), default=None,
                     help="run another measured workload end to end through the scheduler instead")
     ap.add_argument("--window", type=int, default=4096, help="--compare sarudra: positions of the sliding window")
-    ap.add_argument("--compare", choices=["fokedra", "sarudra", "bezutar", "lakadra"], default=None,
+    ap.add_argument("--compare", choices=["fokedra", "sarudra", "bezutar", "lakadra", "fusipel"], default=None,
                     help="time another decoder design beside the Qwen2.5 decoder at equal layer sizes instead")
     ap.add_argument("--sizes", default="", help="--compare: which of 0.5b,7b,14b (default: all)")
     ap.add_argument("--mask-chunk", type=int, default=8192, help="--compare: positions per attention chunk")
@@ -1331,6 +1549,8 @@ def main() -> int:
             return run_compare_bezutar(args)
         if args.compare == "lakadra":
             return run_compare_lakadra(args)
+        if args.compare == "fusipel":
+            return run_compare_fusipel(args)
         return run_compare_sarudra(args) if args.compare == "sarudra" else run_compare(args)
     if args.workload:
         return run_workload(args.workload, args)

@@ -55,7 +55,7 @@ __device__ __forceinline__ void store8f(float* p, const float (&v)[8]) {
 //   values    to theirs: dv elements, zeros behind them.
 // The score of query (head, map m) with such a key row is that of map m alone, so the attention kernels run n_q * M
 // query heads over n_kv key/value heads of D >= max(M * d, dv) elements.  kv: [page][2][kv head][offset][D].
-// A block per token.  VEC 8: bfloat16, 16-byte accesses, pairs of neighbours; VEC 1: any type and size.
+// Two kernels: one with 16-byte accesses (bfloat16, sizes in runs of 8, pairs of neighbours), one for any type and size.
 struct HeadsArgs {
     const void* rows;
     int64_t row_stride;
@@ -72,8 +72,9 @@ struct HeadsArgs {
     int* err;
 };
 
-template <typename T, int VEC>
-__global__ void __launch_bounds__(512) heads_to_pages_kernel(const HeadsArgs a) {
+// Any type and size: a block per token, a thread per element.
+template <typename T>
+__global__ void __launch_bounds__(256) heads_to_pages_kernel(const HeadsArgs a) {
     pdl_launch_dependents();
     pdl_wait();
     __shared__ float cos_s[128], sin_s[128], scratch[2][32];
@@ -91,21 +92,8 @@ __global__ void __launch_bounds__(512) heads_to_pages_kernel(const HeadsArgs a) 
     float q_rstd = 1.f, k_rstd = 1.f;
     if (a.q_weight) {
         float sq = 0.f, sk = 0.f;
-        for (int c = threadIdx.x * VEC; c < q_len + k_len; c += blockDim.x * VEC) {
-            const bool is_q = c < q_len;  // VEC divides q_len
-            const T* p = is_q ? row + c : row + a.k_col + (c - q_len);
-            float s = 0.f;
-            if constexpr (VEC == 8) {
-                float v[8];
-                unpack8(*reinterpret_cast<const uint4*>(p), v);
-#pragma unroll
-                for (int e = 0; e < 8; ++e) s = fmaf(v[e], v[e], s);
-            } else {
-                const float v = to_float(*p);
-                s = v * v;
-            }
-            if (is_q) sq += s; else sk += s;
-        }
+        for (int c = threadIdx.x; c < q_len; c += blockDim.x) sq = fmaf(to_float(row[c]), to_float(row[c]), sq);
+        for (int c = threadIdx.x; c < k_len; c += blockDim.x) sk = fmaf(to_float(row[a.k_col + c]), to_float(row[a.k_col + c]), sk);
         q_rstd = 1.0f / sqrtf(block_sum_once(sq, scratch[0]) / (float)q_len + a.eps);
         k_rstd = 1.0f / sqrtf(block_sum_once(sk, scratch[1]) / (float)k_len + a.eps);
     } else {
@@ -113,20 +101,19 @@ __global__ void __launch_bounds__(512) heads_to_pages_kernel(const HeadsArgs a) 
     }
     const int64_t page = slot >= 0 ? slot / a.page_size : 0;
     const int off = slot >= 0 ? (int)(slot % a.page_size) : 0;
-    // outputs in runs of VEC: queries, then (with a slot) keys and values
-    const int per_head = D / VEC, q_runs = a.n_q * a.maps * per_head, kv_runs = slot >= 0 ? a.n_kv * per_head : 0;
-    T* const q_out = reinterpret_cast<T*>(a.q_out) + (int64_t)t * a.n_q * a.maps * D;
+    const int q_runs = a.n_q * a.maps * D, kv_runs = slot >= 0 ? a.n_kv * D : 0;
+    T* const q_out = reinterpret_cast<T*>(a.q_out) + (int64_t)t * q_runs;
     T* const kv = reinterpret_cast<T*>(a.kv);
     for (int run = threadIdx.x; run < q_runs + 2 * kv_runs; run += blockDim.x) {
         const bool is_q = run < q_runs, is_v = run >= q_runs + kv_runs;
         const int r = is_q ? run : (is_v ? run - q_runs - kv_runs : run - q_runs);
-        const int head = r / per_head, o = (r - head * per_head) * VEC;
+        const int head = r / D, o = r - head * D;
         T* dst;
-        int from = -1;  // place of the run's first element among its projection's; -1: zeros
+        int from = -1;  // place of the element among its projection's; -1: zero
         int in_part = 0;
         if (is_q) {
-            dst = q_out + (int64_t)head * D + o;
-            const int m = a.maps == 1 ? 0 : head % a.maps, h = a.maps == 1 ? head : head / a.maps;
+            dst = q_out + r;
+            const int m = head % a.maps, h = head / a.maps;
             in_part = o - m * a.d;
             if (in_part >= 0 && in_part < a.d) from = h * md + o;
         } else {
@@ -134,57 +121,135 @@ __global__ void __launch_bounds__(512) heads_to_pages_kernel(const HeadsArgs a) 
             if (is_v) {
                 if (o < a.dv) from = head * a.dv + o;
             } else if (o < md) {
-                in_part = a.maps == 1 ? o : o % a.d;
+                in_part = o % a.d;
                 from = head * md + o;
             }
         }
-        const T* src = row + (is_q ? 0 : (is_v ? a.v_col : a.k_col)) + from;
-        const float* w = is_q ? a.q_weight : a.k_weight;
-        const float rstd = is_q ? q_rstd : k_rstd;
-        const bool normed = w != nullptr && !is_v, turned = !is_v && in_part < a.rot_dim;
-        if constexpr (VEC == 8) {
-            float v[8];
-            if (from < 0) {
-                *reinterpret_cast<uint4*>(dst) = make_uint4(0u, 0u, 0u, 0u);
-                continue;
+        float v = 0.f;
+        if (from >= 0) {
+            const T* src = row + (is_q ? 0 : (is_v ? a.v_col : a.k_col)) + from;
+            const float* w = is_q ? a.q_weight : a.k_weight;
+            const float rstd = is_q ? q_rstd : k_rstd;
+            const bool normed = w != nullptr && !is_v;
+            v = to_float(*src);
+            if (normed) v = v * rstd * w[from];
+            if (!is_v && in_part < a.rot_dim) {
+                const int half = a.rot_dim >> 1;
+                const bool second = a.interleaved ? (in_part & 1) != 0 : in_part >= half;
+                const int to = a.interleaved ? (second ? -1 : 1) : (second ? -half : half);
+                const int i = a.interleaved ? in_part >> 1 : (second ? in_part - half : in_part);
+                float other = to_float(src[to]);
+                if (normed) other = other * rstd * w[from + to];
+                // (u, v) -> (u c - v s, v c + u s)
+                v = __fadd_rn(__fmul_rn(v, cos_s[i]), __fmul_rn(second ? other : -other, sin_s[i]));
             }
-            unpack8(*reinterpret_cast<const uint4*>(src), v);
-            if (normed) {
-                float w8[8];
-                load8f(w + from, w8);
-#pragma unroll
-                for (int e = 0; e < 8; ++e) v[e] = v[e] * rstd * w8[e];
-            }
-            if (turned) {
-#pragma unroll
-                for (int e = 0; e < 8; e += 2) {
-                    const int i = (in_part + e) >> 1;
-                    if (in_part + e < a.rot_dim) {
-                        const float c = cos_s[i], s = sin_s[i], x = v[e], y = v[e + 1];
-                        v[e] = __fadd_rn(__fmul_rn(x, c), __fmul_rn(-y, s));
-                        v[e + 1] = __fadd_rn(__fmul_rn(y, c), __fmul_rn(x, s));
-                    }
-                }
-            }
-            *reinterpret_cast<uint4*>(dst) = pack8(v);
-        } else {
-            float v = 0.f;
-            if (from >= 0) {
-                v = to_float(*src);
-                if (normed) v = v * rstd * w[from];
-                if (turned) {
-                    const int half = a.rot_dim >> 1;
-                    const bool second = a.interleaved ? (in_part & 1) != 0 : in_part >= half;
-                    const int to = a.interleaved ? (second ? -1 : 1) : (second ? -half : half);
-                    const int i = a.interleaved ? in_part >> 1 : (second ? in_part - half : in_part);
-                    float other = to_float(src[to]);
-                    if (normed) other = other * rstd * w[from + to];
-                    // (u, v) -> (u c - v s, v c + u s)
-                    v = __fadd_rn(__fmul_rn(v, cos_s[i]), __fmul_rn(second ? other : -other, sin_s[i]));
-                }
-            }
-            *dst = from_float<T>(v);
         }
+        *dst = from_float<T>(v);
+    }
+}
+
+// bfloat16 in runs of 8 elements (16 bytes): a block per token (without a norm the runs of a token may be spread over
+// blocks along y), R runs a thread, read once: a run's source is in registers before the angles and the sums of squares
+// are formed, and every source run serves exactly one run of the queries or keys, so the sums come from the same loads.
+template <int R>
+__global__ void __launch_bounds__(1024) heads_to_pages_bf16x8_kernel(const HeadsArgs a, unsigned per_head_inverse) {
+    pdl_launch_dependents();
+    __shared__ float cos_s[128], sin_s[128], scratch[2][32];
+    const int t = blockIdx.x, D = a.D, md = a.maps * a.d, per_head = D / 8;
+    const int q_runs = a.n_q * a.maps * per_head, kv_runs = a.n_kv * per_head, runs = q_runs + 2 * kv_runs;
+    const int run0 = blockIdx.y * blockDim.x * R + threadIdx.x;
+    int from[R], head_of[R], at[R];  // source (place in the row; -1: zeros), output head, first element in it
+#pragma unroll
+    for (int k = 0; k < R; ++k) {
+        const int run = run0 + k * blockDim.x;
+        const bool is_q = run < q_runs, is_v = run >= q_runs + kv_runs;
+        const int r = is_q ? run : (is_v ? run - q_runs - kv_runs : run - q_runs);
+        const int head = (int)__umulhi((unsigned)r, per_head_inverse), o = (r - head * per_head) * 8;
+        head_of[k] = head;
+        at[k] = o;
+        from[k] = -1;
+        if (run < runs) {
+            if (is_q) {
+                const int m = a.maps == 1 ? 0 : (head & 1), h = a.maps == 1 ? head : head >> 1, in_part = o - m * a.d;
+                if (in_part >= 0 && in_part < a.d) from[k] = h * md + o;
+            } else if (is_v) {
+                if (o < a.dv) from[k] = a.v_col + head * a.dv + o;
+            } else if (o < md) {
+                from[k] = a.k_col + head * md + o;
+            }
+        }
+    }
+    pdl_wait();
+    const bf16* row = reinterpret_cast<const bf16*>(a.rows) + (int64_t)t * a.row_stride;
+    uint4 raw[R];
+#pragma unroll
+    for (int k = 0; k < R; ++k) raw[k] = from[k] >= 0 ? *reinterpret_cast<const uint4*>(row + from[k]) : make_uint4(0u, 0u, 0u, 0u);
+    const float pos = (float)a.positions[t];
+    int64_t slot = (a.slots && a.kv) ? (int64_t)a.slots[t] : -1;
+    for (int i = threadIdx.x; i < a.rot_dim / 2; i += blockDim.x) sincosf(__fmul_rn(pos, a.inv_freq[i]), &sin_s[i], &cos_s[i]);
+    if (slot >= a.pool_slots) {
+        if (threadIdx.x == 0 && blockIdx.y == 0) atomicOr(a.err, SS_ERR_SLOT_RANGE);
+        slot = -1;
+    }
+    float q_rstd = 1.f, k_rstd = 1.f;
+    if (a.q_weight) {
+        float sq = 0.f, sk = 0.f;
+#pragma unroll
+        for (int k = 0; k < R; ++k) {
+            const int run = run0 + k * blockDim.x;
+            if (run >= q_runs + kv_runs) continue;
+            float v[8], s = 0.f;
+            unpack8(raw[k], v);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) s = fmaf(v[e], v[e], s);
+            if (run < q_runs) sq += s; else sk += s;
+        }
+        sq = warp_sum(sq);
+        sk = warp_sum(sk);
+        const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n_warps = (blockDim.x + 31) >> 5;
+        if (lane == 0) { scratch[0][warp] = sq; scratch[1][warp] = sk; }
+        __syncthreads();
+        q_rstd = 1.0f / sqrtf(warp_sum(lane < n_warps ? scratch[0][lane] : 0.f) / (float)(a.n_q * md) + a.eps);
+        k_rstd = 1.0f / sqrtf(warp_sum(lane < n_warps ? scratch[1][lane] : 0.f) / (float)(a.n_kv * md) + a.eps);
+    } else {
+        __syncthreads();
+    }
+    const int page_size = a.page_size, page = slot >= 0 ? (int)slot / page_size : 0, off = slot >= 0 ? (int)slot - page * page_size : 0;
+#pragma unroll
+    for (int k = 0; k < R; ++k) {
+        const int run = run0 + k * blockDim.x;
+        const bool is_q = run < q_runs, is_v = run >= q_runs + kv_runs;
+        if (run >= runs || (!is_q && slot < 0)) continue;
+        bf16* dst;
+        if (is_q) dst = reinterpret_cast<bf16*>(a.q_out) + (int64_t)t * a.n_q * a.maps * D + run * 8;
+        else dst = reinterpret_cast<bf16*>(a.kv) + ((((int64_t)page * 2 + (is_v ? 1 : 0)) * a.n_kv + head_of[k]) * page_size + off) * D + at[k];
+        const int second = a.maps == 2 && (is_q ? (head_of[k] & 1) : at[k] >= a.d) ? a.d : 0, in_part = at[k] - second;
+        const bool turned = in_part < a.rot_dim;
+        if (from[k] < 0 || is_v || (!a.q_weight && !turned)) {
+            *reinterpret_cast<uint4*>(dst) = raw[k];
+            continue;
+        }
+        float v[8];
+        unpack8(raw[k], v);
+        if (a.q_weight) {
+            float w8[8];
+            load8f(is_q ? a.q_weight + from[k] : a.k_weight + from[k] - a.k_col, w8);
+            const float rstd = is_q ? q_rstd : k_rstd;
+#pragma unroll
+            for (int e = 0; e < 8; ++e) v[e] = v[e] * rstd * w8[e];
+        }
+        if (turned) {
+#pragma unroll
+            for (int e = 0; e < 8; e += 2) {
+                if (in_part + e < a.rot_dim) {
+                    const int i = (in_part + e) >> 1;
+                    const float c = cos_s[i], s = sin_s[i], x = v[e], y = v[e + 1];
+                    v[e] = __fadd_rn(__fmul_rn(x, c), __fmul_rn(-y, s));
+                    v[e + 1] = __fadd_rn(__fmul_rn(y, c), __fmul_rn(x, s));
+                }
+            }
+        }
+        *reinterpret_cast<uint4*>(dst) = pack8(v);
     }
 }
 
@@ -194,7 +259,7 @@ extern "C" int ss_heads_to_pages(const void* rows, int64_t row_stride, const int
                                  int rot_dim, int interleaved, float eps, int page_size, int64_t num_pages, int dtype, int* err,
                                  cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
-    if (n_q < 1 || n_kv < 0 || (maps != 1 && maps != 2) || d < 1 || dv < 1 || D % 8 != 0 || maps * d > D || dv > D || rot_dim < 0 ||
+    if (n_q < 1 || n_kv < 0 || (maps != 1 && maps != 2) || d < 1 || dv < 1 || D < 16 || D % 8 != 0 || maps * d > D || dv > D || rot_dim < 0 ||
         rot_dim > d || rot_dim % 2 || rot_dim > 256 || (rot_dim > 0 && !inv_freq) || (!q_weight != !k_weight && n_kv > 0) || page_size < 1)
         return (int)cudaErrorInvalidValue;
     HeadsArgs a;
@@ -202,17 +267,32 @@ extern "C" int ss_heads_to_pages(const void* rows, int64_t row_stride, const int
     a.q_weight = q_weight; a.k_weight = k_weight; a.q_out = q_out; a.kv = kv; a.n_q = n_q; a.n_kv = n_kv; a.maps = maps;
     a.d = d; a.dv = dv; a.D = D; a.k_col = k_col; a.v_col = v_col; a.rot_dim = rot_dim; a.interleaved = interleaved;
     a.page_size = page_size; a.eps = eps; a.pool_slots = num_pages * page_size; a.err = err;
+    if (a.pool_slots > 0x7fffffff) return (int)cudaErrorInvalidValue;  // slots are 32-bit
     const bool wide = dtype == SS_BF16 && (interleaved || rot_dim == 0) && d % 8 == 0 && dv % 8 == 0 && k_col % 8 == 0 &&
                       v_col % 8 == 0 && row_stride % 8 == 0 && ((uintptr_t)rows & 15) == 0 && ((uintptr_t)q_out & 15) == 0 &&
                       ((uintptr_t)kv & 15) == 0 && ((uintptr_t)q_weight & 15) == 0 && ((uintptr_t)k_weight & 15) == 0;
-    if (wide) {
-        const int runs = (n_q * maps + 2 * n_kv) * (D / 8);
-        const int threads = runs >= 1024 ? 512 : (runs >= 512 ? 256 : 128);
-        ss_launch(heads_to_pages_kernel<bf16, 8>, dim3(n_tokens), dim3(threads), 0, stream, a);
+    const int runs = (n_q * maps + 2 * n_kv) * (D / 8);
+    // few tokens want a short chain per thread, many tokens several loads in flight per thread and several blocks an SM
+    const bool many = n_tokens >= 2 * ss_sm_count();
+    if (wide && runs <= 4 * 1024) {
+        const unsigned inverse = (unsigned)((((uint64_t)1 << 32) + D / 8 - 1) / (D / 8));  // exact for the small numbers here (D >= 16)
+        if (!q_weight) {  // nothing is summed over the token: its runs over as many blocks as keep one run a thread
+            const int threads = runs >= 256 ? 256 : 128;
+            if (many && runs > threads)
+                ss_launch(heads_to_pages_bf16x8_kernel<2>, dim3(n_tokens, (runs + 2 * threads - 1) / (2 * threads)), dim3(threads), 0, stream, a, inverse);
+            else
+                ss_launch(heads_to_pages_bf16x8_kernel<1>, dim3(n_tokens, (runs + threads - 1) / threads), dim3(threads), 0, stream, a, inverse);
+        } else {
+            const int r = runs <= 1024 && !many ? 1 : (runs <= 512 || (runs <= 2048 && !many) ? 2 : 4);
+            const int threads = ((runs + r - 1) / r + 31) / 32 * 32;
+            if (r == 1) ss_launch(heads_to_pages_bf16x8_kernel<1>, dim3(n_tokens), dim3(threads), 0, stream, a, inverse);
+            else if (r == 2) ss_launch(heads_to_pages_bf16x8_kernel<2>, dim3(n_tokens), dim3(threads), 0, stream, a, inverse);
+            else ss_launch(heads_to_pages_bf16x8_kernel<4>, dim3(n_tokens), dim3(threads), 0, stream, a, inverse);
+        }
     } else if (dtype == SS_BF16) {
-        ss_launch(heads_to_pages_kernel<bf16, 1>, dim3(n_tokens), dim3(256), 0, stream, a);
+        ss_launch(heads_to_pages_kernel<bf16>, dim3(n_tokens), dim3(256), 0, stream, a);
     } else {
-        ss_launch(heads_to_pages_kernel<float, 1>, dim3(n_tokens), dim3(256), 0, stream, a);
+        ss_launch(heads_to_pages_kernel<float>, dim3(n_tokens), dim3(256), 0, stream, a);
     }
     return SS_LAUNCH_CHECK();
 }
@@ -276,7 +356,9 @@ struct BranchArgs {
     float mult, y_eps, eps;
 };
 
-template <typename T, int VEC>
+// EARLY (few rows): the weights are in registers before the kernels in front are complete; with many rows they are read
+// where they are used, which leaves room for more blocks on an SM.
+template <typename T, int VEC, bool EARLY>
 __global__ void __launch_bounds__(1024) branch_norm_kernel(const BranchArgs a) {
     pdl_launch_dependents();
     __shared__ float scratch[2][32];
@@ -285,7 +367,7 @@ __global__ void __launch_bounds__(1024) branch_norm_kernel(const BranchArgs a) {
         const int j = threadIdx.x * 8;
         const bool on = j < hidden;
         float wy[8], w[8];
-        if (on) {  // weights do not depend on the kernels in front
+        if (EARLY && on) {  // weights do not depend on the kernels in front
             load8f(a.weight + j, w);
             if (a.y) load8f(a.y_weight + j, wy);
         }
@@ -309,6 +391,7 @@ __global__ void __launch_bounds__(1024) branch_norm_kernel(const BranchArgs a) {
             float anchor[8];
             if (on && a.anchor) load8f(a.anchor + src * hidden + j, anchor);
             const float f = 1.0f / sqrtf(block_sum_once(ss, scratch[0]) / (float)hidden + a.y_eps);
+            if (!EARLY && on) load8f(a.y_weight + j, wy);
             if (on) {
 #pragma unroll
                 for (int e = 0; e < 8; ++e) v[e] = fmaf(a.mult, y[e] * f * wy[e], v[e]);
@@ -323,6 +406,7 @@ __global__ void __launch_bounds__(1024) branch_norm_kernel(const BranchArgs a) {
 #pragma unroll
         for (int e = 0; e < 8; ++e) ss = fmaf(v[e], v[e], ss);
         const float f = 1.0f / sqrtf(block_sum_once(ss, scratch[1]) / (float)hidden + a.eps);
+        if (!EARLY && on) load8f(a.weight + j, w);
         if (on) {
 #pragma unroll
             for (int e = 0; e < 8; ++e) v[e] = v[e] * f * w[e];
@@ -376,12 +460,14 @@ extern "C" int ss_branch_norm(float* residual, const void* y, const float* y_wei
     const bool aligned = (((uintptr_t)residual | (uintptr_t)y | (uintptr_t)y_weight | (uintptr_t)anchor | (uintptr_t)weight | (uintptr_t)out) & 15) == 0;
     if (hidden % 8 == 0 && hidden <= 8192 && aligned) {
         const dim3 block((hidden / 8 + 31) / 32 * 32);
-        if (dtype == SS_BF16) ss_launch(branch_norm_kernel<bf16, 8>, dim3(n_rows), block, 0, stream, a);
-        else ss_launch(branch_norm_kernel<float, 8>, dim3(n_rows), block, 0, stream, a);
+        const bool many = n_rows >= 2 * ss_sm_count();
+        if (dtype == SS_BF16 && many) ss_launch(branch_norm_kernel<bf16, 8, false>, dim3(n_rows), block, 0, stream, a);
+        else if (dtype == SS_BF16) ss_launch(branch_norm_kernel<bf16, 8, true>, dim3(n_rows), block, 0, stream, a);
+        else ss_launch(branch_norm_kernel<float, 8, true>, dim3(n_rows), block, 0, stream, a);
     } else {
         const dim3 block(hidden >= 2048 ? 512 : (hidden >= 512 ? 256 : 128));
-        if (dtype == SS_BF16) ss_launch(branch_norm_kernel<bf16, 1>, dim3(n_rows), block, 0, stream, a);
-        else ss_launch(branch_norm_kernel<float, 1>, dim3(n_rows), block, 0, stream, a);
+        if (dtype == SS_BF16) ss_launch(branch_norm_kernel<bf16, 1, false>, dim3(n_rows), block, 0, stream, a);
+        else ss_launch(branch_norm_kernel<float, 1, false>, dim3(n_rows), block, 0, stream, a);
     }
     return SS_LAUNCH_CHECK();
 }

@@ -121,7 +121,7 @@ class LatentAttention(Mixer):
         return n * self.o_weight.element_size()
 
     def capture_variant(self, longest: int, plan: object = None) -> object:
-        return None  # layers with sinks run one form of the decode kernel
+        return None  # captured steps run one form of the decode kernel, however long the contexts
 
     def capture_group(self) -> object:
         return ("latent_attention",)

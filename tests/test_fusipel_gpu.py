@@ -402,7 +402,6 @@ def test_gated_unit_with_the_tanh_form_of_gelu(dtype, n, h, ff):
     """The library product with the activation kernel, the streaming product of decode steps and the two-SM product of
     long portions, the latter two with the unit in their epilogues."""
     from slipstream_b200.parts import GELU_TANH, GatedFeedForward, Runtime
-    from slipstream_b200.parts.base import WeightSpec  # noqa: F401
     g = torch.Generator().manual_seed(n)
     w = {f"m.{r}": (torch.randn(a, b, generator=g) * s * b ** -0.5).to(dtype) for r, a, b, s in
          (("gate", ff, h, 3.0), ("up", ff, h, 1.0), ("down", h, ff, 1.0))}
