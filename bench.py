@@ -371,6 +371,7 @@ def kernel_tables(which: str) -> int:
 # is compared, and the weights of either model are still larger than L2.
 COMPARE_SIZES = {
     "0.5b": dict(vocab=151936, width=896, heads=14, kv_heads=2, dim=64, ff=4864, layers=8),
+    "1.5b": dict(vocab=151936, width=1536, heads=12, kv_heads=2, dim=128, ff=8960, layers=8),
     "7b": dict(vocab=152064, width=3584, heads=28, kv_heads=4, dim=128, ff=18944, layers=8),
     "14b": dict(vocab=152064, width=5120, heads=40, kv_heads=8, dim=128, ff=13824, layers=6),
 }
@@ -1364,6 +1365,7 @@ def run_compare_fusipel(args) -> int:
         with torch.cuda.graph(graph):
             for i in range(copies * 2):
                 run(i % copies)
+        time.sleep(0.25)  # a burst of launches by itself: the clock falls behind seconds of matrix products
         times = []
         for _ in range(8):
             torch.cuda.synchronize()
@@ -1527,7 +1529,7 @@ def main() -> int:
     ap.add_argument("--window", type=int, default=4096, help="--compare sarudra: positions of the sliding window")
     ap.add_argument("--compare", choices=["fokedra", "sarudra", "bezutar", "lakadra", "fusipel"], default=None,
                     help="time another decoder design beside the Qwen2.5 decoder at equal layer sizes instead")
-    ap.add_argument("--sizes", default="", help="--compare: which of 0.5b,7b,14b (default: all)")
+    ap.add_argument("--sizes", default="", help="--compare: which of 0.5b,1.5b,7b,14b (default: all)")
     ap.add_argument("--mask-chunk", type=int, default=8192, help="--compare: positions per attention chunk")
     ap.add_argument("--streams", type=int, default=2, help="--compare: residual streams")
     ap.add_argument("--skip-qwen2", action="store_true", help="--compare: time the other design only")
