@@ -15,16 +15,16 @@ extern "C" int ss_attn_simt(const void* q, int64_t q_stride, void* out, int64_t 
                             const int32_t* tile_req, const int32_t* tile_q0, int n_tiles,
                             const int32_t* q_start, const int32_t* seq_lens, int n_q, int n_kv,
                             int page_size, int64_t num_pages, float scale, int window, int dtype,
-                            const void* gate, int* err, cudaStream_t stream, float softcap, const float* sinks, int keep) {
+                            const void* gate, int* err, cudaStream_t stream, float softcap, const float* sinks, int keep, int across) {
     if (n_tiles <= 0) return 0;
-    if (keep < 0 || (keep > 0 && window <= 0)) return (int)cudaErrorInvalidValue;
+    if (keep < 0 || (keep > 0 && window <= 0) || (across && gate)) return (int)cudaErrorInvalidValue;
     if (dtype == SS_BF16)
         return launch_attn_simt<bf16, HEAD_DIM>(q, q_stride, out, out_stride, kv, block_tables, max_blocks,
                                                 tile_req, tile_q0, n_tiles, q_start, seq_lens, n_q, n_kv,
-                                                page_size, num_pages, scale, window, gate, err, stream, softcap, sinks, keep);
+                                                page_size, num_pages, scale, window, gate, err, stream, softcap, sinks, keep, across);
     return launch_attn_simt<float, HEAD_DIM>(q, q_stride, out, out_stride, kv, block_tables, max_blocks,
                                              tile_req, tile_q0, n_tiles, q_start, seq_lens, n_q, n_kv,
-                                             page_size, num_pages, scale, window, gate, err, stream, softcap, sinks, keep);
+                                             page_size, num_pages, scale, window, gate, err, stream, softcap, sinks, keep, across);
 }
 
 #include "attention_mma.cuh"
@@ -48,19 +48,19 @@ extern "C" int ss_attn_prefill_mma(const void* q, int64_t q_stride, void* out, i
                                    const int32_t* q_start, const int32_t* seq_lens, int n_q, int n_kv,
                                    int page_size, int64_t num_pages, float scale, int window, const void* gate, int* err,
                                    cudaStream_t stream, float softcap, const float* sinks, int keep, int out_f32, int diff_on,
-                                   float diff_lam, float diff_mult, float diff_eps, int diff_dim) {
+                                   float diff_lam, float diff_mult, float diff_eps, int diff_dim, int across) {
     if (n_tiles <= 0) return 0;
     const DiffPair diff = {diff_on, diff_lam, diff_mult, diff_eps, diff_dim};
     if (keep < 0 || (keep > 0 && window <= 0) || !diff_pair_fits(diff, n_q, n_kv, out_stride, out) || (diff_on && (gate || out_f32)) ||
-        (out_f32 && gate))
+        (out_f32 && gate) || (across && (diff_on || gate)))
         return (int)cudaErrorInvalidValue;
     constexpr int smem = mma_smem_bytes<HEAD_DIM>();
     static SsPerDevice opted;
     if (int rc_smem = ss_opt_in_smem(attn_prefill_mma<HEAD_DIM>, smem, opted)) return rc_smem;
-    dim3 grid(n_tiles, n_kv);
+    dim3 grid(n_tiles, across ? n_kv * n_kv : n_kv);
     ss_launch(attn_prefill_mma<HEAD_DIM>, dim3(grid), dim3(MMA_THREADS), smem, stream, 
         (const bf16*)q, q_stride, (bf16*)out, out_stride, (const bf16*)kv, block_tables, max_blocks, tile_req,
-        tile_row0, q_start, seq_lens, n_q, n_kv, page_size, num_pages, scale, window, err, (const bf16*)gate, softcap, sinks, keep, out_f32, diff);
+        tile_row0, q_start, seq_lens, n_q, n_kv, page_size, num_pages, scale, window, err, (const bf16*)gate, softcap, sinks, keep, out_f32, diff, across);
     return SS_LAUNCH_CHECK();
 }
 
@@ -78,8 +78,8 @@ extern "C" int ss_attn_decode_mma(const void* q, int64_t q_stride, void* out, in
                                   int page_size, int64_t num_pages, float scale, int window, int n_slices,
                                   const float* inv_freq, int rot_dim, int fused, float* part_o, float* part_lse, int* counters,
                                   const void* gate, int* err, cudaStream_t stream, float softcap, const float* sinks, int keep,
-                                  int out_f32) {
-    if (keep < 0 || (keep > 0 && window <= 0) || (out_f32 && gate)) return (int)cudaErrorInvalidValue;
+                                  int out_f32, int across) {
+    if (keep < 0 || (keep > 0 && window <= 0) || (out_f32 && gate) || (across && (fused || gate))) return (int)cudaErrorInvalidValue;
     if (n_requests <= 0) return 0;
     const int cluster = n_slices >= 2 && n_slices <= 8;  // the slices are combined through shared memory
     if (fused && (rot_dim < 0 || rot_dim > HEAD_DIM || rot_dim % 2 || (rot_dim > 0 && !inv_freq))) return (int)cudaErrorInvalidValue;
@@ -89,15 +89,15 @@ extern "C" int ss_attn_decode_mma(const void* q, int64_t q_stride, void* out, in
     static SsPerDevice opted;
     if (int rc_smem = ss_opt_in_smem(attn_decode_mma<HEAD_DIM>, smem, opted)) return rc_smem;
     const int G = n_q / n_kv;
-    dim3 grid(n_requests, n_kv * ((G + 15) / 16), n_slices);
+    dim3 grid(n_requests, (across ? n_kv * n_kv : n_kv) * ((G + 15) / 16), n_slices);
     if (cluster)
         ss_launch_cluster(attn_decode_mma<HEAD_DIM>, dim3(grid), dim3(MMA_THREADS), smem, stream, n_slices,
             (const bf16*)q, q_stride, (bf16*)out, out_stride, (const bf16*)kv, block_tables, max_blocks, q_start,
-            seq_lens, n_q, n_kv, page_size, num_pages, scale, window, n_slices, 1, inv_freq, rot_dim, fused, part_o, part_lse, counters, err, (const bf16*)gate, softcap, sinks, keep, out_f32);
+            seq_lens, n_q, n_kv, page_size, num_pages, scale, window, n_slices, 1, inv_freq, rot_dim, fused, part_o, part_lse, counters, err, (const bf16*)gate, softcap, sinks, keep, out_f32, across);
     else
         ss_launch(attn_decode_mma<HEAD_DIM>, dim3(grid), dim3(MMA_THREADS), smem, stream,
             (const bf16*)q, q_stride, (bf16*)out, out_stride, (const bf16*)kv, block_tables, max_blocks, q_start,
-            seq_lens, n_q, n_kv, page_size, num_pages, scale, window, n_slices, 0, inv_freq, rot_dim, fused, part_o, part_lse, counters, err, (const bf16*)gate, softcap, sinks, keep, out_f32);
+            seq_lens, n_q, n_kv, page_size, num_pages, scale, window, n_slices, 0, inv_freq, rot_dim, fused, part_o, part_lse, counters, err, (const bf16*)gate, softcap, sinks, keep, out_f32, across);
     return SS_LAUNCH_CHECK();
 }
 
@@ -116,16 +116,16 @@ extern "C" int ss_attn_prefill_tc5(const void* q, int64_t q_stride, int n_tokens
                                    const int32_t* q_start, const int32_t* seq_lens, int n_q, int n_kv, int page_size,
                                    int64_t num_pages, float scale, int splits, int span, int* err, cudaStream_t stream,
                                    float softcap, const float* sinks, int keep, int out_f32, int diff_on, float diff_lam,
-                                   float diff_mult, float diff_eps, int diff_dim) {
+                                   float diff_mult, float diff_eps, int diff_dim, int across) {
     if (n_tiles <= 0) return 0;
     const DiffPair diff = {diff_on, diff_lam, diff_mult, diff_eps, diff_dim};
-    if (keep < 0 || (keep > 0 && span <= 0) || !diff_pair_fits(diff, n_q, n_kv, out_stride, out) || (diff_on && (splits != 1 || out_f32)) ||
+    if (keep < 0 || (keep > 0 && span <= 0) || !diff_pair_fits(diff, n_q, n_kv, out_stride, out) || (diff_on && (splits != 1 || out_f32 || across)) ||
         (out_f32 && (out_stride % 4 || ((uintptr_t)out & 15))))
         return (int)cudaErrorInvalidValue;
     const int G = n_q / n_kv;
     if (G < 1 || G > 128 || page_size % 8 != 0 || 64 % page_size != 0 || q_stride % 8 != 0) return -3003;
     if (splits != 1 && splits != 2 && splits != 4 && splits != 8) return -3004;
-    const int TOK = 128 / G;
+    const int TOK = 128 / G, n_u = across ? n_kv * n_kv : n_kv;
     CUtensorMap map_q, map_kv;
     int rc = fa::make_map3(&map_q, q, HEAD_DIM, (uint64_t)n_q, (uint64_t)n_tokens, (uint64_t)HEAD_DIM * 2,
                            (uint64_t)q_stride * 2, 64, (uint32_t)G, (uint32_t)TOK);
@@ -137,15 +137,15 @@ extern "C" int ss_attn_prefill_tc5(const void* q, int64_t q_stride, int n_tokens
     a.out = (bf16*)out; a.out_stride = out_stride; a.block_tables = block_tables; a.max_blocks = max_blocks;
     a.tile_req = tile_req; a.tile_tok0 = tile_tok0; a.q_start = q_start; a.seq_lens = seq_lens;
     a.n_q = n_q; a.n_kv = n_kv; a.page_size = page_size; a.num_pages = num_pages; a.scale = scale; a.err = err;
-    a.span = span; a.softcap = softcap; a.sinks = sinks; a.keep = keep; a.out_f32 = out_f32; a.diff = diff;
+    a.span = span; a.softcap = softcap; a.sinks = sinks; a.keep = keep; a.out_f32 = out_f32; a.across = across; a.diff = diff;
     constexpr int smem = fa::smem_bytes<HEAD_DIM>();
     static SsPerDevice opted;
     if (int rc_smem = ss_opt_in_smem(fa::attn_prefill_tc5<HEAD_DIM>, smem, opted)) return rc_smem;
     // splits > 1: the key tiles of every query tile are shared by a thread-block cluster of that many blocks
     if (splits > 1)
-        ss_launch_cluster(fa::attn_prefill_tc5<HEAD_DIM>, dim3(n_tiles * n_kv, 1, splits), dim3(FA_THREADS), smem, stream, splits, map_q, map_kv, a);
+        ss_launch_cluster(fa::attn_prefill_tc5<HEAD_DIM>, dim3(n_tiles * n_u, 1, splits), dim3(FA_THREADS), smem, stream, splits, map_q, map_kv, a);
     else
-        ss_launch(fa::attn_prefill_tc5<HEAD_DIM>, dim3(n_tiles * n_kv), dim3(FA_THREADS), smem, stream, map_q, map_kv, a);
+        ss_launch(fa::attn_prefill_tc5<HEAD_DIM>, dim3(n_tiles * n_u), dim3(FA_THREADS), smem, stream, map_q, map_kv, a);
     return SS_LAUNCH_CHECK();
 }
 
@@ -174,9 +174,9 @@ extern "C" int ss_attn_decode_tma(const void* q, int64_t q_stride, void* out, in
                                   int page_size, int64_t num_pages, float scale, int window, int n_slices,
                                   const float* inv_freq, int rot_dim, int fused, float* part_o,
                                   float* part_lse, int* counters, int stages, const void* gate, int* err, cudaStream_t stream,
-                                  float softcap, const float* sinks, int keep, int out_f32) {
+                                  float softcap, const float* sinks, int keep, int out_f32, int across) {
     if (n_requests <= 0) return 0;
-    if (keep < 0 || (keep > 0 && window <= 0) || (out_f32 && gate)) return (int)cudaErrorInvalidValue;
+    if (keep < 0 || (keep > 0 && window <= 0) || (out_f32 && gate) || (across && (fused || gate))) return (int)cudaErrorInvalidValue;
     if (page_size % 8 != 0 || 64 % page_size != 0) return -3003;
     // up to 8 slices: one cluster; a multiple of 8 beyond: clusters of 8 whose results meet in scratch memory;
     // any other count: single blocks and scratch memory
@@ -194,9 +194,9 @@ extern "C" int ss_attn_decode_tma(const void* q, int64_t q_stride, void* out, in
     a.n_q = n_q; a.n_kv = n_kv; a.page_size = page_size; a.num_pages = num_pages; a.scale = scale; a.softcap = softcap; a.window = window;
     a.n_slices = n_slices; a.cluster = cluster; a.inv_freq = inv_freq; a.rot_dim = rot_dim; a.fused = fused;
     a.part_o = part_o; a.part_lse = part_lse; a.counters = counters; a.err = err; a.gate = (const bf16*)gate;
-    a.sinks = sinks; a.keep = keep; a.out_f32 = out_f32;
+    a.sinks = sinks; a.keep = keep; a.out_f32 = out_f32; a.across = across;
     const int G = n_q / n_kv;
-    dim3 grid(n_requests, n_kv * ((G + 15) / 16), n_slices);
+    dim3 grid(n_requests, (across ? n_kv * n_kv : n_kv) * ((G + 15) / 16), n_slices);
     // the usual decode step (rotation inside, no window, one cluster, a rotary size in steps of 16) has kernels of its own
     const bool usual = fused && window == 0 && gate == nullptr && sinks == nullptr && !out_f32 && softcap <= 0.f && cluster == n_slices && cluster > 1 && rot_dim > 0 && rot_dim % 16 == 0;
     const int smem3 = decode_tma_smem_bytes<HEAD_DIM, 3>(G < 16 ? G : 16, cluster);
@@ -281,7 +281,7 @@ extern "C" int ss_attn_decode_noalloc(const void* q, int64_t q_stride, void* out
     dim3 grid(n_requests, n_kv * ((G + 15) / 16), n_slices);
     ss_launch(attn_decode_mma<HEAD_DIM>, dim3(grid), dim3(MMA_THREADS), smem, stream, 
         (const bf16*)q, q_stride, (bf16*)out, out_stride, (const bf16*)kv, block_tables, max_blocks, q_start,
-        seq_lens, n_q, n_kv, page_size, num_pages, scale, window, n_slices, 0, (const float*)nullptr, 0, 0, part_o, part_lse, counters, err, (const bf16*)nullptr, 0.f, (const float*)nullptr, 0, 0);
+        seq_lens, n_q, n_kv, page_size, num_pages, scale, window, n_slices, 0, (const float*)nullptr, 0, 0, part_o, part_lse, counters, err, (const bf16*)nullptr, 0.f, (const float*)nullptr, 0, 0, 0);
     return SS_LAUNCH_CHECK();
 }
 

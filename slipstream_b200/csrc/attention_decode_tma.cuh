@@ -65,6 +65,7 @@ struct DecodeTmaArgs {
     const float* sinks;  // float32 [n_q] or null: one more term exp(sinks[h]) in the denominator of head h's softmax
     int keep;  // with a sliding window: the request's first `keep` keys stay visible (common.cuh: key_tiles)
     int out_f32;  // `out` is float32
+    int across;  // common.cuh: head_pair
 };
 
 template <int D, int NS = DT_STAGES>
@@ -133,7 +134,10 @@ attn_decode_tma(const __grid_constant__ CUtensorMap map_kv, const DecodeTmaArgs 
     const int keep = FORM == 0 ? a.keep : 0;
     const bool fused = FORM == 0 ? a.fused != 0 : true;
     const int G = n_q / n_kv, hblocks = (G + 15) / 16;
-    const int r = blockIdx.x, kvh = blockIdx.y / hblocks, g0 = (blockIdx.y % hblocks) * 16;
+    const int r = blockIdx.x, u = blockIdx.y / hblocks, g0 = (blockIdx.y % hblocks) * 16;
+    const bool across = FORM == 0 ? a.across != 0 : false;
+    const HeadPair hp = head_pair(u, n_kv, across);
+    const int kvh = hp.key, n_out = across ? n_q * n_kv : n_q;
     const int heads_here = min(16, G - g0);
     const int slice = blockIdx.z;
     // slices per cluster, clusters, this one
@@ -222,10 +226,16 @@ attn_decode_tma(const __grid_constant__ CUtensorMap map_kv, const DecodeTmaArgs 
                         page = -1;
                     }
                     if (page < 0) page = spare;
-                    fa::tma_load_3d_once(Ks + h * (MMA_BN * 64) + p * page_size * 64, &map_kv, h * 64, 0,
-                                         (int)((page * 2 + 0) * n_kv + kvh), &full[bar_of(i)], once);
-                    fa::tma_load_3d_once(Vs + h * (MMA_BN * 64) + p * page_size * 64, &map_kv, h * 64, 0,
-                                         (int)((page * 2 + 1) * n_kv + kvh), &full[bar_of(i)], once);
+                    bf16* kd = Ks + h * (MMA_BN * 64) + p * page_size * 64;
+                    bf16* vd = Vs + h * (MMA_BN * 64) + p * page_size * 64;
+                    const int kz = (int)((page * 2 + 0) * n_kv + kvh), vz = (int)((page * 2 + 1) * n_kv + hp.value);
+                    if (across) {  // the same tiles are read by n_kv blocks: they should stay in L2 meanwhile
+                        fa::tma_load_3d(kd, &map_kv, h * 64, 0, kz, &full[bar_of(i)]);
+                        fa::tma_load_3d(vd, &map_kv, h * 64, 0, vz, &full[bar_of(i)]);
+                    } else {
+                        fa::tma_load_3d_once(kd, &map_kv, h * 64, 0, kz, &full[bar_of(i)], once);
+                        fa::tma_load_3d_once(vd, &map_kv, h * 64, 0, vz, &full[bar_of(i)], once);
+                    }
                 }
             }
         }
@@ -430,7 +440,7 @@ attn_decode_tma(const __grid_constant__ CUtensorMap map_kv, const DecodeTmaArgs 
         Fm[tid] = mm != -INFINITY ? fast_exp2(Mm[tid] - mm) : 0.f;
     }
     __syncthreads();
-    const int64_t head0 = (int64_t)kvh * G + g0;
+    const int64_t head0 = (int64_t)u * G + g0;  // of the output
     const int rank = cs > 1 ? (int)cluster_rank() : 0;
     for (int idx = tid; idx < heads_here * (D / 2); idx += DT_THREADS) {
         const int row = idx / (D / 2), d = (idx - row * (D / 2)) * 2;
@@ -460,10 +470,10 @@ attn_decode_tma(const __grid_constant__ CUtensorMap map_kv, const DecodeTmaArgs 
                 }
                 store_out2(a, (int64_t)row_q * a.out_stride + (head0 + row) * D + d, v0, v1);
             } else {
-                float* po = a.part_o + (((int64_t)r * n_q + head0 + row) * n_groups + group) * D + d;
+                float* po = a.part_o + (((int64_t)r * n_out + head0 + row) * n_groups + group) * D + d;
                 po[0] = acc0 * inv;
                 po[1] = acc1 * inv;
-                if (d == 0) a.part_lse[((int64_t)r * n_q + head0 + row) * n_groups + group] = ll > 0.f ? mm + log2f(ll) : -INFINITY;
+                if (d == 0) a.part_lse[((int64_t)r * n_out + head0 + row) * n_groups + group] = ll > 0.f ? mm + log2f(ll) : -INFINITY;
             }
         }
     }
@@ -501,10 +511,10 @@ attn_decode_tma(const __grid_constant__ CUtensorMap map_kv, const DecodeTmaArgs 
                 if (FORM == 0) store_out2(a, (int64_t)row_q * a.out_stride + (head0 + row) * D + d, v0, v1);
                 else *reinterpret_cast<__nv_bfloat162*>(a.out + (int64_t)row_q * a.out_stride + (head0 + row) * D + d) = __floats2bfloat162_rn(v0, v1);
             } else {  // several clusters share the keys of this head block: the cluster's result goes to scratch
-                float* po = a.part_o + (((int64_t)r * n_q + head0 + row) * n_groups + group) * D + d;
+                float* po = a.part_o + (((int64_t)r * n_out + head0 + row) * n_groups + group) * D + d;
                 po[0] = acc0 * inv;
                 po[1] = acc1 * inv;
-                if (d == 0) a.part_lse[((int64_t)r * n_q + head0 + row) * n_groups + group] = den > 0.f ? mx + log2f(den) : -INFINITY;
+                if (d == 0) a.part_lse[((int64_t)r * n_out + head0 + row) * n_groups + group] = den > 0.f ? mx + log2f(den) : -INFINITY;
             }
         }
         if (n_groups == 1) return;
@@ -526,7 +536,7 @@ attn_decode_tma(const __grid_constant__ CUtensorMap map_kv, const DecodeTmaArgs 
     float* W = reinterpret_cast<float*>(base);  // [16][n_groups]
     for (int idx = tid; idx < heads_here * n_groups; idx += DT_THREADS) {
         const int row = idx / n_groups, sl = idx - row * n_groups;
-        W[row * n_groups + sl] = __ldcg(a.part_lse + ((int64_t)r * n_q + head0 + row) * n_groups + sl);
+        W[row * n_groups + sl] = __ldcg(a.part_lse + ((int64_t)r * n_out + head0 + row) * n_groups + sl);
     }
     __syncthreads();
     if (tid < heads_here) {
@@ -544,7 +554,7 @@ attn_decode_tma(const __grid_constant__ CUtensorMap map_kv, const DecodeTmaArgs 
     __syncthreads();
     for (int idx = tid; idx < heads_here * D; idx += DT_THREADS) {
         const int row = idx / D, d = idx - row * D;
-        const float* po = a.part_o + ((int64_t)r * n_q + head0 + row) * n_groups * D + d;
+        const float* po = a.part_o + ((int64_t)r * n_out + head0 + row) * n_groups * D + d;
         const float* w = W + row * n_groups;
         float acc = 0.f;
 #pragma unroll 8

@@ -17,6 +17,7 @@
 // are float32 (:64-88); with out_f32 the heads' outputs are written as float32, with `diff` (prefill) the two maps of a
 // differential head are combined where they are written; probabilities are rounded to
 // bfloat16 for the second product as the reference's `.to(query.dtype)` does.
+// `across`: common.cuh, head_pair.
 // kv layout: [page][2][kv head][offset in page][D].
 #pragma once
 
@@ -88,15 +89,15 @@ __device__ __forceinline__ TableRef stage_table(int32_t* smem_table, const int32
 
 // Stage keys [k0, k0 + 64) of one kv head: K rows to Ks, V rows to Vs (row stride D + 8).
 // Rows outside [lo, hi] (keys below `keep` count as inside) or without a page are zero-filled; the row of key `skip`
-// is left alone.
+// is left alone.  The values are those of kv head kvh + v_shift.
 template <int D>
 __device__ __forceinline__ void load_kv_tile(bf16* Ks, bf16* Vs, const bf16* __restrict__ kv,
                                              const TableRef table, int k0, int lo, int hi,
                                              int kvh, int n_kv, int page_size, int64_t num_pages, int* err,
-                                             int skip = -1, int keep = 0) {
+                                             int skip = -1, int keep = 0, int v_shift = 0) {
     constexpr int CPR = D / 8;  // 16-byte chunks per row
     constexpr int KSTR = D + 8;
-    const int64_t v_off = (int64_t)n_kv * page_size * D;
+    const int64_t v_off = (int64_t)(n_kv + v_shift) * page_size * D;
     for (int c = threadIdx.x; c < MMA_BN * CPR; c += MMA_THREADS) {
         const int row = c / CPR, col = (c - row * CPR) * 8;
         const int key = k0 + row;
@@ -238,7 +239,7 @@ attn_prefill_mma(const bf16* __restrict__ q, int64_t q_stride, bf16* __restrict_
                  const int32_t* __restrict__ tile_req, const int32_t* __restrict__ tile_row0,
                  const int32_t* __restrict__ q_start, const int32_t* __restrict__ seq_lens, int n_q, int n_kv,
                  int page_size, int64_t num_pages, float scale, int window, int* err, const bf16* __restrict__ gate,
-                 float softcap, const float* __restrict__ sinks, int keep, int out_f32, const DiffPair diff) {
+                 float softcap, const float* __restrict__ sinks, int keep, int out_f32, const DiffPair diff, int across) {
     pdl_launch_dependents();  // the next kernel may be scheduled now; it waits for this one itself
     pdl_wait();               // nothing below runs before the kernels before this one are complete
     constexpr int KSTR = D + 8;
@@ -247,7 +248,9 @@ attn_prefill_mma(const bf16* __restrict__ q, int64_t q_stride, bf16* __restrict_
     bf16* KV = Qs + 64 * KSTR;  // stage s: K at KV + s*2*64*KSTR, V after it
 
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-    const int G = n_q / n_kv, kvh = blockIdx.y;
+    const int G = n_q / n_kv, u = blockIdx.y;
+    const HeadPair hp = head_pair(u, n_kv, across);
+    const int kvh = hp.key, v_shift = hp.value - hp.key;
     const int r = tile_req[blockIdx.x], row0 = tile_row0[blockIdx.x];
     const int qs = q_start[r], q_len = q_start[r + 1] - qs, seq_len = seq_lens[r];
     const int rows_total = q_len * G;
@@ -269,7 +272,7 @@ attn_prefill_mma(const bf16* __restrict__ q, int64_t q_stride, bf16* __restrict_
         const int tok = ok ? gr / G : 0, g = ok ? gr - tok * G : 0;
         cp_async16(Qs + row * KSTR + col, q + (int64_t)(qs + tok) * q_stride + (int64_t)(kvh * G + g) * D + col, ok);
     }
-    load_kv_tile<D>(KV, KV + MMA_BN * KSTR, kv, table, walk.at(0) * MMA_BN, lo, last_pos, kvh, n_kv, page_size, num_pages, err, -1, keep);
+    load_kv_tile<D>(KV, KV + MMA_BN * KSTR, kv, table, walk.at(0) * MMA_BN, lo, last_pos, kvh, n_kv, page_size, num_pages, err, -1, keep, v_shift);
     cp_async_commit();
 
     // this thread's two rows
@@ -302,7 +305,7 @@ attn_prefill_mma(const bf16* __restrict__ q, int64_t q_stride, bf16* __restrict_
         bf16* Vs = Ks + MMA_BN * KSTR;
         if (jt + 1 < walk.count) {
             bf16* Kn = KV + (stage ^ 1) * 2 * MMA_BN * KSTR;
-            load_kv_tile<D>(Kn, Kn + MMA_BN * KSTR, kv, table, walk.at(jt + 1) * MMA_BN, lo, last_pos, kvh, n_kv, page_size, num_pages, err, -1, keep);
+            load_kv_tile<D>(Kn, Kn + MMA_BN * KSTR, kv, table, walk.at(jt + 1) * MMA_BN, lo, last_pos, kvh, n_kv, page_size, num_pages, err, -1, keep, v_shift);
             cp_async_commit();
             cp_async_wait<1>();
         } else {
@@ -365,13 +368,13 @@ attn_prefill_mma(const bf16* __restrict__ q, int64_t q_stride, bf16* __restrict_
         }
         if (row >= rows_here) continue;
         if (out_f32) {
-            float* dst = reinterpret_cast<float*>(out) + (int64_t)(qs + tok) * out_stride + (int64_t)(kvh * G + g) * D + ((lane & 3) << 1);
+            float* dst = reinterpret_cast<float*>(out) + (int64_t)(qs + tok) * out_stride + (int64_t)(u * G + g) * D + ((lane & 3) << 1);
 #pragma unroll
             for (int d = 0; d < D / 8; ++d)
                 *reinterpret_cast<float2*>(dst + d * 8) = make_float2(o[d][2 * h] * inv, o[d][2 * h + 1] * inv);
             continue;
         }
-        bf16* dst = out + (int64_t)(qs + tok) * out_stride + (int64_t)(kvh * G + g) * D + ((lane & 3) << 1);
+        bf16* dst = out + (int64_t)(qs + tok) * out_stride + (int64_t)(u * G + g) * D + ((lane & 3) << 1);
         const bf16* gt = gate ? gate + (int64_t)(qs + tok) * q_stride + (int64_t)(kvh * G + g) * D + ((lane & 3) << 1) : nullptr;
 #pragma unroll
         for (int d = 0; d < D / 8; ++d) {
@@ -398,7 +401,7 @@ attn_decode_mma(const bf16* __restrict__ q, int64_t q_stride, bf16* __restrict__
                 int page_size, int64_t num_pages, float scale, int window, int n_slices, int cluster,
                 const float* __restrict__ inv_freq, int rot_dim, int fused,
                 float* __restrict__ part_o, float* __restrict__ part_lse, int* __restrict__ counters, int* err,
-                const bf16* __restrict__ gate, float softcap, const float* __restrict__ sinks, int keep, int out_f32) {
+                const bf16* __restrict__ gate, float softcap, const float* __restrict__ sinks, int keep, int out_f32, int across) {
     pdl_launch_dependents();  // the next kernel may be scheduled now; it waits for this one itself
     // Until pdl_wait() below, only what no kernel of this step writes is touched: the lengths, the block
     // table, and keys and values at positions before the newest token (earlier steps wrote those).  The
@@ -410,7 +413,9 @@ attn_decode_mma(const bf16* __restrict__ q, int64_t q_stride, bf16* __restrict__
 
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int G = n_q / n_kv, hblocks = (G + 15) / 16;
-    const int r = blockIdx.x, kvh = blockIdx.y / hblocks, g0 = (blockIdx.y % hblocks) * 16;
+    const int r = blockIdx.x, u = blockIdx.y / hblocks, g0 = (blockIdx.y % hblocks) * 16;
+    const HeadPair hp = head_pair(u, n_kv, across);
+    const int kvh = hp.key, v_shift = hp.value - hp.key, n_out = across ? n_q * n_kv : n_q;
     const int heads_here = min(16, G - g0);
     const int slice = blockIdx.z;
     const int row_q = q_start[r], seq_len = seq_lens[r];
@@ -509,7 +514,7 @@ attn_decode_mma(const bf16* __restrict__ q, int64_t q_stride, bf16* __restrict__
         for (int st = 0; st < NS - 1; ++st) {
             if (j_lo + st <= j_hi && j_lo + st < j_last) {
                 bf16* Kn = KV + st * 2 * MMA_BN * KSTR;
-                load_kv_tile<D>(Kn, Kn + MMA_BN * KSTR, kv, table, walk.at(j_lo + st) * MMA_BN, lo, pos, kvh, n_kv, page_size, num_pages, err, -1, keep);
+                load_kv_tile<D>(Kn, Kn + MMA_BN * KSTR, kv, table, walk.at(j_lo + st) * MMA_BN, lo, pos, kvh, n_kv, page_size, num_pages, err, -1, keep, v_shift);
             }
         }
         pdl_wait();
@@ -526,7 +531,7 @@ attn_decode_mma(const bf16* __restrict__ q, int64_t q_stride, bf16* __restrict__
         for (int st = 0; st < NS - 1; ++st) {
             if (j_lo + st <= j_hi && j_lo + st == j_last) {
                 bf16* Kn = KV + st * 2 * MMA_BN * KSTR;
-                load_kv_tile<D>(Kn, Kn + MMA_BN * KSTR, kv, table, walk.at(j_last) * MMA_BN, lo, pos, kvh, n_kv, page_size, num_pages, err, skip, keep);
+                load_kv_tile<D>(Kn, Kn + MMA_BN * KSTR, kv, table, walk.at(j_last) * MMA_BN, lo, pos, kvh, n_kv, page_size, num_pages, err, skip, keep, v_shift);
                 if (fused) put_newest(Kn, Kn + MMA_BN * KSTR);
             }
             cp_async_commit();
@@ -541,7 +546,7 @@ attn_decode_mma(const bf16* __restrict__ q, int64_t q_stride, bf16* __restrict__
             bf16* Vs = Ks + MMA_BN * KSTR;
             if (j + NS - 1 <= j_hi) {
                 bf16* Kn = KV + ((j - j_lo + NS - 1) % NS) * 2 * MMA_BN * KSTR;
-                load_kv_tile<D>(Kn, Kn + MMA_BN * KSTR, kv, table, walk.at(j + NS - 1) * MMA_BN, lo, pos, kvh, n_kv, page_size, num_pages, err, skip, keep);
+                load_kv_tile<D>(Kn, Kn + MMA_BN * KSTR, kv, table, walk.at(j + NS - 1) * MMA_BN, lo, pos, kvh, n_kv, page_size, num_pages, err, skip, keep, v_shift);
                 if (fused && j + NS - 1 == j_last) put_newest(Kn, Kn + MMA_BN * KSTR);
             }
             cp_async_commit();
@@ -625,7 +630,7 @@ attn_decode_mma(const bf16* __restrict__ q, int64_t q_stride, bf16* __restrict__
 #pragma unroll
         for (int w = 0; w < 4; ++w) acc += Om[(w * 16 + row) * OSTR + d] * Fm[w * 16 + row];
         const float val = ll > 0.f ? acc / ll : 0.f;
-        const int head = kvh * G + g0 + row;
+        const int head = u * G + g0 + row;
         if (n_slices == 1) {
             if (out_f32) reinterpret_cast<float*>(out)[(int64_t)row_q * out_stride + (int64_t)head * D + d] = val;
             else out[(int64_t)row_q * out_stride + (int64_t)head * D + d] = __float2bfloat16_rn(
@@ -634,8 +639,8 @@ attn_decode_mma(const bf16* __restrict__ q, int64_t q_stride, bf16* __restrict__
             Pc[row * D + d] = val;
             if (d == 0) Lc[row] = ll > 0.f ? mm + log2f(ll) : -INFINITY;
         } else {
-            part_o[(((int64_t)r * n_q + head) * n_slices + slice) * D + d] = val;
-            if (d == 0) part_lse[((int64_t)r * n_q + head) * n_slices + slice] = ll > 0.f ? mm + log2f(ll) : -INFINITY;
+            part_o[(((int64_t)r * n_out + head) * n_slices + slice) * D + d] = val;
+            if (d == 0) part_lse[((int64_t)r * n_out + head) * n_slices + slice] = ll > 0.f ? mm + log2f(ll) : -INFINITY;
         }
     }
     if (n_slices == 1) return;
@@ -666,7 +671,7 @@ attn_decode_mma(const bf16* __restrict__ q, int64_t q_stride, bf16* __restrict__
 #pragma unroll
             for (int sl = 0; sl < 8; ++sl) acc += p[sl] * (lse[sl] * inv);
             if (gate) acc = gated<true>(acc, to_float(gate[(int64_t)row_q * q_stride + (int64_t)(kvh * G + g0 + row) * D + d]));
-            const int64_t at = (int64_t)row_q * out_stride + (int64_t)(kvh * G + g0 + row) * D + d;
+            const int64_t at = (int64_t)row_q * out_stride + (int64_t)(u * G + g0 + row) * D + d;
             if (out_f32) reinterpret_cast<float*>(out)[at] = acc;
             else out[at] = __float2bfloat16_rn(acc);
         }
@@ -692,7 +697,7 @@ attn_decode_mma(const bf16* __restrict__ q, int64_t q_stride, bf16* __restrict__
     float* W = reinterpret_cast<float*>(smem_raw);  // [16][n_slices]
     for (int idx = tid; idx < heads_here * n_slices; idx += MMA_THREADS) {
         const int row = idx / n_slices, sl = idx - row * n_slices;
-        W[row * n_slices + sl] = __ldcg(part_lse + ((int64_t)r * n_q + kvh * G + g0 + row) * n_slices + sl);
+        W[row * n_slices + sl] = __ldcg(part_lse + ((int64_t)r * n_out + u * G + g0 + row) * n_slices + sl);
     }
     __syncthreads();
     if (tid < heads_here) {
@@ -710,8 +715,8 @@ attn_decode_mma(const bf16* __restrict__ q, int64_t q_stride, bf16* __restrict__
     __syncthreads();
     for (int idx = tid; idx < heads_here * D; idx += MMA_THREADS) {
         const int row = idx / D, d = idx - row * D;
-        const int head = kvh * G + g0 + row;
-        const float* po = part_o + ((int64_t)r * n_q + head) * n_slices * D + d;
+        const int head = u * G + g0 + row;
+        const float* po = part_o + ((int64_t)r * n_out + head) * n_slices * D + d;
         const float* w = W + row * n_slices;
         float acc = 0.f;
 #pragma unroll 8

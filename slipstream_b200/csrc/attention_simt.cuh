@@ -15,6 +15,7 @@
 // loop of slipstream/kernels/attention_ref.py:68-89 and the Triton decode kernel
 // slipstream/kernels/triton_paged.py:97-206.
 //
+// `across`: common.cuh, head_pair.
 // kv layout: [page][2][kv head][offset in page][D], element type T.
 #pragma once
 
@@ -37,7 +38,7 @@ attn_simt_kernel(const T* __restrict__ q, int64_t q_stride, T* __restrict__ out,
                  const int32_t* __restrict__ tile_req, const int32_t* __restrict__ tile_q0,
                  const int32_t* __restrict__ q_start, const int32_t* __restrict__ seq_lens,
                  int n_q, int n_kv, int page_size, int64_t num_pages, float scale, int window,
-                 int* err, const T* __restrict__ gate, float softcap, const float* __restrict__ sinks, int keep) {
+                 int* err, const T* __restrict__ gate, float softcap, const float* __restrict__ sinks, int keep, int across) {
     pdl_launch_dependents();  // the next kernel may be scheduled now; it waits for this one itself
     pdl_wait();               // nothing below runs before the kernels before this one are complete
     constexpr int DPL = (D + 31) / 32;
@@ -49,7 +50,9 @@ attn_simt_kernel(const T* __restrict__ q, int64_t q_stride, T* __restrict__ out,
     float* Ps = Vs + ATT_BN * D;
 
     const int tid = threadIdx.x, lane = tid & 31, w = tid >> 5;
-    const int h = blockIdx.y, kvh = h / (n_q / n_kv);
+    const int G = n_q / n_kv, h_out = blockIdx.y;  // the output's head
+    const HeadPair hp = head_pair(h_out / G, n_kv, across);
+    const int h = hp.key * G + h_out % G;          // the query's
     const int r = tile_req[blockIdx.x], q0 = tile_q0[blockIdx.x];
     const int qs = q_start[r], q_len = q_start[r + 1] - qs, seq_len = seq_lens[r];
     const int rows_here = min(ATT_BM, q_len - q0);
@@ -93,8 +96,8 @@ attn_simt_kernel(const T* __restrict__ q, int64_t q_stride, T* __restrict__ out,
             }
             if (page >= 0) {
                 const int off = key % page_size;
-                const T* kp = kv + ((((page * 2 + 0) * n_kv + kvh) * page_size + off) * (int64_t)D);
-                const T* vp = kv + ((((page * 2 + 1) * n_kv + kvh) * page_size + off) * (int64_t)D);
+                const T* kp = kv + ((((page * 2 + 0) * n_kv + hp.key) * page_size + off) * (int64_t)D);
+                const T* vp = kv + ((((page * 2 + 1) * n_kv + hp.value) * page_size + off) * (int64_t)D);
                 for (int d = lane; d < D; d += 32) {
                     Ks[row * KS + d] = to_float(kp[d]);
                     Vs[row * D + d] = to_float(vp[d]);
@@ -167,7 +170,7 @@ attn_simt_kernel(const T* __restrict__ q, int64_t q_stride, T* __restrict__ out,
         const int row = w * ATT_RPW + i;
         if (row >= rows_here) continue;
         const float inv = l[i] > 0.f ? 1.0f / l[i] : 0.f;
-        T* dst = out + (int64_t)(qs + q0 + row) * out_stride + (int64_t)h * D;
+        T* dst = out + (int64_t)(qs + q0 + row) * out_stride + (int64_t)h_out * D;
 #pragma unroll
         for (int c = 0; c < DPL; ++c) {
             const int d = lane + 32 * c;
@@ -186,14 +189,14 @@ int launch_attn_simt(const void* q, int64_t q_stride, void* out, int64_t out_str
                      const int32_t* tile_q0, int n_tiles, const int32_t* q_start,
                      const int32_t* seq_lens, int n_q, int n_kv, int page_size, int64_t num_pages,
                      float scale, int window, const void* gate, int* err, cudaStream_t stream, float softcap = 0.f,
-                     const float* sinks = nullptr, int keep = 0) {
+                     const float* sinks = nullptr, int keep = 0, int across = 0) {
     static_assert(ATT_RPW == 4, "the kernel packs four rows per warp into a float4");
     constexpr int smem = att_simt_smem_bytes<D>();
     static SsPerDevice opted;
     if (int rc_smem = ss_opt_in_smem(attn_simt_kernel<T, D>, smem, opted)) return rc_smem;
-    dim3 grid(n_tiles, n_q);
+    dim3 grid(n_tiles, across ? n_q * n_kv : n_q);
     ss_launch(attn_simt_kernel<T, D>, dim3(grid), dim3(ATT_WARPS * 32), smem, stream, 
         (const T*)q, q_stride, (T*)out, out_stride, (const T*)kv, block_tables, max_blocks, tile_req,
-        tile_q0, q_start, seq_lens, n_q, n_kv, page_size, num_pages, scale, window, err, (const T*)gate, softcap, sinks, keep);
+        tile_q0, q_start, seq_lens, n_q, n_kv, page_size, num_pages, scale, window, err, (const T*)gate, softcap, sinks, keep, across);
     return SS_LAUNCH_CHECK();
 }

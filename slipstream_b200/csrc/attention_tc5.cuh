@@ -155,6 +155,7 @@ struct Args {
     const float* sinks;  // float32 [n_q] or null: one more term exp(sinks[h]) in the denominator of head h's softmax
     int keep;  // with a sliding window: the request's first `keep` keys stay visible (common.cuh: key_tiles)
     int out_f32;  // `out` is float32
+    int across;  // common.cuh: head_pair
     DiffPair diff;  // one layer of blocks only (gridDim.z == 1), dim a multiple of 8
 };
 
@@ -202,10 +203,12 @@ attn_prefill_tc5(const __grid_constant__ CUtensorMap map_q, const __grid_constan
     // start first, then those of the next longest, whatever their head or request (head by head, the short tiles
     // of one head started before the long ones of the next and left one SM with three times the work of another:
     // a 2,048-token prompt took 45.7 us instead of 37.3)
-    const int G = a.n_q / a.n_kv, kvh = blockIdx.x % a.n_kv;
+    const int G = a.n_q / a.n_kv, n_u = a.across ? a.n_kv * a.n_kv : a.n_kv, u = blockIdx.x % n_u;
+    const HeadPair hp = head_pair(u, a.n_kv, a.across);
+    const int kvh = hp.key;
     const int TOK = 128 / G;
     pdl_wait();  // q, the pages and the tables come from the kernels before this one
-    const int tile = blockIdx.x / a.n_kv;
+    const int tile = blockIdx.x / n_u;
     const int r = a.tile_req[tile], tok0 = a.tile_tok0[tile];
     const int qs = a.q_start[r], q_len = a.q_start[r + 1] - qs, seq_len = a.seq_lens[r];
     const int toks_here = min(TOK, q_len - tok0);
@@ -293,7 +296,7 @@ attn_prefill_tc5(const __grid_constant__ CUtensorMap map_q, const __grid_constan
                 __syncwarp();
                 if (mine)
                     tma_load_3d(Vs + st * KV_BYTES + h * HALF_KV + p * ps * 128, &map_kv, h * 64, 0,
-                                (int)((page * 2 + 1) * a.n_kv + kvh), &v_full[st]);
+                                (int)((page * 2 + 1) * a.n_kv + hp.value), &v_full[st]);
             }
         }
     } else if (warp == 1) {
@@ -499,7 +502,7 @@ attn_prefill_tc5(const __grid_constant__ CUtensorMap map_q, const __grid_constan
                     }
                     diff_scale = a.diff.mult / sqrtf(ss / (float)a.diff.dim + a.diff.eps);
                 }
-                bf16* dst = a.out + (int64_t)(qs + tok0 + tok) * a.out_stride + (int64_t)(kvh * G + g) * D;
+                bf16* dst = a.out + (int64_t)(qs + tok0 + tok) * a.out_stride + (int64_t)(u * G + g) * D;
 #pragma unroll 1
                 for (int c = 0; c < D; c += 32) {
                     uint32_t o[32];
@@ -526,7 +529,7 @@ attn_prefill_tc5(const __grid_constant__ CUtensorMap map_q, const __grid_constan
                         }
                     } else if (a.out_f32) {
                         if (valid) {
-                            float* fdst = reinterpret_cast<float*>(a.out) + (int64_t)(qs + tok0 + tok) * a.out_stride + (int64_t)(kvh * G + g) * D + c;
+                            float* fdst = reinterpret_cast<float*>(a.out) + (int64_t)(qs + tok0 + tok) * a.out_stride + (int64_t)(u * G + g) * D + c;
 #pragma unroll
                             for (int e = 0; e < 32; e += 4)
                                 *reinterpret_cast<float4*>(fdst + e) = make_float4(__uint_as_float(o[e]) * inv, __uint_as_float(o[e + 1]) * inv,
@@ -594,7 +597,7 @@ attn_prefill_tc5(const __grid_constant__ CUtensorMap map_q, const __grid_constan
             if (a.sinks && valid)  // once for the row, whichever block of the cluster writes these columns
                 l_all = m_all == -INFINITY ? 1.f : l_all + ex2(a.sinks[kvh * G + g] * 1.4426950408889634f - m_all);
             const float inv = l_all > 0.f ? 1.f / l_all : 0.f;
-            bf16* dst = a.out + (int64_t)(qs + tok0 + tok) * a.out_stride + (int64_t)(kvh * G + g) * D + c0;
+            bf16* dst = a.out + (int64_t)(qs + tok0 + tok) * a.out_stride + (int64_t)(u * G + g) * D + c0;
 #pragma unroll 1
             for (int c = 0; c < cols; c += 8) {
                 float acc[8];
@@ -608,7 +611,7 @@ attn_prefill_tc5(const __grid_constant__ CUtensorMap map_q, const __grid_constan
                     }
                 }
                 if (valid && a.out_f32) {
-                    float* fdst = reinterpret_cast<float*>(a.out) + (int64_t)(qs + tok0 + tok) * a.out_stride + (int64_t)(kvh * G + g) * D + c0 + c;
+                    float* fdst = reinterpret_cast<float*>(a.out) + (int64_t)(qs + tok0 + tok) * a.out_stride + (int64_t)(u * G + g) * D + c0 + c;
                     *reinterpret_cast<float4*>(fdst) = make_float4(acc[0] * inv, acc[1] * inv, acc[2] * inv, acc[3] * inv);
                     *reinterpret_cast<float4*>(fdst + 4) = make_float4(acc[4] * inv, acc[5] * inv, acc[6] * inv, acc[7] * inv);
                 } else if (valid) {

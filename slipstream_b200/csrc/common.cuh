@@ -66,6 +66,20 @@ __device__ __forceinline__ KeyTiles key_tiles(int lo, int last, int keep, int bn
     return t;
 }
 
+// Which key/value heads a block of an attention kernel reads.  Usually number u is kv head u, for keys and for values.
+// With `across` every query head's weights meet the values of EVERY kv head (what a later mixture over heads needs):
+// there are n_kv * n_kv such numbers, u = (kv head of the keys and of the queries) * n_kv + (kv head of the values), and
+// the outputs are n_kv * n_q heads, those of number u being heads u * G .. u * G + G - 1.
+struct HeadPair {
+    int key, value;
+};
+__device__ __forceinline__ HeadPair head_pair(int u, int n_kv, int across) {
+    HeadPair p;
+    p.key = across ? u / n_kv : u;
+    p.value = across ? u - p.key * n_kv : u;
+    return p;
+}
+
 // What the attention kernels do with the outputs of a head's two softmax maps (query heads 2h and 2h + 1, side by side
 // in a kv group).  on: o = a_2h - lam * a_2h+1 over the first `dim` elements, times mult / sqrt(mean(o^2) + eps), all in
 // float32, is written as one head of `dim` elements.

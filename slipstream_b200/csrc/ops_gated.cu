@@ -1,5 +1,6 @@
 // Kernels of two more recurrent mixers and of the parts that stand around them, beside ops_cells.cu:
-//   * linear attention with a fixed decay per head:  S <- decay_h S + k v^T,  o = S^T q  (q, k, v under silu), and
+//   * linear attention with a fixed decay per head:  S <- decay_h S + k v^T,  o = S^T q  (q, k, v under silu, or q and k
+//     rotated and k scaled), and
 //     the RMS norm of the concatenated heads under a sigmoid gate;
 //   * the real-gated linear recurrent unit:  gates from square blocks of the convolved input,
 //     a = exp(-c r softplus(lam)),  S <- a S + sqrt(1 - a^2) (i u),  output S gelu(y);
@@ -25,8 +26,10 @@ __device__ __forceinline__ float gelu_tanh_f(float z) {
 
 // ---------------------------------------------------------------- linear attention with a decay per head
 //
-// proj row: [q: heads * dim | k: heads * dim | v: heads * vdim | ...] (pre-activations).  Per request and head, token
-// by token:  S <- decay S + silu(k) silu(v)^T,  o = S^T silu(q).  state: float32 [slots][heads][dim][vdim];
+// proj row: [q: heads * dim | k: heads * dim | v: heads * vdim | ...] (as projected).  Per request and head, token
+// by token:  S <- decay S + k' v'^T,  o = S^T q'.  SILU: q', k', v' are silu of what was projected.  Otherwise v' = v,
+// q' is q and k' is k with elements i and i + half of the first 2 half elements turned by position * inv_freq[i], k' also
+// times k_scale; a batch's cosines and sines are formed once, while the batch in front is computed.  state: float32 [slots][heads][dim][vdim];
 // out: float32 [rows][heads * vdim].
 //
 // A block of DA_WARPS warps takes one head of one request and DA_COLS value columns.  A lane is a column; warp w holds rows
@@ -52,11 +55,17 @@ __device__ __forceinline__ float silu_act(float z) {
 template <int RMAX>
 constexpr int da_smem_bytes() { return (2 * DA_BATCH * DA_WARPS * RMAX + DA_BATCH * DA_COLS + DA_WARPS * DA_BATCH * DA_COLS) * 4; }
 
-template <typename T, int RMAX, bool FAST, bool VEC>
+struct DaTurn {
+    const float* inv_freq;  // float32 [half]
+    int half;               // 0: no rotation
+    float k_scale;
+};
+
+template <typename T, int RMAX, bool FAST, bool VEC, bool SILU>
 __global__ void __launch_bounds__(DA_WARPS * 32)
 decay_attention_kernel(const T* __restrict__ proj, int64_t stride, const float* __restrict__ decay, float* __restrict__ state,
                        float* __restrict__ out, const int32_t* __restrict__ q_start, const int32_t* __restrict__ seq_lens,
-                       const int32_t* __restrict__ slots, int heads, int dim, int vdim, int n_slots, int* err) {
+                       const int32_t* __restrict__ slots, int heads, int dim, int vdim, int n_slots, int* err, const DaTurn turn) {
     constexpr int GROUPS = RMAX / 4, W = DA_WARPS * RMAX;  // W: rows of shared memory a token's q (or k) takes
     const int col_blocks = (vdim + DA_COLS - 1) / DA_COLS;
     const int h = blockIdx.x / col_blocks, cb = blockIdx.x % col_blocks, r = blockIdx.y;
@@ -74,6 +83,9 @@ decay_attention_kernel(const T* __restrict__ proj, int64_t stride, const float* 
     float* ks = qs + DA_BATCH * W;             // [DA_BATCH][W]
     float* vs = ks + DA_BATCH * W;             // [DA_BATCH][DA_COLS]
     float* red = vs + DA_BATCH * DA_COLS;      // [DA_WARPS][DA_BATCH][DA_COLS]
+    float2* cs = reinterpret_cast<float2*>(red + DA_WARPS * DA_BATCH * DA_COLS);  // [DA_BATCH][half] (cosine, sine), without SILU
+    const int half = SILU ? 0 : turn.half;
+    const float k_scale = SILU ? 1.f : turn.k_scale;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, j = cb * DA_COLS + lane;
     const bool live = j < vdim;
     const int row0 = warp * RMAX;
@@ -86,7 +98,19 @@ decay_attention_kernel(const T* __restrict__ proj, int64_t stride, const float* 
     const int64_t k_off = (int64_t)heads * dim + (int64_t)h * dim, v_off = 2 * (int64_t)heads * dim + (int64_t)h * vdim;
     // VEC: the items of a batch are 16-byte pieces, per token dim / 8 of q, dim / 8 of k and DA_COLS / 8 of v
     const int dim8 = dim >> 3, ipt = 2 * dim8 + DA_COLS / 8;
-    uint4 raw[DA_MAX_VEC];
+    uint4 raw[DA_MAX_VEC], partner[SILU ? 1 : DA_MAX_VEC];  // partner: the piece half a rotation away
+    const int half8 = half >> 3;
+    const int pos0 = seq_lens[r] - q_len;  // position of the step's first row
+    auto turns = [&](int t0, int nb) {
+        if constexpr (!SILU) {
+            for (int i = tid; i < nb * half; i += DA_WARPS * 32) {
+                const int t = i / half, e = i - t * half;
+                float sn, c;
+                sincosf(__fmul_rn((float)(pos0 + t0 + t), turn.inv_freq[e]), &sn, &c);
+                cs[i] = make_float2(c, sn);
+            }
+        }
+    };
     auto issue = [&](int t0, int nb) {
 #pragma unroll
         for (int w = 0; w < DA_MAX_VEC; ++w) {
@@ -98,6 +122,12 @@ decay_attention_kernel(const T* __restrict__ proj, int64_t stride, const float* 
                 const bf16* src = c < dim8 ? row + (int64_t)h * dim + c * 8
                                 : c < 2 * dim8 ? row + k_off + (c - dim8) * 8 : row + v_off + cb * DA_COLS + (c - 2 * dim8) * 8;
                 if (c < 2 * dim8 || cb * DA_COLS + (c - 2 * dim8) * 8 < vdim) raw[w] = *reinterpret_cast<const uint4*>(src);
+                if constexpr (!SILU) {
+                    const int piece = c < dim8 ? c : c - dim8;
+                    partner[w] = make_uint4(0u, 0u, 0u, 0u);
+                    if (c < 2 * dim8 && piece < 2 * half8)
+                        partner[w] = *reinterpret_cast<const uint4*>(src + (piece < half8 ? half : -half));
+                }
             }
         }
     };
@@ -112,8 +142,29 @@ decay_attention_kernel(const T* __restrict__ proj, int64_t stride, const float* 
                 float f[8];
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
-                    f[2 * e] = silu_act<FAST>(__uint_as_float(q[e] << 16));
-                    f[2 * e + 1] = silu_act<FAST>(__uint_as_float(q[e] & 0xffff0000u));
+                    f[2 * e] = __uint_as_float(q[e] << 16);
+                    f[2 * e + 1] = __uint_as_float(q[e] & 0xffff0000u);
+                }
+                if constexpr (SILU) {
+#pragma unroll
+                    for (int e = 0; e < 8; ++e) f[e] = silu_act<FAST>(f[e]);
+                } else if (c < 2 * dim8) {
+                    const int piece = c < dim8 ? c : c - dim8;
+                    if (piece < 2 * half8) {
+                        const bool low = piece < half8;
+                        const float2* turned = cs + t * half + (low ? piece : piece - half8) * 8;
+                        const uint32_t o[4] = {partner[w].x, partner[w].y, partner[w].z, partner[w].w};
+#pragma unroll
+                        for (int e = 0; e < 8; ++e) {
+                            const float other = __uint_as_float((e & 1) ? o[e >> 1] & 0xffff0000u : o[e >> 1] << 16);
+                            const float2 t2 = turned[e];
+                            f[e] = low ? f[e] * t2.x - other * t2.y : f[e] * t2.x + other * t2.y;
+                        }
+                    }
+                    if (c >= dim8) {
+#pragma unroll
+                        for (int e = 0; e < 8; ++e) f[e] *= k_scale;
+                    }
                 }
                 *reinterpret_cast<float4*>(dst) = make_float4(f[0], f[1], f[2], f[3]);
                 *reinterpret_cast<float4*>(dst + 4) = make_float4(f[4], f[5], f[6], f[7]);
@@ -121,6 +172,7 @@ decay_attention_kernel(const T* __restrict__ proj, int64_t stride, const float* 
         }
     };
     if (VEC) issue(0, min(DA_BATCH, q_len));
+    if (half > 0) turns(0, min(DA_BATCH, q_len));
     for (int t0 = 0; t0 < q_len; t0 += DA_BATCH) {
         const int nb = min(DA_BATCH, q_len - t0);
         __syncthreads();  // the batch in front is done with shared memory (and, the first time, the zeros are in place)
@@ -131,16 +183,21 @@ decay_attention_kernel(const T* __restrict__ proj, int64_t stride, const float* 
         } else {
             const int n_qk = nb * dim, n_all = n_qk + nb * DA_COLS;
             for (int i0 = tid; i0 < n_all; i0 += 4 * blockDim.x) {  // four loads (pairs, for q and k) in flight
-                float a[4], b[4];
+                float a[4], b[4], pa[4], pb[4];
 #pragma unroll
                 for (int w = 0; w < 4; ++w) {
                     const int i = i0 + w * blockDim.x;
-                    a[w] = b[w] = 0.f;
+                    a[w] = b[w] = pa[w] = pb[w] = 0.f;
                     if (i < n_qk) {
                         const int t = i / dim, e = i - t * dim;
                         const T* row = proj + (int64_t)(q0 + t0 + t) * stride;
                         a[w] = to_float(row[(int64_t)h * dim + e]);
                         b[w] = to_float(row[k_off + e]);
+                        if (e < 2 * half) {
+                            const int p = e < half ? e + half : e - half;
+                            pa[w] = to_float(row[(int64_t)h * dim + p]);
+                            pb[w] = to_float(row[k_off + p]);
+                        }
                     } else if (i < n_all) {
                         const int t = (i - n_qk) / DA_COLS, e = (i - n_qk) - t * DA_COLS;
                         if (cb * DA_COLS + e < vdim) a[w] = to_float(proj[(int64_t)(q0 + t0 + t) * stride + v_off + cb * DA_COLS + e]);
@@ -151,16 +208,29 @@ decay_attention_kernel(const T* __restrict__ proj, int64_t stride, const float* 
                     const int i = i0 + w * blockDim.x;
                     if (i < n_qk) {
                         const int t = i / dim, e = i - t * dim;
-                        qs[t * W + e] = silu_act<FAST>(a[w]);
-                        ks[t * W + e] = silu_act<FAST>(b[w]);
+                        if constexpr (SILU) {
+                            qs[t * W + e] = silu_act<FAST>(a[w]);
+                            ks[t * W + e] = silu_act<FAST>(b[w]);
+                        } else {
+                            float x = a[w], y = b[w];
+                            if (e < 2 * half) {
+                                const float2 t2 = cs[t * half + (e < half ? e : e - half)];
+                                const float sn = e < half ? -t2.y : t2.y;
+                                x = x * t2.x + pa[w] * sn;
+                                y = y * t2.x + pb[w] * sn;
+                            }
+                            qs[t * W + e] = x;
+                            ks[t * W + e] = y * k_scale;
+                        }
                     } else if (i < n_all) {
                         const int t = (i - n_qk) / DA_COLS, e = (i - n_qk) - t * DA_COLS;
-                        vs[t * DA_COLS + e] = silu_act<FAST>(a[w]);  // silu(0) = 0 behind the last column
+                        vs[t * DA_COLS + e] = SILU ? silu_act<FAST>(a[w]) : a[w];  // (0 behind the last column)
                     }
                 }
             }
             __syncthreads();
         }
+        if (half > 0 && t0 + DA_BATCH < q_len) turns(t0 + DA_BATCH, min(DA_BATCH, q_len - t0 - DA_BATCH));  // read behind the next barrier
         if (row0 < dim) {  // (a warp whose rows lie behind the head's last one has nothing to add)
             for (int t = 0; t < nb; t += 2) {  // two tokens' loads in flight; their updates in order
                 const int t1 = min(t + 1, nb - 1);
@@ -212,40 +282,50 @@ decay_attention_kernel(const T* __restrict__ proj, int64_t stride, const float* 
     }
 }
 
-template <typename T, int RMAX, bool FAST, bool VEC>
+template <typename T, int RMAX, bool FAST, bool VEC, bool SILU>
 static int launch_decay_attention(const void* proj, int64_t stride, const float* decay, float* state, float* out,
                                   const int32_t* q_start, const int32_t* seq_lens, const int32_t* slots, int R, int heads,
-                                  int dim, int vdim, int n_slots, int* err, cudaStream_t stream) {
-    constexpr int smem = da_smem_bytes<RMAX>();
+                                  int dim, int vdim, int n_slots, int* err, cudaStream_t stream, const DaTurn& turn) {
+    constexpr int most = da_smem_bytes<RMAX>() + (SILU ? 0 : DA_BATCH * (DA_MAX_DIM / 2) * 8);
+    const int smem = da_smem_bytes<RMAX>() + (SILU ? 0 : DA_BATCH * turn.half * 8);
     static SsPerDevice opted;
-    if (int rc = ss_opt_in_smem(decay_attention_kernel<T, RMAX, FAST, VEC>, smem, opted)) return rc;
+    if (int rc = ss_opt_in_smem(decay_attention_kernel<T, RMAX, FAST, VEC, SILU>, most, opted)) return rc;
     const dim3 grid(heads * ((vdim + DA_COLS - 1) / DA_COLS), R), block(DA_WARPS * 32);
-    ss_launch(decay_attention_kernel<T, RMAX, FAST, VEC>, grid, block, smem, stream, (const T*)proj, stride, decay, state, out,
-              q_start, seq_lens, slots, heads, dim, vdim, n_slots, err);
+    ss_launch(decay_attention_kernel<T, RMAX, FAST, VEC, SILU>, grid, block, smem, stream, (const T*)proj, stride, decay, state, out,
+              q_start, seq_lens, slots, heads, dim, vdim, n_slots, err, turn);
     return SS_LAUNCH_CHECK();
 }
 
 extern "C" int ss_decay_attention(const void* proj, int64_t stride, const float* decay, float* state, float* out,
                                   const int32_t* q_start, const int32_t* seq_lens, const int32_t* slots, int R, int heads,
-                                  int dim, int vdim, int n_slots, int dtype, int* err, cudaStream_t stream) {
+                                  int dim, int vdim, int n_slots, int dtype, int* err, cudaStream_t stream, int silu,
+                                  const float* inv_freq, int half, float k_scale) {
     if (R <= 0) return 0;
     if (heads < 1 || dim < 1 || dim > DA_MAX_DIM || vdim < 1) return (int)cudaErrorInvalidValue;
-#define DA_GO(T, RMAX, FAST, VEC)                                                                                         \
-    return launch_decay_attention<T, RMAX, FAST, VEC>(proj, stride, decay, state, out, q_start, seq_lens, slots, R, heads, \
-                                                      dim, vdim, n_slots, err, stream)
+    if (half < 0 || 2 * half > dim || (half > 0 && (silu || !inv_freq))) return (int)cudaErrorInvalidValue;
+    const DaTurn turn = {inv_freq, half, k_scale};
+#define DA_GO(T, RMAX, FAST, VEC, SILU)                                                                                    \
+    return launch_decay_attention<T, RMAX, FAST, VEC, SILU>(proj, stride, decay, state, out, q_start, seq_lens, slots, R, \
+                                                            heads, dim, vdim, n_slots, err, stream, turn)
+#define DA_SIZES(T, FAST, VEC, SILU)                                                                                    \
+    do {                                                                                                                \
+        if (dim <= 4 * DA_WARPS) DA_GO(T, 4, FAST, VEC, SILU);                                                          \
+        else if (dim <= 8 * DA_WARPS) DA_GO(T, 8, FAST, VEC, SILU);                                                     \
+        else DA_GO(T, 16, FAST, VEC, SILU);                                                                             \
+    } while (0)
 #define DA_PICK(T, FAST, VEC)                                                                                           \
     do {                                                                                                                \
-        if (dim <= 4 * DA_WARPS) DA_GO(T, 4, FAST, VEC);                                                                \
-        else if (dim <= 8 * DA_WARPS) DA_GO(T, 8, FAST, VEC);                                                           \
-        else DA_GO(T, 16, FAST, VEC);                                                                                   \
+        if (silu) DA_SIZES(T, FAST, VEC, true);                                                                         \
+        else DA_SIZES(T, FAST, VEC, false);                                                                             \
     } while (0)
-    const bool vec = dtype == SS_BF16 && dim % 8 == 0 && vdim % 8 == 0 && stride % 8 == 0 && ((uintptr_t)proj & 15) == 0;
+    const bool vec = dtype == SS_BF16 && dim % 8 == 0 && vdim % 8 == 0 && half % 8 == 0 && stride % 8 == 0 && ((uintptr_t)proj & 15) == 0;
     if (dtype == SS_BF16) {
         if (vec) DA_PICK(bf16, true, true); else DA_PICK(bf16, true, false);
     } else {
         DA_PICK(float, false, false);
     }
 #undef DA_PICK
+#undef DA_SIZES
 #undef DA_GO
     return 0;
 }

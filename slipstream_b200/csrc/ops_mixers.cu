@@ -675,7 +675,7 @@ extern "C" int ss_ssm_scan(const void* xbc, int C, const void* dt_raw, int64_t d
 
 // ---------------------------------------------------------------- router of the routed experts
 //
-// z = W_router x in float32 (x and W in the compute type); scores s = sigmoid(z), or, with `softmax`, the softmax of
+// z = W_router x (+ bias) in float32 (x and W in the compute type, the bias float32); scores s = sigmoid(z), or, with `softmax`, the softmax of
 // z over all experts; choice scores c = s + correction (no correction: c = s).  With `groups` > 1 the experts form
 // that many equal groups of neighbours, a group's score is its largest choice score, and only experts of the `keep`
 // best groups can be chosen (the others' choice scores count as -infinity).  The `top` largest choice scores are
@@ -718,7 +718,8 @@ template <typename T>
 __global__ void __launch_bounds__(ROUTER_THREADS)
 router_kernel(const T* __restrict__ x, const T* __restrict__ w_router, int32_t* __restrict__ ids,
               float* __restrict__ weights, int hidden, int experts, int top, int renormalize, int softmax,
-              const float* __restrict__ correction, int groups, int keep, float* __restrict__ extra_out, int extra) {
+              const float* __restrict__ correction, int groups, int keep, float* __restrict__ extra_out, int extra,
+              const float* __restrict__ bias) {
     pdl_wait();
     extern __shared__ __align__(16) float rsm[];
     float* xs = rsm;                  // [hidden] (rounded up to a multiple of 4)
@@ -734,6 +735,7 @@ router_kernel(const T* __restrict__ x, const T* __restrict__ w_router, int32_t* 
         float acc = router_dot(w, xs, hidden, lane);
         acc = warp_sum(acc);
         if (lane == 0) {
+            if (e < experts && bias) acc += bias[e];
             if (e >= experts) extra_out[(int64_t)t * extra + (e - experts)] = acc;
             else z[e] = softmax ? acc : 1.0f / (1.0f + expf(-acc));  // the choice below is among scores
         }
@@ -814,7 +816,7 @@ router_kernel(const T* __restrict__ x, const T* __restrict__ w_router, int32_t* 
 
 extern "C" int ss_router(const void* x, const void* w_router, int32_t* ids, float* weights, int n_tokens, int hidden,
                          int experts, int top, int renormalize, int dtype, cudaStream_t stream, int softmax,
-                         const float* correction, int groups, int keep, float* extra_out, int extra) {
+                         const float* correction, int groups, int keep, float* extra_out, int extra, const float* bias) {
     if (n_tokens <= 0) return 0;
     if (experts < 1 || experts > ROUTER_MAX_EXPERTS || top < 1 || top > experts) return (int)cudaErrorInvalidValue;
     if (groups < 1 || experts % groups || keep < 1 || keep > groups || extra < 0 || (extra > 0 && !extra_out))
@@ -823,10 +825,10 @@ extern "C" int ss_router(const void* x, const void* w_router, int32_t* ids, floa
     if (smem > 48 * 1024) return (int)cudaErrorInvalidValue;
     if (dtype == SS_BF16)
         ss_launch(router_kernel<bf16>, dim3(n_tokens), dim3(ROUTER_THREADS), smem, stream, (const bf16*)x, (const bf16*)w_router, ids,
-                  weights, hidden, experts, top, renormalize, softmax, correction, groups, keep, extra_out, extra);
+                  weights, hidden, experts, top, renormalize, softmax, correction, groups, keep, extra_out, extra, bias);
     else
         ss_launch(router_kernel<float>, dim3(n_tokens), dim3(ROUTER_THREADS), smem, stream, (const float*)x, (const float*)w_router,
-                  ids, weights, hidden, experts, top, renormalize, softmax, correction, groups, keep, extra_out, extra);
+                  ids, weights, hidden, experts, top, renormalize, softmax, correction, groups, keep, extra_out, extra, bias);
     return SS_LAUNCH_CHECK();
 }
 

@@ -259,7 +259,7 @@ extern "C" int ss_hc_norm(float* streams, const void* y, const float* mix, const
 //   then (norm_dim > 0) the head is divided by sqrt(sum(x^2) / norm_dim + eps): a unit RMS norm over the head's
 //   norm_dim real elements (elements beyond them are padding and zero);
 //   queries are written back in place, keys to their page (or in place when the token has no slot), values are
-//   copied to their page as they are.
+//   copied to their page as they are, or (value_norm_dim > 0) divided by sqrt(sum(v^2) / value_norm_dim + eps).
 // kv layout: [page][2][kv head][offset in page][D].  D even, at most 256.
 // Two neighbouring elements with one load or store.
 __device__ __forceinline__ void load_pair(const float* p, float& a, float& b) {
@@ -282,7 +282,7 @@ __global__ void __launch_bounds__(256)
 rope_norm_cache_kernel(T* __restrict__ rows, int64_t row_stride, const int32_t* __restrict__ positions,
                        const int32_t* __restrict__ slots, const float* __restrict__ inv_freq, float mscale,
                        T* __restrict__ kv, int n_q, int n_kv, int D, int rot_dim, int interleaved, int norm_dim,
-                       float eps, int page_size, int64_t pool_slots, int write_cache, int* err) {
+                       float eps, int page_size, int64_t pool_slots, int write_cache, int* err, int value_norm_dim) {
     pdl_wait();
     __shared__ float cos_s[128], sin_s[128];
     const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n_warps = blockDim.x >> 5;
@@ -304,10 +304,15 @@ rope_norm_cache_kernel(T* __restrict__ rows, int64_t row_stride, const int32_t* 
     __syncthreads();
     for (int h = blockIdx.y * n_warps + warp; h < n_q + 2 * n_kv; h += gridDim.y * n_warps) {
         T* src = rows + (int64_t)t * row_stride + (int64_t)h * D;
-        if (h >= n_q + n_kv) {  // a value head: copied to its page as it is
+        if (h >= n_q + n_kv) {  // a value head: to its page, as it is or divided by its root mean square
             if (slot < 0) continue;
             T* dst = kv + ((((page * 2 + 1) * n_kv + (h - n_q - n_kv)) * page_size + off) * (int64_t)D);
-            if ((D * sizeof(T)) % 16 == 0 && (((uintptr_t)src | (uintptr_t)dst) & 15) == 0) {
+            if (value_norm_dim > 0) {
+                float ss = 0.f;
+                for (int d = lane; d < D; d += 32) ss = fmaf(to_float(src[d]), to_float(src[d]), ss);
+                const float f = 1.0f / sqrtf(warp_sum(ss) / (float)value_norm_dim + eps);
+                for (int d = lane; d < D; d += 32) dst[d] = from_float<T>(to_float(src[d]) * f);
+            } else if ((D * sizeof(T)) % 16 == 0 && (((uintptr_t)src | (uintptr_t)dst) & 15) == 0) {
                 for (int c = lane; c < (int)(D * sizeof(T) / 16); c += 32)
                     reinterpret_cast<uint4*>(dst)[c] = reinterpret_cast<const uint4*>(src)[c];
             } else {
@@ -363,13 +368,13 @@ rope_norm_cache_kernel(T* __restrict__ rows, int64_t row_stride, const int32_t* 
 
 // bfloat16 with 16-byte accesses (neighbouring pairs, D a multiple of 8, 16-byte aligned rows): LPH lanes share a
 // head, 8 elements (4 pairs) each, so a warp holds 32 / LPH heads at a time and two such sets are in flight per
-// thread; value heads are copied 16 bytes a thread.  A block per token.
+// thread; value heads are copied 16 bytes a thread, or, under a norm, walked behind the keys.  A block per token.
 template <int LPH>
 __global__ void __launch_bounds__(256)
 rope_norm_cache_bf16x8_kernel(bf16* __restrict__ rows, int64_t row_stride, const int32_t* __restrict__ positions,
                               const int32_t* __restrict__ slots, const float* __restrict__ inv_freq, float mscale,
                               bf16* __restrict__ kv, int n_q, int n_kv, int D, int rot_dim, int norm_dim, float eps,
-                              int page_size, int64_t pool_slots, int write_cache, int* err) {
+                              int page_size, int64_t pool_slots, int write_cache, int* err, int value_norm_dim) {
     pdl_wait();
     __shared__ float cos_s[128], sin_s[128];
     const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n_warps = blockDim.x >> 5;
@@ -390,7 +395,7 @@ rope_norm_cache_bf16x8_kernel(bf16* __restrict__ rows, int64_t row_stride, const
     const int off = slot >= 0 ? (int)(slot % page_size) : 0;
     bf16* row = rows + (int64_t)t * row_stride;
     // values first: their copies are in flight while the sines are formed
-    if (slot >= 0) {
+    if (slot >= 0 && value_norm_dim == 0) {
         const int cpr = D / 8;
         for (int idx = threadIdx.x; idx < n_kv * cpr; idx += blockDim.x) {
             const int h = idx / cpr, c = idx - h * cpr;
@@ -402,7 +407,7 @@ rope_norm_cache_bf16x8_kernel(bf16* __restrict__ rows, int64_t row_stride, const
     constexpr int HPW = 32 / LPH, U = 2;
     const int sub = lane / LPH, l = lane % LPH;
     const bool lane_on = l * 8 < D;
-    const int heads = n_q + n_kv, stride = n_warps * HPW;
+    const int turned = n_q + n_kv, heads = turned + (value_norm_dim > 0 && slot >= 0 ? n_kv : 0), stride = n_warps * HPW;
     for (int hb = warp * HPW; hb < heads; hb += stride * U) {  // the same trips for every lane of a warp (shuffles below)
         const int h0 = hb + sub;
         uint4 raw[U];
@@ -425,7 +430,7 @@ rope_norm_cache_bf16x8_kernel(bf16* __restrict__ rows, int64_t row_stride, const
                     const __nv_bfloat162 v = *reinterpret_cast<const __nv_bfloat162*>(&w[e]);
                     float x1 = __low2float(v), x2 = __high2float(v);
                     const int p = l * 4 + e;
-                    if (p < half) {
+                    if (p < half && h < turned) {
                         const float cs = cos_s[p], sn = sin_s[p];
                         const float r1 = __fadd_rn(__fmul_rn(x1, cs), __fmul_rn(-x2, sn));
                         const float r2 = __fadd_rn(__fmul_rn(x2, cs), __fmul_rn(x1, sn));
@@ -439,14 +444,16 @@ rope_norm_cache_bf16x8_kernel(bf16* __restrict__ rows, int64_t row_stride, const
                 }
             }
             float scale = 1.f;
-            if (norm_dim > 0) {  // the whole warp takes part in the shuffles
+            if (norm_dim > 0 || value_norm_dim > 0) {  // the whole warp takes part in the shuffles
 #pragma unroll
                 for (int o = LPH / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-                scale = 1.0f / sqrtf(ss / (float)norm_dim + eps);
+                const int over = h < turned ? norm_dim : value_norm_dim;
+                if (over > 0) scale = 1.0f / sqrtf(ss / (float)over + eps);
             }
             if (on[u]) {
+                const int side = h < turned ? 0 : 1;  // a value head is walked only when it has a slot
                 bf16* dst = (h < n_q || slot < 0) ? row + (int64_t)h * D
-                                                  : kv + ((((page * 2 + 0) * n_kv + (h - n_q)) * page_size + off) * (int64_t)D);
+                                                  : kv + ((((page * 2 + side) * n_kv + (h - n_q - side * n_kv)) * page_size + off) * (int64_t)D);
                 uint32_t o4[4];
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
@@ -462,9 +469,9 @@ rope_norm_cache_bf16x8_kernel(bf16* __restrict__ rows, int64_t row_stride, const
 extern "C" int ss_rope_norm_cache(void* rows, int64_t row_stride, const int32_t* positions, const int32_t* slots,
                                   const float* inv_freq, float mscale, void* kv, int n_tokens, int n_q, int n_kv,
                                   int D, int rot_dim, int interleaved, int norm_dim, float eps, int page_size,
-                                  int64_t num_pages, int write_cache, int dtype, int* err, cudaStream_t stream) {
+                                  int64_t num_pages, int write_cache, int dtype, int* err, cudaStream_t stream, int value_norm_dim) {
     if (n_tokens <= 0) return 0;
-    if (D < 2 || D > 256 || D % 2 || rot_dim < 0 || rot_dim > D || rot_dim % 2 || (rot_dim > 0 && !inv_freq) ||
+    if (D < 2 || D > 256 || D % 2 || value_norm_dim < 0 || value_norm_dim > D || rot_dim < 0 || rot_dim > D || rot_dim % 2 || (rot_dim > 0 && !inv_freq) ||
         row_stride % 2 || ((uintptr_t)rows & 7) || ((uintptr_t)kv & 7))
         return (int)cudaErrorInvalidValue;
     const int heads = n_q + 2 * n_kv;
@@ -476,7 +483,7 @@ extern "C" int ss_rope_norm_cache(void* rows, int64_t row_stride, const int32_t*
         const int lph = D <= 32 ? 4 : (D <= 64 ? 8 : (D <= 128 ? 16 : 32));
 #define RN_GO(LPH)                                                                                                      \
     ss_launch(rope_norm_cache_bf16x8_kernel<LPH>, dim3(n_tokens), dim3(256), 0, stream, (bf16*)rows, row_stride, positions, \
-              slots, inv_freq, mscale, (bf16*)kv, n_q, n_kv, D, rot_dim, norm_dim, eps, page_size, pool, write_cache, err)
+              slots, inv_freq, mscale, (bf16*)kv, n_q, n_kv, D, rot_dim, norm_dim, eps, page_size, pool, write_cache, err, value_norm_dim)
         if (lph == 4) RN_GO(4);
         else if (lph == 8) RN_GO(8);
         else if (lph == 16) RN_GO(16);
@@ -487,11 +494,11 @@ extern "C" int ss_rope_norm_cache(void* rows, int64_t row_stride, const int32_t*
     if (dtype == SS_BF16)
         ss_launch(rope_norm_cache_kernel<bf16>, grid, dim3(warps * 32), 0, stream, (bf16*)rows, row_stride,
                   positions, slots, inv_freq, mscale, (bf16*)kv, n_q, n_kv, D, rot_dim, interleaved, norm_dim, eps,
-                  page_size, pool, write_cache, err);
+                  page_size, pool, write_cache, err, value_norm_dim);
     else
         ss_launch(rope_norm_cache_kernel<float>, grid, dim3(warps * 32), 0, stream, (float*)rows, row_stride,
                   positions, slots, inv_freq, mscale, (float*)kv, n_q, n_kv, D, rot_dim, interleaved, norm_dim, eps,
-                  page_size, pool, write_cache, err);
+                  page_size, pool, write_cache, err, value_norm_dim);
     return SS_LAUNCH_CHECK();
 }
 

@@ -20,7 +20,7 @@ from ctypes import c_float, c_int, c_int64, c_void_p
 import numpy as np
 import torch
 
-from .library import KernelBuildError, load_library, require_cuda
+from .library import OPS_SOURCES, KernelBuildError, load_library, require_cuda
 
 SS_F32, SS_BF16 = 0, 1
 
@@ -56,7 +56,7 @@ _OPS_SIGNATURES = {
     "ss_hc_norm": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int,
                    c_int, c_float, c_int, c_void_p, c_void_p],
     "ss_rope_norm_cache": [c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_int, c_int, c_int, c_int,
-                           c_int, c_int, c_int, c_float, c_int, c_int64, c_int, c_int, c_void_p, c_void_p],
+                           c_int, c_int, c_int, c_float, c_int, c_int64, c_int, c_int, c_void_p, c_void_p, c_int],
     "ss_glu_limited": [c_void_p, c_void_p, c_int64, c_int, c_int, c_float, c_float, c_float, c_float, c_int, c_void_p],
     "ss_sigmoid_gate": [c_void_p, c_int64, c_void_p, c_int64, c_int64, c_int, c_int, c_void_p],
     "ss_group_norm": [c_void_p, c_int, c_int64, c_int, c_void_p, c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_void_p,
@@ -67,7 +67,7 @@ _OPS_SIGNATURES = {
     "ss_ssm_scan": [c_void_p, c_int, c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                     c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int],
     "ss_router": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p,
-                  c_int, c_int, c_void_p, c_int],
+                  c_int, c_int, c_void_p, c_int, c_void_p],
     "ss_moe_plan": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int],
     "ss_moe_gemm": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
                     c_int, c_int, c_int, c_int, c_int, c_void_p, c_int],
@@ -93,7 +93,7 @@ _OPS_SIGNATURES = {
     "ss_latent_rows": [c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_void_p,
                        c_int, c_int, c_int, c_int, c_int, c_int, c_int64, c_float, c_int, c_void_p, c_void_p],
     "ss_decay_attention": [c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
-                           c_int, c_int, c_int, c_void_p, c_void_p],
+                           c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_float],
     "ss_gated_rmsnorm": [c_void_p, c_void_p, c_int64, c_void_p, c_void_p, c_int, c_int, c_float, c_int, c_void_p],
     "ss_block_gates": [c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p],
     "ss_gated_linear_recurrence": [c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_float, c_void_p, c_void_p,
@@ -111,27 +111,31 @@ _OPS_SIGNATURES = {
     "ss_diff_combine": [c_void_p, c_void_p, c_int64, c_int, c_int, c_int, c_float, c_float, c_float, c_int, c_void_p],
     "ss_branch_norm": [c_void_p, c_void_p, c_void_p, c_float, c_float, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_int,
                        c_int, c_int, c_void_p],
+    "ss_embedding_norm": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_float, c_void_p, c_void_p],
+    "ss_head_norm_gate": [c_void_p, c_void_p, c_int64, c_void_p, c_int, c_int, c_int, c_float, c_int, c_void_p],
+    "ss_talk_heads": [c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p],
+    "ss_normed_pair": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_float, c_int, c_void_p],
 }
 
 _ATTN_SIGNATURES = {
     "ss_attn_simt": [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_void_p, c_int, c_void_p,
                      c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int64, c_float,
-                     c_int, c_int, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_int],
+                     c_int, c_int, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_int, c_int],
     "ss_attn_prefill_mma": [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_void_p, c_int, c_void_p,
                             c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int64, c_float,
                             c_int, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_int, c_int, c_int, c_float, c_float,
-                            c_float, c_int],
+                            c_float, c_int, c_int],
     "ss_attn_prefill_tc5": [c_void_p, c_int64, c_int, c_void_p, c_int64, c_void_p, c_void_p, c_int, c_void_p,
                             c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int64, c_float, c_int, c_int,
-                            c_void_p, c_void_p, c_float, c_void_p, c_int, c_int, c_int, c_float, c_float, c_float, c_int],
+                            c_void_p, c_void_p, c_float, c_void_p, c_int, c_int, c_int, c_float, c_float, c_float, c_int, c_int],
     "ss_attn_decode_tma": [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_void_p, c_int, c_int,
                            c_void_p, c_void_p, c_int, c_int, c_int, c_int64, c_float, c_int, c_int,
                            c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_float,
-                           c_void_p, c_int, c_int],
+                           c_void_p, c_int, c_int, c_int],
     "ss_attn_decode_mma": [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_void_p, c_int, c_int,
                            c_void_p, c_void_p, c_int, c_int, c_int, c_int64, c_float, c_int, c_int,
                            c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_int,
-                           c_int],
+                           c_int, c_int],
 }
 
 _GEMM_SIGNATURES = {
@@ -177,7 +181,7 @@ def ops_library() -> ctypes.CDLL:
     lib = _state.get("ops")
     if lib is None:
         require_cuda()
-        lib = load_library("slipstream_ops", ["ops.cu", "ops_streams.cu", "ops_mixers.cu", "ops_cells.cu", "ops_gated.cu", "ops_heads.cu", "sampling.cu"])
+        lib = load_library("slipstream_ops", OPS_SOURCES)
         _declare(lib, _OPS_SIGNATURES)
         _state["ops"] = lib
     return lib  # type: ignore[return-value]
@@ -417,13 +421,14 @@ def hc_norm(streams: torch.Tensor, y: torch.Tensor | None, mix: torch.Tensor | N
 def rope_norm_cache(rows: torch.Tensor, positions: torch.Tensor, slots: torch.Tensor | None,
                     inv_freq: torch.Tensor | None, kv: torch.Tensor | None, n_q: int, n_kv: int, head_dim: int,
                     rotary_dim: int, *, interleaved: bool = False, mscale: float = 1.0, norm_dim: int = 0,
-                    eps: float = 0.0, write_cache: bool = True) -> None:
+                    eps: float = 0.0, write_cache: bool = True, value_norm_dim: int = 0) -> None:
     """Rotation, unit norm and page write for one layer's projected heads.  ``rows`` [N, width]: each row starts
     with ``n_q`` query heads, then ``n_kv`` key heads and ``n_kv`` value heads (``n_kv`` 0: queries only) of
     ``head_dim`` elements; whatever follows them in a row is left alone.  The first ``rotary_dim`` elements of
     queries and keys are rotated by position * ``inv_freq`` in pairs (2i, 2i+1) (``interleaved``) or
     (i, i + rotary_dim / 2), cosines and sines times ``mscale``; with ``norm_dim`` > 0 each query and key head is
-    then divided by ``sqrt(sum(x^2) / norm_dim + eps)``.  Queries change in place; keys and values go to their
+    then divided by ``sqrt(sum(x^2) / norm_dim + eps)``, with ``value_norm_dim`` > 0 each value head likewise over that many
+    elements.  Queries change in place; keys and values go to their
     pages ``kv`` [pages, 2, n_kv, page_size, head_dim] at ``slots`` (-1 or ``write_cache`` False: keys in place)."""
     _need(rows, None, "projected rows")
     _need(positions, torch.int32, "positions")
@@ -449,7 +454,7 @@ def rope_norm_cache(rows: torch.Tensor, positions: torch.Tensor, slots: torch.Te
                                             _ptr(kv) if write else None, n, n_q, n_kv, head_dim, rotary_dim,
                                             int(interleaved), int(norm_dim), float(eps), max(page_size, 1), pages,
                                             int(write), _code(rows.dtype), error_word(rows.device).data_ptr(),
-                                            _stream()), "rope_norm_cache")
+                                            _stream(), int(value_norm_dim)), "rope_norm_cache")
 
 
 def glu_limited(gate_up: torch.Tensor, block: int | None = None, alpha: float = 1.0, limit: float = 0.0,
@@ -618,7 +623,7 @@ def paged_attention_simt(q: torch.Tensor, q_stride: int, out: torch.Tensor, kv: 
                          q_start: torch.Tensor, seq_lens: torch.Tensor, n_q: int, n_kv: int,
                          head_dim: int, scale: float, window: int = 0, chunk: int = 0,
                          gate: torch.Tensor | None = None, softcap: float = 0.0,
-                         sinks: torch.Tensor | None = None, keep: int = 0) -> None:
+                         sinks: torch.Tensor | None = None, keep: int = 0, across: bool = False) -> None:
     """Causal grouped-query attention of the step's query rows over the pages (``window`` / ``chunk``: `key_span`).
     ``softcap`` c > 0 (in every attention entry point but the tcgen05 one): a scaled score s enters the softmax as
     ``c * tanh(s / c)``.
@@ -630,7 +635,9 @@ def paged_attention_simt(q: torch.Tensor, q_stride: int, out: torch.Tensor, kv: 
     of one request (request index, first token within the request's rows of this step).
     ``keep`` (in every attention entry point; with ``window``): the request's first ``keep`` keys stay visible.
     ``sinks`` (in every attention entry point; float32 [n_q]): the softmax's denominator of head h also
-    holds ``exp(sinks[h])``, a term of its own with neither key nor value, which the scale does not touch."""
+    holds ``exp(sinks[h])``, a term of its own with neither key nor value, which the scale does not touch.
+    ``across`` (in every attention entry point; without a gate): every query head's weights meet the values of every kv head:
+    ``out`` is [N, n_kv * n_q * D], head (a * n_kv + c) * G + r holding query head a * G + r over the values of kv head c."""
     _need(out, q.dtype, "attention output")
     _check_sinks(sinks, n_q)
     _need(kv, q.dtype, "kv pages")
@@ -643,7 +650,7 @@ def paged_attention_simt(q: torch.Tensor, q_stride: int, out: torch.Tensor, kv: 
                             tile_q0.data_ptr(), tile_req.numel(), q_start.data_ptr(), seq_lens.data_ptr(),
                             n_q, n_kv, kv.shape[3], kv.shape[0], float(scale), key_span(window, chunk),
                             _code(q.dtype), _gate_ptr(gate, q, q_stride), error_word(q.device).data_ptr(), _stream(),
-                            float(softcap or 0.0), _ptr(sinks), _kept(keep, window)),
+                            float(softcap or 0.0), _ptr(sinks), _kept(keep, window), int(across)),
            "paged_attention_simt")
 
 
@@ -652,7 +659,7 @@ def paged_attention_prefill(q: torch.Tensor, q_stride: int, out: torch.Tensor, k
                             q_start: torch.Tensor, seq_lens: torch.Tensor, n_q: int, n_kv: int, head_dim: int,
                             scale: float, window: int = 0, chunk: int = 0, gate: torch.Tensor | None = None,
                             softcap: float = 0.0, sinks: torch.Tensor | None = None, keep: int = 0,
-                            diff: DiffPair | None = None) -> None:
+                            diff: DiffPair | None = None, across: bool = False) -> None:
     """bfloat16 tensor-core attention for prompt portions and mixed batches.  A tile is 64 consecutive
     rows of one request, a row being a (query token, head of the kv group) pair in token-major order:
     ``tile_req`` / ``tile_row0`` list (request index, first row).  ``out`` bfloat16, or float32 without ``gate`` and
@@ -672,7 +679,7 @@ def paged_attention_prefill(q: torch.Tensor, q_stride: int, out: torch.Tensor, k
                                    tile_row0.data_ptr(), tile_req.numel(), q_start.data_ptr(), seq_lens.data_ptr(),
                                    n_q, n_kv, kv.shape[3], kv.shape[0], float(scale), key_span(window, chunk),
                                    _gate_ptr(gate, q, q_stride), error_word(q.device).data_ptr(), _stream(),
-                                   float(softcap or 0.0), _ptr(sinks), _kept(keep, window), out_f32, *_diff_args(diff)),
+                                   float(softcap or 0.0), _ptr(sinks), _kept(keep, window), out_f32, *_diff_args(diff), int(across)),
            "paged_attention_prefill")
 
 
@@ -695,7 +702,7 @@ def paged_attention_prefill_tcgen05(q: torch.Tensor, q_stride: int, out: torch.T
                                     q_start: torch.Tensor, seq_lens: torch.Tensor, n_q: int, n_kv: int,
                                     head_dim: int, scale: float, key_parts: int = 1, chunk: int = 0, window: int = 0,
                                     softcap: float = 0.0, sinks: torch.Tensor | None = None, keep: int = 0,
-                                    diff: DiffPair | None = None) -> None:
+                                    diff: DiffPair | None = None, across: bool = False) -> None:
     """bfloat16 causal attention for prompt portions and mixed batches on the tcgen05 tensor cores (Q, K, V
     tiles by TMA, S and O in tensor memory).  A tile is ``128 // (n_q // n_kv)`` consecutive query tokens of
     one request: ``tile_req`` / ``tile_tok0`` list (request index, first token within the request's rows); blocks
@@ -721,7 +728,7 @@ def paged_attention_prefill_tcgen05(q: torch.Tensor, q_stride: int, out: torch.T
                                    tile_tok0.data_ptr(), tile_req.numel(), q_start.data_ptr(), seq_lens.data_ptr(),
                                    n_q, n_kv, kv.shape[3], kv.shape[0], float(scale), int(key_parts),
                                    key_span(window, chunk), error_word(q.device).data_ptr(), _stream(),
-                                   float(softcap or 0.0), _ptr(sinks), _kept(keep, window), out_f32, *_diff_args(diff)),
+                                   float(softcap or 0.0), _ptr(sinks), _kept(keep, window), out_f32, *_diff_args(diff), int(across)),
            "paged_attention_prefill_tcgen05")
 
 
@@ -776,7 +783,8 @@ def paged_attention_decode(q: torch.Tensor, q_stride: int, out: torch.Tensor, kv
                            n_slices: int = 1, scratch: tuple[torch.Tensor, torch.Tensor] | None = None,
                            rope: tuple[torch.Tensor | None, int] | None = None, tma: bool | None = None,
                            stages: int = 2, chunk: int = 0, gate: torch.Tensor | None = None,
-                           softcap: float = 0.0, sinks: torch.Tensor | None = None, keep: int = 0) -> None:
+                           softcap: float = 0.0, sinks: torch.Tensor | None = None, keep: int = 0,
+                           across: bool = False) -> None:
     """bfloat16 attention for requests that bring ONE token each, the keys of every request cut into
     ``n_slices`` slices that run in parallel.  Up to 8 slices form a thread-block cluster and are combined
     through shared memory; with more, the partial results (of every cluster of 8 in the TMA-fed kernel when the
@@ -804,14 +812,15 @@ def paged_attention_decode(q: torch.Tensor, q_stride: int, out: torch.Tensor, kv
     for name, t in (("block_tables", block_tables), ("q_start", q_start), ("seq_lens", seq_lens)):
         _need(t, torch.int32, name)
     part_o = part_lse = counters = None
+    n_blocks, n_out = (n_kv * n_kv, n_kv * n_q) if across else (n_kv, n_q)
     if n_slices > 8:
         counters = decode_counters(q.device)
-        if n_requests * n_kv * ((n_q // n_kv + 15) // 16) > _DECODE_COUNTERS:
+        if n_requests * n_blocks * ((n_q // n_kv + 15) // 16) > _DECODE_COUNTERS:
             raise KernelError("too many (request, head block) pairs for the decode counters")
         if scratch is None:
-            scratch = decode_scratch(n_requests, n_q, n_slices, head_dim, q.device)
+            scratch = decode_scratch(n_requests, n_out, n_slices, head_dim, q.device)
         part_o, part_lse = scratch
-        if part_o.numel() < n_requests * n_q * n_slices * head_dim or part_lse.numel() < n_requests * n_q * n_slices:
+        if part_o.numel() < n_requests * n_out * n_slices * head_dim or part_lse.numel() < n_requests * n_out * n_slices:
             raise KernelError("decode scratch is too small")
     inv_freq, rotary_dim = rope if rope is not None else (None, 0)
     if rope is not None:
@@ -832,10 +841,10 @@ def paged_attention_decode(q: torch.Tensor, q_stride: int, out: torch.Tensor, kv
         raise KernelError("a gated layer does not rotate inside the decode kernel")
     tail = (_gate_ptr(gate, q, q_stride), error_word(q.device).data_ptr(), _stream(), float(softcap or 0.0))
     if tma:
-        _check(lib.ss_attn_decode_tma(*args, int(stages), *tail, _ptr(sinks), _kept(keep, window), out_f32),
+        _check(lib.ss_attn_decode_tma(*args, int(stages), *tail, _ptr(sinks), _kept(keep, window), out_f32, int(across)),
                "paged_attention_decode")
     else:
-        _check(lib.ss_attn_decode_mma(*args, *tail, _ptr(sinks), _kept(keep, window), out_f32), "paged_attention_decode")
+        _check(lib.ss_attn_decode_mma(*args, *tail, _ptr(sinks), _kept(keep, window), out_f32, int(across)), "paged_attention_decode")
 
 
 WIDE_CONTEXT = 8192  # from this many cached tokens a decode step of few requests may use more than 8 slices
@@ -891,7 +900,7 @@ def paged_attention(qkv: torch.Tensor, out: torch.Tensor, kv: torch.Tensor, bloc
                     ctx, n_q: int, n_kv: int, head_dim: int, scale: float, window: int = 0,
                     rope: tuple[torch.Tensor | None, int] | None = None, chunk: int = 0,
                     gate: torch.Tensor | None = None, softcap: float = 0.0, sinks: torch.Tensor | None = None,
-                    keep: int = 0, diff: DiffPair | None = None) -> None:
+                    keep: int = 0, diff: DiffPair | None = None, across: bool = False) -> None:
     """Attention of the step's rows over the pages, choosing the kernel for the batch.
 
     ``qkv`` is the stacked projection output [N, (n_q + 2 n_kv) * D] whose first n_q heads are the
@@ -912,16 +921,22 @@ def paged_attention(qkv: torch.Tensor, out: torch.Tensor, kv: torch.Tensor, bloc
     ``diff``: query heads 2h and 2h + 1 are the two maps of a differential head and ``out`` [N, n_q / 2 * diff.dim] takes
     the combined heads.  The prefill kernels combine them as they write; where they cannot (decode steps, keys cut into
     parts, float32), the heads are written in float32 and `diff_combine` follows, so the difference is formed from
-    unrounded outputs either way."""
+    unrounded outputs either way.
+
+    ``across``: every query head over the values of every kv head (see `paged_attention_simt`), ``out`` float32; `talk_heads`
+    is what mixes them."""
     if diff is not None and gate is not None:
         raise KernelError("a gate on differential heads is not built")
+    if across and (diff is not None or gate is not None or rope is not None):
+        raise KernelError("attention across all values comes without gates, differential heads and rotation inside")
+    n_blocks = n_kv * n_kv if across else n_kv  # (keys' kv head, values' kv head) pairs the kernels walk
     if rope is not None and not (qkv.dtype == torch.bfloat16 and ctx.is_decode_only):
         raise KernelError("only bfloat16 decode steps rotate inside the attention kernel")
     if qkv.dtype == torch.float32:
         tile_req, tile_q0 = ctx.query_tiles(16)
         heads = out if diff is None else _heads_f32(out, n_q, head_dim)
         paged_attention_simt(qkv, qkv.shape[1], heads, kv, block_tables, tile_req, tile_q0, ctx.q_start,
-                             ctx.seq_lens, n_q, n_kv, head_dim, scale, window, chunk, gate, softcap, sinks, keep)
+                             ctx.seq_lens, n_q, n_kv, head_dim, scale, window, chunk, gate, softcap, sinks, keep, across)
         if diff is not None:
             diff_combine(heads, diff, n_q // 2, out)
         return
@@ -931,29 +946,30 @@ def paged_attention(qkv: torch.Tensor, out: torch.Tensor, kv: torch.Tensor, bloc
         longest = static or ctx.max_seq_len
         wide = ctx.extras.get("decode_wide", False) if static else is_long_context(ctx.max_seq_len)
         wide = bool(wide) and tcgen05_attention_fits(head_dim, n_q, n_kv, kv.shape[3], 0)
-        slices = decode_slices(ctx.num_requests, n_kv, group, min(longest, (window or chunk or longest) + keep), wide,
+        slices = decode_slices(ctx.num_requests, n_blocks, group, min(longest, (window or chunk or longest) + keep), wide,
                                sm_count(qkv.device))
-        scratch = ctx.extras.get(("decode_scratch", n_q, head_dim))
+        scratch = ctx.extras.get(("decode_scratch", n_q, head_dim)) if not across else None
         heads = out if diff is None else _heads_f32(out, n_q, head_dim)
         paged_attention_decode(qkv, qkv.shape[1], heads, kv, block_tables, ctx.q_start, ctx.seq_lens,
                                ctx.num_requests, n_q, n_kv, head_dim, scale, window, slices, scratch, rope,
-                               stages=DECODE_RING_STAGES, chunk=chunk, gate=gate, softcap=softcap, sinks=sinks, keep=keep)
+                               stages=DECODE_RING_STAGES, chunk=chunk, gate=gate, softcap=softcap, sinks=sinks, keep=keep,
+                               across=across)
         if diff is not None:
             diff_combine(heads, diff, n_q // 2, out)
         return
     fused = diff is None or diff_in_attention(diff, n_q, n_kv)
     if tcgen05_prefill_fits(head_dim, n_q, n_kv, kv.shape[3]):
         tile_req, tile_tok0 = ctx.query_tiles_longest_first(128 // group)
-        key = ("prefill_key_parts", 128 // group, n_kv, (window or chunk) + keep)
+        key = ("prefill_key_parts", 128 // group, n_blocks, (window or chunk) + keep)
         parts = ctx.extras.get(key)
         if parts is None:  # the same for every layer of the step that sees as far
-            parts = ctx.extras[key] = prefill_key_parts(ctx.q_lens_host, ctx.seq_lens_host, 128 // group, n_kv,
+            parts = ctx.extras[key] = prefill_key_parts(ctx.q_lens_host, ctx.seq_lens_host, 128 // group, n_blocks,
                                                         sm_count(qkv.device), (window or chunk) + keep)
         fused = fused and (diff is None or parts == 1)
         heads = out if fused else _heads_f32(out, n_q, head_dim)
         paged_attention_prefill_tcgen05(qkv, qkv.shape[1], heads, kv, block_tables, tile_req, tile_tok0, ctx.q_start,
                                         ctx.seq_lens, n_q, n_kv, head_dim, scale, parts, chunk, window, softcap, sinks, keep,
-                                        diff if fused else None)
+                                        diff if fused else None, across)
         if not fused:
             diff_combine(heads, diff, n_q // 2, out)
         if gate is not None:
@@ -963,7 +979,7 @@ def paged_attention(qkv: torch.Tensor, out: torch.Tensor, kv: torch.Tensor, bloc
     heads = out if fused else _heads_f32(out, n_q, head_dim)
     paged_attention_prefill(qkv, qkv.shape[1], heads, kv, block_tables, tile_req, tile_row0, ctx.q_start,
                             ctx.seq_lens, n_q, n_kv, head_dim, scale, window, chunk, gate, softcap, sinks, keep,
-                            diff if fused else None)
+                            diff if fused else None, across)
     if not fused:
         diff_combine(heads, diff, n_q // 2, out)
 
@@ -1719,8 +1735,8 @@ def ssm_scan(xbc: torch.Tensor, dt: torch.Tensor, dt_bias: torch.Tensor, a_log: 
 
 def router(x: torch.Tensor, weight: torch.Tensor, top: int, renormalize: bool = False, *, softmax: bool = False,
            correction: torch.Tensor | None = None, groups: int = 1, keep: int = 1,
-           extra: int = 0) -> "tuple[torch.Tensor, torch.Tensor] | tuple[torch.Tensor, torch.Tensor, torch.Tensor]":
-    """Router: logits ``x @ weight.T`` in float32, scores their sigmoid (or, with ``softmax``, their softmax over all
+           extra: int = 0, bias: torch.Tensor | None = None) -> "tuple[torch.Tensor, torch.Tensor] | tuple[torch.Tensor, torch.Tensor, torch.Tensor]":
+    """Router: logits ``x @ weight.T + bias`` (``bias`` float32 [experts] or None) in float32, scores their sigmoid (or, with ``softmax``, their softmax over all
     experts), the ``top`` largest per token chosen (the lower index on a tie).  ``correction`` (float32 [experts]) is
     added to the scores for the choice only.  ``groups`` > 1: the experts form that many equal groups of neighbours, a
     group's score is its largest choice score, and only experts of the ``keep`` best groups can be chosen.  Returns
@@ -1740,12 +1756,16 @@ def router(x: torch.Tensor, weight: torch.Tensor, top: int, renormalize: bool = 
         _need(correction, torch.float32, "correction")
         if correction.numel() != experts:
             raise KernelError("router: one correction per expert")
+    if bias is not None:
+        _need(bias, torch.float32, "router bias")
+        if bias.numel() != experts:
+            raise KernelError("router: one bias per expert")
     ids = torch.empty((n, top), dtype=torch.int32, device=x.device)
     scores = torch.empty((n, top), dtype=torch.float32, device=x.device)
     rest = torch.empty((n, extra), dtype=torch.float32, device=x.device) if extra else None
     _check(ops_library().ss_router(x.data_ptr(), weight.data_ptr(), ids.data_ptr(), scores.data_ptr(), n, hidden, experts,
                                    int(top), int(renormalize), _code(x.dtype), _stream(), int(softmax), _ptr(correction),
-                                   int(groups), int(keep), _ptr(rest), int(extra)), "router")
+                                   int(groups), int(keep), _ptr(rest), int(extra), _ptr(bias)), "router")
     return (ids, scores, rest) if extra else (ids, scores)
 
 
@@ -1755,11 +1775,11 @@ MOE_TILE = 64  # rows of one expert that a block of the grouped products takes
 GROUPED_TCGEN05_ROWS = 1024  # from this many (token, choice) pairs the experts' products run the two-SM tcgen05 kernel
 
 
-def moe_experts(x: torch.Tensor, ids: torch.Tensor, scores: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor,
+def moe_experts(x: torch.Tensor, ids: torch.Tensor, scores: torch.Tensor | None, gate_up: torch.Tensor, down: torch.Tensor,
                 run: int | None = None) -> tuple[torch.Tensor, torch.Tensor | None]:
     """The chosen experts of every token: ``y[t, k] = W_down[e] (silu(W_gate[e] a) * (W_up[e] a))`` with
     ``e = ids[t, k]`` and ``a = scores[t, k] * x[t]`` (the score multiplies the expert's INPUT), rounded to the
-    compute dtype.  ``gate_up`` [experts, 2 ff, hidden]: gate and up rows alternating in runs of ``run`` (default ff:
+    compute dtype; ``scores`` None: ``a = x[t]`` (`moe_mix` may weigh the outputs).  ``gate_up`` [experts, 2 ff, hidden]: gate and up rows alternating in runs of ``run`` (default ff:
     all gate rows, then all up rows); ``down`` [experts, hidden, ff].
 
     Returns (terms, term_rows): either float32 [N, top, hidden] and None, or, from the tcgen05 path, bfloat16
@@ -1777,7 +1797,8 @@ def moe_experts(x: torch.Tensor, ids: torch.Tensor, scores: torch.Tensor, gate_u
     _need(gate_up, x.dtype, "gate_up")
     _need(down, x.dtype, "down")
     _need(ids, torch.int32, "ids")
-    _need(scores, torch.float32, "scores")
+    if scores is not None:
+        _need(scores, torch.float32, "scores")
     if tuple(down.shape) != (experts, hidden, ff) or gate_up.shape[2] != hidden or run < 1 or ff % run:
         raise KernelError("moe_experts: weights of the wrong shape")
     a = n * top
@@ -1795,7 +1816,7 @@ def moe_experts(x: torch.Tensor, ids: torch.Tensor, scores: torch.Tensor, gate_u
     lists = (perm.data_ptr(), tile_expert.data_ptr(), tile_row0.data_ptr(), tile_rows.data_ptr())
     if tensor_cores:
         gathered = torch.empty((a, hidden), dtype=x.dtype, device=x.device)
-        _check(lib.ss_moe_gather(x.data_ptr(), scores.data_ptr(), perm.data_ptr(), gathered.data_ptr(), a, top, hidden,
+        _check(lib.ss_moe_gather(x.data_ptr(), _ptr(scores), perm.data_ptr(), gathered.data_ptr(), a, top, hidden,
                                  _stream()), "moe_gather")
     if tcgen05:
         err = error_word(x.device).data_ptr()
@@ -1814,7 +1835,7 @@ def moe_experts(x: torch.Tensor, ids: torch.Tensor, scores: torch.Tensor, gate_u
         _check(lib.ss_moe_gemm_mma(hidden_act.data_ptr(), down.data_ptr(), *lists, None, y.data_ptr(), ff, hidden,
                                    max_tiles, tile, 0, 0, int(a <= 4), _stream()), "moe_down")
         return y, None
-    _check(lib.ss_moe_gemm(x.data_ptr(), scores.data_ptr(), gate_up.data_ptr(), *lists, hidden_act.data_ptr(), None, top,
+    _check(lib.ss_moe_gemm(x.data_ptr(), _ptr(scores), gate_up.data_ptr(), *lists, hidden_act.data_ptr(), None, top,
                            hidden, ff, max_tiles, 1, _code(x.dtype), run, _stream(), 0), "moe_up")
     _check(lib.ss_moe_gemm(hidden_act.data_ptr(), None, down.data_ptr(), *lists, None, y.data_ptr(), top, ff, hidden,
                            max_tiles, 0, _code(x.dtype), 0, _stream(), 0), "moe_down")
@@ -2117,11 +2138,15 @@ def head_product(x: torch.Tensor, x_head: int, weight: torch.Tensor, out: torch.
 # --------------------------------------------------------------------------- decayed linear attention, gated linear recurrence
 
 def decay_attention(proj: torch.Tensor, decay: torch.Tensor, state: torch.Tensor, ctx, heads: int, dim: int,
-                    value_dim: int) -> torch.Tensor:
+                    value_dim: int, *, silu: bool = True, inv_freq: torch.Tensor | None = None, k_scale: float = 1.0) -> torch.Tensor:
     """Linear attention with a fixed decay per head over each request's tokens, continued from and left in ``state``
     (float32 [slots, heads, dim, value_dim]).  A row of ``proj`` starts with the heads' queries, then keys (``dim``
     each), then values (``value_dim``), all before their activation; whatever follows is left alone.  Per head h, token
-    by token: ``S <- decay[h] S + silu(k) silu(v)^T``, ``o = S^T silu(q)``.  Returns o float32 [N, heads * value_dim]."""
+    by token: ``S <- decay[h] S + silu(k) silu(v)^T``, ``o = S^T silu(q)``.  Returns o float32 [N, heads * value_dim].
+
+    ``silu`` False: no activation; the first ``2 * len(inv_freq)`` elements of queries and keys are rotated by the row's
+    position * ``inv_freq`` in pairs (i, i + len(inv_freq)) (None: not at all), in float32, and keys are multiplied by
+    ``k_scale``."""
     _need(proj, None, "projected rows")
     _need(decay, torch.float32, "decay")
     _need(state, torch.float32, "state")
@@ -2130,11 +2155,18 @@ def decay_attention(proj: torch.Tensor, decay: torch.Tensor, state: torch.Tensor
         raise KernelError("decay_attention: the rows are narrower than their heads, or sizes out of range")
     if tuple(state.shape[1:]) != (heads, dim, value_dim):
         raise KernelError("decay_attention: the state must be [slots, heads, dim, value_dim]")
+    half = 0
+    if inv_freq is not None:
+        _need(inv_freq, torch.float32, "inv_freq")
+        half = inv_freq.numel()
+        if silu or not 0 < 2 * half <= dim:
+            raise KernelError("decay_attention: a rotation comes without the activation and covers at most the head")
     out = torch.empty((n, heads * value_dim), dtype=torch.float32, device=proj.device)
     _check(ops_library().ss_decay_attention(proj.data_ptr(), proj.stride(0), decay.data_ptr(), state.data_ptr(),
                                             out.data_ptr(), ctx.q_start.data_ptr(), ctx.seq_lens.data_ptr(),
                                             ctx.state_slots.data_ptr(), ctx.num_requests, heads, dim, value_dim,
-                                            state.shape[0], _code(proj.dtype), error_word(proj.device).data_ptr(), _stream()),
+                                            state.shape[0], _code(proj.dtype), error_word(proj.device).data_ptr(), _stream(),
+                                            int(silu), _ptr(inv_freq), half, float(k_scale)),
            "decay_attention")
     return out
 
@@ -2341,6 +2373,75 @@ def moe_mix(y: torch.Tensor, term_rows: torch.Tensor | None, ids: torch.Tensor, 
     return out
 
 
+# --------------------------------------------------------------------------- embedding under a norm, retention, talking heads
+
+def embedding_norm(token_ids: torch.Tensor, table: torch.Tensor, weight: torch.Tensor, eps: float, scale: float = 1.0) -> torch.Tensor:
+    """Rows of ``table`` at ``token_ids`` (int32 [N]), times ``scale``, under an RMS norm with ``weight`` (float32 [hidden]),
+    as float32 [N, hidden]."""
+    _need(token_ids, torch.int32, "token_ids")
+    _need(table, None, "embedding table")
+    _need(weight, torch.float32, "norm weight")
+    n, (vocab, hidden) = token_ids.numel(), table.shape
+    if weight.numel() != hidden:
+        raise KernelError("norm weight has the wrong size")
+    out = torch.empty((n, hidden), dtype=torch.float32, device=table.device)
+    _check(ops_library().ss_embedding_norm(token_ids.data_ptr(), table.data_ptr(), weight.data_ptr(), out.data_ptr(), n, hidden,
+                                           vocab, _code(table.dtype), float(scale), float(eps),
+                                           error_word(table.device).data_ptr(), _stream()), "embedding_norm")
+    return out
+
+
+def head_norm_gate(x: torch.Tensor, gate: torch.Tensor, heads: int, eps: float, out_dtype: torch.dtype) -> torch.Tensor:
+    """Every head of ``x`` (float32 [N, heads * dim]) divided by its root mean square (``eps`` inside the root, no weight), times
+    ``silu(gate)`` (a view of that shape in ``out_dtype`` with unit inner stride); float32 arithmetic, one rounding."""
+    _need(x, torch.float32, "x")
+    n, c = x.shape
+    if gate.dtype != out_dtype or tuple(gate.shape) != (n, c) or gate.stride(1) != 1 or heads < 1 or c % heads:
+        raise KernelError("head_norm_gate: x must split into heads and the gate be [N, heads * dim] with unit inner stride")
+    out = torch.empty((n, c), dtype=out_dtype, device=x.device)
+    _check(ops_library().ss_head_norm_gate(x.data_ptr(), gate.data_ptr(), gate.stride(0), out.data_ptr(), n, heads, c // heads,
+                                           float(eps), _code(out_dtype), _stream()), "head_norm_gate")
+    return out
+
+
+def talk_heads(x: torch.Tensor, table_t: torch.Tensor, n_kv: int, out_dtype: torch.dtype,
+               gate: torch.Tensor | None = None) -> torch.Tensor:
+    """Mixtures over heads of attention weights, applied to what `paged_attention` leaves with ``across``.  ``x`` float32
+    [N, n_kv * H * D]: entry (a, c, r) is query head ``a * G + r`` (G = H / n_kv) over the values of kv head c; ``table_t``
+    float32 [H, H], ``table_t[g, h]`` the weight with which head h's mixture takes head g's.  Returns [N, H * D]:
+    ``sigmoid(gate[:, h]) * sum_g table_t[g, h] x[(g // G, h // G, g % G)]`` (``gate`` a view of the result's shape in
+    ``out_dtype`` with unit inner stride, or None), formed in float32 and rounded once."""
+    _need(x, torch.float32, "x")
+    _need(table_t, torch.float32, "table")
+    n, h = x.shape[0], table_t.shape[0]
+    d = x.shape[1] // (n_kv * h)
+    if tuple(table_t.shape) != (h, h) or h % n_kv or x.shape[1] != n_kv * h * d or d % 4:
+        raise KernelError("talk_heads: sizes do not match")
+    if gate is not None and (gate.dtype != out_dtype or tuple(gate.shape) != (n, h * d) or gate.stride(1) != 1):
+        raise KernelError("talk_heads: the gate must be a view [N, H * D] in the compute dtype with unit inner stride")
+    out = torch.empty((n, h * d), dtype=out_dtype, device=x.device)
+    _check(ops_library().ss_talk_heads(x.data_ptr(), table_t.data_ptr(), _ptr(gate), gate.stride(0) if gate is not None else 0,
+                                       out.data_ptr(), n, n_kv, h // n_kv, d, _code(out_dtype), _stream()), "talk_heads")
+    return out
+
+
+def normed_pair(a: torch.Tensor, a_weight: torch.Tensor, b: torch.Tensor, b_weight: torch.Tensor, eps: float,
+                scale: float) -> torch.Tensor:
+    """``scale * (rmsnorm(a) * a_weight + rmsnorm(b) * b_weight)`` row by row: ``a``, ``b`` [N, C] of one dtype, weights float32
+    [C]; float32 arithmetic, one rounding."""
+    _need(a, None, "a")
+    _need(b, a.dtype, "b")
+    _need(a_weight, torch.float32, "a's norm weight")
+    _need(b_weight, torch.float32, "b's norm weight")
+    n, c = a.shape
+    if b.shape != a.shape or a_weight.numel() != c or b_weight.numel() != c:
+        raise KernelError("normed_pair: shapes differ")
+    out = torch.empty_like(a)
+    _check(ops_library().ss_normed_pair(a.data_ptr(), a_weight.data_ptr(), b.data_ptr(), b_weight.data_ptr(), out.data_ptr(), n, c,
+                                        float(eps), float(scale), _code(a.dtype), _stream()), "normed_pair")
+    return out
+
+
 def set_programmatic_launch(enabled: bool) -> None:
     """Turn programmatic dependent launch of this package's kernels on or off (on by default)."""
     libs = [ops_library(), gemm_library()] + [lib for key, lib in _state.items() if isinstance(key, str) and key.startswith("attn")]
@@ -2357,4 +2458,5 @@ __all__ = ["KernelError", "KernelBuildError", "embedding", "add_rmsnorm", "hc_no
            "norm_rope_cache", "turn_heads", "soft_cap", "embed_sum", "matrix_cell", "cell_output", "gated_recurrence", "xielu",
            "DiffPair", "diff_in_attention", "diff_combine", "heads_to_pages", "branch_norm",
            "latent_rows", "head_product", "decay_attention", "gated_rmsnorm", "block_gates", "gated_linear_recurrence", "head_gate",
+           "embedding_norm", "head_norm_gate", "talk_heads", "normed_pair",
            "scaled_sum", "relu_square", "moe_experts_single", "moe_mix"]

@@ -25,6 +25,9 @@ import threading
 import time
 from pathlib import Path
 
+# the row-wise operations and recurrences of every design: one library
+OPS_SOURCES = ["ops.cu", "ops_streams.cu", "ops_mixers.cu", "ops_cells.cu", "ops_gated.cu", "ops_heads.cu", "ops_retention.cu",
+               "sampling.cu"]
 CSRC = Path(__file__).resolve().parent.parent / "csrc"
 ARCH_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a"]
 BASE_FLAGS = ["-O3", "-std=c++17", "-lineinfo", "--shared", "-Xcompiler", "-fPIC",

@@ -27,8 +27,14 @@ score s enters the softmax as ``c tanh(s / c)``.  ``head_gate``: head h's output
 the scale does not touch.  ``keep_first`` K (with ``window``): a query also sees the request's first K keys, at their true
 positions.  ``joint_norm_eps``: before the rotation ONE RMS norm over all query heads of a token together, and one over
 all its key heads, with weights of the whole projections' sizes (tensors ``q_norm`` / ``k_norm``).  ``tied_values``: the
-values are the keys as projected, before norm and rotation; there is no v.  ``names``: the checkpoint's tensor names by
-role (q, k, v, o, g, q_bias, k_bias, v_bias, o_bias, q_norm, k_norm, sink).
+values are the keys as projected, before norm and rotation; there is no v.  ``value_norm_eps``: every value head is divided
+by its root mean square (no weight) and cached so.  ``talk``: TALKING HEADS: behind the softmax, head h's weights become
+``sum_g T[h, g] weights_g`` over all query heads g (tensor ``talk`` [heads, heads]), and those are applied to the values of
+h's own key/value head.  How it runs: mixing the weights before they meet the values is the same sum as mixing, per
+key/value head, what every head's own weights make of its values, so the attention kernels walk pairs of (keys' head,
+values' head) and leave every query head over the values of every key/value head in float32, and `ops.talk_heads` forms the
+mixture and applies the gate; the softmax stays inside the kernels and no weights are ever written.  ``names``: the checkpoint's tensor names by
+role (q, k, v, o, g, q_bias, k_bias, v_bias, o_bias, q_norm, k_norm, sink, talk).
 
 Heads of a size the kernels do not take (they take multiples of 16), or values of another size than keys, are
 padded with zeros where the weights are bound: q/k/v/g rows and o columns of the padding are zero, so the
@@ -57,12 +63,13 @@ class PagedAttention(Mixer):
                  gate: bool = False, has_kv: bool = True, names: dict[str, str] | None = None,
                  qk_norm_eps: float | None = None, rotate_values: bool = False, softcap: float | None = None,
                  head_gate: bool = False, unit_sink: bool = False, learned_sinks: bool = False, keep_first: int = 0,
-                 joint_norm_eps: float | None = None, tied_values: bool = False) -> None:
+                 joint_norm_eps: float | None = None, tied_values: bool = False, value_norm_eps: float | None = None,
+                 talk: bool = False) -> None:
         if num_heads % num_kv_heads != 0:
             raise ValueError(f"num_heads ({num_heads}) must be divisible by num_kv_heads ({num_kv_heads})")
         value_dim = head_dim if value_dim is None else int(value_dim)
-        if head_dim % 2 or not 2 <= head_dim <= 256 or not 1 <= value_dim <= 256:
-            raise ValueError(f"head sizes are even and at most 256 (values: at most 256), not {head_dim} / {value_dim}")
+        if not 1 <= head_dim <= 256 or not 1 <= value_dim <= 256 or (head_dim % 2 and position_encoding.rotary_table()[1]):
+            raise ValueError(f"head sizes are at most 256, and even where they are rotated, not {head_dim} / {value_dim}")
         if window is not None and window < 1:
             raise ValueError("window must be >= 1")
         if chunk is not None and chunk < 1:
@@ -107,6 +114,13 @@ class PagedAttention(Mixer):
             raise ValueError("values that are the keys have the keys' size")
         if self.qk_norm_eps is not None and unit_norm_eps is not None:
             raise ValueError("a layer norms its heads before the rotation or after it, not both")
+        self.talk = bool(talk)
+        self.value_norm_eps = None if value_norm_eps is None else float(value_norm_eps)
+        if self.value_norm_eps is not None and (self.spread or qk_norm_eps is not None or rotate_values
+                                                or self.value_norm_eps != (self.unit_norm_eps if unit_norm_eps is not None else self.value_norm_eps)):
+            raise ValueError("a norm on the values comes beside unit norms of the same eps, or alone, without other norms")
+        if self.talk and (head_gate or rotate_values):
+            raise ValueError("talking heads come without a gate per head and without rotated values")
         self.has_kv = bool(has_kv)
         self.page_size = page_size  # tokens per cache page this layer wants; None: the engine's default
         self.scale = head_dim ** -0.5 if scale is None else float(scale)
@@ -114,7 +128,7 @@ class PagedAttention(Mixer):
         self.names = {"q": f"{n}.q_proj.weight", "k": f"{n}.k_proj.weight", "v": f"{n}.v_proj.weight",
                       "o": f"{n}.o_proj.weight", "g": f"{n}.g_proj.weight", "q_bias": f"{n}.q_proj.bias",
                       "k_bias": f"{n}.k_proj.bias", "v_bias": f"{n}.v_proj.bias", "o_bias": f"{n}.o_proj.bias",
-                      "q_norm": f"{n}.q_norm.weight", "k_norm": f"{n}.k_norm.weight", "sink": f"{n}.sink"}
+                      "q_norm": f"{n}.q_norm.weight", "k_norm": f"{n}.k_norm.weight", "sink": f"{n}.sink", "talk": f"{n}.talk"}
         self.names.update(names or {})
 
     @property
@@ -122,6 +136,12 @@ class PagedAttention(Mixer):
         """Heads go from the projection to the attention kernels' forms by `ops.heads_to_pages`: the projection is
         stacked without padding, and queries get rows of their own."""
         return self.joint_norm_eps is not None or self.tied_values
+
+    @property
+    def kernel_blocks(self) -> int:
+        """Heads of keys and values the attention kernels walk: one number per key/value head, or per pair of a head of
+        keys and a head of values."""
+        return self.num_kv_heads ** 2 if self.talk else self.num_kv_heads
 
     @property
     def sees(self) -> int:
@@ -135,7 +155,7 @@ class PagedAttention(Mixer):
         rotary_plain = getattr(self.position_encoding, "plain", True)
         return (rotary_plain and self.unit_norm_eps is None and not self.gate and self.has_kv
                 and not self.head_gate and not self.unit_sink and not self.learned_sinks and not self.keep_first
-                and not self.spread
+                and not self.spread and not self.talk and self.value_norm_eps is None
                 and self.qk_norm_eps is None and not self.rotate_values and self.softcap is None
                 and self.key_dim == self.value_dim == self.head_dim)
 
@@ -165,6 +185,8 @@ class PagedAttention(Mixer):
         if self.joint_norm_eps is not None:
             specs += [WeightSpec(names["q_norm"], (self.num_heads * d,), kind="vector", init=("one_plus_normal", 0.1)),
                       WeightSpec(names["k_norm"], (self.num_kv_heads * d,), kind="vector", init=("one_plus_normal", 0.1))]
+        if self.talk:
+            specs.append(WeightSpec(names["talk"], (self.num_heads, self.num_heads), kind="vector", init=("normal", 0.5)))
         if self.learned_sinks:
             specs.append(WeightSpec(names["sink"], (self.num_heads,), kind="vector", init=("normal", 1.0)))
         return specs
@@ -233,6 +255,8 @@ class PagedAttention(Mixer):
         self.sinks = torch.zeros(nq, dtype=torch.float32, device=runtime.device) if self.unit_sink else None
         if self.learned_sinks:
             self.sinks = weights[names["sink"]].to(torch.float32).contiguous()
+        if self.talk:  # transposed: [taken head, mixture]
+            self.talk_table = weights[names["talk"]].to(torch.float32).t().contiguous()
         ops.attention_library(self.head_dim)  # compile now, not inside the first step
 
     # ------------------------------------------------------------------ decode steps replayed from a graph
@@ -246,7 +270,7 @@ class PagedAttention(Mixer):
         group = self.num_heads // self.num_kv_heads
         if not bf16 or not ops.tcgen05_prefill_fits(self.head_dim, self.num_heads, self.num_kv_heads, self.page_size or 16):
             return None
-        return int(ops.prefill_key_parts(plan.q_lens, plan.seq_lens, 128 // group, self.num_kv_heads,
+        return int(ops.prefill_key_parts(plan.q_lens, plan.seq_lens, 128 // group, self.kernel_blocks,
                                          ops.sm_count(self.runtime.device), self.sees))
 
     def capture_group(self) -> object:
@@ -257,7 +281,7 @@ class PagedAttention(Mixer):
         if not ctx.is_decode_only:
             # a captured step with prompt portions: the number of key parts is the variant's (the choice follows the
             # lengths of the step, which a replay does not know on the host)
-            ctx.extras[("prefill_key_parts", 128 // (self.num_heads // self.num_kv_heads), self.num_kv_heads,
+            ctx.extras[("prefill_key_parts", 128 // (self.num_heads // self.num_kv_heads), self.kernel_blocks,
                         self.sees)] = int(variant or 1)
             return
         # the number of slices must not follow the lengths of the step that happens to be captured
@@ -326,16 +350,22 @@ class PagedAttention(Mixer):
                                 interleaved=getattr(encoding, "interleaved", False),
                                 mscale=getattr(encoding, "mscale", 1.0),
                                 norm_dim=self.key_dim if self.unit_norm_eps is not None else 0,
-                                eps=self.unit_norm_eps or 0.0, write_cache=layer.writes_cache)
+                                eps=self.unit_norm_eps or self.value_norm_eps or 0.0, write_cache=layer.writes_cache,
+                            value_norm_dim=self.value_dim if self.value_norm_eps is not None else 0)
         elif not fused:
             ops.rope_and_cache(qkv, ctx.positions, meta.slot_mapping, inv_freq, layer.kv, self.num_heads,
                                self.num_kv_heads, self.head_dim, rotary_dim, write_cache=layer.writes_cache)
-        out = torch.empty((x.shape[0], self.num_heads * self.head_dim), dtype=x.dtype, device=x.device)
+        width = self.num_heads * self.head_dim
+        gate = qkv[:, qkv.shape[1] - width:] if self.gate else None
+        out = torch.empty((x.shape[0], self.num_kv_heads * width if self.talk else width),
+                          dtype=torch.float32 if self.talk else x.dtype, device=x.device)
         ops.paged_attention(q, out, layer.kv, meta.block_tables, ctx, self.num_heads, self.num_kv_heads,
                             self.head_dim, self.scale, self.window or 0,
                             rope=(inv_freq, rotary_dim) if fused else None, chunk=self.chunk or 0,
-                            gate=qkv[:, qkv.shape[1] - out.shape[1]:] if self.gate else None, softcap=self.softcap or 0.0,
-                            sinks=self.sinks, keep=self.keep_first)
+                            gate=None if self.talk else gate, softcap=self.softcap or 0.0,
+                            sinks=self.sinks, keep=self.keep_first, across=self.talk)
+        if self.talk:
+            out = ops.talk_heads(out, self.talk_table, self.num_kv_heads, x.dtype, gate)
         if self.head_gate:
             ops.head_gate(out, qkv[:, self.head_gate_col: self.head_gate_col + self.num_heads], self.num_heads, self.head_dim)
         if self.rotate_values:

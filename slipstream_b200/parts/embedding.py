@@ -8,7 +8,7 @@ import torch
 
 from slipstream_b200 import ops
 
-from .base import EMBEDDINGS, HEADS, Embedding, Head, Runtime, StateSpec, WeightSpec
+from .base import EMBEDDINGS, HEADS, Embedding, Head, Norm, Runtime, StateSpec, WeightSpec
 
 
 @EMBEDDINGS.register("token_table")
@@ -16,10 +16,14 @@ class TokenEmbedding(Embedding):
     cuda_graph_safe = True
 
     def __init__(self, name: str, vocab_size: int, hidden_size: int, scale: float = 1.0, copies: int = 1,
-                 tensor: str | None = None) -> None:
+                 tensor: str | None = None, norm: Norm | None = None) -> None:
         """``scale``: a constant the table's rows are multiplied by (in float32).  ``copies``: how many residual
         streams the model keeps; above 1 the result is [N, copies, hidden], every stream starting as the same
-        row.  ``tensor``: the checkpoint's name of the table (default ``<name>.weight``)."""
+        row.  ``tensor``: the checkpoint's name of the table (default ``<name>.weight``).  ``norm``: an RMS norm (a part with
+        ``weight`` float32 [hidden] and ``eps``) on the scaled rows, in the kernel that gathers them."""
+        if norm is not None and copies != 1:
+            raise ValueError("a norm on the embedding comes with one residual stream")
+        self.norm = norm
         self.name = name
         self.vocab_size = vocab_size
         self.hidden_size = hidden_size
@@ -28,13 +32,18 @@ class TokenEmbedding(Embedding):
         self.tensor = tensor or f"{name}.weight"
 
     def weight_specs(self) -> list[WeightSpec]:
-        return [WeightSpec(self.tensor, (self.vocab_size, self.hidden_size))]
+        specs = [WeightSpec(self.tensor, (self.vocab_size, self.hidden_size))]
+        return specs + (self.norm.weight_specs() if self.norm is not None else [])
 
     def bind(self, weights: dict[str, torch.Tensor], runtime: Runtime) -> None:
         super().bind(weights, runtime)
         self.weight = weights[self.tensor]
+        if self.norm is not None:
+            self.norm.bind(weights, runtime)
 
     def forward(self, token_ids: torch.Tensor) -> torch.Tensor:
+        if self.norm is not None:
+            return ops.embedding_norm(token_ids, self.weight, self.norm.weight, self.norm.eps, self.scale)
         return ops.embedding(token_ids, self.weight, scale=self.scale, copies=self.copies)
 
 

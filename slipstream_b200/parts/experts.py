@@ -1,7 +1,7 @@
 """Routed experts: a router picks ``top`` of ``experts`` small feed-forwards per token; a shared expert may run
 for every token beside them.
 
-Router: logits ``W_r x`` in float32, scores ``sigmoid(logits)`` (or, ``scores="softmax"``, their softmax over all
+Router: logits ``W_r x`` (plus ``router_bias``, a tensor [experts], in choice and weight) in float32, scores ``sigmoid(logits)`` (or, ``scores="softmax"``, their softmax over all
 experts), the ``top`` largest chosen; the chosen scores are the weights (divided by their sum only with
 ``renormalize``).  ``correction``: a tensor [experts] added to the scores for the CHOICE only.  ``groups`` = (count,
 keep): the experts form ``count`` equal groups of neighbours, a group's score is its largest choice score, and only
@@ -10,7 +10,7 @@ experts', which take part in scores, groups and choice like experts; such an exp
 its input.
 
 Two forms of expert.  ``gated`` (the default): ``W_down (silu(W_gate a) * (W_up a))`` fed ``a = score * x``
-(``weight_on_input``), its output added as it is.  Not ``gated``: ``W_down relu(W_up x)^2`` fed ``x``, its output
+(``weight_on_input``), its output added as it is, or, without ``weight_on_input``, fed ``x``, its output times the score.  Not ``gated``: ``W_down relu(W_up x)^2`` fed ``x``, its output
 times the score.  No biases.  ``shared_gate``: a tensor [1, hidden]; the shared expert's output is multiplied by
 ``sigmoid(shared_gate . x)``, one number per token (its logit rides along in the router's product, in float32).
 
@@ -32,21 +32,21 @@ from .base import FEED_FORWARDS, FeedForward, Part, Runtime, WeightSpec
 class RoutedExperts(FeedForward):
     cuda_graph_safe = True
     can_return_terms = True  # ``forward(..., as_terms=True)`` leaves the sum over the choices to the caller's kernel
-    # (the gated form; the un-gated form always forms its weighted sum itself)
+    # (gated experts with their weight on the input; the other forms always form their weighted sum themselves)
 
     def __init__(self, name: str, hidden_size: int, expert_size: int, experts: int, top: int,
                  shared: FeedForward | None = None, renormalize: bool = False, weight_on_input: bool = True,
                  router_tensor: str | None = None, expert_names: str | None = None, *, gated: bool = True,
                  scores: str = "sigmoid", correction: str | None = None, groups: tuple[int, int] | None = None,
-                 identity: int = 0, shared_gate: str | None = None) -> None:
+                 identity: int = 0, shared_gate: str | None = None, router_bias: str | None = None) -> None:
         """``expert_names``: a pattern with ``{e}`` and ``{role}`` (gate, up, down) for the experts' tensors
         (default ``<name>.experts.{e}.{role}_proj.weight``); ``router_tensor``: the router's (``<name>.gate.weight``);
-        ``correction`` and ``shared_gate``: tensor names."""
+        ``correction``, ``shared_gate`` and ``router_bias``: tensor names."""
         slots = experts + int(identity)
         if not 1 <= top <= slots or slots > 1024 or identity < 0:
             raise ValueError(f"top ({top}) must be between 1 and experts + identity ({slots}), that at most 1024")
-        if gated != bool(weight_on_input):
-            raise ValueError("built: gated experts with their weight on the input, un-gated ones with it on the output")
+        if weight_on_input and not gated:
+            raise ValueError("un-gated experts have their weight on the output")
         if gated and identity:
             raise ValueError("experts that hand their input on come with the un-gated form")
         if scores not in ("sigmoid", "softmax"):
@@ -57,6 +57,7 @@ class RoutedExperts(FeedForward):
         if shared_gate is not None and shared is None:
             raise ValueError("a gate on the shared expert comes with a shared expert")
         self.gated, self.scores, self.correction, self.groups = bool(gated), scores, correction, groups
+        self.weight_on_input, self.router_bias = bool(weight_on_input), router_bias
         self.identity, self.slots, self.shared_gate = int(identity), slots, shared_gate
         self.name = name
         self.hidden_size, self.expert_size, self.experts, self.top = hidden_size, expert_size, experts, top
@@ -73,6 +74,8 @@ class RoutedExperts(FeedForward):
         specs = [WeightSpec(self.router_tensor, (self.slots, h), init=("normal", 0.2))]
         if self.correction is not None:
             specs.append(WeightSpec(self.correction, (self.slots,), kind="vector", init=("normal", 0.02)))
+        if self.router_bias is not None:
+            specs.append(WeightSpec(self.router_bias, (self.slots,), kind="vector", init=("normal", 0.5)))
         if self.shared_gate is not None:
             specs.append(WeightSpec(self.shared_gate, (1, h), init=("normal", 0.2)))
         for e in range(self.experts):
@@ -90,6 +93,8 @@ class RoutedExperts(FeedForward):
             self.router_weight = torch.cat([self.router_weight, weights[self.shared_gate].reshape(1, -1)]).contiguous()
         self.correction_weight = (weights[self.correction].to(torch.float32).contiguous()
                                   if self.correction is not None else None)
+        self.router_bias_weight = (weights[self.router_bias].to(torch.float32).contiguous()
+                                   if self.router_bias is not None else None)
         self.down = torch.stack([weights[name(e=e, role="down")] for e in range(self.experts)]).contiguous()
         if not self.gated:
             self.up = torch.stack([weights[name(e=e, role="up")] for e in range(self.experts)]).contiguous()
@@ -115,11 +120,15 @@ class RoutedExperts(FeedForward):
         count, keep = self.groups or (1, 1)
         routed = ops.router(x, self.router_weight, self.top, self.renormalize, softmax=self.scores == "softmax",
                             correction=self.correction_weight, groups=count, keep=keep,
-                            extra=1 if self.shared_gate is not None else 0)
+                            extra=1 if self.shared_gate is not None else 0, bias=self.router_bias_weight)
         ids, scores = routed[0], routed[1]
         shared = self.shared.forward(x, ctx) if self.shared is not None else None
-        if not self.gated:  # the weights, the experts that hand their input on and the shared expert's gate meet in one sum
-            y, term_rows = ops.moe_experts_single(x, ids, self.up, self.down, self.slots)
+        if not self.weight_on_input:
+            # the weights, the experts that hand their input on and the shared expert's gate meet in one sum
+            if self.gated:
+                y, term_rows = ops.moe_experts(x, ids, None, self.gate_up, self.down, self.run)
+            else:
+                y, term_rows = ops.moe_experts_single(x, ids, self.up, self.down, self.slots)
             return ops.moe_mix(y, term_rows, ids, scores, self.experts, x, shared,
                                routed[2] if self.shared_gate is not None else None)
         y, term_rows = ops.moe_experts(x, ids, scores, self.gate_up, self.down, self.run)

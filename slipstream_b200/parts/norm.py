@@ -119,22 +119,23 @@ class NormedBranch:
 
 @NORMS.register("joining_rmsnorm")
 class JoiningNorm(Norm):
-    """RMS norm ``x / sqrt(mean(x^2) + eps) * weight``, formed in float32 and rounded once, for blocks that norm a branch
+    """RMS norm ``x / sqrt(mean(x^2) + eps) * weight`` (``scalar``: the weight is ONE number for all coordinates, a tensor
+    without axes), formed in float32 and rounded once, for blocks that norm a branch
     on both sides (`SandwichBlock`).  In front of a branch (and as the model's last norm) it is ``add_norm``, whose kernel
     first lets the pending branch output join the stream, under that output's own norm; behind a branch it is
     ``branch(y, mult)``, which leaves its work to the next ``add_norm``."""
 
     cuda_graph_safe = True
 
-    def __init__(self, tensor: str, size: int, eps: float) -> None:
-        self.tensor, self.size, self.eps = tensor, size, float(eps)
+    def __init__(self, tensor: str, size: int, eps: float, scalar: bool = False) -> None:
+        self.tensor, self.size, self.eps, self.scalar = tensor, size, float(eps), bool(scalar)
 
     def weight_specs(self) -> list[WeightSpec]:
-        return [WeightSpec(self.tensor, (self.size,), kind="vector", init=("one_plus_normal", 0.1))]
+        return [WeightSpec(self.tensor, () if self.scalar else (self.size,), kind="vector", init=("one_plus_normal", 0.1))]
 
     def bind(self, weights: dict[str, torch.Tensor], runtime: Runtime) -> None:
         super().bind(weights, runtime)
-        self.weight = weights[self.tensor].to(torch.float32).contiguous()
+        self.weight = weights[self.tensor].to(torch.float32).expand(self.size).contiguous()  # the kernels read a row
 
     def weight_bytes(self) -> int:
         return self.weight.numel() * self.weight.element_size()

@@ -20,7 +20,9 @@ over ``taps`` tokens whose last ``taps - 1`` inputs live in the request's state 
 `DecayedLinearAttention`: linear attention with a fixed decay per head.  With q, k of ``dim`` elements and v of
 ``value_dim`` per head, all three under silu: ``S <- decay_h S + k v^T``, ``o = S^T q`` (no other scale).  The
 concatenated heads of o pass one RMS norm with a weight, are multiplied by ``sigmoid(W_g x)`` and projected back.  S
-lives in the request's state slot.
+lives in the request's state slot.  With ``retention`` the form of retentive networks: no activations; q and k are rotated by
+a position encoding (half-split pairs) and k is multiplied by ``dim ** -0.5``; EVERY head of o is divided by its root mean
+square (no weight), and the gate is ``silu(W_g x)``.
 
 `GatedLinearRecurrenceMixer`: the recurrent block around a real-gated linear recurrent unit.  Two branches of
 ``width`` channels: ``y = gelu_tanh(W_y x + b_y)`` and ``u = conv(W_x x + b_x)``, a causal convolution per channel with a
@@ -29,7 +31,8 @@ bias and no activation.  u is cut into ``blocks`` equal parts; in part b ``r = s
 ``S <- a S + sqrt(1 - a^2) (i u)`` element by element from S = 0; output ``W_o (S y)``.  S and the convolution's last
 inputs live in the request's state slot.
 
-`ParallelMixers`: two mixers that read the same input; the result is ``left_scale * left + right_scale * right``.
+`ParallelMixers`: two mixers that read the same input; the result is ``left_scale * left + right_scale * right``, or, with
+``out_norms``, ``scale * (norm_left(left) + norm_right(right))``.
 
 Gates, biases, decays, states and norms are float32; the projections are in the compute dtype, except the two
 gate rows of the matrix memory, whose product leaves in float32.
@@ -41,7 +44,7 @@ import torch
 
 from slipstream_b200 import ops
 
-from .base import MIXERS, CacheSpec, IntoNorm, LayerBinding, Mixer, Part, Runtime, StateSpec, WeightSpec
+from .base import MIXERS, CacheSpec, IntoNorm, LayerBinding, Mixer, Part, PositionEncoding, Runtime, StateSpec, WeightSpec
 
 
 def _f32(t: torch.Tensor) -> torch.Tensor:
@@ -197,10 +200,15 @@ class DecayedLinearAttention(Mixer):
     takes_pending_norm = True  # the input goes to one product and nowhere else
 
     def __init__(self, name: str, hidden_size: int, heads: int, dim: int, value_dim: int, decay: "tuple[float, ...]",
-                 norm_eps: float = 1e-6, names: dict[str, str] | None = None) -> None:
-        """``decay``: one number per head.  ``names``: the checkpoint's tensor names by role (q, k, v, g, o, norm)."""
+                 norm_eps: float = 1e-6, names: dict[str, str] | None = None, *, retention: bool = False,
+                 position_encoding: PositionEncoding | None = None) -> None:
+        """``decay``: one number per head.  ``names``: the checkpoint's tensor names by role (q, k, v, g, o, norm).
+        ``position_encoding``: what rotates q and k with ``retention`` (None: nothing)."""
         if heads < 1 or not 1 <= dim <= 256 or value_dim < 1 or len(decay) != heads:
             raise ValueError("heads and value_dim must be >= 1, dim between 1 and 256, one decay per head")
+        if position_encoding is not None and (not retention or not getattr(position_encoding, "plain", True)):
+            raise ValueError("a rotation comes with the retention form, in half-split pairs with unscaled sines")
+        self.retention, self.position_encoding = bool(retention), position_encoding
         self.name, self.hidden_size = name, hidden_size
         self.heads, self.dim, self.value_dim = heads, dim, value_dim
         self.decay, self.norm_eps = tuple(float(d) for d in decay), float(norm_eps)
@@ -210,8 +218,9 @@ class DecayedLinearAttention(Mixer):
     def weight_specs(self) -> list[WeightSpec]:
         n, w, h, d, v = self.names, self.hidden_size, self.heads, self.dim, self.value_dim
         return [WeightSpec(n["q"], (h * d, w)), WeightSpec(n["k"], (h * d, w)), WeightSpec(n["v"], (h * v, w)),
-                WeightSpec(n["g"], (h * v, w)), WeightSpec(n["o"], (w, h * v)),
-                WeightSpec(n["norm"], (h * v,), kind="vector", init=("one_plus_normal", 0.1))]
+                WeightSpec(n["g"], (h * v, w)), WeightSpec(n["o"], (w, h * v))] + (
+                    [] if self.retention else
+                    [WeightSpec(n["norm"], (h * v,), kind="vector", init=("one_plus_normal", 0.1))])
 
     def state_specs(self) -> list[StateSpec]:
         return [StateSpec("memory", (self.heads, self.dim, self.value_dim))]  # S, row by row
@@ -221,7 +230,9 @@ class DecayedLinearAttention(Mixer):
         n = self.names
         self.qkvg_weight = _pad_rows(torch.cat([weights[n[r]] for r in ("q", "k", "v", "g")], dim=0))
         self.decay_weight = torch.tensor(self.decay, dtype=torch.float64).to(torch.float32).to(runtime.device)
-        self.norm_weight = _f32(weights[n["norm"]])
+        self.norm_weight = None if self.retention else _f32(weights[n["norm"]])
+        if self.position_encoding is not None:
+            self.position_encoding.bind(weights, runtime)
         self.o_weight = weights[n["o"]]
 
     def weight_bytes(self) -> int:
@@ -230,9 +241,15 @@ class DecayedLinearAttention(Mixer):
     def forward(self, x: torch.Tensor, ctx, layer: LayerBinding, into: IntoNorm | None = None) -> torch.Tensor:
         h, d, v = self.heads, self.dim, self.value_dim
         proj = ops.linear(x, self.qkvg_weight)
-        mixed = ops.decay_attention(proj, self.decay_weight, layer.state["memory"], ctx, h, d, v)
-        g0 = h * (2 * d + v)
-        out = ops.gated_rmsnorm(mixed, proj[:, g0: g0 + h * v], self.norm_weight, self.norm_eps, self.runtime.dtype)
+        gate = proj[:, h * (2 * d + v): h * (2 * d + 2 * v)]
+        if self.retention:
+            inv_freq = self.position_encoding.rotary_table()[0] if self.position_encoding is not None else None
+            mixed = ops.decay_attention(proj, self.decay_weight, layer.state["memory"], ctx, h, d, v, silu=False,
+                                        inv_freq=inv_freq, k_scale=d ** -0.5)
+            out = ops.head_norm_gate(mixed, gate, h, self.norm_eps, self.runtime.dtype)
+        else:
+            mixed = ops.decay_attention(proj, self.decay_weight, layer.state["memory"], ctx, h, d, v)
+            out = ops.gated_rmsnorm(mixed, gate, self.norm_weight, self.norm_eps, self.runtime.dtype)
         if into is not None:
             return into.close(out, self.o_weight, None)
         return ops.linear(out, self.o_weight)
@@ -302,12 +319,17 @@ class ParallelMixers(Mixer):
     """``left_scale * left(x) + right_scale * right(x)``: two mixers side by side on the same input.  At most one of
     them keeps pages (its `cache_spec` is the pair's); both may keep state, which the pair declares under the names
     ``left.<name>`` and ``right.<name>`` and hands to each side under its own names.  The sum is formed in float32 and
-    rounded once."""
+    rounded once.  ``out_norms`` = (left's tensor, right's tensor, eps): each output first passes an RMS norm over the model
+    width with a weight of its own; both scales are then equal."""
 
     takes_into = False
     takes_pending_norm = False  # two products read the input
 
-    def __init__(self, left: Mixer, right: Mixer, left_scale: float = 1.0, right_scale: float = 1.0) -> None:
+    def __init__(self, left: Mixer, right: Mixer, left_scale: float = 1.0, right_scale: float = 1.0,
+                 out_norms: tuple[str, str, float] | None = None, hidden_size: int | None = None) -> None:
+        if out_norms is not None and (left_scale != right_scale or hidden_size is None):
+            raise ValueError("normed outputs are scaled alike, and their norms need the model's width")
+        self.out_norms, self.hidden_size = out_norms, hidden_size
         if left.cache_spec() is not None and right.cache_spec() is not None:
             raise ValueError("at most one side of a pair of mixers keeps pages")
         self.left, self.right = left, right
@@ -316,6 +338,15 @@ class ParallelMixers(Mixer):
 
     def children(self) -> list[Part]:
         return [self.left, self.right]
+
+    def weight_specs(self) -> list[WeightSpec]:
+        return [WeightSpec(name, (self.hidden_size,), kind="vector", init=("one_plus_normal", 0.1))
+                for name in (self.out_norms or ())[:2]]
+
+    def bind(self, weights: dict[str, torch.Tensor], runtime: Runtime) -> None:
+        super().bind(weights, runtime)
+        if self.out_norms is not None:
+            self.norm_weights = [_f32(weights[name]) for name in self.out_norms[:2]]
 
     def cache_spec(self) -> CacheSpec | None:
         return self.left.cache_spec() or self.right.cache_spec()
@@ -335,4 +366,6 @@ class ParallelMixers(Mixer):
         left_pages = self.left.cache_spec() is not None
         a = self.left.forward(x, ctx, self._side(layer, "left", left_pages))
         b = self.right.forward(x, ctx, self._side(layer, "right", not left_pages and self.right.cache_spec() is not None))
+        if self.out_norms is not None:
+            return ops.normed_pair(a, self.norm_weights[0], b, self.norm_weights[1], self.out_norms[2], self.left_scale)
         return ops.scaled_sum(a, self.left_scale, b, self.right_scale)

@@ -83,6 +83,8 @@ def _register_builtin() -> None:
     from slipstream_b200.config.sarudra_config import SarudraConfig
     from slipstream_b200.models.qwen2 import build_qwen2
     from slipstream_b200.models.sarudra import build_sarudra
+    from slipstream_b200.config.sazepel_config import SazepelConfig
+    from slipstream_b200.models.sazepel import build_sazepel
 
     register_architecture("Qwen2ForCausalLM", Qwen2Config, build_qwen2, model_types=("qwen2", "qwen"))
     register_architecture("Fokedra", FokedraConfig, build_fokedra)
@@ -90,6 +92,7 @@ def _register_builtin() -> None:
     register_architecture("Bezutar", BezutarConfig, build_bezutar)
     register_architecture("Lakadra", LakadraConfig, build_lakadra)
     register_architecture("Fusipel", FusipelConfig, build_fusipel)
+    register_architecture("Sazepel", SazepelConfig, build_sazepel)
 
 
 _register_builtin()
