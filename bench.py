@@ -1508,6 +1508,224 @@ def run_compare_fusipel(args) -> int:
     return 0
 
 
+def sazepel_config(z: dict) -> dict:
+    """config.json of a Sazepel decoder at the layer sizes ``z``: a retention layer (the attention's heads and head size) and
+    a pair of talking-heads attention (the dense model's heads) and a retention of half as many heads, in turn; every
+    feed-forward routed, two of eight gated experts of half the dense layer's size, so that a token's feed-forward does the
+    dense layer's work."""
+    def retention(heads):
+        return dict(heads=heads, dim=z["dim"], vdim=z["dim"], rot=dict(base=1000000.0, dims=z["dim"]),
+                    decay=[1.0 - 2.0 ** -(5 + 5 * i / heads) for i in range(heads)])
+
+    mlp = dict(kind="moe", expert=dict(ff=z["ff"] // 2 // 64 * 64), router=dict(experts=8, top=2))
+    left = dict(heads=z["heads"], kv_heads=z["kv_heads"], dim=z["dim"], vdim=z["dim"], scale=z["dim"] ** -0.5)
+    layers = [dict(type="parallel", mixer=dict(left=left, right=retention(z["heads"] // 2)), mlp=mlp) if i % 2 else
+              dict(type="retention", mixer=retention(z["heads"]), mlp=mlp) for i in range(z["layers"])]
+    return dict(architecture="Sazepel", vocab=z["vocab"], width=z["width"], norm=dict(eps=1e-6), logit_scale=0.5, layers=layers,
+                max_position_embeddings=8192)
+
+
+def run_compare_sazepel(args) -> int:
+    """The Sazepel decoder beside the Qwen2.5 decoder at equal layer sizes (whole steps), then every kernel the design adds
+    or runs in a form of its own, alone at the 7B layer sizes, beside the like kernel of the Qwen2.5 path or its nearest
+    relative among the other decoders'."""
+    import numpy as np
+    import torch
+
+    from slipstream_b200 import ops
+    from slipstream_b200.engine.context import query_tiles_host, query_tiles_longest_first_host
+
+    pk, pk_kind = peaks()
+    rng = np.random.default_rng(0)
+    dev = torch.device("cuda:0")
+    batch, ctx_tokens, T, page = args.batch, args.prompt_len, args.chunk, 16
+    result: dict = {"compare": "sazepel", "peaks": pk_kind, "batch": batch, "context": ctx_tokens, "prefill_tokens": T, "sizes": {}}
+    for name in (args.sizes.split(",") if args.sizes else ("0.5b", "1.5b", "7b")):
+        qwen, _ = compare_configs(COMPARE_SIZES[name], 8192, 1, False)
+        result["sizes"][name] = {}
+        for which, config in (("qwen2", qwen), ("sazepel", sazepel_config(COMPARE_SIZES[name]))):
+            if which == "qwen2" and args.skip_qwen2:
+                continue
+            print(f"[bench] {name} {which} ...", file=sys.stderr, flush=True)
+            result["sizes"][name][which] = measure_model(config, args, pk, rng)
+            print(f"[bench] {name} {which}: {result['sizes'][name][which]}", file=sys.stderr, flush=True)
+    if args.no_kernels:
+        print(json.dumps(result))
+        return 0
+
+    print("[bench] single kernels ...", file=sys.stderr, flush=True)
+    gen = torch.Generator(device=dev).manual_seed(1)
+    kernels: dict = {}
+
+    def rand(*shape, dtype=torch.bfloat16, std=0.5):
+        return (torch.randn(*shape, generator=gen, device=dev) * std).to(dtype)
+
+    def sweep(run, copies: int = 6) -> float:
+        """Microseconds a launch, the operands rotating through ``copies`` sets; replayed from a graph, as an engine's
+        steps are, so that launches of a few microseconds are not timed at the speed of the host."""
+        for i in range(copies):
+            run(i)
+        torch.cuda.synchronize()  # the operands are complete before another stream captures launches that read them
+        graph = torch.cuda.CUDAGraph()
+        with torch.cuda.graph(graph):
+            for i in range(copies * 2):
+                run(i % copies)
+        time.sleep(0.25)  # a burst of launches by itself: the clock falls behind seconds of matrix products
+        times = []
+        for _ in range(8):
+            torch.cuda.synchronize()
+            start, stop = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            start.record()
+            graph.replay()
+            stop.record()
+            torch.cuda.synchronize()
+            times.append(start.elapsed_time(stop) * 1e3 / (2 * copies))
+        return sorted(times[3:])[2]
+
+    def hbm(name: str, us: float, nbytes: float, **more) -> None:
+        gbs = nbytes / us / 1e3
+        kernels[name] = {"us": round(us, 2), "gbs": round(gbs, 1), "hbm_frac": round(gbs / pk["hbm_gbs"], 3), **more}
+
+    def tensor(name: str, us: float, flops: float) -> None:
+        tf = flops / us / 1e6
+        kernels[name] = {"us": round(us, 2), "tflops": round(tf, 1), "bf16_frac": round(tf / pk["bf16_tflops"], 3)}
+
+    def step(q_lens, seq_lens):
+        starts = np.concatenate([[0], np.cumsum(q_lens)]).astype(np.int32)
+        as_dev = lambda v: torch.tensor(np.asarray(v), dtype=torch.int32, device=dev)  # noqa: E731
+        positions = np.concatenate([np.arange(s - n, s) for n, s in zip(q_lens, seq_lens)])
+        return types.SimpleNamespace(q_start=as_dev(starts), seq_lens=as_dev(seq_lens), state_slots=as_dev(np.arange(len(q_lens))),
+                                     positions=as_dev(positions), num_requests=len(q_lens), max_q_len=max(q_lens),
+                                     is_decode_only=all(n == 1 for n in q_lens))
+
+    z = COMPARE_SIZES["7b"]
+    h, n_q, n_kv, d, eps = z["width"], z["heads"], z["kv_heads"], z["dim"], 1e-6
+    ff = z["ff"] // 2 // 64 * 64
+    inv = torch.rand(d // 2, device=dev)
+    table_rows = rand(20000, h)
+    for tokens, tag, ctx in ((T, "prefill", step([T], [T])), (batch, "decode", step([1] * batch, [ctx_tokens] * batch))):
+        R = ctx.num_requests
+        ids = [torch.randint(0, 20000, (tokens,), generator=gen, device=dev, dtype=torch.int32) for _ in range(6)]
+        w, wb = rand(h, dtype=torch.float32), rand(h, dtype=torch.float32)
+        hbm(f"{tag}_embedding (qwen2)", sweep(lambda i: ops.embedding(ids[i], table_rows)), tokens * h * 6.0)
+        hbm(f"{tag}_embedding under a norm", sweep(lambda i: ops.embedding_norm(ids[i], table_rows, w, eps)), tokens * h * 6.0)
+        streams = [rand(tokens, h, dtype=torch.float32) for _ in range(6)]
+        ys, y2s = [rand(tokens, h) for _ in range(6)], [rand(tokens, h) for _ in range(6)]
+        hbm(f"{tag}_add_rmsnorm (qwen2)", sweep(lambda i: ops.add_rmsnorm(streams[i], ys[i], w, eps, torch.bfloat16)), tokens * h * 12.0)
+        hbm(f"{tag}_branch_norm (fusipel)",
+            sweep(lambda i: ops.branch_norm(streams[i], ys[i], wb, eps, 1.0, w, eps, torch.bfloat16)), tokens * h * 12.0)
+        hbm(f"{tag}_scaled_sum of two mixers (lakadra)", sweep(lambda i: ops.scaled_sum(ys[i], 0.5, y2s[i], 0.5)), tokens * h * 6.0)
+        hbm(f"{tag}_normed_pair (alone)", sweep(lambda i: ops.normed_pair(ys[i], w, y2s[i], wb, eps, 0.5)), tokens * h * 6.0)
+        del streams
+        # queries, keys and values to their norms and pages
+        rows = [rand(tokens, (2 * n_q + 2 * n_kv) * d) for _ in range(6)]
+        qkv = [r[:, : (n_q + 2 * n_kv) * d].contiguous() for r in rows]
+        kvs = [torch.zeros(max(tokens // page, 1), 2, n_kv, page, d, dtype=torch.bfloat16, device=dev) for _ in range(6)]
+        slots = torch.arange(tokens, dtype=torch.int32, device=dev)
+        hbm(f"{tag}_rope_and_cache (qwen2)", sweep(lambda i: ops.rope_and_cache(qkv[i], slots, slots, inv, kvs[i], n_q, n_kv, d, d)),
+            tokens * d * 2.0 * (2 * n_q + 4 * n_kv))
+        for what, over in (("unit norms of queries and keys (fokedra's norm)", 0), ("unit norms of queries, keys and values", d)):
+            hbm(f"{tag}_{what}", sweep(lambda i: ops.rope_norm_cache(rows[i], slots, slots, None, kvs[i], n_q, n_kv, d, 0, norm_dim=d,
+                                                                     eps=eps, value_norm_dim=over)), tokens * d * 2.0 * (2 * n_q + 4 * n_kv))
+        del rows, qkv, kvs
+        # retention beside linear attention under silu: the same state, the same bytes
+        proj = [rand(tokens, n_q * 4 * d) for _ in range(6)]
+        decay = torch.full((n_q,), 0.99, device=dev)
+        memory = [torch.zeros(R, n_q, d, d, device=dev) for _ in range(6)]
+        moved = R * n_q * d * d * 8.0 + tokens * n_q * d * (3 * 2.0 + 4.0)
+        for what, more in (("decay_attention (lakadra)", {}), ("retention", dict(silu=False, inv_freq=inv, k_scale=d ** -0.5)),
+                           ("retention token by token", dict(silu=False, inv_freq=inv, k_scale=d ** -0.5, chunks=False))):
+            us = sweep(lambda i: ops.decay_attention(proj[i], decay, memory[i], ctx, n_q, d, d, **more))
+            hbm(f"{tag}_{what}", us, moved, fp32_tflops=round(4.0 * tokens * n_q * d * d / us / 1e6, 2))
+        mixed = [ops.decay_attention(p, decay, m, ctx, n_q, d, d) for p, m in zip(proj, memory)]
+        w_all = rand(n_q * d, dtype=torch.float32)
+        hbm(f"{tag}_gated_rmsnorm (lakadra)", sweep(lambda i: ops.gated_rmsnorm(mixed[i], proj[i][:, 3 * n_q * d:], w_all, eps, torch.bfloat16)),
+            tokens * n_q * d * 8.0)
+        hbm(f"{tag}_head_norm_gate", sweep(lambda i: ops.head_norm_gate(mixed[i], proj[i][:, 3 * n_q * d:], n_q, eps, torch.bfloat16)),
+            tokens * n_q * d * 8.0)
+        del proj, memory, mixed
+        # the routed feed-forward
+        w_router, bias = rand(8, h, std=0.05), rand(8, dtype=torch.float32)
+        kernels[f"{tag}_router (lakadra's softmax)"] = {"us": round(sweep(lambda i: ops.router(ys[i], w_router, 2, softmax=True)), 2)}
+        kernels[f"{tag}_router (softmax over the chosen, bias)"] = {
+            "us": round(sweep(lambda i: ops.router(ys[i], w_router, 2, True, softmax=True, bias=bias)), 2)}
+        chosen, scores = ops.router(ys[0], w_router, 2, True, softmax=True, bias=bias)
+        gate_up, down = rand(8, 2 * ff, h, std=0.02), rand(8, h, ff, std=0.02)
+        touched = int(torch.unique(chosen).numel())
+        for what, weight in (("gated experts, weight on the input (sarudra)", scores), ("gated experts, weight on the output", None)):
+            us = sweep(lambda i: ops.moe_experts(ys[i], chosen, weight, gate_up, down, 64))
+            flops, moved = 6.0 * tokens * 2 * h * ff, touched * 3 * ff * h * 2.0
+            kernels[f"{tag}_{what}"] = {
+                "us": round(us, 2), "tflops": round(flops / us / 1e6, 1), "bf16_frac": round(flops / us / 1e6 / pk["bf16_tflops"], 3),
+                "gbs": round(moved / us / 1e3, 1), "hbm_frac": round(moved / us / 1e3 / pk["hbm_gbs"], 3), "experts_touched": touched}
+        y, place = ops.moe_experts(ys[0], chosen, None, gate_up, down, 64)
+        each = 2.0 if place is not None else 4.0
+        hbm(f"{tag}_moe_combine (sarudra)", sweep(lambda i: ops.moe_combine(y, None, torch.bfloat16, place, 2)), tokens * h * (2 * each + 2.0))
+        hbm(f"{tag}_moe_mix (alone)", sweep(lambda i: ops.moe_mix(y, place, chosen, scores, 8, ys[i])), tokens * h * (2 * each + 2.0))
+        del gate_up, down, y, ys, y2s
+
+    # attention of a prompt in one step.  The operations counted are the design's own: scores, the mixture of the heads'
+    # weights, values
+    def pages_for(n_req: int, tokens: int):
+        per = (tokens + page - 1) // page
+        return torch.arange(n_req * per, dtype=torch.int32, device=dev).view(n_req, per)
+
+    one_q = torch.tensor([0, T], dtype=torch.int32, device=dev)
+    one_len = torch.tensor([T], dtype=torch.int32, device=dev)
+    for name in ("0.5b", "1.5b", "7b"):
+        z = COMPARE_SIZES[name]
+        n_q, n_kv, d = z["heads"], z["kv_heads"], z["dim"]
+        group, keys = n_q // n_kv, T * (T + 1) / 2
+        table = pages_for(1, T)
+        kv_pages = [rand(T // page + 1, 2, n_kv, page, d) for _ in range(6)]
+        qs, gate, talk = rand(T, n_q * d), rand(T, n_q * d), rand(n_q, n_q, dtype=torch.float32)
+        out = torch.empty(T, n_q * d, dtype=torch.bfloat16, device=dev)
+        wide = [torch.empty(T, n_kv * n_q * d, dtype=torch.float32, device=dev) for _ in range(2)]
+        req, tok0 = (torch.from_numpy(a).to(dev) for a in query_tiles_longest_first_host(
+            np.asarray([T], dtype=np.int32), np.asarray([T], dtype=np.int32), 128 // group))
+        args_of = lambda i: (kv_pages[i], table, req, tok0, one_q, one_len, n_q, n_kv, d, d ** -0.5)  # noqa: E731
+        us = sweep(lambda i: ops.paged_attention_prefill_tcgen05(qs, n_q * d, out, *args_of(i)))
+        tensor(f"prefill_attention {name} (qwen2)", us, keys * 4.0 * n_q * d)
+        us = sweep(lambda i: ops.paged_attention_prefill_tcgen05(qs, n_q * d, wide[i % 2], *args_of(i), across=True))
+        kernels[f"prefill_attention {name} over every head's values"] = {"us": round(us, 2)}
+        us2 = sweep(lambda i: ops.talk_heads(wide[i % 2], talk, n_kv, torch.bfloat16, gate))
+        hbm(f"prefill_talk_heads {name}", us2, T * n_q * d * (4.0 * n_kv + 4.0))
+        tensor(f"prefill_attention {name} with talking heads (both)", us + us2, keys * (4.0 * n_q * d + 2.0 * n_q * n_q))
+        req, row0 = (torch.from_numpy(a).to(dev) for a in query_tiles_host(np.asarray([T * group], dtype=np.int32), 64))
+        args_of = lambda i: (kv_pages[i], table, req, row0, one_q, one_len, n_q, n_kv, d, d ** -0.5)  # noqa: E731
+        us = sweep(lambda i: ops.paged_attention_prefill(qs, n_q * d, out, *args_of(i)), 2)
+        tensor(f"prefill_attention {name} mma.sync (qwen2's heads)", us, keys * 4.0 * n_q * d)
+        us = sweep(lambda i: ops.paged_attention_prefill(qs, n_q * d, wide[i % 2], *args_of(i), across=True), 2)
+        tensor(f"prefill_attention {name} mma.sync with talking heads (both)", us + us2, keys * (4.0 * n_q * d + 2.0 * n_q * n_q))
+        del kv_pages, wide
+
+        for n_req, tokens in ((batch, ctx_tokens), (batch, 8000), (64, 4000)):
+            copies = 6 if n_req * tokens < 20000 else 3
+            kv_pages = [rand(n_req * ((tokens + page - 1) // page), 2, n_kv, page, d) for _ in range(copies)]
+            table = pages_for(n_req, tokens)
+            starts = torch.arange(n_req + 1, dtype=torch.int32, device=dev)
+            lens = torch.full((n_req,), tokens, dtype=torch.int32, device=dev)
+            q, gate = rand(n_req, n_q * d), rand(n_req, n_q * d)
+            out = torch.empty_like(q)
+            wide1 = torch.empty(n_req, n_kv * n_q * d, dtype=torch.float32, device=dev)
+            moved = n_req * tokens * 4.0 * n_kv * d + n_req * n_q * d * 4.0
+
+            def decode(into, across):
+                slices = ops.decode_slices(n_req, n_kv * n_kv if across else n_kv, group, tokens, False, ops.sm_count(dev))
+                return sweep(lambda i: ops.paged_attention_decode(q, q.shape[1], into, kv_pages[i], table, starts, lens, n_req, n_q, n_kv, d,
+                                                                  d ** -0.5, 0, slices, stages=ops.functions.DECODE_RING_STAGES, across=across), copies)
+
+            hbm(f"decode_attention {name} {n_req} x {tokens} (qwen2, rotation outside)", decode(out, False), moved)
+            us = decode(wide1, True)
+            us2 = sweep(lambda i: ops.talk_heads(wide1, talk, n_kv, torch.bfloat16, gate))
+            hbm(f"decode_attention {name} {n_req} x {tokens} with talking heads (both)", us + us2, moved, talk_us=round(us2, 2))
+            del kv_pages
+    ops.check_errors(dev)
+    result["kernels"] = kernels
+    print(json.dumps(result))
+    return 0
+
+
 def main() -> int:
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -1527,7 +1745,7 @@ def main() -> int:
     ap.add_argument("--workload", choices=sorted(WORKLOADS), default=None,
                     help="run another measured workload end to end through the scheduler instead")
     ap.add_argument("--window", type=int, default=4096, help="--compare sarudra: positions of the sliding window")
-    ap.add_argument("--compare", choices=["fokedra", "sarudra", "bezutar", "lakadra", "fusipel"], default=None,
+    ap.add_argument("--compare", choices=["fokedra", "sarudra", "bezutar", "lakadra", "fusipel", "sazepel"], default=None,
                     help="time another decoder design beside the Qwen2.5 decoder at equal layer sizes instead")
     ap.add_argument("--sizes", default="", help="--compare: which of 0.5b,1.5b,7b,14b (default: all)")
     ap.add_argument("--mask-chunk", type=int, default=8192, help="--compare: positions per attention chunk")
@@ -1553,6 +1771,8 @@ def main() -> int:
             return run_compare_lakadra(args)
         if args.compare == "fusipel":
             return run_compare_fusipel(args)
+        if args.compare == "sazepel":
+            return run_compare_sazepel(args)
         return run_compare_sarudra(args) if args.compare == "sarudra" else run_compare(args)
     if args.workload:
         return run_workload(args.workload, args)

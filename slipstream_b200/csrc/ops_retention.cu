@@ -1,10 +1,11 @@
 // Kernels around retention layers and heads that share their attention weights, beside ops_gated.cu:
 //   * the embedding rows under an RMS norm, straight into the float32 stream;
+//   * retention over prompt portions on the tensor cores, a chunk of tokens at a time;
 //   * the output of a retention layer: every head over its root mean square, under a silu gate;
 //   * talking heads: each head's output as a mixture over the heads' attention weights, under a sigmoid gate;
 //   * the weighted sum of two branches, each under an RMS norm of its own.
 // Norms, gates and mixtures are float32; T is the compute type of projections and activations.
-#include "common.cuh"
+#include "mma_sync.cuh"
 
 namespace {
 
@@ -267,4 +268,395 @@ extern "C" int ss_normed_pair(const void* a, const float* wa, const void* b, con
     else
         ss_launch(normed_pair_kernel<float>, dim3(n_rows), dim3(256), 0, stream, (const float*)a, wa, (const float*)b, wb, (float*)out, hidden, eps, scale);
     return SS_LAUNCH_CHECK();
+}
+
+// ---------------------------------------------------------------- retention over prompt portions, a chunk at a time
+//
+// The recurrence S <- g S + k v^T, o = S^T q of a head (g its decay) over a chunk of C tokens from the state S_0 in front
+// of it is, exactly:
+//   o_t = g^(t+1) S_0^T q_t + sum_{s <= t} g^(t-s) (q_t . k_s) v_s,        S_C = g^C S_0 + sum_s g^(C-1-s) k_s v_s^T,
+// products of matrices instead of C dependent steps.  q and k are rotated (pairs (i, i + half), k times k_scale) and the
+// state is kept in float32; every float32 operand of a product is cut into two bfloat16 parts, x = hi + lo with a remainder
+// below 2^-17 |x|, and the products hi hi + hi lo + lo hi are accumulated in float32 (the values v are bfloat16 as projected).
+//
+// A block of 8 warps takes RC_COLS value columns of a head of a request and walks its tokens in chunks of RC_T:
+//   * the chunk's rows arrive in shared memory by asynchronous copies issued while the chunk in front is computed;
+//   * they are rotated and cut in two (cosines and sines of a row's offset in the chunk come from a table made once, those
+//     of the chunk's first position are formed once a chunk);
+//   * warps w and w + 4 take rows 16 w .. 16 w + 15: every other 16 keys of the scores and half of the state's rows each,
+//     their sums meet in shared memory;
+//   * the state stays in registers as accumulators, cut in two in shared memory once a chunk.
+// proj, state, out as for the token-by-token kernel (ops_gated.cu).  D: 64 or 128, at least the head's dim; zeros behind it.
+#define RC_T 64
+#define RC_COLS 32
+#define RC_THREADS 256
+
+template <int D>
+struct RcSmem {
+    static constexpr int S = D + 8, V = RC_COLS + 8;          // strides that spread ldmatrix over all banks
+    static constexpr int raw_qk = 0;                          // bf16 [2][RC_T][D]
+    static constexpr int raw_v = raw_qk + 2 * RC_T * D * 2;   // bf16 [RC_T][RC_COLS]
+    static constexpr int qk = raw_v + RC_T * RC_COLS * 2;     // bf16 [q hi, q lo, k hi, k lo][RC_T][S]
+    static constexpr int v = qk + 4 * RC_T * S * 2;           // bf16 [v, g^(n-1-s) v: hi, lo][RC_T][V]
+    static constexpr int st = v + 3 * RC_T * V * 2;           // bf16 [state hi, lo][D][V]
+    static constexpr int sum = st + 2 * D * V * 2;            // float [RC_T][V]
+    static constexpr int pw = sum + RC_T * V * 4;             // float [RC_T + 4]: powers of the decay
+    static constexpr int base = pw + (RC_T + 4) * 4;          // float2 [D / 2]: the chunk's first position
+    static constexpr int turn = base + D / 2 * 8;             // float2 [RC_T][D / 2]: offsets in the chunk
+    static constexpr int bytes = turn + RC_T * (D / 2) * 8;
+};
+
+__device__ __forceinline__ void cut_in_two(const float (&x)[8], uint4& hi, uint4& lo) {
+    uint32_t h[4], l[4];
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+        h[e] = pack_bf16(x[2 * e], x[2 * e + 1]);
+        l[e] = pack_bf16(x[2 * e] - __uint_as_float(h[e] << 16), x[2 * e + 1] - __uint_as_float(h[e] & 0xffff0000u));
+    }
+    hi = make_uint4(h[0], h[1], h[2], h[3]);
+    lo = make_uint4(l[0], l[1], l[2], l[3]);
+}
+__device__ __forceinline__ void eight(const uint4& r, float (&v)[8]) {
+    const uint32_t w[4] = {r.x, r.y, r.z, r.w};
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+        v[2 * e] = __uint_as_float(w[e] << 16);
+        v[2 * e + 1] = __uint_as_float(w[e] & 0xffff0000u);
+    }
+}
+
+template <int D>
+__global__ void __launch_bounds__(RC_THREADS)
+retention_chunks_kernel(const bf16* __restrict__ proj, int64_t stride, const float* __restrict__ decay, float* __restrict__ state,
+                        float* __restrict__ out, const int32_t* __restrict__ q_start, const int32_t* __restrict__ seq_lens,
+                        const int32_t* __restrict__ slots, int heads, int dim, int vdim, int n_slots, int* err,
+                        const float* __restrict__ inv_freq, int half, float k_scale) {
+    using M = RcSmem<D>;
+    constexpr int S = M::S, V = M::V, KS = D / 16, NT = RC_COLS / 8;
+    constexpr int UT = D == 128 ? NT : NT / 2;  // column tiles of the state a warp holds (of 16 rows)
+    extern __shared__ __align__(16) unsigned char smem[];
+    bf16* raw = reinterpret_cast<bf16*>(smem + M::raw_qk);
+    bf16* raw_v = reinterpret_cast<bf16*>(smem + M::raw_v);
+    bf16* Qh = reinterpret_cast<bf16*>(smem + M::qk);
+    bf16* Ql = Qh + RC_T * S;
+    bf16* Kh = Ql + RC_T * S;
+    bf16* Kl = Kh + RC_T * S;
+    bf16* Vs = reinterpret_cast<bf16*>(smem + M::v);
+    bf16* Wh = Vs + RC_T * V;
+    bf16* Wl = Wh + RC_T * V;
+    bf16* Sh = reinterpret_cast<bf16*>(smem + M::st);
+    bf16* Sl = Sh + D * V;
+    float* sums = reinterpret_cast<float*>(smem + M::sum);
+    float* pw = reinterpret_cast<float*>(smem + M::pw);
+    float2* base = reinterpret_cast<float2*>(smem + M::base);
+    float2* turn = reinterpret_cast<float2*>(smem + M::turn);
+
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int col_blocks = (vdim + RC_COLS - 1) / RC_COLS;
+    const int h = blockIdx.x / col_blocks, c0 = (blockIdx.x % col_blocks) * RC_COLS, r = blockIdx.y;
+    const float g = decay[h];
+    pdl_launch_dependents();
+    for (int i = tid; i < RC_T * half; i += RC_THREADS) {  // offsets of the rows of a chunk: constants of the layer
+        const int t = i / half, e = i - t * half;
+        float sn, cs;
+        sincosf(__fmul_rn((float)t, inv_freq[e]), &sn, &cs);
+        turn[t * (D / 2) + e] = make_float2(cs, sn);
+    }
+    for (int i = tid; i <= RC_T; i += RC_THREADS) pw[i] = powf(g, (float)i);
+    pdl_wait();
+    const int q0 = q_start[r], q_len = q_start[r + 1] - q0, seq_len = seq_lens[r];
+    if (q_len <= 0 || seq_len <= 0) return;
+    const int slot = slots[r];
+    if (slot < 0 || slot >= n_slots) {
+        if (tid == 0) atomicOr(err, SS_ERR_SLOT_RANGE);
+        return;
+    }
+    const int pos0 = seq_len - q_len;
+    const int64_t k_off = (int64_t)heads * dim, v_off = 2 * k_off + (int64_t)h * vdim + c0;
+
+    // a chunk's rows into shared memory, 16 bytes a copy; zeros behind the last row, the head's last element and its last column
+    auto fetch = [&](int t0) {
+        for (int i = tid; i < 2 * RC_T * (D / 8); i += RC_THREADS) {
+            const int which = i / (RC_T * (D / 8)), rest = i - which * (RC_T * (D / 8)), t = rest / (D / 8), c = (rest % (D / 8)) * 8;
+            const bool ok = t0 + t < q_len && c < dim;
+            const bf16* src = proj + (int64_t)(q0 + (ok ? t0 + t : 0)) * stride + which * k_off + (int64_t)h * dim + (ok ? c : 0);
+            cp_async16(raw + (which * RC_T + t) * D + c, src, ok);
+        }
+        for (int i = tid; i < RC_T * (RC_COLS / 8); i += RC_THREADS) {
+            const int t = i / (RC_COLS / 8), c = (i % (RC_COLS / 8)) * 8;
+            const bool ok = t0 + t < q_len && c0 + c < vdim;
+            const bf16* src = proj + (int64_t)(q0 + (ok ? t0 + t : 0)) * stride + v_off + (ok ? c : 0);
+            cp_async16(raw_v + t * RC_COLS + c, ok ? src : proj, ok);
+        }
+        cp_async_commit();
+    };
+    fetch(0);
+
+    // the state as accumulators: this warp's 16 rows and UT column tiles
+    const int s_row = (D == 128 ? warp : warp & 3) * 16 + (lane >> 2), s_nt = D == 128 ? 0 : (warp >> 2) * UT;
+    float* sp = state + ((int64_t)slot * heads + h) * dim * vdim;
+    float acc_s[UT][4];
+#pragma unroll
+    for (int n = 0; n < UT; ++n)
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+            const int row = s_row + e * 8, col = c0 + (s_nt + n) * 8 + (lane & 3) * 2;
+            float2 x = make_float2(0.f, 0.f);
+            if (row < dim && col < vdim) x = *reinterpret_cast<const float2*>(sp + (int64_t)row * vdim + col);
+            acc_s[n][2 * e] = x.x;
+            acc_s[n][2 * e + 1] = x.y;
+        }
+    const int rt = warp & 3, part = warp >> 2;  // rows 16 rt .. of the chunk; which half of the keys and of the state's rows
+    const int half8 = half / 8;
+
+    for (int t0 = 0; t0 < q_len; t0 += RC_T) {
+        const int nb = min(RC_T, q_len - t0);
+        for (int i = tid; i < half; i += RC_THREADS) {
+            float sn, cs;
+            sincosf(__fmul_rn((float)(pos0 + t0), inv_freq[i]), &sn, &cs);
+            base[i] = make_float2(cs, sn);
+        }
+        cp_async_wait<0>();
+        __syncthreads();  // the rows and the chunk's first angles; and the chunk in front is done with everything below
+        // rotated pairs, eight at a time
+        for (int i = tid; i < 2 * RC_T * half8; i += RC_THREADS) {
+            const int which = i / (RC_T * half8), rest = i - which * (RC_T * half8), t = rest / half8, c = (rest - t * half8) * 8;
+            const bf16* src = raw + (which * RC_T + t) * D;
+            float u[8], v[8];
+            eight(*reinterpret_cast<const uint4*>(src + c), u);
+            eight(*reinterpret_cast<const uint4*>(src + c + half), v);
+            const float f = which ? k_scale : 1.f;
+#pragma unroll
+            for (int e = 0; e < 8; ++e) {
+                const float2 a = turn[t * (D / 2) + c + e], b = base[c + e];
+                const float cs = (a.x * b.x - a.y * b.y) * f, sn = (a.y * b.x + a.x * b.y) * f;
+                const float x = u[e] * cs - v[e] * sn;
+                v[e] = v[e] * cs + u[e] * sn;
+                u[e] = x;
+            }
+            bf16* hi = which ? Kh : Qh;
+            bf16* lo = which ? Kl : Ql;
+            uint4 ph, pl;
+            cut_in_two(u, ph, pl);
+            *reinterpret_cast<uint4*>(hi + t * S + c) = ph;
+            *reinterpret_cast<uint4*>(lo + t * S + c) = pl;
+            cut_in_two(v, ph, pl);
+            *reinterpret_cast<uint4*>(hi + t * S + c + half) = ph;
+            *reinterpret_cast<uint4*>(lo + t * S + c + half) = pl;
+        }
+        // elements that are not rotated (and the zeros behind the head)
+        const int rest8 = D / 8 - 2 * half8;
+        for (int i = tid; i < 2 * RC_T * rest8; i += RC_THREADS) {
+            const int which = i / (RC_T * rest8), rest = i - which * (RC_T * rest8), t = rest / rest8, c = 2 * half + (rest - t * rest8) * 8;
+            float u[8];
+            eight(*reinterpret_cast<const uint4*>(raw + (which * RC_T + t) * D + c), u);
+            const float f = which ? k_scale : 1.f;
+#pragma unroll
+            for (int e = 0; e < 8; ++e) u[e] *= f;
+            uint4 ph, pl;
+            cut_in_two(u, ph, pl);
+            *reinterpret_cast<uint4*>((which ? Kh : Qh) + t * S + c) = ph;
+            *reinterpret_cast<uint4*>((which ? Kl : Ql) + t * S + c) = pl;
+        }
+        for (int i = tid; i < RC_T * (RC_COLS / 8); i += RC_THREADS) {
+            const int t = i / (RC_COLS / 8), c = (i % (RC_COLS / 8)) * 8;
+            const uint4 w = *reinterpret_cast<const uint4*>(raw_v + t * RC_COLS + c);
+            *reinterpret_cast<uint4*>(Vs + t * V + c) = w;
+            float u[8];
+            eight(w, u);
+            const float f = t < nb ? pw[nb - 1 - t] : 0.f;
+#pragma unroll
+            for (int e = 0; e < 8; ++e) u[e] *= f;
+            uint4 ph, pl;
+            cut_in_two(u, ph, pl);
+            *reinterpret_cast<uint4*>(Wh + t * V + c) = ph;
+            *reinterpret_cast<uint4*>(Wl + t * V + c) = pl;
+        }
+#pragma unroll
+        for (int n = 0; n < UT; ++n)
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                const int at = (s_row + e * 8) * V + (s_nt + n) * 8 + (lane & 3) * 2;
+                const float x = acc_s[n][2 * e], y = acc_s[n][2 * e + 1];
+                const uint32_t hi = pack_bf16(x, y);
+                *reinterpret_cast<uint32_t*>(Sh + at) = hi;
+                *reinterpret_cast<uint32_t*>(Sl + at) = pack_bf16(x - __uint_as_float(hi << 16), y - __uint_as_float(hi & 0xffff0000u));
+            }
+        __syncthreads();
+        if (t0 + RC_T < q_len) fetch(t0 + RC_T);  // the rows as they came have been used up
+
+        // scores of 16 rows with every other 16 keys up to the diagonal, and half of q S_0
+        const bool rows_on = rt * 16 < nb;
+        float sc[2][2][4], o[NT][4];
+#pragma unroll
+        for (int n = 0; n < NT; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
+#pragma unroll
+        for (int b = 0; b < 2; ++b)
+#pragma unroll
+            for (int n = 0; n < 2; ++n) sc[b][n][0] = sc[b][n][1] = sc[b][n][2] = sc[b][n][3] = 0.f;
+        if (rows_on) {
+#pragma unroll
+            for (int ks = 0; ks < KS; ++ks) {
+                uint32_t qh[4], ql[4];
+                const int qa = (rt * 16 + (lane & 15)) * S + ks * 16 + ((lane >> 4) << 3);
+                ldmatrix_x4(qh, Qh + qa);
+                ldmatrix_x4(ql, Ql + qa);
+#pragma unroll
+                for (int b = 0; b < 2; ++b) {
+                    const int kb = part + 2 * b;
+                    if (kb <= rt) {
+                        uint32_t kh[4], kl[4];
+                        const int ka = (kb * 16 + (lane & 7) + ((lane >> 4) << 3)) * S + ks * 16 + (((lane >> 3) & 1) << 3);
+                        ldmatrix_x4(kh, Kh + ka);
+                        ldmatrix_x4(kl, Kl + ka);
+#pragma unroll
+                        for (int n = 0; n < 2; ++n) {
+                            mma_bf16(sc[b][n], qh, kh[2 * n], kh[2 * n + 1]);
+                            mma_bf16(sc[b][n], qh, kl[2 * n], kl[2 * n + 1]);
+                            mma_bf16(sc[b][n], ql, kh[2 * n], kh[2 * n + 1]);
+                        }
+                    }
+                }
+                if (ks / (KS / 2) == part) {
+#pragma unroll
+                    for (int n = 0; n < NT; n += 2) {
+                        uint32_t sh[4], sl[4];
+                        const int sa = (ks * 16 + (lane & 7) + (((lane >> 3) & 1) << 3)) * V + n * 8 + ((lane >> 4) << 3);
+                        ldmatrix_x4_trans(sh, Sh + sa);
+                        ldmatrix_x4_trans(sl, Sl + sa);
+#pragma unroll
+                        for (int m = 0; m < 2; ++m) {
+                            mma_bf16(o[n + m], qh, sh[2 * m], sh[2 * m + 1]);
+                            mma_bf16(o[n + m], qh, sl[2 * m], sl[2 * m + 1]);
+                            mma_bf16(o[n + m], ql, sh[2 * m], sh[2 * m + 1]);
+                        }
+                    }
+                }
+            }
+            const int row_lo = rt * 16 + (lane >> 2), row_hi = row_lo + 8;
+            const float f_lo = pw[row_lo + 1], f_hi = pw[row_hi + 1];
+#pragma unroll
+            for (int n = 0; n < NT; ++n) {
+                o[n][0] *= f_lo; o[n][1] *= f_lo;
+                o[n][2] *= f_hi; o[n][3] *= f_hi;
+            }
+#pragma unroll
+            for (int b = 0; b < 2; ++b) {
+                const int kb = part + 2 * b;
+                if (kb <= rt) {
+                    uint32_t ah[4], al[4];
+#pragma unroll
+                    for (int n = 0; n < 2; ++n) {
+                        const int key = kb * 16 + n * 8 + ((lane & 3) << 1);
+                        float x[4];
+#pragma unroll
+                        for (int e = 0; e < 4; ++e) {
+                            const int back = (e < 2 ? row_lo : row_hi) - (key + (e & 1));
+                            x[e] = back >= 0 ? sc[b][n][e] * pw[back] : 0.f;
+                        }
+#pragma unroll
+                        for (int e = 0; e < 2; ++e) {
+                            const uint32_t hi = pack_bf16(x[2 * e], x[2 * e + 1]);
+                            ah[2 * n + e] = hi;
+                            al[2 * n + e] = pack_bf16(x[2 * e] - __uint_as_float(hi << 16), x[2 * e + 1] - __uint_as_float(hi & 0xffff0000u));
+                        }
+                    }
+#pragma unroll
+                    for (int n = 0; n < NT; n += 2) {
+                        uint32_t vv[4];
+                        ldmatrix_x4_trans(vv, Vs + (kb * 16 + (lane & 7) + (((lane >> 3) & 1) << 3)) * V + n * 8 + ((lane >> 4) << 3));
+#pragma unroll
+                        for (int m = 0; m < 2; ++m) {
+                            mma_bf16(o[n + m], ah, vv[2 * m], vv[2 * m + 1]);
+                            mma_bf16(o[n + m], al, vv[2 * m], vv[2 * m + 1]);
+                        }
+                    }
+                }
+            }
+        }
+        // the state behind the chunk
+        if (s_row - (lane >> 2) < dim) {
+            const float f = pw[nb];
+#pragma unroll
+            for (int n = 0; n < UT; ++n)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) acc_s[n][e] *= f;
+            const int m0 = s_row - (lane >> 2);
+#pragma unroll
+            for (int ks = 0; ks < RC_T / 16; ++ks) {
+                if (ks * 16 >= nb) break;
+                uint32_t kh[4], kl[4];
+                const int ka = (ks * 16 + (lane & 7) + ((lane >> 4) << 3)) * S + m0 + (((lane >> 3) & 1) << 3);
+                ldmatrix_x4_trans(kh, Kh + ka);
+                ldmatrix_x4_trans(kl, Kl + ka);
+#pragma unroll
+                for (int n = 0; n < UT; n += 2) {
+                    uint32_t wh[4], wl[4];
+                    const int wa = (ks * 16 + (lane & 7) + (((lane >> 3) & 1) << 3)) * V + (s_nt + n) * 8 + ((lane >> 4) << 3);
+                    ldmatrix_x4_trans(wh, Wh + wa);
+                    ldmatrix_x4_trans(wl, Wl + wa);
+#pragma unroll
+                    for (int m = 0; m < 2; ++m) {
+                        mma_bf16(acc_s[n + m], kh, wh[2 * m], wh[2 * m + 1]);
+                        mma_bf16(acc_s[n + m], kh, wl[2 * m], wl[2 * m + 1]);
+                        mma_bf16(acc_s[n + m], kl, wh[2 * m], wh[2 * m + 1]);
+                    }
+                }
+            }
+        }
+        if (part == 1 && rows_on) {
+#pragma unroll
+            for (int n = 0; n < NT; ++n)
+#pragma unroll
+                for (int e = 0; e < 2; ++e)
+                    *reinterpret_cast<float2*>(sums + (rt * 16 + (lane >> 2) + e * 8) * V + n * 8 + (lane & 3) * 2) = make_float2(o[n][2 * e], o[n][2 * e + 1]);
+        }
+        __syncthreads();
+        if (part == 0 && rows_on) {
+#pragma unroll
+            for (int n = 0; n < NT; ++n)
+#pragma unroll
+                for (int e = 0; e < 2; ++e) {
+                    const int t = rt * 16 + (lane >> 2) + e * 8, c = n * 8 + (lane & 3) * 2;
+                    const float2 other = *reinterpret_cast<const float2*>(sums + t * V + c);
+                    if (t < nb && c0 + c < vdim)
+                        *reinterpret_cast<float2*>(out + ((int64_t)(q0 + t0 + t) * heads + h) * vdim + c0 + c) =
+                            make_float2(o[n][2 * e] + other.x, o[n][2 * e + 1] + other.y);
+                }
+        }
+    }
+#pragma unroll
+    for (int n = 0; n < UT; ++n)
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+            const int row = s_row + e * 8, col = c0 + (s_nt + n) * 8 + (lane & 3) * 2;
+            if (row < dim && col < vdim) *reinterpret_cast<float2*>(sp + (int64_t)row * vdim + col) = make_float2(acc_s[n][2 * e], acc_s[n][2 * e + 1]);
+        }
+}
+
+template <int D>
+static int launch_retention_chunks(const bf16* proj, int64_t stride, const float* decay, float* state, float* out, const int32_t* q_start,
+                                   const int32_t* seq_lens, const int32_t* slots, int R, int heads, int dim, int vdim, int n_slots, int* err,
+                                   cudaStream_t stream, const float* inv_freq, int half, float k_scale) {
+    constexpr int smem = RcSmem<D>::bytes;
+    static SsPerDevice opted;
+    if (int rc = ss_opt_in_smem(retention_chunks_kernel<D>, smem, opted)) return rc;
+    ss_launch(retention_chunks_kernel<D>, dim3(heads * ((vdim + RC_COLS - 1) / RC_COLS), R), dim3(RC_THREADS), smem, stream, proj, stride, decay,
+              state, out, q_start, seq_lens, slots, heads, dim, vdim, n_slots, err, inv_freq, half, k_scale);
+    return SS_LAUNCH_CHECK();
+}
+
+// bfloat16 rows; dim at most 128, dim, vdim, stride and half in steps of 8, proj, state and out on 16-byte boundaries.
+extern "C" int ss_retention_chunks(const void* proj, int64_t stride, const float* decay, float* state, float* out, const int32_t* q_start,
+                                   const int32_t* seq_lens, const int32_t* slots, int R, int heads, int dim, int vdim, int n_slots, int* err,
+                                   cudaStream_t stream, const float* inv_freq, int half, float k_scale) {
+    if (R <= 0) return 0;
+    if (heads < 1 || dim < 8 || dim > 128 || vdim < 8 || dim % 8 || vdim % 8 || stride % 8 || half < 0 || half % 8 || 2 * half > dim ||
+        (half > 0 && !inv_freq) || (((uintptr_t)proj | (uintptr_t)state | (uintptr_t)out) & 15))
+        return (int)cudaErrorInvalidValue;
+    if (dim <= 64)
+        return launch_retention_chunks<64>((const bf16*)proj, stride, decay, state, out, q_start, seq_lens, slots, R, heads, dim, vdim, n_slots, err,
+                                           stream, inv_freq, half, k_scale);
+    return launch_retention_chunks<128>((const bf16*)proj, stride, decay, state, out, q_start, seq_lens, slots, R, heads, dim, vdim, n_slots, err,
+                                        stream, inv_freq, half, k_scale);
 }

@@ -113,6 +113,8 @@ _OPS_SIGNATURES = {
                        c_int, c_int, c_void_p],
     "ss_embedding_norm": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_float, c_void_p, c_void_p],
     "ss_head_norm_gate": [c_void_p, c_void_p, c_int64, c_void_p, c_int, c_int, c_int, c_float, c_int, c_void_p],
+    "ss_retention_chunks": [c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
+                            c_int, c_void_p, c_void_p, c_void_p, c_int, c_float],
     "ss_talk_heads": [c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p],
     "ss_normed_pair": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_float, c_int, c_void_p],
 }
@@ -2138,7 +2140,8 @@ def head_product(x: torch.Tensor, x_head: int, weight: torch.Tensor, out: torch.
 # --------------------------------------------------------------------------- decayed linear attention, gated linear recurrence
 
 def decay_attention(proj: torch.Tensor, decay: torch.Tensor, state: torch.Tensor, ctx, heads: int, dim: int,
-                    value_dim: int, *, silu: bool = True, inv_freq: torch.Tensor | None = None, k_scale: float = 1.0) -> torch.Tensor:
+                    value_dim: int, *, silu: bool = True, inv_freq: torch.Tensor | None = None, k_scale: float = 1.0,
+                    chunks: bool = True) -> torch.Tensor:
     """Linear attention with a fixed decay per head over each request's tokens, continued from and left in ``state``
     (float32 [slots, heads, dim, value_dim]).  A row of ``proj`` starts with the heads' queries, then keys (``dim``
     each), then values (``value_dim``), all before their activation; whatever follows is left alone.  Per head h, token
@@ -2146,7 +2149,8 @@ def decay_attention(proj: torch.Tensor, decay: torch.Tensor, state: torch.Tensor
 
     ``silu`` False: no activation; the first ``2 * len(inv_freq)`` elements of queries and keys are rotated by the row's
     position * ``inv_freq`` in pairs (i, i + len(inv_freq)) (None: not at all), in float32, and keys are multiplied by
-    ``k_scale``."""
+    ``k_scale``.  Steps with prompt portions then run the kernel that takes chunks of tokens on the tensor cores where it can
+    (``chunks`` False: never): bfloat16 rows, ``dim`` at most 128, sizes in steps of 8."""
     _need(proj, None, "projected rows")
     _need(decay, torch.float32, "decay")
     _need(state, torch.float32, "state")
@@ -2162,6 +2166,14 @@ def decay_attention(proj: torch.Tensor, decay: torch.Tensor, state: torch.Tensor
         if silu or not 0 < 2 * half <= dim:
             raise KernelError("decay_attention: a rotation comes without the activation and covers at most the head")
     out = torch.empty((n, heads * value_dim), dtype=torch.float32, device=proj.device)
+    if (chunks and not silu and not ctx.is_decode_only and proj.dtype == torch.bfloat16 and dim <= 128
+            and dim % 8 == value_dim % 8 == half % 8 == proj.stride(0) % 8 == proj.data_ptr() % 16 == 0):
+        _check(ops_library().ss_retention_chunks(proj.data_ptr(), proj.stride(0), decay.data_ptr(), state.data_ptr(), out.data_ptr(),
+                                                 ctx.q_start.data_ptr(), ctx.seq_lens.data_ptr(), ctx.state_slots.data_ptr(),
+                                                 ctx.num_requests, heads, dim, value_dim, state.shape[0],
+                                                 error_word(proj.device).data_ptr(), _stream(), _ptr(inv_freq), half, float(k_scale)),
+               "retention_chunks")
+        return out
     _check(ops_library().ss_decay_attention(proj.data_ptr(), proj.stride(0), decay.data_ptr(), state.data_ptr(),
                                             out.data_ptr(), ctx.q_start.data_ptr(), ctx.seq_lens.data_ptr(),
                                             ctx.state_slots.data_ptr(), ctx.num_requests, heads, dim, value_dim,
