@@ -279,31 +279,32 @@ extern "C" int ss_normed_pair(const void* a, const float* wa, const void* b, con
 // state is kept in float32; every float32 operand of a product is cut into two bfloat16 parts, x = hi + lo with a remainder
 // below 2^-17 |x|, and the products hi hi + hi lo + lo hi are accumulated in float32 (the values v are bfloat16 as projected).
 //
-// A block of 8 warps takes RC_COLS value columns of a head of a request and walks its tokens in chunks of RC_T:
+// A block of 16 warps takes RC_COLS value columns of a head of a request and walks its tokens in chunks of RC_T:
 //   * the chunk's rows arrive in shared memory by asynchronous copies issued while the chunk in front is computed;
 //   * they are rotated and cut in two (cosines and sines of a row's offset in the chunk come from a table made once, those
 //     of the chunk's first position are formed once a chunk);
-//   * warps w and w + 4 take rows 16 w .. 16 w + 15: every other 16 keys of the scores and half of the state's rows each,
-//     their sums meet in shared memory;
+//   * four warps share 16 rows: each takes 16 keys of the scores and a quarter of the state's rows, and their sums meet in
+//     shared memory;
 //   * the state stays in registers as accumulators, cut in two in shared memory once a chunk.
 // proj, state, out as for the token-by-token kernel (ops_gated.cu).  D: 64 or 128, at least the head's dim; zeros behind it.
 #define RC_T 64
 #define RC_COLS 32
-#define RC_THREADS 256
+#define RC_THREADS 512
 
 template <int D>
 struct RcSmem {
     static constexpr int S = D + 8, V = RC_COLS + 8;          // strides that spread ldmatrix over all banks
+    static constexpr int A = D / 2 + 8;                       // stride of the table of angles, for the same reason
     static constexpr int raw_qk = 0;                          // bf16 [2][RC_T][D]
     static constexpr int raw_v = raw_qk + 2 * RC_T * D * 2;   // bf16 [RC_T][RC_COLS]
     static constexpr int qk = raw_v + RC_T * RC_COLS * 2;     // bf16 [q hi, q lo, k hi, k lo][RC_T][S]
     static constexpr int v = qk + 4 * RC_T * S * 2;           // bf16 [v, g^(n-1-s) v: hi, lo][RC_T][V]
     static constexpr int st = v + 3 * RC_T * V * 2;           // bf16 [state hi, lo][D][V]
-    static constexpr int sum = st + 2 * D * V * 2;            // float [RC_T][V]
-    static constexpr int pw = sum + RC_T * V * 4;             // float [RC_T + 4]: powers of the decay
+    static constexpr int sum = st + 2 * D * V * 2;            // float [4][RC_T][V]
+    static constexpr int pw = sum + 4 * RC_T * V * 4;         // float [RC_T + 4]: powers of the decay
     static constexpr int base = pw + (RC_T + 4) * 4;          // float2 [D / 2]: the chunk's first position
     static constexpr int turn = base + D / 2 * 8;             // float2 [RC_T][D / 2]: offsets in the chunk
-    static constexpr int bytes = turn + RC_T * (D / 2) * 8;
+    static constexpr int bytes = turn + RC_T * A * 8;
 };
 
 __device__ __forceinline__ void cut_in_two(const float (&x)[8], uint4& hi, uint4& lo) {
@@ -332,8 +333,8 @@ retention_chunks_kernel(const bf16* __restrict__ proj, int64_t stride, const flo
                         const int32_t* __restrict__ slots, int heads, int dim, int vdim, int n_slots, int* err,
                         const float* __restrict__ inv_freq, int half, float k_scale) {
     using M = RcSmem<D>;
-    constexpr int S = M::S, V = M::V, KS = D / 16, NT = RC_COLS / 8;
-    constexpr int UT = D == 128 ? NT : NT / 2;  // column tiles of the state a warp holds (of 16 rows)
+    constexpr int S = M::S, V = M::V, A = M::A, KS = D / 16, NT = RC_COLS / 8;
+    constexpr int UT = NT / 2;  // column tiles of the state a warp holds (of 16 rows); with D = 64 half of the warps hold any
     extern __shared__ __align__(16) unsigned char smem[];
     bf16* raw = reinterpret_cast<bf16*>(smem + M::raw_qk);
     bf16* raw_v = reinterpret_cast<bf16*>(smem + M::raw_v);
@@ -355,12 +356,13 @@ retention_chunks_kernel(const bf16* __restrict__ proj, int64_t stride, const flo
     const int col_blocks = (vdim + RC_COLS - 1) / RC_COLS;
     const int h = blockIdx.x / col_blocks, c0 = (blockIdx.x % col_blocks) * RC_COLS, r = blockIdx.y;
     const float g = decay[h];
+    const int half8 = half / 8;
     pdl_launch_dependents();
     for (int i = tid; i < RC_T * half; i += RC_THREADS) {  // offsets of the rows of a chunk: constants of the layer
         const int t = i / half, e = i - t * half;
         float sn, cs;
         sincosf(__fmul_rn((float)t, inv_freq[e]), &sn, &cs);
-        turn[t * (D / 2) + e] = make_float2(cs, sn);
+        turn[t * A + (e & 7) * half8 + (e >> 3)] = make_float2(cs, sn);  // (as the loop below reads: runs of 8 side by side)
     }
     for (int i = tid; i <= RC_T; i += RC_THREADS) pw[i] = powf(g, (float)i);
     pdl_wait();
@@ -393,7 +395,8 @@ retention_chunks_kernel(const bf16* __restrict__ proj, int64_t stride, const flo
     fetch(0);
 
     // the state as accumulators: this warp's 16 rows and UT column tiles
-    const int s_row = (D == 128 ? warp : warp & 3) * 16 + (lane >> 2), s_nt = D == 128 ? 0 : (warp >> 2) * UT;
+    const int s_row = (warp % (D / 16)) * 16 + (lane >> 2), s_nt = warp / (D / 16) * UT;
+    const bool s_mine = s_nt < NT && s_row - (lane >> 2) < dim;
     float* sp = state + ((int64_t)slot * heads + h) * dim * vdim;
     float acc_s[UT][4];
 #pragma unroll
@@ -402,19 +405,18 @@ retention_chunks_kernel(const bf16* __restrict__ proj, int64_t stride, const flo
         for (int e = 0; e < 2; ++e) {
             const int row = s_row + e * 8, col = c0 + (s_nt + n) * 8 + (lane & 3) * 2;
             float2 x = make_float2(0.f, 0.f);
-            if (row < dim && col < vdim) x = *reinterpret_cast<const float2*>(sp + (int64_t)row * vdim + col);
+            if (s_mine && row < dim && col < vdim) x = *reinterpret_cast<const float2*>(sp + (int64_t)row * vdim + col);
             acc_s[n][2 * e] = x.x;
             acc_s[n][2 * e + 1] = x.y;
         }
-    const int rt = warp & 3, part = warp >> 2;  // rows 16 rt .. of the chunk; which half of the keys and of the state's rows
-    const int half8 = half / 8;
+    const int rt = warp & 3, part = warp >> 2;  // rows 16 rt .. of the chunk; which keys and which of the state's rows
 
     for (int t0 = 0; t0 < q_len; t0 += RC_T) {
         const int nb = min(RC_T, q_len - t0);
         for (int i = tid; i < half; i += RC_THREADS) {
             float sn, cs;
             sincosf(__fmul_rn((float)(pos0 + t0), inv_freq[i]), &sn, &cs);
-            base[i] = make_float2(cs, sn);
+            base[(i & 7) * half8 + (i >> 3)] = make_float2(cs, sn);
         }
         cp_async_wait<0>();
         __syncthreads();  // the rows and the chunk's first angles; and the chunk in front is done with everything below
@@ -428,7 +430,7 @@ retention_chunks_kernel(const bf16* __restrict__ proj, int64_t stride, const flo
             const float f = which ? k_scale : 1.f;
 #pragma unroll
             for (int e = 0; e < 8; ++e) {
-                const float2 a = turn[t * (D / 2) + c + e], b = base[c + e];
+                const float2 a = turn[t * A + e * half8 + (c >> 3)], b = base[e * half8 + (c >> 3)];
                 const float cs = (a.x * b.x - a.y * b.y) * f, sn = (a.y * b.x + a.x * b.y) * f;
                 const float x = u[e] * cs - v[e] * sn;
                 v[e] = v[e] * cs + u[e] * sn;
@@ -472,52 +474,50 @@ retention_chunks_kernel(const bf16* __restrict__ proj, int64_t stride, const flo
             *reinterpret_cast<uint4*>(Wh + t * V + c) = ph;
             *reinterpret_cast<uint4*>(Wl + t * V + c) = pl;
         }
+        if (s_nt < NT) {
 #pragma unroll
-        for (int n = 0; n < UT; ++n)
+            for (int n = 0; n < UT; ++n)
 #pragma unroll
-            for (int e = 0; e < 2; ++e) {
-                const int at = (s_row + e * 8) * V + (s_nt + n) * 8 + (lane & 3) * 2;
-                const float x = acc_s[n][2 * e], y = acc_s[n][2 * e + 1];
-                const uint32_t hi = pack_bf16(x, y);
-                *reinterpret_cast<uint32_t*>(Sh + at) = hi;
-                *reinterpret_cast<uint32_t*>(Sl + at) = pack_bf16(x - __uint_as_float(hi << 16), y - __uint_as_float(hi & 0xffff0000u));
-            }
+                for (int e = 0; e < 2; ++e) {
+                    const int at = (s_row + e * 8) * V + (s_nt + n) * 8 + (lane & 3) * 2;
+                    const float x = acc_s[n][2 * e], y = acc_s[n][2 * e + 1];
+                    const uint32_t hi = pack_bf16(x, y);
+                    *reinterpret_cast<uint32_t*>(Sh + at) = hi;
+                    *reinterpret_cast<uint32_t*>(Sl + at) = pack_bf16(x - __uint_as_float(hi << 16), y - __uint_as_float(hi & 0xffff0000u));
+                }
+        }
         __syncthreads();
         if (t0 + RC_T < q_len) fetch(t0 + RC_T);  // the rows as they came have been used up
 
-        // scores of 16 rows with every other 16 keys up to the diagonal, and half of q S_0
-        const bool rows_on = rt * 16 < nb;
-        float sc[2][2][4], o[NT][4];
+        // scores of 16 rows with 16 keys up to the diagonal, and a quarter of q S_0
+        const bool rows_on = rt * 16 < nb, keys_on = part <= rt;
+        float sc[2][4], o[NT][4];
 #pragma unroll
         for (int n = 0; n < NT; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
 #pragma unroll
-        for (int b = 0; b < 2; ++b)
-#pragma unroll
-            for (int n = 0; n < 2; ++n) sc[b][n][0] = sc[b][n][1] = sc[b][n][2] = sc[b][n][3] = 0.f;
+        for (int n = 0; n < 2; ++n) sc[n][0] = sc[n][1] = sc[n][2] = sc[n][3] = 0.f;
         if (rows_on) {
 #pragma unroll
             for (int ks = 0; ks < KS; ++ks) {
+                const bool state_on = ks / (KS / 4) == part;
+                if (!keys_on && !state_on) continue;
                 uint32_t qh[4], ql[4];
                 const int qa = (rt * 16 + (lane & 15)) * S + ks * 16 + ((lane >> 4) << 3);
                 ldmatrix_x4(qh, Qh + qa);
                 ldmatrix_x4(ql, Ql + qa);
+                if (keys_on) {
+                    uint32_t kh[4], kl[4];
+                    const int ka = (part * 16 + (lane & 7) + ((lane >> 4) << 3)) * S + ks * 16 + (((lane >> 3) & 1) << 3);
+                    ldmatrix_x4(kh, Kh + ka);
+                    ldmatrix_x4(kl, Kl + ka);
 #pragma unroll
-                for (int b = 0; b < 2; ++b) {
-                    const int kb = part + 2 * b;
-                    if (kb <= rt) {
-                        uint32_t kh[4], kl[4];
-                        const int ka = (kb * 16 + (lane & 7) + ((lane >> 4) << 3)) * S + ks * 16 + (((lane >> 3) & 1) << 3);
-                        ldmatrix_x4(kh, Kh + ka);
-                        ldmatrix_x4(kl, Kl + ka);
-#pragma unroll
-                        for (int n = 0; n < 2; ++n) {
-                            mma_bf16(sc[b][n], qh, kh[2 * n], kh[2 * n + 1]);
-                            mma_bf16(sc[b][n], qh, kl[2 * n], kl[2 * n + 1]);
-                            mma_bf16(sc[b][n], ql, kh[2 * n], kh[2 * n + 1]);
-                        }
+                    for (int n = 0; n < 2; ++n) {
+                        mma_bf16(sc[n], qh, kh[2 * n], kh[2 * n + 1]);
+                        mma_bf16(sc[n], qh, kl[2 * n], kl[2 * n + 1]);
+                        mma_bf16(sc[n], ql, kh[2 * n], kh[2 * n + 1]);
                     }
                 }
-                if (ks / (KS / 2) == part) {
+                if (state_on) {
 #pragma unroll
                     for (int n = 0; n < NT; n += 2) {
                         uint32_t sh[4], sl[4];
@@ -540,42 +540,43 @@ retention_chunks_kernel(const bf16* __restrict__ proj, int64_t stride, const flo
                 o[n][0] *= f_lo; o[n][1] *= f_lo;
                 o[n][2] *= f_hi; o[n][3] *= f_hi;
             }
+            if (keys_on) {
+                uint32_t ah[4], al[4];
 #pragma unroll
-            for (int b = 0; b < 2; ++b) {
-                const int kb = part + 2 * b;
-                if (kb <= rt) {
-                    uint32_t ah[4], al[4];
+                for (int n = 0; n < 2; ++n) {
+                    const int key = part * 16 + n * 8 + ((lane & 3) << 1);
+                    float x[4];
 #pragma unroll
-                    for (int n = 0; n < 2; ++n) {
-                        const int key = kb * 16 + n * 8 + ((lane & 3) << 1);
-                        float x[4];
-#pragma unroll
-                        for (int e = 0; e < 4; ++e) {
-                            const int back = (e < 2 ? row_lo : row_hi) - (key + (e & 1));
-                            x[e] = back >= 0 ? sc[b][n][e] * pw[back] : 0.f;
-                        }
-#pragma unroll
-                        for (int e = 0; e < 2; ++e) {
-                            const uint32_t hi = pack_bf16(x[2 * e], x[2 * e + 1]);
-                            ah[2 * n + e] = hi;
-                            al[2 * n + e] = pack_bf16(x[2 * e] - __uint_as_float(hi << 16), x[2 * e + 1] - __uint_as_float(hi & 0xffff0000u));
-                        }
+                    for (int e = 0; e < 4; ++e) {
+                        const int back = (e < 2 ? row_lo : row_hi) - (key + (e & 1));
+                        x[e] = back >= 0 ? sc[n][e] * pw[back] : 0.f;
                     }
 #pragma unroll
-                    for (int n = 0; n < NT; n += 2) {
-                        uint32_t vv[4];
-                        ldmatrix_x4_trans(vv, Vs + (kb * 16 + (lane & 7) + (((lane >> 3) & 1) << 3)) * V + n * 8 + ((lane >> 4) << 3));
+                    for (int e = 0; e < 2; ++e) {
+                        const uint32_t hi = pack_bf16(x[2 * e], x[2 * e + 1]);
+                        ah[2 * n + e] = hi;
+                        al[2 * n + e] = pack_bf16(x[2 * e] - __uint_as_float(hi << 16), x[2 * e + 1] - __uint_as_float(hi & 0xffff0000u));
+                    }
+                }
 #pragma unroll
-                        for (int m = 0; m < 2; ++m) {
-                            mma_bf16(o[n + m], ah, vv[2 * m], vv[2 * m + 1]);
-                            mma_bf16(o[n + m], al, vv[2 * m], vv[2 * m + 1]);
-                        }
+                for (int n = 0; n < NT; n += 2) {
+                    uint32_t vv[4];
+                    ldmatrix_x4_trans(vv, Vs + (part * 16 + (lane & 7) + (((lane >> 3) & 1) << 3)) * V + n * 8 + ((lane >> 4) << 3));
+#pragma unroll
+                    for (int m = 0; m < 2; ++m) {
+                        mma_bf16(o[n + m], ah, vv[2 * m], vv[2 * m + 1]);
+                        mma_bf16(o[n + m], al, vv[2 * m], vv[2 * m + 1]);
                     }
                 }
             }
+#pragma unroll
+            for (int n = 0; n < NT; ++n)
+#pragma unroll
+                for (int e = 0; e < 2; ++e)
+                    *reinterpret_cast<float2*>(sums + (part * RC_T + row_lo + e * 8) * V + n * 8 + (lane & 3) * 2) = make_float2(o[n][2 * e], o[n][2 * e + 1]);
         }
         // the state behind the chunk
-        if (s_row - (lane >> 2) < dim) {
+        if (s_mine) {
             const float f = pw[nb];
 #pragma unroll
             for (int n = 0; n < UT; ++n)
@@ -604,25 +605,19 @@ retention_chunks_kernel(const bf16* __restrict__ proj, int64_t stride, const flo
                 }
             }
         }
-        if (part == 1 && rows_on) {
-#pragma unroll
-            for (int n = 0; n < NT; ++n)
-#pragma unroll
-                for (int e = 0; e < 2; ++e)
-                    *reinterpret_cast<float2*>(sums + (rt * 16 + (lane >> 2) + e * 8) * V + n * 8 + (lane & 3) * 2) = make_float2(o[n][2 * e], o[n][2 * e + 1]);
-        }
         __syncthreads();
-        if (part == 0 && rows_on) {
+        {
+            const int t = tid / (RC_COLS / 4), c = (tid % (RC_COLS / 4)) * 4;
+            static_assert(RC_THREADS == RC_T * (RC_COLS / 4), "a thread adds four neighbouring sums");
+            if (t < nb && c0 + c < vdim) {
+                float4 x = *reinterpret_cast<const float4*>(sums + t * V + c);
 #pragma unroll
-            for (int n = 0; n < NT; ++n)
-#pragma unroll
-                for (int e = 0; e < 2; ++e) {
-                    const int t = rt * 16 + (lane >> 2) + e * 8, c = n * 8 + (lane & 3) * 2;
-                    const float2 other = *reinterpret_cast<const float2*>(sums + t * V + c);
-                    if (t < nb && c0 + c < vdim)
-                        *reinterpret_cast<float2*>(out + ((int64_t)(q0 + t0 + t) * heads + h) * vdim + c0 + c) =
-                            make_float2(o[n][2 * e] + other.x, o[n][2 * e + 1] + other.y);
+                for (int p = 1; p < 4; ++p) {
+                    const float4 y = *reinterpret_cast<const float4*>(sums + (p * RC_T + t) * V + c);
+                    x.x += y.x; x.y += y.y; x.z += y.z; x.w += y.w;
                 }
+                *reinterpret_cast<float4*>(out + ((int64_t)(q0 + t0 + t) * heads + h) * vdim + c0 + c) = x;
+            }
         }
     }
 #pragma unroll
@@ -630,7 +625,7 @@ retention_chunks_kernel(const bf16* __restrict__ proj, int64_t stride, const flo
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
             const int row = s_row + e * 8, col = c0 + (s_nt + n) * 8 + (lane & 3) * 2;
-            if (row < dim && col < vdim) *reinterpret_cast<float2*>(sp + (int64_t)row * vdim + col) = make_float2(acc_s[n][2 * e], acc_s[n][2 * e + 1]);
+            if (s_mine && row < dim && col < vdim) *reinterpret_cast<float2*>(sp + (int64_t)row * vdim + col) = make_float2(acc_s[n][2 * e], acc_s[n][2 * e + 1]);
         }
 }
 
