@@ -1615,8 +1615,10 @@ def run_compare_sazepel(args) -> int:
         hbm(f"{tag}_branch_norm (fusipel)",
             sweep(lambda i: ops.branch_norm(streams[i], ys[i], wb, eps, 1.0, w, eps, torch.bfloat16)), tokens * h * 12.0)
         hbm(f"{tag}_scaled_sum of two mixers (lakadra)", sweep(lambda i: ops.scaled_sum(ys[i], 0.5, y2s[i], 0.5)), tokens * h * 6.0)
+        hbm(f"{tag}_branch_norm that forms a normed pair",
+            sweep(lambda i: ops.branch_norm(streams[i], ops.PairedOutput(ys[i], w, y2s[i], wb, eps, 0.5), wb, eps, 1.0, w, eps, torch.bfloat16)),
+            tokens * h * 14.0)
         hbm(f"{tag}_normed_pair (alone)", sweep(lambda i: ops.normed_pair(ys[i], w, y2s[i], wb, eps, 0.5)), tokens * h * 6.0)
-        del streams
         # queries, keys and values to their norms and pages
         rows = [rand(tokens, (2 * n_q + 2 * n_kv) * d) for _ in range(6)]
         qkv = [r[:, : (n_q + 2 * n_kv) * d].contiguous() for r in rows]
@@ -1637,6 +1639,9 @@ def run_compare_sazepel(args) -> int:
                            ("retention token by token", dict(silu=False, inv_freq=inv, k_scale=d ** -0.5, chunks=False))):
             us = sweep(lambda i: ops.decay_attention(proj[i], decay, memory[i], ctx, n_q, d, d, **more))
             hbm(f"{tag}_{what}", us, moved, fp32_tflops=round(4.0 * tokens * n_q * d * d / us / 1e6, 2))
+        hbm(f"{tag}_retention with its norm and gate", sweep(lambda i: ops.retention(proj[i], decay, memory[i], ctx, n_q, d, d, eps, inv_freq=inv,
+                                                                                       k_scale=d ** -0.5)),
+            R * n_q * d * d * 8.0 + tokens * n_q * d * (4 * 2.0 + 2.0))
         mixed = [ops.decay_attention(p, decay, m, ctx, n_q, d, d) for p, m in zip(proj, memory)]
         w_all = rand(n_q * d, dtype=torch.float32)
         hbm(f"{tag}_gated_rmsnorm (lakadra)", sweep(lambda i: ops.gated_rmsnorm(mixed[i], proj[i][:, 3 * n_q * d:], w_all, eps, torch.bfloat16)),
@@ -1661,8 +1666,11 @@ def run_compare_sazepel(args) -> int:
         y, place = ops.moe_experts(ys[0], chosen, None, gate_up, down, 64)
         each = 2.0 if place is not None else 4.0
         hbm(f"{tag}_moe_combine (sarudra)", sweep(lambda i: ops.moe_combine(y, None, torch.bfloat16, place, 2)), tokens * h * (2 * each + 2.0))
+        hbm(f"{tag}_branch_norm that sums the chosen experts",
+            sweep(lambda i: ops.branch_norm(streams[i], ops.WeighedTerms(y, place, scores), wb, eps, 1.0, w, eps, torch.bfloat16)),
+            tokens * h * (2 * each + 10.0))
         hbm(f"{tag}_moe_mix (alone)", sweep(lambda i: ops.moe_mix(y, place, chosen, scores, 8, ys[i])), tokens * h * (2 * each + 2.0))
-        del gate_up, down, y, ys, y2s
+        del gate_up, down, y, ys, y2s, streams
 
     # attention of a prompt in one step.  The operations counted are the design's own: scores, the mixture of the heads'
     # weights, values

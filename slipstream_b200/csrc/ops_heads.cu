@@ -342,6 +342,9 @@ extern "C" int ss_diff_combine(const float* x, void* out, int64_t n_tokens, int 
 // ---------------------------------------------------------------- a branch's normed output, and the next norm
 //
 // residual += mult * (y / sqrt(mean(y^2) + eps_y) * w_y) [+ anchor], then out = residual / sqrt(mean(residual^2) + eps) * w.
+// y is a branch's output, or one that has not been formed yet (SRC): the weighted sum of two outputs under norms of their
+// own, pair_scale * (a / rms(a) * wa + b / rms(b) * wb), or the sum over a token's chosen experts of weight * output (float32
+// [token][choice][hidden], or bfloat16 rows in sorted order with the place of every (token, choice)).
 // y null: the second half only.  With `rows` only those rows are produced and the stream stays as it is.  Weights are
 // float32.  A block per row.  VEC 8: hidden a multiple of 8, at most 8 elements a thread, each row read once; VEC 1: any.
 struct BranchArgs {
@@ -354,14 +357,21 @@ struct BranchArgs {
     const int32_t* rows;
     int hidden;
     float mult, y_eps, eps;
+    const void* y2;  // SRC_PAIR: y is a, y2 is b
+    const float* pair_weight[2];
+    float pair_eps, pair_scale;
+    const float* term_weight;  // SRC_TERMS: [token][top]
+    const int32_t* place;      // y holds sorted rows (of type T); null: y is float32 in order
+    int top;
 };
+enum { SRC_PLAIN = 0, SRC_PAIR = 1, SRC_TERMS = 2 };
 
 // EARLY (few rows): the weights are in registers before the kernels in front are complete; with many rows they are read
 // where they are used, which leaves room for more blocks on an SM.
-template <typename T, int VEC, bool EARLY>
+template <typename T, int VEC, bool EARLY, int SRC>
 __global__ void __launch_bounds__(1024) branch_norm_kernel(const BranchArgs a) {
     pdl_launch_dependents();
-    __shared__ float scratch[2][32];
+    __shared__ float scratch[4][32];
     const int hidden = a.hidden;
     if constexpr (VEC == 8) {
         const int j = threadIdx.x * 8;
@@ -382,12 +392,47 @@ __global__ void __launch_bounds__(1024) branch_norm_kernel(const BranchArgs a) {
 #pragma unroll
             for (int e = 0; e < 8; ++e) y[e] = 0.f;
             float ss = 0.f;
-            if (on) {
-                if constexpr (sizeof(T) == 2) unpack8(*reinterpret_cast<const uint4*>(reinterpret_cast<const T*>(a.y) + src * hidden + j), y);
-                else load8f(reinterpret_cast<const float*>(a.y) + src * hidden + j, y);
+            auto row8 = [&](const void* p, int64_t row, float (&x)[8]) {
+                if constexpr (sizeof(T) == 2) unpack8(*reinterpret_cast<const uint4*>(reinterpret_cast<const T*>(p) + row * hidden + j), x);
+                else load8f(reinterpret_cast<const float*>(p) + row * hidden + j, x);
+            };
+            if constexpr (SRC == SRC_PLAIN) {
+                if (on) row8(a.y, src, y);
+            } else if constexpr (SRC == SRC_PAIR) {
+                float b[8], sa = 0.f, sb = 0.f;
 #pragma unroll
-                for (int e = 0; e < 8; ++e) ss = fmaf(y[e], y[e], ss);
+                for (int e = 0; e < 8; ++e) b[e] = 0.f;
+                if (on) {
+                    row8(a.y, src, y);
+                    row8(a.y2, src, b);
+                }
+#pragma unroll
+                for (int e = 0; e < 8; ++e) {
+                    sa = fmaf(y[e], y[e], sa);
+                    sb = fmaf(b[e], b[e], sb);
+                }
+                const float fa = a.pair_scale / sqrtf(block_sum_once(sa, scratch[2]) / (float)hidden + a.pair_eps);
+                const float fb = a.pair_scale / sqrtf(block_sum_once(sb, scratch[3]) / (float)hidden + a.pair_eps);
+                if (on) {
+                    float wa[8], wb[8];
+                    load8f(a.pair_weight[0] + j, wa);
+                    load8f(a.pair_weight[1] + j, wb);
+#pragma unroll
+                    for (int e = 0; e < 8; ++e) y[e] = fmaf(y[e] * fa, wa[e], b[e] * fb * wb[e]);
+                }
+            } else if (on) {
+                for (int k = 0; k < a.top; ++k) {
+                    const int64_t at = src * a.top + k;
+                    float t[8];
+                    if (a.place) row8(a.y, a.place[at], t);
+                    else load8f(reinterpret_cast<const float*>(a.y) + at * hidden + j, t);
+                    const float w = a.term_weight[at];
+#pragma unroll
+                    for (int e = 0; e < 8; ++e) y[e] = fmaf(w, t[e], y[e]);
+                }
             }
+#pragma unroll
+            for (int e = 0; e < 8; ++e) ss = fmaf(y[e], y[e], ss);
             float anchor[8];
             if (on && a.anchor) load8f(a.anchor + src * hidden + j, anchor);
             const float f = 1.0f / sqrtf(block_sum_once(ss, scratch[0]) / (float)hidden + a.y_eps);
@@ -418,19 +463,49 @@ __global__ void __launch_bounds__(1024) branch_norm_kernel(const BranchArgs a) {
         pdl_wait();
         const int64_t src = a.rows ? a.rows[blockIdx.x] : blockIdx.x;
         float* res = a.residual + src * hidden;
-        const T* y = a.y ? reinterpret_cast<const T*>(a.y) + src * hidden : nullptr;
+        float fa = 0.f, fb = 0.f;
+        auto branch = [&](int j) -> float {  // element j of the branch's output
+            const T* y = reinterpret_cast<const T*>(a.y);
+            if constexpr (SRC == SRC_PLAIN) {
+                return to_float(y[src * hidden + j]);
+            } else if constexpr (SRC == SRC_PAIR) {
+                return fmaf(to_float(y[src * hidden + j]) * fa, a.pair_weight[0][j],
+                            to_float(reinterpret_cast<const T*>(a.y2)[src * hidden + j]) * fb * a.pair_weight[1][j]);
+            } else {
+                float sum = 0.f;
+                for (int k = 0; k < a.top; ++k) {
+                    const int64_t at = src * a.top + k;
+                    const float t = a.place ? to_float(y[(int64_t)a.place[at] * hidden + j]) : reinterpret_cast<const float*>(a.y)[at * hidden + j];
+                    sum = fmaf(a.term_weight[at], t, sum);
+                }
+                return sum;
+            }
+        };
+        if constexpr (SRC == SRC_PAIR) {
+            float sa = 0.f, sb = 0.f;
+            for (int j = threadIdx.x; j < hidden; j += blockDim.x) {
+                const float x = to_float(reinterpret_cast<const T*>(a.y)[src * hidden + j]), z = to_float(reinterpret_cast<const T*>(a.y2)[src * hidden + j]);
+                sa = fmaf(x, x, sa);
+                sb = fmaf(z, z, sb);
+            }
+            fa = a.pair_scale / sqrtf(block_sum_once(sa, scratch[2]) / (float)hidden + a.pair_eps);
+            fb = a.pair_scale / sqrtf(block_sum_once(sb, scratch[3]) / (float)hidden + a.pair_eps);
+        }
         const float* anchor = a.anchor ? a.anchor + src * hidden : nullptr;
         T* out = reinterpret_cast<T*>(a.out) + (int64_t)blockIdx.x * hidden;
         float fy = 0.f;
-        if (y) {
+        if (a.y) {
             float ss = 0.f;
-            for (int j = threadIdx.x; j < hidden; j += blockDim.x) ss = fmaf(to_float(y[j]), to_float(y[j]), ss);
+            for (int j = threadIdx.x; j < hidden; j += blockDim.x) {
+                const float v = branch(j);
+                ss = fmaf(v, v, ss);
+            }
             fy = 1.0f / sqrtf(block_sum_once(ss, scratch[0]) / (float)hidden + a.y_eps);
         }
         auto joined = [&](int j) {
             float v = res[j];
-            if (y) {
-                v = fmaf(a.mult, to_float(y[j]) * fy * a.y_weight[j], v);
+            if (a.y) {
+                v = fmaf(a.mult, branch(j) * fy * a.y_weight[j], v);
                 if (anchor) v += anchor[j];
             }
             return v;
@@ -443,31 +518,45 @@ __global__ void __launch_bounds__(1024) branch_norm_kernel(const BranchArgs a) {
         const float f = 1.0f / sqrtf(block_sum_once(ss, scratch[1]) / (float)hidden + a.eps);
         for (int j = threadIdx.x; j < hidden; j += blockDim.x) {  // every thread meets its own elements again
             const float v = joined(j);
-            if (y && !a.rows) res[j] = v;
+            if (a.y && !a.rows) res[j] = v;
             out[j] = from_float<T>(v * f * a.weight[j]);
         }
     }
 }
 
-extern "C" int ss_branch_norm(float* residual, const void* y, const float* y_weight, float y_eps, float mult, const float* anchor,
-                              const float* weight, float eps, void* out, const int32_t* rows, int n_rows, int hidden, int dtype,
-                              cudaStream_t stream) {
-    if (n_rows <= 0) return 0;
-    if (hidden < 1 || (y && !y_weight) || (!y && anchor)) return (int)cudaErrorInvalidValue;
-    BranchArgs a;
-    a.residual = residual; a.y = y; a.y_weight = y_weight; a.anchor = anchor; a.weight = weight; a.out = out; a.rows = rows;
-    a.hidden = hidden; a.mult = mult; a.y_eps = y_eps; a.eps = eps;
-    const bool aligned = (((uintptr_t)residual | (uintptr_t)y | (uintptr_t)y_weight | (uintptr_t)anchor | (uintptr_t)weight | (uintptr_t)out) & 15) == 0;
+template <int SRC>
+static int launch_branch_norm(const BranchArgs& a, int n_rows, int dtype, bool aligned, cudaStream_t stream) {
+    const int hidden = a.hidden;
     if (hidden % 8 == 0 && hidden <= 8192 && aligned) {
         const dim3 block((hidden / 8 + 31) / 32 * 32);
         const bool many = n_rows >= 2 * ss_sm_count();
-        if (dtype == SS_BF16 && many) ss_launch(branch_norm_kernel<bf16, 8, false>, dim3(n_rows), block, 0, stream, a);
-        else if (dtype == SS_BF16) ss_launch(branch_norm_kernel<bf16, 8, true>, dim3(n_rows), block, 0, stream, a);
-        else ss_launch(branch_norm_kernel<float, 8, true>, dim3(n_rows), block, 0, stream, a);
+        if (dtype == SS_BF16 && many) ss_launch(branch_norm_kernel<bf16, 8, false, SRC>, dim3(n_rows), block, 0, stream, a);
+        else if (dtype == SS_BF16) ss_launch(branch_norm_kernel<bf16, 8, true, SRC>, dim3(n_rows), block, 0, stream, a);
+        else ss_launch(branch_norm_kernel<float, 8, true, SRC>, dim3(n_rows), block, 0, stream, a);
     } else {
         const dim3 block(hidden >= 2048 ? 512 : (hidden >= 512 ? 256 : 128));
-        if (dtype == SS_BF16) ss_launch(branch_norm_kernel<bf16, 1, false>, dim3(n_rows), block, 0, stream, a);
-        else ss_launch(branch_norm_kernel<float, 1, false>, dim3(n_rows), block, 0, stream, a);
+        if (dtype == SS_BF16) ss_launch(branch_norm_kernel<bf16, 1, false, SRC>, dim3(n_rows), block, 0, stream, a);
+        else ss_launch(branch_norm_kernel<float, 1, false, SRC>, dim3(n_rows), block, 0, stream, a);
     }
     return SS_LAUNCH_CHECK();
+}
+
+// y2 with pair_a, pair_b: SRC_PAIR.  term_weight: SRC_TERMS.
+extern "C" int ss_branch_norm(float* residual, const void* y, const float* y_weight, float y_eps, float mult, const float* anchor,
+                              const float* weight, float eps, void* out, const int32_t* rows, int n_rows, int hidden, int dtype,
+                              cudaStream_t stream, const void* y2, const float* pair_a, const float* pair_b, float pair_eps, float pair_scale,
+                              const float* term_weight, const int32_t* place, int top) {
+    if (n_rows <= 0) return 0;
+    if (hidden < 1 || (y && !y_weight) || (!y && anchor) || (y2 && (!y || !pair_a || !pair_b || term_weight)) || (term_weight && (!y || top < 1)))
+        return (int)cudaErrorInvalidValue;
+    BranchArgs a;
+    a.residual = residual; a.y = y; a.y_weight = y_weight; a.anchor = anchor; a.weight = weight; a.out = out; a.rows = rows;
+    a.hidden = hidden; a.mult = mult; a.y_eps = y_eps; a.eps = eps;
+    a.y2 = y2; a.pair_weight[0] = pair_a; a.pair_weight[1] = pair_b; a.pair_eps = pair_eps; a.pair_scale = pair_scale;
+    a.term_weight = term_weight; a.place = place; a.top = top;
+    const bool aligned = (((uintptr_t)residual | (uintptr_t)y | (uintptr_t)y_weight | (uintptr_t)anchor | (uintptr_t)weight | (uintptr_t)out |
+                           (uintptr_t)y2 | (uintptr_t)pair_a | (uintptr_t)pair_b) & 15) == 0;
+    if (y2) return launch_branch_norm<SRC_PAIR>(a, n_rows, dtype, aligned, stream);
+    if (term_weight) return launch_branch_norm<SRC_TERMS>(a, n_rows, dtype, aligned, stream);
+    return launch_branch_norm<SRC_PLAIN>(a, n_rows, dtype, aligned, stream);
 }

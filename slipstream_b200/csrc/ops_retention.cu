@@ -655,3 +655,112 @@ extern "C" int ss_retention_chunks(const void* proj, int64_t stride, const float
     return launch_retention_chunks<128>((const bf16*)proj, stride, decay, state, out, q_start, seq_lens, slots, R, heads, dim, vdim, n_slots, err,
                                         stream, inv_freq, half, k_scale);
 }
+
+// ---------------------------------------------------------------- retention of single tokens, head norm and gate included
+//
+// A decode step: every request brings one token.  S <- g S + k v^T, o = S^T q as above, then o / sqrt(mean(o^2) + eps) *
+// silu(gate) head by head, in T.  A block takes a head of a request whole: a thread holds four neighbouring columns of every
+// RG-th row of the state, all its loads in flight before the first is used; the row groups' sums meet in shared memory.
+// vdim a multiple of 4 up to 256.
+#define RD_THREADS 512
+#define RD_ROWS 8  // rows of the state a thread has in flight
+template <typename T>
+__global__ void __launch_bounds__(RD_THREADS, 2)
+retention_token_kernel(const T* __restrict__ proj, int64_t stride, const float* __restrict__ decay, float* __restrict__ state,
+                       T* __restrict__ out, const int32_t* __restrict__ q_start, const int32_t* __restrict__ seq_lens,
+                       const int32_t* __restrict__ slots, int heads, int dim, int vdim, int n_slots, int* err,
+                       const float* __restrict__ inv_freq, int half, float k_scale, float eps) {
+    __shared__ float qs[256], ks[256], scratch[33];
+    __shared__ __align__(16) float sums[4 * RD_THREADS];
+    const int tid = threadIdx.x, h = blockIdx.x, r = blockIdx.y;
+    const int cols4 = vdim >> 2, groups = RD_THREADS / cols4;
+    const int c4 = tid % cols4, rg = tid / cols4;
+    const bool on = rg < groups;
+    const float g = decay[h];
+    pdl_launch_dependents();
+    pdl_wait();
+    const int seq_len = seq_lens[r];
+    if (q_start[r + 1] <= q_start[r] || seq_len <= 0) return;
+    const int slot = slots[r];
+    if (slot < 0 || slot >= n_slots) {
+        if (tid == 0) atomicOr(err, SS_ERR_SLOT_RANGE);
+        return;
+    }
+    float4* sp = reinterpret_cast<float4*>(state + ((int64_t)slot * heads + h) * dim * vdim) + c4;
+    float4 s[RD_ROWS];
+#pragma unroll
+    for (int i = 0; i < RD_ROWS; ++i) {
+        const int row = rg + i * groups;
+        if (on && row < dim) s[i] = sp[(int64_t)row * cols4];
+    }
+    const int64_t row_q = q_start[r];
+    const T* src = proj + row_q * stride;
+    const int64_t k_off = (int64_t)heads * dim;
+    for (int i = tid; i < dim; i += RD_THREADS) {
+        if (i < half) {
+            float sn, cs;
+            sincosf(__fmul_rn((float)(seq_len - 1), inv_freq[i]), &sn, &cs);
+            const float q1 = to_float(src[(int64_t)h * dim + i]), q2 = to_float(src[(int64_t)h * dim + i + half]);
+            const float k1 = to_float(src[k_off + (int64_t)h * dim + i]), k2 = to_float(src[k_off + (int64_t)h * dim + i + half]);
+            qs[i] = q1 * cs - q2 * sn;
+            qs[i + half] = q2 * cs + q1 * sn;
+            ks[i] = (k1 * cs - k2 * sn) * k_scale;
+            ks[i + half] = (k2 * cs + k1 * sn) * k_scale;
+        } else if (i >= 2 * half) {
+            qs[i] = to_float(src[(int64_t)h * dim + i]);
+            ks[i] = to_float(src[k_off + (int64_t)h * dim + i]) * k_scale;
+        }
+    }
+    float v[4] = {0.f, 0.f, 0.f, 0.f};
+    const T* vp = src + 2 * k_off + (int64_t)h * vdim;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) v[e] = to_float(vp[c4 * 4 + e]);
+    __syncthreads();
+    float o[4] = {0.f, 0.f, 0.f, 0.f};
+    auto row_of = [&](const float4& old, int row) {
+        const float k = ks[row], q = qs[row];
+        float4 n;
+        n.x = fmaf(k, v[0], g * old.x); n.y = fmaf(k, v[1], g * old.y);
+        n.z = fmaf(k, v[2], g * old.z); n.w = fmaf(k, v[3], g * old.w);
+        o[0] = fmaf(n.x, q, o[0]); o[1] = fmaf(n.y, q, o[1]);
+        o[2] = fmaf(n.z, q, o[2]); o[3] = fmaf(n.w, q, o[3]);
+        sp[(int64_t)row * cols4] = n;
+    };
+    if (on) {
+#pragma unroll
+        for (int i = 0; i < RD_ROWS; ++i) {
+            const int row = rg + i * groups;
+            if (row < dim) row_of(s[i], row);
+        }
+        for (int row = rg + RD_ROWS * groups; row < dim; row += groups) row_of(sp[(int64_t)row * cols4], row);
+        *reinterpret_cast<float4*>(sums + (rg * cols4 + c4) * 4) = make_float4(o[0], o[1], o[2], o[3]);
+    }
+    __syncthreads();
+    float x = 0.f;
+    if (tid < vdim)
+        for (int i = 0; i < groups; ++i) x += sums[i * vdim + tid];
+    const float f = 1.0f / sqrtf(block_sum(x * x, scratch) / (float)vdim + eps);
+    if (tid < vdim) {
+        const int64_t at = (int64_t)h * vdim + tid;
+        const float gate = to_float(src[2 * k_off + (int64_t)heads * vdim + at]);
+        out[row_q * heads * vdim + at] = from_float<T>(x * f * silu_of<T>(gate));
+    }
+}
+
+// proj row: [q | k | v | gate], heads * (2 dim + 2 vdim) elements; out [rows][heads * vdim] in the type of proj.
+extern "C" int ss_retention_token(const void* proj, int64_t stride, const float* decay, float* state, void* out, const int32_t* q_start,
+                                  const int32_t* seq_lens, const int32_t* slots, int R, int heads, int dim, int vdim, int n_slots, int dtype,
+                                  int* err, cudaStream_t stream, const float* inv_freq, int half, float k_scale, float eps) {
+    if (R <= 0) return 0;
+    if (heads < 1 || dim < 1 || dim > 256 || vdim < 4 || vdim > 256 || vdim % 4 || half < 0 || 2 * half > dim || (half > 0 && !inv_freq) ||
+        ((uintptr_t)state & 15))
+        return (int)cudaErrorInvalidValue;
+    const dim3 grid(heads, R), block(RD_THREADS);
+    if (dtype == SS_BF16)
+        ss_launch(retention_token_kernel<bf16>, grid, block, 0, stream, (const bf16*)proj, stride, decay, state, (bf16*)out, q_start, seq_lens,
+                  slots, heads, dim, vdim, n_slots, err, inv_freq, half, k_scale, eps);
+    else
+        ss_launch(retention_token_kernel<float>, grid, block, 0, stream, (const float*)proj, stride, decay, state, (float*)out, q_start, seq_lens,
+                  slots, heads, dim, vdim, n_slots, err, inv_freq, half, k_scale, eps);
+    return SS_LAUNCH_CHECK();
+}

@@ -110,11 +110,13 @@ _OPS_SIGNATURES = {
                           c_void_p, c_void_p],
     "ss_diff_combine": [c_void_p, c_void_p, c_int64, c_int, c_int, c_int, c_float, c_float, c_float, c_int, c_void_p],
     "ss_branch_norm": [c_void_p, c_void_p, c_void_p, c_float, c_float, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_int,
-                       c_int, c_int, c_void_p],
+                       c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_float, c_void_p, c_void_p, c_int],
     "ss_embedding_norm": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_float, c_void_p, c_void_p],
     "ss_head_norm_gate": [c_void_p, c_void_p, c_int64, c_void_p, c_int, c_int, c_int, c_float, c_int, c_void_p],
     "ss_retention_chunks": [c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
                             c_int, c_void_p, c_void_p, c_void_p, c_int, c_float],
+    "ss_retention_token": [c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
+                           c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_float, c_float],
     "ss_talk_heads": [c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p],
     "ss_normed_pair": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_float, c_int, c_void_p],
 }
@@ -1052,21 +1054,73 @@ def heads_to_pages(rows: torch.Tensor, positions: torch.Tensor, slots: torch.Ten
     return q
 
 
-def branch_norm(residual: torch.Tensor, y: torch.Tensor | None, y_weight: torch.Tensor | None, y_eps: float, mult: float,
+@dataclasses.dataclass(frozen=True)
+class PairedOutput:
+    """The output of two branches side by side that has not been formed: ``scale * (rmsnorm(a) * a_weight + rmsnorm(b) *
+    b_weight)`` (`normed_pair`).  `branch_norm` forms it where it adds a branch to the stream."""
+
+    a: torch.Tensor
+    a_weight: torch.Tensor
+    b: torch.Tensor
+    b_weight: torch.Tensor
+    eps: float
+    scale: float
+
+    def materialize(self) -> torch.Tensor:
+        return normed_pair(self.a, self.a_weight, self.b, self.b_weight, self.eps, self.scale)
+
+
+@dataclasses.dataclass(frozen=True)
+class WeighedTerms:
+    """The output of routed experts that has not been summed: ``sum_k weights[t, k] * term(t, k)`` with the terms in either form
+    that `moe_experts` returns.  `branch_norm` forms it where it adds a branch to the stream."""
+
+    terms: torch.Tensor
+    rows: torch.Tensor | None
+    weights: torch.Tensor
+
+
+def branch_norm(residual: torch.Tensor, y: "torch.Tensor | PairedOutput | WeighedTerms | None", y_weight: torch.Tensor | None, y_eps: float, mult: float,
                 weight: torch.Tensor, eps: float, out_dtype: torch.dtype, *, anchor: torch.Tensor | None = None,
                 rows: torch.Tensor | None = None) -> torch.Tensor:
     """``residual`` (float32 [N, H]) += ``mult * rmsnorm(y) * y_weight`` (+ ``anchor``, float32 [N, H]) in place, then
     the RMS norm of the new stream times ``weight`` in ``out_dtype``.  Weights are float32, the arithmetic too, and the
-    result is rounded once.  With ``rows`` (int32 [M]) only those rows are produced and the stream stays as it is."""
+    result is rounded once.  With ``rows`` (int32 [M]) only those rows are produced and the stream stays as it is.  ``y`` may
+    be a `PairedOutput` or `WeighedTerms`, which is then formed inside, in float32."""
+    more: tuple = (None, None, None, 0.0, 0.0, None, None, 0)
+    if isinstance(y, PairedOutput):
+        pair = y
+        y = pair.a
+        _need(pair.b, out_dtype, "second output of a pair")
+        for w in (pair.a_weight, pair.b_weight):
+            _need(w, torch.float32, "norm weight of a pair")
+        if pair.b.shape != y.shape or pair.a_weight.numel() != y.shape[-1] or pair.b_weight.numel() != y.shape[-1]:
+            raise KernelError("the two outputs of a pair or their norms' weights differ in size")
+        more = (pair.b.data_ptr(), pair.a_weight.data_ptr(), pair.b_weight.data_ptr(), float(pair.eps), float(pair.scale), None, None, 0)
+    elif isinstance(y, WeighedTerms):
+        terms = y
+        n, top = terms.weights.shape
+        _need(terms.weights, torch.float32, "weights of the terms")
+        if terms.rows is None:
+            _need(terms.terms, torch.float32, "terms")
+        else:
+            _need(terms.terms, out_dtype, "sorted terms")
+            _need(terms.rows, torch.int32, "places of the terms")
+        if (n != residual.shape[0] or terms.terms.shape[-1] != residual.shape[-1]
+                or (terms.rows.numel() if terms.rows is not None else terms.terms.numel() // residual.shape[-1]) != n * top):
+            raise KernelError("the terms do not match the stream")
+        more = (None, None, None, 0.0, 0.0, terms.weights.data_ptr(), _ptr(terms.rows), top)
+        y = terms.terms
     _need(residual, torch.float32, "residual")
     hidden = residual.shape[-1]
     _need(weight, torch.float32, "norm weight")
     if weight.numel() != hidden:
         raise KernelError("norm weight has the wrong size")
     if y is not None:
-        _need(y, out_dtype, "branch output")
+        if more[5] is None:
+            _need(y, out_dtype, "branch output")
         _need(y_weight, torch.float32, "branch norm weight")
-        if y.shape != residual.shape or y_weight.numel() != hidden:
+        if (more[5] is None and y.shape != residual.shape) or y_weight.numel() != hidden:
             raise KernelError("branch output or its norm's weight does not match the stream")
     if anchor is not None:
         _need(anchor, torch.float32, "anchor")
@@ -1078,7 +1132,7 @@ def branch_norm(residual: torch.Tensor, y: torch.Tensor | None, y_weight: torch.
     out = torch.empty((n_out, hidden), dtype=out_dtype, device=residual.device)
     _check(ops_library().ss_branch_norm(residual.data_ptr(), _ptr(y), _ptr(y_weight) if y is not None else None, float(y_eps),
                                         float(mult), _ptr(anchor), weight.data_ptr(), float(eps), out.data_ptr(), _ptr(rows),
-                                        n_out, hidden, _code(out_dtype), _stream()), "branch_norm")
+                                        n_out, hidden, _code(out_dtype), _stream(), *more), "branch_norm")
     return out
 
 
@@ -2416,6 +2470,34 @@ def head_norm_gate(x: torch.Tensor, gate: torch.Tensor, heads: int, eps: float, 
     return out
 
 
+def retention(proj: torch.Tensor, decay: torch.Tensor, state: torch.Tensor, ctx, heads: int, dim: int, value_dim: int, eps: float,
+              *, inv_freq: torch.Tensor | None = None, k_scale: float = 1.0) -> torch.Tensor:
+    """A retention layer between its projections: `decay_attention` without activations, then `head_norm_gate`.  A row of
+    ``proj`` is [queries | keys | values | gate].  Returns [N, heads * value_dim] in the dtype of ``proj``.  Decode steps
+    (``value_dim`` a multiple of 4 up to 256) do all of it in one kernel."""
+    gate0 = heads * (2 * dim + value_dim)
+    if proj.dim() != 2 or proj.shape[1] < gate0 + heads * value_dim:
+        raise KernelError("retention: the rows are narrower than queries, keys, values and gate")
+    if not ctx.is_decode_only or value_dim % 4 or value_dim > 256:
+        mixed = decay_attention(proj, decay, state, ctx, heads, dim, value_dim, silu=False, inv_freq=inv_freq, k_scale=k_scale)
+        return head_norm_gate(mixed, proj[:, gate0: gate0 + heads * value_dim], heads, eps, proj.dtype)
+    _need(proj, None, "projected rows")
+    _need(decay, torch.float32, "decay")
+    _need(state, torch.float32, "state")
+    half = 0
+    if inv_freq is not None:
+        _need(inv_freq, torch.float32, "inv_freq")
+        half = inv_freq.numel()
+    if decay.numel() != heads or not 1 <= dim <= 256 or 2 * half > dim or tuple(state.shape[1:]) != (heads, dim, value_dim):
+        raise KernelError("retention: one decay per head, the state [slots, heads, dim, value_dim], a rotation of at most the head")
+    out = torch.empty((proj.shape[0], heads * value_dim), dtype=proj.dtype, device=proj.device)
+    _check(ops_library().ss_retention_token(proj.data_ptr(), proj.stride(0), decay.data_ptr(), state.data_ptr(), out.data_ptr(),
+                                            ctx.q_start.data_ptr(), ctx.seq_lens.data_ptr(), ctx.state_slots.data_ptr(), ctx.num_requests,
+                                            heads, dim, value_dim, state.shape[0], _code(proj.dtype), error_word(proj.device).data_ptr(),
+                                            _stream(), _ptr(inv_freq), half, float(k_scale), float(eps)), "retention_token")
+    return out
+
+
 def talk_heads(x: torch.Tensor, table_t: torch.Tensor, n_kv: int, out_dtype: torch.dtype,
                gate: torch.Tensor | None = None) -> torch.Tensor:
     """Mixtures over heads of attention weights, applied to what `paged_attention` leaves with ``across``.  ``x`` float32
@@ -2468,7 +2550,7 @@ __all__ = ["KernelError", "KernelBuildError", "embedding", "add_rmsnorm", "hc_no
            "gemm_simt", "paged_attention_simt", "paged_attention", "fuses_rope", "paged_attention_prefill", "paged_attention_prefill_tcgen05", "prefill_key_parts", "tcgen05_attention_fits", "tcgen05_prefill_fits", "paged_attention_decode", "decode_scratch", "decode_slices", "is_long_context", "require_cuda", "argmax", "sample", "mark_seen", "gather_tokens", "prepare_decode", "gemm_tcgen05", "gemm_tcgen05_many", "many_tokens_fits", "many_tokens_swiglu_fits", "gemm_plan", "gemm_library", "gate_up_swiglu", "set_programmatic_launch", "launch_count", "count_launches", "sm_count", "linear", "linear_add_rmsnorm", "adds_to_stream", "takes_pending_norm", "PendingNorm", "set_norm_fusion", "check_errors", "raise_for_status", "error_word", "ops_library",
            "attention_library", "group_norm", "round_stream", "conv_silu", "ssm_scan", "router", "moe_experts", "moe_combine",
            "norm_rope_cache", "turn_heads", "soft_cap", "embed_sum", "matrix_cell", "cell_output", "gated_recurrence", "xielu",
-           "DiffPair", "diff_in_attention", "diff_combine", "heads_to_pages", "branch_norm",
+           "DiffPair", "diff_in_attention", "diff_combine", "heads_to_pages", "branch_norm", "PairedOutput", "WeighedTerms",
            "latent_rows", "head_product", "decay_attention", "gated_rmsnorm", "block_gates", "gated_linear_recurrence", "head_gate",
-           "embedding_norm", "head_norm_gate", "talk_heads", "normed_pair",
+           "embedding_norm", "head_norm_gate", "retention", "talk_heads", "normed_pair",
            "scaled_sum", "relu_square", "moe_experts_single", "moe_mix"]

@@ -131,7 +131,7 @@ class SandwichBlock(Block):
     """``x + m * norm1b(mixer(norm1(x)))`` then ``x + m * norm2b(ffn(norm2(x)))``: a norm on both sides of each branch
     and a multiplier on what joins the stream.  ``feed_forward`` may be None.  All norms are `JoiningNorm`: a branch's
     output stays pending, and the kernel of the next norm, of this block or of the next one, norms it, adds it and norms
-    the new stream in one pass."""
+    the new stream in one pass; a branch whose output is a sum (``can_return_unformed``) leaves that to the same kernel."""
 
     cuda_graph_safe = True
 
@@ -150,8 +150,10 @@ class SandwichBlock(Block):
 
     def forward(self, residual: torch.Tensor, pending, ctx, layer: LayerBinding):
         x = self.mixer_norm.add_norm(residual, pending)
-        pending = self.mixer_out_norm.branch(self.mixer.forward(x, ctx, layer), self.residual_mult)
+        more = {"unformed": True} if getattr(self.mixer, "can_return_unformed", False) else {}
+        pending = self.mixer_out_norm.branch(self.mixer.forward(x, ctx, layer, **more), self.residual_mult)
         if self.feed_forward is not None:
             x = self.ffn_norm.add_norm(residual, pending)
-            pending = self.ffn_out_norm.branch(self.feed_forward.forward(x, ctx), self.residual_mult)
+            more = {"unformed": True} if getattr(self.feed_forward, "can_return_unformed", False) else {}
+            pending = self.ffn_out_norm.branch(self.feed_forward.forward(x, ctx, **more), self.residual_mult)
         return residual, pending

@@ -58,6 +58,8 @@ class RoutedExperts(FeedForward):
             raise ValueError("a gate on the shared expert comes with a shared expert")
         self.gated, self.scores, self.correction, self.groups = bool(gated), scores, correction, groups
         self.weight_on_input, self.router_bias = bool(weight_on_input), router_bias
+        # ``forward(..., unformed=True)``: `ops.WeighedTerms`, the sum over the choices left to the caller's kernel
+        self.can_return_unformed = not self.weight_on_input and shared is None and not identity
         self.identity, self.slots, self.shared_gate = int(identity), slots, shared_gate
         self.name = name
         self.hidden_size, self.expert_size, self.experts, self.top = hidden_size, expert_size, experts, top
@@ -116,7 +118,7 @@ class RoutedExperts(FeedForward):
         per_expert = (first[0].numel() + self.down[0].numel()) * self.down.element_size()
         return self.router_weight.numel() * self.router_weight.element_size() + self.top * per_expert
 
-    def forward(self, x: torch.Tensor, ctx, as_terms: bool = False):
+    def forward(self, x: torch.Tensor, ctx, as_terms: bool = False, unformed: bool = False):
         count, keep = self.groups or (1, 1)
         routed = ops.router(x, self.router_weight, self.top, self.renormalize, softmax=self.scores == "softmax",
                             correction=self.correction_weight, groups=count, keep=keep,
@@ -129,6 +131,8 @@ class RoutedExperts(FeedForward):
                 y, term_rows = ops.moe_experts(x, ids, None, self.gate_up, self.down, self.run)
             else:
                 y, term_rows = ops.moe_experts_single(x, ids, self.up, self.down, self.slots)
+            if unformed and self.can_return_unformed:
+                return ops.WeighedTerms(y, term_rows, scores)
             return ops.moe_mix(y, term_rows, ids, scores, self.experts, x, shared,
                                routed[2] if self.shared_gate is not None else None)
         y, term_rows = ops.moe_experts(x, ids, scores, self.gate_up, self.down, self.run)

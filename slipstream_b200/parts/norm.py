@@ -108,7 +108,7 @@ class NormedBranch:
     """A branch output that has not joined the stream yet: the next norm's kernel adds ``mult * norm(y)`` (and
     ``anchor``, float32, if there is one) where it reads the stream."""
 
-    y: torch.Tensor
+    y: "torch.Tensor | ops.PairedOutput | ops.WeighedTerms"  # formed, or left to be formed by that kernel
     norm: "JoiningNorm"
     mult: float
     anchor: torch.Tensor | None = None
@@ -140,7 +140,7 @@ class JoiningNorm(Norm):
     def weight_bytes(self) -> int:
         return self.weight.numel() * self.weight.element_size()
 
-    def branch(self, y: torch.Tensor, mult: float = 1.0) -> NormedBranch:
+    def branch(self, y: "torch.Tensor | ops.PairedOutput | ops.WeighedTerms", mult: float = 1.0) -> NormedBranch:
         return NormedBranch(y, self, mult)
 
     def add_norm(self, residual: torch.Tensor, delta: "NormedBranch | None",

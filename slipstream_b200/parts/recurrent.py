@@ -241,15 +241,14 @@ class DecayedLinearAttention(Mixer):
     def forward(self, x: torch.Tensor, ctx, layer: LayerBinding, into: IntoNorm | None = None) -> torch.Tensor:
         h, d, v = self.heads, self.dim, self.value_dim
         proj = ops.linear(x, self.qkvg_weight)
-        gate = proj[:, h * (2 * d + v): h * (2 * d + 2 * v)]
         if self.retention:
             inv_freq = self.position_encoding.rotary_table()[0] if self.position_encoding is not None else None
-            mixed = ops.decay_attention(proj, self.decay_weight, layer.state["memory"], ctx, h, d, v, silu=False,
-                                        inv_freq=inv_freq, k_scale=d ** -0.5)
-            out = ops.head_norm_gate(mixed, gate, h, self.norm_eps, self.runtime.dtype)
+            out = ops.retention(proj, self.decay_weight, layer.state["memory"], ctx, h, d, v, self.norm_eps, inv_freq=inv_freq,
+                                k_scale=d ** -0.5)
         else:
             mixed = ops.decay_attention(proj, self.decay_weight, layer.state["memory"], ctx, h, d, v)
-            out = ops.gated_rmsnorm(mixed, gate, self.norm_weight, self.norm_eps, self.runtime.dtype)
+            g0 = h * (2 * d + v)
+            out = ops.gated_rmsnorm(mixed, proj[:, g0: g0 + h * v], self.norm_weight, self.norm_eps, self.runtime.dtype)
         if into is not None:
             return into.close(out, self.o_weight, None)
         return ops.linear(out, self.o_weight)
@@ -330,6 +329,7 @@ class ParallelMixers(Mixer):
         if out_norms is not None and (left_scale != right_scale or hidden_size is None):
             raise ValueError("normed outputs are scaled alike, and their norms need the model's width")
         self.out_norms, self.hidden_size = out_norms, hidden_size
+        self.can_return_unformed = out_norms is not None  # ``forward(..., unformed=True)``: an `ops.PairedOutput`
         if left.cache_spec() is not None and right.cache_spec() is not None:
             raise ValueError("at most one side of a pair of mixers keeps pages")
         self.left, self.right = left, right
@@ -362,10 +362,11 @@ class ParallelMixers(Mixer):
             return LayerBinding(kv=layer.kv, group=layer.group, writes_cache=layer.writes_cache, state=state)
         return LayerBinding(state=state)
 
-    def forward(self, x: torch.Tensor, ctx, layer: LayerBinding) -> torch.Tensor:
+    def forward(self, x: torch.Tensor, ctx, layer: LayerBinding, unformed: bool = False) -> "torch.Tensor | ops.PairedOutput":
         left_pages = self.left.cache_spec() is not None
         a = self.left.forward(x, ctx, self._side(layer, "left", left_pages))
         b = self.right.forward(x, ctx, self._side(layer, "right", not left_pages and self.right.cache_spec() is not None))
         if self.out_norms is not None:
-            return ops.normed_pair(a, self.norm_weights[0], b, self.norm_weights[1], self.out_norms[2], self.left_scale)
+            pair = ops.PairedOutput(a, self.norm_weights[0], b, self.norm_weights[1], self.out_norms[2], self.left_scale)
+            return pair if unformed else pair.materialize()
         return ops.scaled_sum(a, self.left_scale, b, self.right_scale)

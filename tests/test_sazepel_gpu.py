@@ -292,7 +292,8 @@ def step_ctx(q_lens, seq_lens, slots):
 
 PLANS = [  # two requests of 200 and 37 rows: whole; portions down to two tokens and single ones; at the edges of tiles
     [[("a", 200), ("b", 37)]],
-    [[("a", 33)], [("a", 2), ("b", 17)], [("a", 1), ("b", 1)], [("a", 34), ("b", 2)], [("b", 16)], [("b", 1)], [("a", 127)], [("a", 3)]],
+    [[("a", 33)], [("a", 2), ("b", 17)], [("a", 1), ("b", 1)], [("a", 34), ("b", 2)], [("b", 16)], [("b", 1)], [("a", 120)]]
+    + [[("a", 1)] for _ in range(10)],
     [[("b", 37)], [("a", 16)], [("a", 64)], [("a", 63)], [("a", 57)]],
 ]
 
@@ -325,9 +326,7 @@ def test_retention_whole_and_cut_with_slots_used_again(heads, dim, vdim, dims, d
         for step in plan:
             ctx = step_ctx([n for _, n in step], [done[k] + n for k, n in step], [slots[k] for k, _ in step])
             x = torch.cat([rows[k][done[k]: done[k] + n] for k, n in step]).to(DEV)
-            mixed = ops.decay_attention(x, torch.tensor(decay, device=DEV), state, ctx, heads, dim, vdim, silu=False, inv_freq=inv,
-                                        k_scale=dim ** -0.5)
-            out = ops.head_norm_gate(mixed, x[:, at[3]: at[4]], heads, 1e-6, dtype)
+            out = ops.retention(x, torch.tensor(decay, device=DEV), state, ctx, heads, dim, vdim, 1e-6, inv_freq=inv, k_scale=dim ** -0.5)
             row = 0
             for k, n in step:
                 got[k].append(out[row: row + n].double().cpu())
@@ -591,7 +590,23 @@ def test_norms_with_one_number_normed_embedding_and_normed_pair(width, dtype):
     a, b = (torch.randn(n, width, generator=g).to(dtype) for _ in range(2))
     wa, wb = torch.randn(width, generator=g), torch.randn(width, generator=g)
     want = 0.5 * (plain.norm(a.double(), wa.double(), eps) + plain.norm(b.double() * 1.0, wb.double(), eps))
-    assert rel(ops.normed_pair(a.to(DEV), wa.to(DEV), b.to(DEV), wb.to(DEV), eps, 0.5), want) < tol
+    unformed = ops.PairedOutput(a.to(DEV), wa.to(DEV), b.to(DEV), wb.to(DEV), eps, 0.5)
+    assert rel(unformed.materialize(), want) < tol
+    # the pair's output formed where it joins the stream, and chosen experts' outputs summed there, in both their forms
+    got = norm_in.add_norm(stream, norm_out.branch(unformed))
+    x = x + plain.norm(want, w["n.out"].double(), eps)
+    assert rel(stream, x) < 3e-6 and rel(got, plain.norm(x, w["n.in"].double(), eps)) < tol
+    terms, weights = torch.randn(n, 3, width, generator=g), torch.rand(n, 3, generator=g)
+    place = torch.randperm(3 * n, generator=g).to(torch.int32)
+    in_order = torch.empty(3 * n, width)
+    in_order[place.long()] = terms.reshape(3 * n, width)
+    for y, value in ((ops.WeighedTerms(terms.to(DEV), None, weights.to(DEV)), terms.double()),
+                     (ops.WeighedTerms(in_order.to(dtype).to(DEV), place.to(DEV), weights.to(DEV)), terms.to(dtype).double())):
+        chosen = norm_in.add_norm(stream, norm_out.branch(y), rows=torch.tensor([7, 2], dtype=torch.int32, device=DEV))
+        got = norm_in.add_norm(stream, norm_out.branch(y))
+        x = x + plain.norm((weights.double()[:, :, None] * value).sum(1), w["n.out"].double(), eps)
+        want = plain.norm(x, w["n.in"].double(), eps)
+        assert rel(stream, x) < 3e-6 and rel(got, want) < tol and rel(chosen, want[[7, 2]]) < tol
     ops.check_errors(DEV)
     out_of_range = torch.tensor([3, vocab], dtype=torch.int32, device=DEV)  # flagged by the kernel, nothing is read there
     embed.forward_step(out_of_range, None, {})
