@@ -1715,18 +1715,16 @@ def run_compare_sazepel(args) -> int:
             lens = torch.full((n_req,), tokens, dtype=torch.int32, device=dev)
             q, gate = rand(n_req, n_q * d), rand(n_req, n_q * d)
             out = torch.empty_like(q)
-            wide1 = torch.empty(n_req, n_kv * n_q * d, dtype=torch.float32, device=dev)
             moved = n_req * tokens * 4.0 * n_kv * d + n_req * n_q * d * 4.0
 
-            def decode(into, across):
-                slices = ops.decode_slices(n_req, n_kv * n_kv if across else n_kv, group, tokens, False, ops.sm_count(dev))
-                return sweep(lambda i: ops.paged_attention_decode(q, q.shape[1], into, kv_pages[i], table, starts, lens, n_req, n_q, n_kv, d,
-                                                                  d ** -0.5, 0, slices, stages=ops.functions.DECODE_RING_STAGES, across=across), copies)
-
-            hbm(f"decode_attention {name} {n_req} x {tokens} (qwen2, rotation outside)", decode(out, False), moved)
-            us = decode(wide1, True)
-            us2 = sweep(lambda i: ops.talk_heads(wide1, talk, n_kv, torch.bfloat16, gate))
-            hbm(f"decode_attention {name} {n_req} x {tokens} with talking heads (both)", us + us2, moved, talk_us=round(us2, 2))
+            slices = ops.decode_slices(n_req, n_kv, group, tokens, False, ops.sm_count(dev))
+            us = sweep(lambda i: ops.paged_attention_decode(q, q.shape[1], out, kv_pages[i], table, starts, lens, n_req, n_q, n_kv, d, d ** -0.5, 0,
+                                                            slices, stages=ops.functions.DECODE_RING_STAGES), copies)
+            hbm(f"decode_attention {name} {n_req} x {tokens} (qwen2, rotation outside)", us, moved)
+            slices = ops.across_slices(n_req, n_kv, tokens, ops.sm_count(dev))
+            us = sweep(lambda i: ops.talking_attention_decode(q, q.shape[1], kv_pages[i], table, starts, lens, n_req, n_q, n_kv, d, d ** -0.5, talk,
+                                                              gate, slices), copies)
+            hbm(f"decode_attention {name} {n_req} x {tokens} with talking heads (both kernels)", us, moved)
             del kv_pages
     ops.check_errors(dev)
     result["kernels"] = kernels

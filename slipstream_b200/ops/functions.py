@@ -142,6 +142,11 @@ _ATTN_SIGNATURES = {
                            c_int, c_int],
 }
 
+_ATTN_SIGNATURES["ss_attn_decode_across_sets"] = [c_int, c_int, c_int]
+_ATTN_SIGNATURES["ss_attn_decode_across"] = [c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int,
+                                             c_int, c_int64, c_float, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_void_p,
+                                             c_void_p]
+
 _GEMM_SIGNATURES = {
     "ss_gemm_tc5_many": [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int64, c_int64, c_int64,
                          c_int, c_int, c_int, c_void_p, c_void_p],
@@ -2519,6 +2524,67 @@ def talk_heads(x: torch.Tensor, table_t: torch.Tensor, n_kv: int, out_dtype: tor
     return out
 
 
+@functools.lru_cache(maxsize=None)
+def across_decode_sets(head_dim: int, n_q: int, n_kv: int, page_size: int) -> int:
+    """Parts per slice that the decode kernel over all kv heads' values leaves, or 0 where it does not take the layer (head
+    size 64 or 128, 2 to 8 kv heads of at most 16 query heads, pages of 8, 16, 32 or 64 tokens)."""
+    if head_dim not in (64, 128):
+        return 0
+    return int(attention_library(head_dim).ss_attn_decode_across_sets(int(n_q), int(n_kv), int(page_size)))
+
+
+def across_slices(n_requests: int, n_kv: int, longest: int, sms: int | None = None) -> int:
+    """Into how many slices that kernel cuts the keys: a block per SM (its ring of tiles takes the SM's shared memory)."""
+    blocks = n_requests * (1 if n_kv <= 4 else (n_kv + 1) // 2)
+    return max(1, min((sms or sm_count()) // blocks, (longest + 31) // 32, 64))
+
+
+def talking_attention_decode(q: torch.Tensor, q_stride: int, kv: torch.Tensor, block_tables: torch.Tensor, q_start: torch.Tensor,
+                             seq_lens: torch.Tensor, n_requests: int, n_q: int, n_kv: int, head_dim: int, scale: float, table_t: torch.Tensor,
+                             gate: torch.Tensor | None, n_slices: int) -> torch.Tensor:
+    """Attention with talking heads for requests that bring ONE token each (bfloat16), where `across_decode_sets`: every tile of
+    keys and values is fetched once for all heads; the slices' sums are combined, mixed and gated by a second kernel."""
+    sets = across_decode_sets(head_dim, n_q, n_kv, kv.shape[3])
+    if not sets or q.dtype != torch.bfloat16:
+        raise KernelError("the decode kernel over all values does not take this layer")
+    _need(kv, torch.bfloat16, "kv pages")
+    _need(table_t, torch.float32, "table")
+    for name, t in (("block_tables", block_tables), ("q_start", q_start), ("seq_lens", seq_lens)):
+        _need(t, torch.int32, name)
+    rows = q.shape[0]
+    if tuple(table_t.shape) != (n_q, n_q) or (gate is not None and (gate.dtype != q.dtype or tuple(gate.shape) != (rows, n_q * head_dim)
+                                                                    or gate.stride(1) != 1)):
+        raise KernelError("talking_attention_decode: the table must be [H, H], the gate a view [N, H * D] with unit inner stride")
+    parts = n_slices * sets
+    part_o = torch.empty((n_requests, parts, n_kv, n_q, head_dim), dtype=torch.float32, device=q.device)
+    part_ml = torch.empty((n_requests, parts, n_q, 2), dtype=torch.float32, device=q.device)
+    out = torch.empty((rows, n_q * head_dim), dtype=q.dtype, device=q.device)
+    _check(attention_library(head_dim).ss_attn_decode_across(
+        q.data_ptr(), q_stride, out.data_ptr(), kv.data_ptr(), block_tables.data_ptr(), block_tables.shape[1], n_requests, q_start.data_ptr(),
+        seq_lens.data_ptr(), n_q, n_kv, kv.shape[3], kv.shape[0], float(scale), int(n_slices), part_o.data_ptr(), part_ml.data_ptr(),
+        table_t.data_ptr(), _ptr(gate), gate.stride(0) if gate is not None else 0, error_word(q.device).data_ptr(), _stream()),
+        "talking_attention_decode")
+    _launches[0] += 1  # two kernels
+    return out
+
+
+def talking_attention(q: torch.Tensor, kv: torch.Tensor, block_tables: torch.Tensor, ctx, n_q: int, n_kv: int, head_dim: int, scale: float,
+                      table_t: torch.Tensor, gate: torch.Tensor | None = None, **mask) -> torch.Tensor:
+    """Attention whose heads' weights are mixed behind the softmax: head h applies ``sum_g table_t[g, h] weights_g`` to the values
+    of its own kv head; the result [N, H * D] is multiplied by ``sigmoid(gate)``.  ``q``: rows that start with the queries.
+    ``mask``: `paged_attention`'s window, chunk, keep, softcap and sinks.  bfloat16 decode steps without these run the kernel
+    that walks all kv heads together; everything else `paged_attention` across all values and `talk_heads`."""
+    if (q.dtype == torch.bfloat16 and ctx.is_decode_only and not any(v is not None and v for v in mask.values())
+            and across_decode_sets(head_dim, n_q, n_kv, kv.shape[3])):
+        longest = ctx.extras.get("static_max_seq_len") or ctx.max_seq_len
+        slices = across_slices(ctx.num_requests, n_kv, longest, sm_count(q.device))
+        return talking_attention_decode(q, q.shape[1], kv, block_tables, ctx.q_start, ctx.seq_lens, ctx.num_requests, n_q, n_kv, head_dim, scale,
+                                        table_t, gate, slices)
+    wide = torch.empty((q.shape[0], n_kv * n_q * head_dim), dtype=torch.float32, device=q.device)
+    paged_attention(q, wide, kv, block_tables, ctx, n_q, n_kv, head_dim, scale, across=True, **mask)
+    return talk_heads(wide, table_t, n_kv, q.dtype, gate)
+
+
 def normed_pair(a: torch.Tensor, a_weight: torch.Tensor, b: torch.Tensor, b_weight: torch.Tensor, eps: float,
                 scale: float) -> torch.Tensor:
     """``scale * (rmsnorm(a) * a_weight + rmsnorm(b) * b_weight)`` row by row: ``a``, ``b`` [N, C] of one dtype, weights float32
@@ -2552,5 +2618,5 @@ __all__ = ["KernelError", "KernelBuildError", "embedding", "add_rmsnorm", "hc_no
            "norm_rope_cache", "turn_heads", "soft_cap", "embed_sum", "matrix_cell", "cell_output", "gated_recurrence", "xielu",
            "DiffPair", "diff_in_attention", "diff_combine", "heads_to_pages", "branch_norm", "PairedOutput", "WeighedTerms",
            "latent_rows", "head_product", "decay_attention", "gated_rmsnorm", "block_gates", "gated_linear_recurrence", "head_gate",
-           "embedding_norm", "head_norm_gate", "retention", "talk_heads", "normed_pair",
+           "embedding_norm", "head_norm_gate", "retention", "talk_heads", "talking_attention", "talking_attention_decode", "across_decode_sets", "across_slices", "normed_pair",
            "scaled_sum", "relu_square", "moe_experts_single", "moe_mix"]

@@ -32,8 +32,8 @@ by its root mean square (no weight) and cached so.  ``talk``: TALKING HEADS: beh
 ``sum_g T[h, g] weights_g`` over all query heads g (tensor ``talk`` [heads, heads]), and those are applied to the values of
 h's own key/value head.  How it runs: mixing the weights before they meet the values is the same sum as mixing, per
 key/value head, what every head's own weights make of its values, so the attention kernels walk pairs of (keys' head,
-values' head) and leave every query head over the values of every key/value head in float32, and `ops.talk_heads` forms the
-mixture and applies the gate; the softmax stays inside the kernels and no weights are ever written.  ``names``: the checkpoint's tensor names by
+values' head) and leave every query head over the values of every key/value head in float32, and a kernel behind them forms
+the mixture and applies the gate (decode steps: one walk over all key/value heads, `ops.talking_attention`); the softmax stays inside the kernels and no weights are ever written.  ``names``: the checkpoint's tensor names by
 role (q, k, v, o, g, q_bias, k_bias, v_bias, o_bias, q_norm, k_norm, sink, talk).
 
 Heads of a size the kernels do not take (they take multiples of 16), or values of another size than keys, are
@@ -357,15 +357,14 @@ class PagedAttention(Mixer):
                                self.num_kv_heads, self.head_dim, rotary_dim, write_cache=layer.writes_cache)
         width = self.num_heads * self.head_dim
         gate = qkv[:, qkv.shape[1] - width:] if self.gate else None
-        out = torch.empty((x.shape[0], self.num_kv_heads * width if self.talk else width),
-                          dtype=torch.float32 if self.talk else x.dtype, device=x.device)
-        ops.paged_attention(q, out, layer.kv, meta.block_tables, ctx, self.num_heads, self.num_kv_heads,
-                            self.head_dim, self.scale, self.window or 0,
-                            rope=(inv_freq, rotary_dim) if fused else None, chunk=self.chunk or 0,
-                            gate=None if self.talk else gate, softcap=self.softcap or 0.0,
-                            sinks=self.sinks, keep=self.keep_first, across=self.talk)
+        mask = dict(window=self.window or 0, chunk=self.chunk or 0, softcap=self.softcap or 0.0, sinks=self.sinks, keep=self.keep_first)
         if self.talk:
-            out = ops.talk_heads(out, self.talk_table, self.num_kv_heads, x.dtype, gate)
+            out = ops.talking_attention(q, layer.kv, meta.block_tables, ctx, self.num_heads, self.num_kv_heads, self.head_dim, self.scale,
+                                        self.talk_table, gate, **mask)
+        else:
+            out = torch.empty((x.shape[0], width), dtype=x.dtype, device=x.device)
+            ops.paged_attention(q, out, layer.kv, meta.block_tables, ctx, self.num_heads, self.num_kv_heads, self.head_dim, self.scale,
+                                rope=(inv_freq, rotary_dim) if fused else None, gate=gate, **mask)
         if self.head_gate:
             ops.head_gate(out, qkv[:, self.head_gate_col: self.head_gate_col + self.num_heads], self.num_heads, self.head_dim)
         if self.rotate_values:

@@ -397,7 +397,8 @@ def across_reference(q, kv, table, starts, lens, n_kv, page, scale):
 
 @pytest.mark.gpu
 @pytest.mark.parametrize("n_q,n_kv,d,page", [(6, 3, 64, 16), (8, 1, 128, 16), (6, 3, 48, 8), (2, 2, 64, 8), (28, 4, 128, 64), (4, 1, 32, 5),
-                                             (2, 2, 256, 16), (4, 2, 64, 32), (20, 1, 64, 16), (34, 2, 80, 16), (16, 8, 128, 16)])
+                                             (2, 2, 256, 16), (4, 2, 64, 32), (20, 1, 64, 16), (34, 2, 80, 16), (16, 8, 128, 16),
+                                             (10, 5, 64, 8), (3, 3, 128, 64), (32, 2, 128, 8), (7, 7, 64, 64), (36, 6, 128, 32)])
 def test_every_head_over_all_values_in_every_attention_kernel_and_the_mixture_behind(n_q, n_kv, d, page):
     from slipstream_b200 import ops
     from slipstream_b200.engine.context import query_tiles_host
@@ -447,7 +448,14 @@ def test_every_head_over_all_values_in_every_attention_kernel_and_the_mixture_be
         got = ops.talk_heads(flat.float().to(DEV), table_t, n_kv, dtype)
         assert rel(got, want) < (5e-6 if dtype == torch.float32 else 6e-3)
         got = ops.talk_heads(flat.float().to(DEV), table_t, n_kv, dtype, gate.to(DEV)[:, 8:])
-        assert rel(got, want * torch.sigmoid(gate[:, 8:].double())) < (5e-6 if dtype == torch.float32 else 8e-3)
+        gated = want * torch.sigmoid(gate[:, 8:].double())
+        assert rel(got, gated) < (5e-6 if dtype == torch.float32 else 8e-3)
+        if dtype == torch.bfloat16 and max(q_lens) == 1 and ops.across_decode_sets(d, n_q, n_kv, page):
+            for slices in (1, 2, 5, 18, 64):  # all kv heads in one walk, mixture and gate behind it
+                got = ops.talking_attention_decode(*args, dev[1], dev[2], dev[3], dev[4], n, n_q, n_kv, d, scale, table_t, gate.to(DEV)[:, 8:], slices)
+                assert rel(got, gated) < 1.5e-2, slices
+                got = ops.talking_attention_decode(*args, dev[1], dev[2], dev[3], dev[4], n, n_q, n_kv, d, scale, table_t, None, slices)
+                assert rel(got, want) < 1.5e-2, slices
     ops.check_errors(DEV)
 
 
@@ -491,6 +499,14 @@ def test_one_key_that_stands_out_is_found_wherever_it_lies(target):
                 ops.paged_attention_decode(dev[0][:1].contiguous(), n_q * d, out, dev[1], dev[2], one, length, 1, n_q, n_kv, d, 1.0, n_slices=slices,
                                            tma=tma, across=True)
                 assert rel(out[:1], ref[:1].reshape(1, -1)) < 1e-2, (tma, slices)
+        behind = (int(table[0, 37]), n % page)  # what a page's last owner left behind the newest token reaches nobody
+        kv[behind[0], :, :, behind[1]:] = float("inf")
+        eye = torch.eye(n_q, device=DEV)
+        want = torch.stack([ref[0, h // 2, h // 2, h % 2] for h in range(n_q)]).reshape(1, -1)
+        for slices in (1, 7):
+            got = ops.talking_attention_decode(dev[0][:1].contiguous(), n_q * d, kv.to(DEV), dev[2], one, length, 1, n_q, n_kv, d, 1.0, eye, None, slices)
+            assert target > 299 or rel(got, want) < 1e-2, slices
+            assert bool(torch.isfinite(got).all())
 
 
 @pytest.mark.gpu
