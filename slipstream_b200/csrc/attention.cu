@@ -209,65 +209,59 @@ extern "C" int ss_attn_decode_tma(const void* q, int64_t q_stride, void* out, in
 
 #include "attention_decode_across.cuh"
 
-// How a decode step over all kv heads' values is laid out: kv heads of values per block, warp sets, stages of the ring (0: not
-// taken by this kernel).
-static void across_layout(int n_q, int n_kv, int* nc, int* sets, int* stages) {
-    *stages = 0;
-    if (n_kv < 2 || n_kv > 8 || n_q % n_kv || n_q / n_kv > 16) return;
-    *nc = n_kv <= 4 ? n_kv : 2;
-    *sets = n_kv == 2 ? 4 : 1;
-    const int stage = across_stage_bytes(HEAD_DIM, n_kv, *nc, *sets);
-    for (int st = 4; st >= 2; --st)
-        if (across_smem_bytes(HEAD_DIM, n_kv, stage, st) <= 220 * 1024) { *stages = st; return; }
+// What a layer needs of ss_attn_decode_across's scratch: parts per slice (the return value; 0 where the kernel does not take
+// the layer) and columns of heads per kv head.
+extern "C" int ss_attn_decode_across_sets(int n_q, int n_kv, int page_size, int* head_cols) {
+    if (page_size % 8 != 0 || 64 % page_size != 0) return 0;
+    const AcrossLayout y = across_layout(HEAD_DIM, n_q, n_kv);
+    if (head_cols) *head_cols = y.nh * 8;
+    return y.stages ? y.sets : 0;
 }
 
-// Parts per slice (the scratch of ss_attn_decode_across holds n_slices times as many), or 0 where the kernel does not fit.
-extern "C" int ss_attn_decode_across_sets(int n_q, int n_kv, int page_size) {
-    int nc = 0, sets = 0, stages = 0;
-    if (page_size % 8 != 0 || 64 % page_size != 0) return 0;
-    across_layout(n_q, n_kv, &nc, &sets, &stages);
-    return stages ? sets : 0;
+template <int BN, int NK, int NH, int CPW>
+static int launch_across(const CUtensorMap& map_kv, const AcrossArgs& a, dim3 grid, int smem, cudaStream_t stream) {
+    static SsPerDevice opted;
+    if (int rc = ss_opt_in_smem(attn_decode_across<HEAD_DIM, BN, NK, NH, CPW>, 220 * 1024, opted)) return rc;
+    ss_launch(attn_decode_across<HEAD_DIM, BN, NK, NH, CPW>, grid, dim3(AX_THREADS), smem, stream, map_kv, a);
+    return SS_LAUNCH_CHECK();
 }
 
 // A decode step with talking heads.  q: rotated or normed queries, n_q heads of HEAD_DIM a row; part_o (float32
-// [requests][parts][n_kv][n_q][HEAD_DIM]) and part_ml ([requests][parts][n_q][2]) scratch of the caller, parts = n_slices *
-// sets; table_t, gate and out as ss_talk_heads (bfloat16).  Two launches.
+// [requests][parts][n_kv][n_kv][HEAD_DIM][head columns]) and part_ml ([requests][parts][n_q][2]) scratch of the caller, parts =
+// n_slices * sets; table_t, gate and out as ss_talk_heads (bfloat16).  Two launches.
 extern "C" int ss_attn_decode_across(const void* q, int64_t q_stride, void* out, const void* kv, const int32_t* block_tables, int max_blocks,
                                      int n_requests, const int32_t* q_start, const int32_t* seq_lens, int n_q, int n_kv, int page_size,
                                      int64_t num_pages, float scale, int n_slices, float* part_o, float* part_ml, const float* table_t,
                                      const void* gate, int64_t gate_stride, int* err, cudaStream_t stream) {
     if (n_requests <= 0) return 0;
-    int nc = 0, sets = 0, stages = 0;
     if (page_size % 8 != 0 || 64 % page_size != 0 || n_slices < 1 || n_slices > SS_DECODE_MAX_SLICES || q_stride % 8) return (int)cudaErrorInvalidValue;
-    across_layout(n_q, n_kv, &nc, &sets, &stages);
-    if (!stages) return (int)cudaErrorInvalidValue;
-    const int bn = across_tile_keys(sets), box = page_size < bn ? page_size : bn;
+    const AcrossLayout y = across_layout(HEAD_DIM, n_q, n_kv);
+    if (!y.stages) return (int)cudaErrorInvalidValue;
     CUtensorMap map_kv;
     int rc = fa::make_map3(&map_kv, kv, HEAD_DIM, (uint64_t)page_size, (uint64_t)num_pages * 2 * n_kv, (uint64_t)HEAD_DIM * 2,
-                           (uint64_t)page_size * HEAD_DIM * 2, 64, (uint32_t)box, 1);
+                           (uint64_t)page_size * HEAD_DIM * 2, 64, (uint32_t)(page_size < y.bn ? page_size : y.bn), 1);
     if (rc) return rc;
     AcrossArgs a;
     a.q = (const bf16*)q; a.q_stride = q_stride; a.block_tables = block_tables; a.max_blocks = max_blocks; a.q_start = q_start;
     a.seq_lens = seq_lens; a.n_q = n_q; a.n_kv = n_kv; a.page_size = page_size; a.num_pages = num_pages; a.scale = scale;
-    a.n_slices = n_slices; a.stages = stages; a.nc = nc; a.sets = sets; a.part_o = part_o; a.part_ml = part_ml; a.err = err;
-    const int smem = across_smem_bytes(HEAD_DIM, n_kv, across_stage_bytes(HEAD_DIM, n_kv, nc, sets), stages);
-    const dim3 grid(n_slices, (n_kv + nc - 1) / nc, n_requests);
-    if (sets == 4) {
-        static SsPerDevice opted;
-        if (int rc_smem = ss_opt_in_smem(attn_decode_across<HEAD_DIM, 64, 16>, 224 * 1024, opted)) return rc_smem;
-        ss_launch(attn_decode_across<HEAD_DIM, 64, 16>, grid, dim3(AX_THREADS), smem, stream, map_kv, a);
+    a.n_slices = n_slices; a.stages = y.stages; a.nc = y.nc; a.sets = y.sets; a.part_o = part_o; a.part_ml = part_ml; a.err = err;
+    const int smem = across_smem_bytes(HEAD_DIM, n_kv, y);
+    const dim3 grid(n_slices, (n_kv + y.nc - 1) / y.nc, n_requests);
+    if (y.nh == 1) {
+        if (y.bn == 64) rc = launch_across<64, 16, 1, 4>(map_kv, a, grid, smem, stream);
+        else if (y.nk == 16) rc = launch_across<32, 16, 1, 4>(map_kv, a, grid, smem, stream);
+        else rc = launch_across<32, 32, 1, 4>(map_kv, a, grid, smem, stream);
     } else {
-        static SsPerDevice opted;
-        if (int rc_smem = ss_opt_in_smem(attn_decode_across<HEAD_DIM, 32, 32>, 224 * 1024, opted)) return rc_smem;
-        ss_launch(attn_decode_across<HEAD_DIM, 32, 32>, grid, dim3(AX_THREADS), smem, stream, map_kv, a);
+        rc = y.bn == 64 ? launch_across<64, 16, 2, 2>(map_kv, a, grid, smem, stream) : launch_across<32, 32, 2, 2>(map_kv, a, grid, smem, stream);
     }
-    if (int rc_launch = SS_LAUNCH_CHECK()) return rc_launch;
+    if (rc) return rc;
     TalkMergeArgs t;
     t.part_o = part_o; t.part_ml = part_ml; t.table_t = table_t; t.gate = (const bf16*)gate; t.gate_stride = gate_stride; t.out = (bf16*)out;
-    t.q_start = q_start; t.seq_lens = seq_lens; t.n_q = n_q; t.n_kv = n_kv; t.n_parts = n_slices * sets;
-    const int merge_smem = n_q * (AM_COLS + t.n_parts) * 4;
+    t.q_start = q_start; t.seq_lens = seq_lens; t.n_q = n_q; t.n_kv = n_kv; t.nh = y.nh; t.n_parts = n_slices * y.sets;
+    t.n_slices = n_slices; t.tile_keys = y.bn; t.splits = talk_merge_splits(n_kv, y.nh);
+    const int merge_smem = (n_kv * y.nh * 8 * (t.splits * (AM_COLS + 1) + t.n_parts) + 4) * 4;
     static SsPerDevice opted_merge;
-    if (int rc_smem = ss_opt_in_smem(talk_merge_kernel<HEAD_DIM>, 160 * 1024, opted_merge)) return rc_smem;
+    if (int rc_smem = ss_opt_in_smem(talk_merge_kernel<HEAD_DIM>, 200 * 1024, opted_merge)) return rc_smem;
     ss_launch(talk_merge_kernel<HEAD_DIM>, dim3(n_kv * (HEAD_DIM / AM_COLS), n_requests), dim3(AM_THREADS), merge_smem, stream, t);
     return SS_LAUNCH_CHECK();
 }

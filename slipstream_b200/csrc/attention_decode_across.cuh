@@ -4,12 +4,14 @@
 // Heads whose softmax weights are mixed before they meet the values (talking heads) need every query head's weights at the
 // values of every kv head.  A block per pair of kv heads would read every key and value n_kv times.  Here a block takes a
 // slice of a request's keys for all of its kv heads at once, so that every tile of keys and values is fetched once:
-//   * a tile is AX_BN keys: their K rows of all n_kv heads and their V rows of the block's `nc` heads (all of them up to four;
-//     more than four are shared by blocks along grid.y), moved by TMA, one box per page, head and 64-element half, into a ring;
-//   * a consumer warp has one kv head of keys (whose query heads are the 16 rows of its products) and AX_CPW = 2 kv heads of
-//     values: scores once, online softmax in float32, two products with values (mma.sync m16n8k16).  With two kv heads the
-//     eight warps are four such sets, a 16-key part of each 64-key tile each.
-// Nothing is merged here: every (slice, part) leaves its unnormalised sums, maxima and sums of exponentials in scratch memory,
+//   * a tile is BN keys: their K rows of all n_kv heads and their V rows of the block's `nc` heads (all of them up to four;
+//     more than four are shared by blocks along grid.y), moved by TMA, one box per page, head and 64-element half, issued by
+//     the lanes of a producer warp into a ring of stages;
+//   * a consumer warp has one kv head of keys and up to CPW kv heads of values, and a set of NK of a tile's keys (where there
+//     are fewer kv heads than warps several sets share a tile).  Its products are turned over so that the few query heads of
+//     a kv head are the narrow side: scores as keys x heads, outputs as head dims x heads (mma.sync m16n8k16; 7 heads fill 7
+//     of 8 columns where they would fill 7 of 16 rows), the weights turned by movmatrix in between.
+// Nothing is merged here: every (slice, set) leaves its unnormalised sums, maxima and sums of exponentials in scratch memory,
 // and talk_merge_kernel, which reads them once, combines the parts, mixes the heads and applies the gate.
 //
 // Masking and the clearing of value rows behind the newest token as in attention_decode_tma.cuh.  Every mbarrier wait is
@@ -21,8 +23,39 @@
 
 #define AX_WARPS 8
 #define AX_THREADS (32 * (AX_WARPS + 1))
-#define AX_CPW 2
 #define AX_TABLE_MAX 512
+
+// How a layer's heads are laid out over a block.
+struct AcrossLayout {
+    int nh;      // columns of heads in steps of 8
+    int nc;      // kv heads of values a block takes
+    int cpw;     // kv heads of values a warp takes at most
+    int sets;    // warp sets that share a tile's keys
+    int bn, nk;  // keys of a tile, and of a set
+    int stages;  // 0: the kernel does not take the layer
+};
+
+constexpr int across_stage_bytes(int D, int n_kv, const AcrossLayout& y) { return y.bn * (n_kv + y.nc) * D * 2; }
+constexpr int across_smem_bytes(int D, int n_kv, const AcrossLayout& y) {
+    return 1024 + y.stages * across_stage_bytes(D, n_kv, y) + n_kv * y.nh * 8 * (D + 8) * 2 + 256;
+}
+
+static AcrossLayout across_layout(int D, int n_q, int n_kv) {
+    AcrossLayout y = {};
+    if (n_kv < 2 || n_kv > 8 || n_q % n_kv || n_q / n_kv > 16) return y;
+    y.nh = n_q / n_kv > 8 ? 2 : 1;
+    y.cpw = y.nh == 1 ? 4 : 2;
+    y.nc = n_kv <= 4 ? n_kv : y.cpw;
+    y.sets = n_kv == 2 ? 4 : (y.nh == 1 && n_kv <= 4 ? 2 : 1);
+    y.bn = n_kv == 2 ? 64 : 32;
+    y.nk = y.bn / y.sets;
+    for (int st = 4; st >= 2; --st) {
+        y.stages = st;
+        if (across_smem_bytes(D, n_kv, y) <= 220 * 1024) return y;
+    }
+    y.stages = 0;
+    return y;
+}
 
 struct AcrossArgs {
     const bf16* q;
@@ -34,21 +67,19 @@ struct AcrossArgs {
     int n_q, n_kv, page_size;
     int64_t num_pages;
     float scale;
-    int n_slices, stages, nc, sets;  // nc: kv heads of values a block takes; sets: warp sets that share a tile's keys
-    float* part_o;   // [request][slice * sets + set][n_kv (values)][n_q][D], unnormalised
+    int n_slices, stages, nc, sets;
+    float* part_o;   // [request][slice * sets + set][kv head of values][kv head of keys][D][8 nh], unnormalised
     float* part_ml;  // [request][slice * sets + set][n_q][2]: maximum (in units of log2 e) and sum of exponentials
     int* err;
 };
 
-// keys of a tile: 16 per warp set with four sets, else 32
-__host__ __device__ constexpr int across_tile_keys(int sets) { return sets == 4 ? 64 : 32; }
-constexpr int across_stage_bytes(int D, int n_kv, int nc, int sets) { return across_tile_keys(sets) * (n_kv + nc) * D * 2; }
-constexpr int across_smem_bytes(int D, int n_kv, int stage_bytes, int stages) {
-    return 1024 + stages * stage_bytes + n_kv * 16 * (D + 8) * 2 + 256;
+__device__ __forceinline__ uint32_t turn_8x8(uint32_t x) {
+    uint32_t y;
+    asm volatile("movmatrix.sync.aligned.m8n8.trans.b16 %0, %1;" : "=r"(y) : "r"(x));
+    return y;
 }
 
-// BN: keys of a tile.  NK: keys of a tile a warp set takes.
-template <int D, int BN, int NK>
+template <int D, int BN, int NK, int NH, int CPW>
 __global__ void __launch_bounds__(AX_THREADS, 1)
 attn_decode_across(const __grid_constant__ CUtensorMap map_kv, const AcrossArgs a) {
     pdl_launch_dependents();
@@ -59,8 +90,8 @@ attn_decode_across(const __grid_constant__ CUtensorMap map_kv, const AcrossArgs 
     const int c0 = blockIdx.y * a.nc, nc = min(a.nc, G - c0);  // this block's kv heads of values
     const int stage_elems = (G + a.nc) * HEAD;
     bf16* ring = reinterpret_cast<bf16*>(base);
-    bf16* Qs = ring + stages * stage_elems;  // [kv head][16][KSTR]
-    uint64_t* full = reinterpret_cast<uint64_t*>(Qs + G * 16 * KSTR);
+    bf16* Qs = ring + stages * stage_elems;  // [kv head][8 NH][KSTR]
+    uint64_t* full = reinterpret_cast<uint64_t*>(Qs + G * NH * 8 * KSTR);
     uint64_t* empty = full + 4;
     volatile int* gave_up = reinterpret_cast<volatile int*>(empty + 4);
     __shared__ int32_t table_s[AX_TABLE_MAX];
@@ -72,12 +103,12 @@ attn_decode_across(const __grid_constant__ CUtensorMap map_kv, const AcrossArgs 
     const int each = (tiles + n_slices - 1) / n_slices;
     const int j_lo = slice * each, j_hi = min(tiles, j_lo + each) - 1, j_last = tiles - 1;
     const bool work = j_lo <= j_hi;
-    // consumer warps: key head, pair of value heads, warp set
-    const int pairs = (nc + AX_CPW - 1) / AX_CPW, slots = G * ((a.nc + AX_CPW - 1) / AX_CPW);
+    // consumer warps: key head, run of value heads, warp set
+    const int runs = (nc + CPW - 1) / CPW, slots = G * ((a.nc + CPW - 1) / CPW);
     const int set = warp / slots, in_set = warp - set * slots;
     const int ka = in_set % G, cp = in_set / G;
-    const bool consumer = warp < AX_WARPS && set < a.sets && cp < pairs;
-    const int active = a.sets * G * pairs;  // consumer warps that use a tile
+    const bool consumer = warp < AX_WARPS && set < a.sets && cp < runs;
+    const int active = a.sets * G * runs;  // consumer warps that use a tile
 
     if (tid == 0) {
         for (int s = 0; s < stages; ++s) { fa::mbar_init(&full[s], 1); fa::mbar_init(&empty[s], active); }
@@ -133,16 +164,10 @@ attn_decode_across(const __grid_constant__ CUtensorMap map_kv, const AcrossArgs 
     } else {
         pdl_wait();
         const int part = slice * a.sets + set, n_parts = n_slices * a.sets;
-        float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
-        float o[AX_CPW][D / 8][4];
-#pragma unroll
-        for (int c = 0; c < AX_CPW; ++c)
-#pragma unroll
-            for (int d = 0; d < D / 8; ++d) o[c][d][0] = o[c][d][1] = o[c][d][2] = o[c][d][3] = 0.f;
         if (work) {
-            // the queries: 16 rows per kv head, rows behind its heads are zero
-            for (int c = tid; c < G * 16 * (D / 8); c += AX_WARPS * 32) {
-                const int row = c / (D / 8), col = (c - row * (D / 8)) * 8, g = row >> 4, hr = row & 15;
+            // the queries: 8 NH rows per kv head, rows behind its heads are zero
+            for (int c = tid; c < G * NH * 8 * (D / 8); c += AX_WARPS * 32) {
+                const int row = c / (D / 8), col = (c - row * (D / 8)) * 8, g = row / (NH * 8), hr = row % (NH * 8);
                 const bool ok = hr < per;
                 cp_async16(Qs + row * KSTR + col, a.q + (int64_t)row_q * a.q_stride + (int64_t)(g * per + (ok ? hr : 0)) * D + col, ok);
             }
@@ -151,10 +176,23 @@ attn_decode_across(const __grid_constant__ CUtensorMap map_kv, const AcrossArgs 
             asm volatile("bar.sync 1, 256;" ::: "memory");  // the consumer warps
         }
         if (work && consumer) {
+            // a thread's heads of column tile t: 8 t + 2 (lane % 4) and the next; its keys lane / 4 and 8 further
+            float m[NH][2], l[NH][2], o[CPW][D / 16][NH][4];
+#pragma unroll
+            for (int t = 0; t < NH; ++t) {
+                m[t][0] = m[t][1] = -INFINITY;
+                l[t][0] = l[t][1] = 0.f;
+            }
+#pragma unroll
+            for (int c = 0; c < CPW; ++c)
+#pragma unroll
+                for (int d = 0; d < D / 16; ++d)
+#pragma unroll
+                    for (int t = 0; t < NH; ++t) o[c][d][t][0] = o[c][d][t][1] = o[c][d][t][2] = o[c][d][t][3] = 0.f;
             const float scale_log2 = a.scale * 1.4426950408889634f;
             const int key_off = set * NK;
-            const int v0 = cp * AX_CPW, n_v = min(AX_CPW, nc - v0);
-            const bf16* Qa = Qs + ka * 16 * KSTR;
+            const int v0 = cp * CPW, n_v = min(CPW, nc - v0);
+            const bf16* Qa = Qs + ka * NH * 8 * KSTR;
             // a row of a head in a tile: halves of 64 elements, BN rows of 128 bytes each, 16-byte chunks permuted by the row
             auto at = [](const bf16* tile, int row, int col) { return tile + (col >> 6) * (BN * 64) + row * 64 + ((((col >> 3) & 7) ^ (row & 7)) << 3); };
             for (int j = j_lo; j <= j_hi; ++j) {
@@ -174,72 +212,94 @@ attn_decode_across(const __grid_constant__ CUtensorMap map_kv, const AcrossArgs 
                         }
                         __syncwarp();
                     }
-                    float s[NK / 8][4];
+                    float s[NK / 16][NH][4];
+                    {
+                        float s2[NK / 16][NH][4];  // two chains of products: even and odd steps
 #pragma unroll
-                    for (int n = 0; n < NK / 8; ++n) s[n][0] = s[n][1] = s[n][2] = s[n][3] = 0.f;
+                        for (int k = 0; k < NK / 16; ++k)
 #pragma unroll
-                    for (int ks = 0; ks < D / 16; ++ks) {
-                        uint32_t qf[4];
-                        ldmatrix_x4(qf, Qa + (lane & 15) * KSTR + ks * 16 + ((lane >> 4) << 3));
+                            for (int t = 0; t < NH; ++t)
 #pragma unroll
-                        for (int n = 0; n < NK / 8; n += 2) {
-                            uint32_t b[4];
-                            ldmatrix_x4(b, at(Ks, key_off + n * 8 + (lane & 7) + ((lane >> 4) << 3), ks * 16 + (((lane >> 3) & 1) << 3)));
-                            mma_bf16(s[n], qf, b[0], b[1]);
-                            mma_bf16(s[n + 1], qf, b[2], b[3]);
-                        }
-                    }
-                    float mx[2] = {-INFINITY, -INFINITY};
+                                for (int e = 0; e < 4; ++e) s[k][t][e] = s2[k][t][e] = 0.f;
 #pragma unroll
-                    for (int n = 0; n < NK / 8; ++n)
+                        for (int ks = 0; ks < D / 16; ks += 2) {
+                            uint32_t q[NH][4];
 #pragma unroll
-                        for (int e = 0; e < 4; ++e) {
-                            const int key = key0 + n * 8 + ((lane & 3) << 1) + (e & 1);
-                            const float v = key <= pos ? s[n][e] * scale_log2 : -INFINITY;
-                            s[n][e] = v;
-                            mx[e >> 1] = fmaxf(mx[e >> 1], v);
-                        }
-                    float alpha[2];
+                            for (int t = 0; t < NH; ++t) ldmatrix_x4(q[t], Qa + (t * 8 + (lane & 7)) * KSTR + ks * 16 + ((lane >> 3) << 3));
 #pragma unroll
-                    for (int h = 0; h < 2; ++h) {
-                        mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], 1));
-                        mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], 2));
-                        mx[h] = fmaxf(m[h], mx[h]);  // finite: the tile's first key is seen
-                        alpha[h] = fast_exp2(m[h] - mx[h]);
-                        m[h] = mx[h];
-                        l[h] *= alpha[h];
-                    }
+                            for (int k = 0; k < NK / 16; ++k) {
+                                uint32_t x[4], y[4];
+                                ldmatrix_x4(x, at(Ks, key_off + k * 16 + (lane & 15), ks * 16 + ((lane >> 4) << 3)));
+                                ldmatrix_x4(y, at(Ks, key_off + k * 16 + (lane & 15), (ks + 1) * 16 + ((lane >> 4) << 3)));
 #pragma unroll
-                    for (int n = 0; n < NK / 8; ++n)
-#pragma unroll
-                        for (int e = 0; e < 4; ++e) {
-                            s[n][e] = fast_exp2(s[n][e] - m[e >> 1]);
-                            l[e >> 1] += s[n][e];
-                        }
-                    if (__any_sync(0xffffffffu, alpha[0] != 1.f || alpha[1] != 1.f)) {
-#pragma unroll
-                        for (int c = 0; c < AX_CPW; ++c)
-#pragma unroll
-                            for (int d = 0; d < D / 8; ++d) {
-                                o[c][d][0] *= alpha[0]; o[c][d][1] *= alpha[0];
-                                o[c][d][2] *= alpha[1]; o[c][d][3] *= alpha[1];
-                            }
-                    }
-#pragma unroll
-                    for (int kk = 0; kk < NK / 16; ++kk) {
-                        const uint32_t p[4] = {pack_bf16(s[2 * kk][0], s[2 * kk][1]), pack_bf16(s[2 * kk][2], s[2 * kk][3]),
-                                               pack_bf16(s[2 * kk + 1][0], s[2 * kk + 1][1]), pack_bf16(s[2 * kk + 1][2], s[2 * kk + 1][3])};
-#pragma unroll
-                        for (int c = 0; c < AX_CPW; ++c) {
-                            if (c >= n_v) break;
-#pragma unroll
-                            for (int d = 0; d < D / 8; d += 2) {
-                                uint32_t b[4];
-                                ldmatrix_x4_trans(b, at(Vs + c * HEAD, key_off + kk * 16 + (lane & 7) + (((lane >> 3) & 1) << 3), d * 8 + ((lane >> 4) << 3)));
-                                mma_bf16(o[c][d], p, b[0], b[1]);
-                                mma_bf16(o[c][d + 1], p, b[2], b[3]);
+                                for (int t = 0; t < NH; ++t) {
+                                    mma_bf16(s[k][t], x, q[t][0], q[t][1]);
+                                    mma_bf16(s2[k][t], y, q[t][2], q[t][3]);
+                                }
                             }
                         }
+#pragma unroll
+                        for (int k = 0; k < NK / 16; ++k)
+#pragma unroll
+                            for (int t = 0; t < NH; ++t)
+#pragma unroll
+                                for (int e = 0; e < 4; ++e) {
+                                    const int key = key0 + k * 16 + (lane >> 2) + (e >> 1) * 8;
+                                    s[k][t][e] = key <= pos ? (s[k][t][e] + s2[k][t][e]) * scale_log2 : -INFINITY;
+                                }
+                    }
+                    bool moved = false;
+                    float alpha[NH][2];
+#pragma unroll
+                    for (int t = 0; t < NH; ++t)
+#pragma unroll
+                        for (int b = 0; b < 2; ++b) {
+                            float mx = m[t][b];
+#pragma unroll
+                            for (int k = 0; k < NK / 16; ++k) mx = fmaxf(mx, fmaxf(s[k][t][b], s[k][t][2 + b]));
+                            mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 4));
+                            mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 8));
+                            mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 16));  // finite: the set's first key is seen
+                            alpha[t][b] = fast_exp2(m[t][b] - mx);
+                            moved |= mx != m[t][b];
+                            m[t][b] = mx;
+                            l[t][b] *= alpha[t][b];
+                        }
+                    uint32_t p[NK / 16][NH][2];  // the weights as the second product reads them: keys by pairs, heads
+#pragma unroll
+                    for (int k = 0; k < NK / 16; ++k)
+#pragma unroll
+                        for (int t = 0; t < NH; ++t) {
+#pragma unroll
+                            for (int e = 0; e < 4; ++e) {
+                                s[k][t][e] = fast_exp2(s[k][t][e] - m[t][e & 1]);
+                                l[t][e & 1] += s[k][t][e];
+                            }
+                            p[k][t][0] = turn_8x8(pack_bf16(s[k][t][0], s[k][t][1]));
+                            p[k][t][1] = turn_8x8(pack_bf16(s[k][t][2], s[k][t][3]));
+                        }
+                    if (__any_sync(0xffffffffu, moved)) {
+#pragma unroll
+                        for (int c = 0; c < CPW; ++c)
+#pragma unroll
+                            for (int d = 0; d < D / 16; ++d)
+#pragma unroll
+                                for (int t = 0; t < NH; ++t)
+#pragma unroll
+                                    for (int e = 0; e < 4; ++e) o[c][d][t][e] *= alpha[t][e & 1];
+                    }
+#pragma unroll
+                    for (int c = 0; c < CPW; ++c) {
+                        if (c >= n_v) break;
+#pragma unroll
+                        for (int k = 0; k < NK / 16; ++k)
+#pragma unroll
+                            for (int d = 0; d < D / 16; ++d) {
+                                uint32_t v[4];
+                                ldmatrix_x4_trans(v, at(Vs + c * HEAD, key_off + k * 16 + (lane & 7) + ((lane >> 4) << 3), d * 16 + (((lane >> 3) & 1) << 3)));
+#pragma unroll
+                                for (int t = 0; t < NH; ++t) mma_bf16(o[c][d][t], v, p[k][t][0], p[k][t][1]);
+                            }
                     }
                 }
                 __syncwarp();
@@ -248,28 +308,32 @@ attn_decode_across(const __grid_constant__ CUtensorMap map_kv, const AcrossArgs 
                     fa::mbar_arrive(&empty[st]);
                 }
             }
-            // the part's results, for the rows that hold a head
+            // the part's results (the columns behind the kv head's last query head are not read)
 #pragma unroll
-            for (int h = 0; h < 2; ++h) {
-                l[h] += __shfl_xor_sync(0xffffffffu, l[h], 1);
-                l[h] += __shfl_xor_sync(0xffffffffu, l[h], 2);
-                const int row = (lane >> 2) + h * 8;
-                if (row >= per) continue;
-                const int head = ka * per + row;
-                if ((lane & 3) == 0 && c0 + v0 == 0)
-                    *reinterpret_cast<float2*>(a.part_ml + (((int64_t)r * n_parts + part) * a.n_q + head) * 2) = make_float2(m[h], l[h]);
+            for (int t = 0; t < NH; ++t)
 #pragma unroll
-                for (int c = 0; c < AX_CPW; ++c) {
-                    if (c >= n_v) break;
-                    float* dst = a.part_o + ((((int64_t)r * n_parts + part) * G + c0 + v0 + c) * a.n_q + head) * D + ((lane & 3) << 1);
-#pragma unroll
-                    for (int d = 0; d < D / 8; ++d) *reinterpret_cast<float2*>(dst + d * 8) = make_float2(o[c][d][2 * h], o[c][d][2 * h + 1]);
+                for (int b = 0; b < 2; ++b) {
+                    l[t][b] += __shfl_xor_sync(0xffffffffu, l[t][b], 4);
+                    l[t][b] += __shfl_xor_sync(0xffffffffu, l[t][b], 8);
+                    l[t][b] += __shfl_xor_sync(0xffffffffu, l[t][b], 16);
+                    const int hr = t * 8 + (lane & 3) * 2 + b;
+                    if (lane < 4 && hr < per && c0 + v0 == 0)
+                        *reinterpret_cast<float2*>(a.part_ml + (((int64_t)r * n_parts + part) * a.n_q + ka * per + hr) * 2) = make_float2(m[t][b], l[t][b]);
                 }
+#pragma unroll
+            for (int c = 0; c < CPW; ++c) {
+                if (c >= n_v) break;
+                float* dst = a.part_o + ((((int64_t)r * n_parts + part) * G + c0 + v0 + c) * G + ka) * D * (NH * 8) + (lane & 3) * 2;
+#pragma unroll
+                for (int d = 0; d < D / 16; ++d)
+#pragma unroll
+                    for (int t = 0; t < NH; ++t)
+#pragma unroll
+                        for (int e = 0; e < 2; ++e)
+                            *reinterpret_cast<float2*>(dst + (d * 16 + (lane >> 2) + e * 8) * (NH * 8) + t * 8) = make_float2(o[c][d][t][2 * e], o[c][d][t][2 * e + 1]);
             }
-        } else if (consumer && c0 == 0 && cp == 0) {  // an empty slice says so
-            const int row = lane;
-            if (row < per)
-                *reinterpret_cast<float2*>(a.part_ml + (((int64_t)r * n_parts + part) * a.n_q + ka * per + row) * 2) = make_float2(-INFINITY, 0.f);
+        } else if (!work && consumer && c0 == 0 && cp == 0 && lane < per) {  // an empty slice says so
+            *reinterpret_cast<float2*>(a.part_ml + (((int64_t)r * n_parts + part) * a.n_q + ka * per + lane) * 2) = make_float2(-INFINITY, 0.f);
         }
     }
     if (*gave_up && lane == 0) atomicOr(a.err, SS_ERR_WAIT_LIMIT);
@@ -279,9 +343,9 @@ attn_decode_across(const __grid_constant__ CUtensorMap map_kv, const AcrossArgs 
 //
 // With w_p(g) = 2^(m_p(g) - max) / sum over the parts of head g, a_g,c = sum_p w_p(g) O_p(g, c):
 //   out[r][h] = sigmoid(gate[r][h]) * sum_g table_t[g][h] a_g,c(h),   c(h) = h / per.
-// A block takes AM_COLS columns of one kv head of values of one request.
+// A block takes AM_COLS head dims of one kv head of values of one request.
 #define AM_COLS 32
-#define AM_THREADS 256
+#define AM_THREADS 512
 struct TalkMergeArgs {
     const float* part_o;
     const float* part_ml;
@@ -291,61 +355,91 @@ struct TalkMergeArgs {
     bf16* out;
     const int32_t* q_start;
     const int32_t* seq_lens;
-    int n_q, n_kv, n_parts;
+    int n_q, n_kv, nh, n_parts, n_slices, tile_keys, splits;  // splits: threads that share the parts of an element
 };
+
+// float4 items (four heads of one head dim) of a block's columns, and how many threads share each
+constexpr int talk_merge_items(int n_kv, int nh) { return n_kv * AM_COLS * nh * 2; }
+constexpr int talk_merge_splits(int n_kv, int nh) { return talk_merge_items(n_kv, nh) >= AM_THREADS ? 1 : AM_THREADS / talk_merge_items(n_kv, nh); }
 
 template <int D>
 __global__ void __launch_bounds__(AM_THREADS)
 talk_merge_kernel(const TalkMergeArgs a) {
     extern __shared__ __align__(16) float am_smem[];
-    float* A = am_smem;                    // [n_q][AM_COLS]
-    float* W = A + a.n_q * AM_COLS;        // [n_q][n_parts]
+    const int slots = a.n_kv * a.nh * 8;             // heads with the padding of every kv head
+    float* A = am_smem;                              // [splits][slots][AM_COLS + 1]
+    float* W = A + a.splits * slots * (AM_COLS + 1); // [n_parts][slots]
+    W += (4 - (a.splits * slots * (AM_COLS + 1)) % 4) % 4;
     pdl_launch_dependents();
-    pdl_wait();
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int c = blockIdx.x / (D / AM_COLS), d0 = (blockIdx.x % (D / AM_COLS)) * AM_COLS, r = blockIdx.y;
-    if (a.seq_lens[r] <= 0) return;
-    const int per = a.n_q / a.n_kv;
-    for (int g = warp; g < a.n_q; g += AM_THREADS / 32) {  // a warp per head: the weights of its parts
+    const int seq_len = a.seq_lens[r], row = a.q_start[r];
+    pdl_wait();
+    if (seq_len <= 0) return;
+    const int per = a.n_q / a.n_kv, wide = a.nh * 8;
+    // the parts that hold keys: those of the first slices (as the kernel in front cut them)
+    const int tiles = (seq_len - 1) / a.tile_keys + 1, each = (tiles + a.n_slices - 1) / a.n_slices;
+    const int parts = (tiles + each - 1) / each * (a.n_parts / a.n_slices);
+    for (int s = warp; s < slots; s += AM_THREADS / 32) {  // a warp per head: the weights of its parts
+        const int hr = s % wide, g = s / wide * per + hr;
+        float2 v[8];  // at most 256 parts
         float mx = -INFINITY, den = 0.f;
-        for (int p = lane; p < a.n_parts; p += 32) mx = fmaxf(mx, a.part_ml[(((int64_t)r * a.n_parts + p) * a.n_q + g) * 2]);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+            const int p = lane + 32 * i;
+            v[i] = p < parts && hr < per ? __ldcg(reinterpret_cast<const float2*>(a.part_ml) + ((int64_t)r * a.n_parts + p) * a.n_q + g)
+                                         : make_float2(-INFINITY, 0.f);
+        }
+#pragma unroll
+        for (int i = 0; i < 8; ++i) mx = fmaxf(mx, v[i].x);
         mx = warp_max(mx);
-        for (int p = lane; p < a.n_parts; p += 32) {
-            const float2 ml = *reinterpret_cast<const float2*>(a.part_ml + (((int64_t)r * a.n_parts + p) * a.n_q + g) * 2);
-            const float e = ml.x == -INFINITY ? 0.f : exp2f(ml.x - mx);
-            W[g * a.n_parts + p] = e;
-            den = fmaf(e, ml.y, den);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+            v[i].x = v[i].x == -INFINITY ? 0.f : exp2f(v[i].x - mx);
+            den = fmaf(v[i].x, v[i].y, den);
         }
         den = warp_sum(den);
         const float inv = den > 0.f ? 1.f / den : 0.f;
-        __syncwarp();
-        for (int p = lane; p < a.n_parts; p += 32) W[g * a.n_parts + p] *= inv;
+#pragma unroll
+        for (int i = 0; i < 8; ++i)
+            if (lane + 32 * i < parts) W[(lane + 32 * i) * slots + s] = v[i].x * inv;
     }
     __syncthreads();
-    const int64_t part_stride = (int64_t)a.n_kv * a.n_q * D;
-    const float* o = a.part_o + ((int64_t)r * a.n_parts * a.n_kv + c) * a.n_q * D + d0;
-    for (int i = tid; i < a.n_q * (AM_COLS / 4); i += AM_THREADS) {
-        const int g = i / (AM_COLS / 4), d = (i % (AM_COLS / 4)) * 4;
-        const float* src = o + (int64_t)g * D + d;
+    const int64_t head_stride = (int64_t)D * wide, part_stride = (int64_t)a.n_kv * a.n_kv * head_stride;
+    const float* o = a.part_o + (int64_t)r * a.n_parts * part_stride + (int64_t)c * a.n_kv * head_stride + (int64_t)d0 * wide;
+    const int run4 = wide / 4, items = a.n_kv * AM_COLS * run4;
+    for (int i = tid; i < items * a.splits; i += AM_THREADS) {
+        const int sp = i / items, rest = i - sp * items, ka = rest / (AM_COLS * run4), at = rest - ka * (AM_COLS * run4);
+        const int d = at / run4, s0 = ka * wide + (at % run4) * 4;
+        const float* src = o + ka * head_stride + at * 4;
         float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll 8
-        for (int p = 0; p < a.n_parts; ++p) {
-            const float w = W[g * a.n_parts + p];
-            if (w != 0.f) {  // (an empty part has written nothing)
-                const float4 v = __ldcg(reinterpret_cast<const float4*>(src + p * part_stride));
-                acc.x = fmaf(w, v.x, acc.x); acc.y = fmaf(w, v.y, acc.y); acc.z = fmaf(w, v.z, acc.z); acc.w = fmaf(w, v.w, acc.w);
-            }
+        for (int p = sp; p < parts; p += a.splits) {
+            const float4 w = *reinterpret_cast<const float4*>(W + p * slots + s0);
+            const float4 v = __ldcg(reinterpret_cast<const float4*>(src + p * part_stride));
+            acc.x = fmaf(w.x, v.x, acc.x); acc.y = fmaf(w.y, v.y, acc.y); acc.z = fmaf(w.z, v.z, acc.z); acc.w = fmaf(w.w, v.w, acc.w);
         }
-        *reinterpret_cast<float4*>(A + g * AM_COLS + d) = acc;
+        float* dst = A + (sp * slots + s0) * (AM_COLS + 1) + d;
+        dst[0] = acc.x;
+        dst[AM_COLS + 1] = acc.y;
+        dst[2 * (AM_COLS + 1)] = acc.z;
+        dst[3 * (AM_COLS + 1)] = acc.w;
     }
     __syncthreads();
     for (int i = tid; i < per * AM_COLS; i += AM_THREADS) {
         const int hr = i / AM_COLS, d = i % AM_COLS, h = c * per + hr;
         float v = 0.f;
+        for (int ka = 0; ka < a.n_kv; ++ka) {
 #pragma unroll 4
-        for (int g = 0; g < a.n_q; ++g) v = fmaf(__ldg(a.table_t + (int64_t)g * a.n_q + h), A[g * AM_COLS + d], v);
-        const int64_t col = (int64_t)h * D + d0 + d, row = a.q_start[r];
+            for (int k = 0; k < per; ++k) {
+                const int s = ka * wide + k;
+                float x = A[s * (AM_COLS + 1) + d];
+                for (int sp = 1; sp < a.splits; ++sp) x += A[(sp * slots + s) * (AM_COLS + 1) + d];
+                v = fmaf(__ldg(a.table_t + (int64_t)(ka * per + k) * a.n_q + h), x, v);
+            }
+        }
+        const int64_t col = (int64_t)h * D + d0 + d;
         if (a.gate) v = gated<true>(v, to_float(a.gate[row * a.gate_stride + col]));
-        a.out[row * a.n_q * D + col] = __float2bfloat16_rn(v);
+        a.out[(int64_t)row * a.n_q * D + col] = __float2bfloat16_rn(v);
     }
 }

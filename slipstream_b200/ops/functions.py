@@ -142,7 +142,7 @@ _ATTN_SIGNATURES = {
                            c_int, c_int],
 }
 
-_ATTN_SIGNATURES["ss_attn_decode_across_sets"] = [c_int, c_int, c_int]
+_ATTN_SIGNATURES["ss_attn_decode_across_sets"] = [c_int, c_int, c_int, c_void_p]
 _ATTN_SIGNATURES["ss_attn_decode_across"] = [c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int,
                                              c_int, c_int64, c_float, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_void_p,
                                              c_void_p]
@@ -2525,12 +2525,15 @@ def talk_heads(x: torch.Tensor, table_t: torch.Tensor, n_kv: int, out_dtype: tor
 
 
 @functools.lru_cache(maxsize=None)
-def across_decode_sets(head_dim: int, n_q: int, n_kv: int, page_size: int) -> int:
-    """Parts per slice that the decode kernel over all kv heads' values leaves, or 0 where it does not take the layer (head
-    size 64 or 128, 2 to 8 kv heads of at most 16 query heads, pages of 8, 16, 32 or 64 tokens)."""
+def across_decode_sets(head_dim: int, n_q: int, n_kv: int, page_size: int) -> tuple[int, int]:
+    """(parts per slice that the decode kernel over all kv heads' values leaves, columns of heads it keeps per kv head);
+    (0, 0) where it does not take the layer (head size 64 or 128, 2 to 8 kv heads of at most 16 query heads, pages of 8, 16, 32
+    or 64 tokens)."""
     if head_dim not in (64, 128):
-        return 0
-    return int(attention_library(head_dim).ss_attn_decode_across_sets(int(n_q), int(n_kv), int(page_size)))
+        return 0, 0
+    cols = c_int(0)
+    sets = int(attention_library(head_dim).ss_attn_decode_across_sets(int(n_q), int(n_kv), int(page_size), ctypes.addressof(cols)))
+    return (sets, int(cols.value)) if sets else (0, 0)
 
 
 def across_slices(n_requests: int, n_kv: int, longest: int, sms: int | None = None) -> int:
@@ -2544,7 +2547,7 @@ def talking_attention_decode(q: torch.Tensor, q_stride: int, kv: torch.Tensor, b
                              gate: torch.Tensor | None, n_slices: int) -> torch.Tensor:
     """Attention with talking heads for requests that bring ONE token each (bfloat16), where `across_decode_sets`: every tile of
     keys and values is fetched once for all heads; the slices' sums are combined, mixed and gated by a second kernel."""
-    sets = across_decode_sets(head_dim, n_q, n_kv, kv.shape[3])
+    sets, head_cols = across_decode_sets(head_dim, n_q, n_kv, kv.shape[3])
     if not sets or q.dtype != torch.bfloat16:
         raise KernelError("the decode kernel over all values does not take this layer")
     _need(kv, torch.bfloat16, "kv pages")
@@ -2556,7 +2559,7 @@ def talking_attention_decode(q: torch.Tensor, q_stride: int, kv: torch.Tensor, b
                                                                     or gate.stride(1) != 1)):
         raise KernelError("talking_attention_decode: the table must be [H, H], the gate a view [N, H * D] with unit inner stride")
     parts = n_slices * sets
-    part_o = torch.empty((n_requests, parts, n_kv, n_q, head_dim), dtype=torch.float32, device=q.device)
+    part_o = torch.empty((n_requests, parts, n_kv, n_kv, head_dim, head_cols), dtype=torch.float32, device=q.device)
     part_ml = torch.empty((n_requests, parts, n_q, 2), dtype=torch.float32, device=q.device)
     out = torch.empty((rows, n_q * head_dim), dtype=q.dtype, device=q.device)
     _check(attention_library(head_dim).ss_attn_decode_across(
@@ -2575,7 +2578,7 @@ def talking_attention(q: torch.Tensor, kv: torch.Tensor, block_tables: torch.Ten
     ``mask``: `paged_attention`'s window, chunk, keep, softcap and sinks.  bfloat16 decode steps without these run the kernel
     that walks all kv heads together; everything else `paged_attention` across all values and `talk_heads`."""
     if (q.dtype == torch.bfloat16 and ctx.is_decode_only and not any(v is not None and v for v in mask.values())
-            and across_decode_sets(head_dim, n_q, n_kv, kv.shape[3])):
+            and across_decode_sets(head_dim, n_q, n_kv, kv.shape[3])[0]):
         longest = ctx.extras.get("static_max_seq_len") or ctx.max_seq_len
         slices = across_slices(ctx.num_requests, n_kv, longest, sm_count(q.device))
         return talking_attention_decode(q, q.shape[1], kv, block_tables, ctx.q_start, ctx.seq_lens, ctx.num_requests, n_q, n_kv, head_dim, scale,

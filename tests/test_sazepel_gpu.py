@@ -450,7 +450,7 @@ def test_every_head_over_all_values_in_every_attention_kernel_and_the_mixture_be
         got = ops.talk_heads(flat.float().to(DEV), table_t, n_kv, dtype, gate.to(DEV)[:, 8:])
         gated = want * torch.sigmoid(gate[:, 8:].double())
         assert rel(got, gated) < (5e-6 if dtype == torch.float32 else 8e-3)
-        if dtype == torch.bfloat16 and max(q_lens) == 1 and ops.across_decode_sets(d, n_q, n_kv, page):
+        if dtype == torch.bfloat16 and max(q_lens) == 1 and ops.across_decode_sets(d, n_q, n_kv, page)[0]:
             for slices in (1, 2, 5, 18, 64):  # all kv heads in one walk, mixture and gate behind it
                 got = ops.talking_attention_decode(*args, dev[1], dev[2], dev[3], dev[4], n, n_q, n_kv, d, scale, table_t, gate.to(DEV)[:, 8:], slices)
                 assert rel(got, gated) < 1.5e-2, slices
