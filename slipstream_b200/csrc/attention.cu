@@ -219,10 +219,10 @@ extern "C" int ss_attn_decode_across_sets(int n_q, int n_kv, int page_size, int*
 }
 
 template <int BN, int NK, int NH, int CPW>
-static int launch_across(const CUtensorMap& map_kv, const AcrossArgs& a, dim3 grid, int smem, cudaStream_t stream) {
+static int launch_across(const CUtensorMap& map_k, const CUtensorMap& map_v, const AcrossArgs& a, dim3 grid, int smem, cudaStream_t stream) {
     static SsPerDevice opted;
     if (int rc = ss_opt_in_smem(attn_decode_across<HEAD_DIM, BN, NK, NH, CPW>, 220 * 1024, opted)) return rc;
-    ss_launch(attn_decode_across<HEAD_DIM, BN, NK, NH, CPW>, grid, dim3(AX_THREADS), smem, stream, map_kv, a);
+    ss_launch(attn_decode_across<HEAD_DIM, BN, NK, NH, CPW>, grid, dim3(AX_THREADS), smem, stream, map_k, map_v, a);
     return SS_LAUNCH_CHECK();
 }
 
@@ -237,9 +237,11 @@ extern "C" int ss_attn_decode_across(const void* q, int64_t q_stride, void* out,
     if (page_size % 8 != 0 || 64 % page_size != 0 || n_slices < 1 || n_slices > SS_DECODE_MAX_SLICES || q_stride % 8) return (int)cudaErrorInvalidValue;
     const AcrossLayout y = across_layout(HEAD_DIM, n_q, n_kv);
     if (!y.stages) return (int)cudaErrorInvalidValue;
-    CUtensorMap map_kv;
-    int rc = fa::make_map3(&map_kv, kv, HEAD_DIM, (uint64_t)page_size, (uint64_t)num_pages * 2 * n_kv, (uint64_t)HEAD_DIM * 2,
-                           (uint64_t)page_size * HEAD_DIM * 2, 64, (uint32_t)(page_size < y.bn ? page_size : y.bn), 1);
+    CUtensorMap map_k, map_v;
+    int rc = 0;
+    for (int v = 0; v < 2 && !rc; ++v)
+        rc = fa::make_map3(v ? &map_v : &map_k, kv, HEAD_DIM, (uint64_t)page_size, (uint64_t)num_pages * 2 * n_kv, (uint64_t)HEAD_DIM * 2,
+                           (uint64_t)page_size * HEAD_DIM * 2, 64, (uint32_t)(page_size < y.bn ? page_size : y.bn), (uint32_t)(v ? y.nc : n_kv));
     if (rc) return rc;
     AcrossArgs a;
     a.q = (const bf16*)q; a.q_stride = q_stride; a.block_tables = block_tables; a.max_blocks = max_blocks; a.q_start = q_start;
@@ -248,21 +250,28 @@ extern "C" int ss_attn_decode_across(const void* q, int64_t q_stride, void* out,
     const int smem = across_smem_bytes(HEAD_DIM, n_kv, y);
     const dim3 grid(n_slices, (n_kv + y.nc - 1) / y.nc, n_requests);
     if (y.nh == 1) {
-        if (y.bn == 64) rc = launch_across<64, 16, 1, 4>(map_kv, a, grid, smem, stream);
-        else if (y.nk == 16) rc = launch_across<32, 16, 1, 4>(map_kv, a, grid, smem, stream);
-        else rc = launch_across<32, 32, 1, 4>(map_kv, a, grid, smem, stream);
+        if (y.bn == 64) rc = launch_across<64, 16, 1, 4>(map_k, map_v, a, grid, smem, stream);
+        else if (y.nk == 16) rc = launch_across<32, 16, 1, 4>(map_k, map_v, a, grid, smem, stream);
+        else rc = launch_across<32, 32, 1, 4>(map_k, map_v, a, grid, smem, stream);
     } else {
-        rc = y.bn == 64 ? launch_across<64, 16, 2, 2>(map_kv, a, grid, smem, stream) : launch_across<32, 32, 2, 2>(map_kv, a, grid, smem, stream);
+        rc = y.bn == 64 ? launch_across<64, 16, 2, 2>(map_k, map_v, a, grid, smem, stream) : launch_across<32, 32, 2, 2>(map_k, map_v, a, grid, smem, stream);
     }
     if (rc) return rc;
     TalkMergeArgs t;
     t.part_o = part_o; t.part_ml = part_ml; t.table_t = table_t; t.gate = (const bf16*)gate; t.gate_stride = gate_stride; t.out = (bf16*)out;
     t.q_start = q_start; t.seq_lens = seq_lens; t.n_q = n_q; t.n_kv = n_kv; t.nh = y.nh; t.n_parts = n_slices * y.sets;
     t.n_slices = n_slices; t.tile_keys = y.bn; t.splits = talk_merge_splits(n_kv, y.nh);
-    const int merge_smem = (n_kv * y.nh * 8 * (t.splits * (AM_COLS + 1) + t.n_parts) + 4) * 4;
-    static SsPerDevice opted_merge;
-    if (int rc_smem = ss_opt_in_smem(talk_merge_kernel<HEAD_DIM>, 200 * 1024, opted_merge)) return rc_smem;
-    ss_launch(talk_merge_kernel<HEAD_DIM>, dim3(n_kv * (HEAD_DIM / AM_COLS), n_requests), dim3(AM_THREADS), merge_smem, stream, t);
+    const int merge_smem = talk_merge_smem(n_q, n_kv, y.nh, t.n_parts);
+    const dim3 merge_grid(n_kv * (HEAD_DIM / AM_COLS), n_requests);
+    if (y.nh == 1) {
+        static SsPerDevice opted;
+        if (int rc_smem = ss_opt_in_smem(talk_merge_kernel<HEAD_DIM, 1>, 100 * 1024, opted)) return rc_smem;
+        ss_launch(talk_merge_kernel<HEAD_DIM, 1>, merge_grid, dim3(AM_THREADS), merge_smem, stream, t);
+    } else {
+        static SsPerDevice opted;
+        if (int rc_smem = ss_opt_in_smem(talk_merge_kernel<HEAD_DIM, 2>, 100 * 1024, opted)) return rc_smem;
+        ss_launch(talk_merge_kernel<HEAD_DIM, 2>, merge_grid, dim3(AM_THREADS), merge_smem, stream, t);
+    }
     return SS_LAUNCH_CHECK();
 }
 #else

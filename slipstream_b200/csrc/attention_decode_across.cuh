@@ -5,8 +5,9 @@
 // values of every kv head.  A block per pair of kv heads would read every key and value n_kv times.  Here a block takes a
 // slice of a request's keys for all of its kv heads at once, so that every tile of keys and values is fetched once:
 //   * a tile is BN keys: their K rows of all n_kv heads and their V rows of the block's `nc` heads (all of them up to four;
-//     more than four are shared by blocks along grid.y), moved by TMA, one box per page, head and 64-element half, issued by
-//     the lanes of a producer warp into a ring of stages;
+//     more than four are shared by blocks along grid.y), moved by TMA into a ring of stages by a producer warp: a box is the
+//     rows of a page and a 64-element half for all heads at once, since a box costs the same however large it is (one box per
+//     head took 2.4 us for a tile of 64 KB);
 //   * a consumer warp has one kv head of keys and up to CPW kv heads of values, and a set of NK of a tile's keys (where there
 //     are fewer kv heads than warps several sets share a tile).  Its products are turned over so that the few query heads of
 //     a kv head are the narrow side: scores as keys x heads, outputs as head dims x heads (mma.sync m16n8k16; 7 heads fill 7
@@ -73,6 +74,12 @@ struct AcrossArgs {
     int* err;
 };
 
+// Tiles a slice takes: an equal share of the request's, but at least 128 keys, since a part costs the combining kernel more
+// than that (a request of 1,024 tokens fills 8 slices, whatever the launch has).
+__device__ __forceinline__ int across_tiles_per_slice(int tiles, int n_slices, int tile_keys) {
+    return max(128 / tile_keys, (tiles + n_slices - 1) / n_slices);
+}
+
 __device__ __forceinline__ uint32_t turn_8x8(uint32_t x) {
     uint32_t y;
     asm volatile("movmatrix.sync.aligned.m8n8.trans.b16 %0, %1;" : "=r"(y) : "r"(x));
@@ -81,7 +88,7 @@ __device__ __forceinline__ uint32_t turn_8x8(uint32_t x) {
 
 template <int D, int BN, int NK, int NH, int CPW>
 __global__ void __launch_bounds__(AX_THREADS, 1)
-attn_decode_across(const __grid_constant__ CUtensorMap map_kv, const AcrossArgs a) {
+attn_decode_across(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v, const AcrossArgs a) {
     pdl_launch_dependents();
     constexpr int KSTR = D + 8, HALVES = D / 64, HEAD = BN * D;  // elements of one head's rows in a tile
     extern __shared__ unsigned char smem_raw[];
@@ -89,6 +96,7 @@ attn_decode_across(const __grid_constant__ CUtensorMap map_kv, const AcrossArgs 
     const int G = a.n_kv, per = a.n_q / G, n_slices = a.n_slices, stages = a.stages;
     const int c0 = blockIdx.y * a.nc, nc = min(a.nc, G - c0);  // this block's kv heads of values
     const int stage_elems = (G + a.nc) * HEAD;
+    const int rows = min(a.page_size, BN), row_shift = __ffs(rows) - 1;  // keys of a box
     bf16* ring = reinterpret_cast<bf16*>(base);
     bf16* Qs = ring + stages * stage_elems;  // [kv head][8 NH][KSTR]
     uint64_t* full = reinterpret_cast<uint64_t*>(Qs + G * NH * 8 * KSTR);
@@ -100,7 +108,7 @@ attn_decode_across(const __grid_constant__ CUtensorMap map_kv, const AcrossArgs 
     const int slice = blockIdx.x, r = blockIdx.z;
     const int row_q = a.q_start[r], seq_len = a.seq_lens[r], pos = seq_len - 1;
     const int tiles = seq_len > 0 ? (seq_len - 1) / BN + 1 : 0;
-    const int each = (tiles + n_slices - 1) / n_slices;
+    const int each = across_tiles_per_slice(tiles, n_slices, BN);
     const int j_lo = slice * each, j_hi = min(tiles, j_lo + each) - 1, j_last = tiles - 1;
     const bool work = j_lo <= j_hi;
     // consumer warps: key head, run of value heads, warp set
@@ -122,10 +130,11 @@ attn_decode_across(const __grid_constant__ CUtensorMap map_kv, const AcrossArgs 
     __syncthreads();
 
     if (warp == AX_WARPS) {
-        // ---------------- producer: a lane per box (page, half, head)
+        // ---------------- producer: a lane per box (page, half, keys or values)
         if (work) {
-            if (lane == 0) asm volatile("prefetch.tensormap [%0];" ::"l"(&map_kv) : "memory");
-            const int rows = min(a.page_size, BN), boxes = BN / rows, total = boxes * HALVES * (G + nc);
+            if (lane == 0) asm volatile("prefetch.tensormap [%0];" ::"l"(&map_k) : "memory");
+            if (lane == 0) asm volatile("prefetch.tensormap [%0];" ::"l"(&map_v) : "memory");
+            const int boxes = BN / rows, total = boxes * HALVES * 2;
             const int b_first = j_lo * BN / a.page_size, b_last = min(pos, j_hi * BN + BN - 1) / a.page_size;
             int64_t spare = table.p[b_first - table.base];  // a page of this request, for blocks that have none
             if (spare < 0 || spare >= a.num_pages) {
@@ -142,10 +151,11 @@ attn_decode_across(const __grid_constant__ CUtensorMap map_kv, const AcrossArgs 
                     pdl_wait();  // the newest key and value are written by the kernel before this one
                     waited = true;
                 }
-                if (lane == 0) fa::mbar_expect_tx(&full[st], (G + nc) * HEAD * 2);
+                if (lane == 0) fa::mbar_expect_tx(&full[st], stage_elems * 2);  // (a box may reach past the last head: what it brings is not read)
                 __syncwarp();
                 for (int b = lane; b < total; b += 32) {
-                    const int h = b % HALVES, p = (b / HALVES) % boxes, head = b / (HALVES * boxes);
+                    const int h = b % HALVES, p = (b / HALVES) % boxes;
+                    const bool keys = b < boxes * HALVES;
                     const int key = j * BN + p * rows, blk = key / a.page_size, off = key - blk * a.page_size;
                     int64_t page = (blk >= b_first && blk <= b_last) ? (int64_t)table.p[blk - table.base] : -1;
                     if (page >= a.num_pages) {
@@ -153,10 +163,12 @@ attn_decode_across(const __grid_constant__ CUtensorMap map_kv, const AcrossArgs 
                         page = -1;
                     }
                     if (page < 0) page = spare;
-                    bf16* dst = ring + st * stage_elems + head * HEAD + h * (BN * 64) + p * rows * 64;
-                    const int z = head < G ? (int)((page * 2 + 0) * G + head) : (int)((page * 2 + 1) * G + c0 + head - G);
-                    if (gridDim.y > 1) fa::tma_load_3d(dst, &map_kv, h * 64, off, z, &full[st]);  // the keys are read by several blocks
-                    else fa::tma_load_3d_once(dst, &map_kv, h * 64, off, z, &full[st], once);
+                    const int heads = keys ? G : a.nc;
+                    bf16* dst = ring + st * stage_elems + (keys ? 0 : G * HEAD) + (h * BN + p * rows) * heads * 64;
+                    const CUtensorMap* map = keys ? &map_k : &map_v;
+                    const int z = keys ? (int)((page * 2 + 0) * G) : (int)((page * 2 + 1) * G + c0);
+                    if (gridDim.y > 1) fa::tma_load_3d(dst, map, h * 64, off, z, &full[st]);  // the keys are read by several blocks
+                    else fa::tma_load_3d_once(dst, map, h * 64, off, z, &full[st], once);
                 }
             }
         }
@@ -193,13 +205,23 @@ attn_decode_across(const __grid_constant__ CUtensorMap map_kv, const AcrossArgs 
             const int key_off = set * NK;
             const int v0 = cp * CPW, n_v = min(CPW, nc - v0);
             const bf16* Qa = Qs + ka * NH * 8 * KSTR;
-            // a row of a head in a tile: halves of 64 elements, BN rows of 128 bytes each, 16-byte chunks permuted by the row
-            auto at = [](const bf16* tile, int row, int col) { return tile + (col >> 6) * (BN * 64) + row * 64 + ((((col >> 3) & 7) ^ (row & 7)) << 3); };
+            // where a row of a tile lies: the box's rows of all heads (rows of 128 bytes, 16-byte chunks permuted by the row)
+            // behind those of the boxes in front, the second 64 elements behind the whole tile's first
+            auto row_at = [&](int row, int heads, int head) { return ((((row >> row_shift) * heads + head) << row_shift) + (row & (rows - 1))) * 64; };
+            const int swz = lane & 7;  // (every row a lane addresses is its lane number mod 8)
+            int k_row[NK / 16], v_row[NK / 16];
+#pragma unroll
+            for (int k = 0; k < NK / 16; ++k) {
+                k_row[k] = row_at(key_off + k * 16 + (lane & 15), G, ka);
+                v_row[k] = row_at(key_off + k * 16 + (lane & 7) + ((lane >> 4) << 3), a.nc, v0);
+            }
+            const int k_half = G * BN * 64, v_half = a.nc * BN * 64, v_head = rows * 64;
+            auto col_at = [&](int col, int half_stride) { return (col >> 6) * half_stride + ((((col >> 3) & 7) ^ swz) << 3); };
             for (int j = j_lo; j <= j_hi; ++j) {
                 const int i = j - j_lo, st = i % stages;
                 const bool ok = fa::mbar_wait(&full[st], (i / stages) & 1, gave_up);
-                const bf16* Ks = ring + st * stage_elems + ka * HEAD;
-                bf16* Vs = ring + st * stage_elems + (G + v0) * HEAD;
+                const bf16* Ks = ring + st * stage_elems;
+                bf16* Vs = ring + st * stage_elems + G * HEAD;
                 const int key0 = j * BN + key_off;
                 if (ok && key0 <= pos) {
                     if (j == j_last && pos < key0 + NK - 1) {
@@ -208,7 +230,8 @@ attn_decode_across(const __grid_constant__ CUtensorMap map_kv, const AcrossArgs 
                         const int first = pos + 1 - j * BN, last = key_off + NK;
                         for (int c = lane; c < (last - first) * (D / 8) * n_v; c += 32) {
                             const int v = c / ((last - first) * (D / 8)), rest = c - v * ((last - first) * (D / 8));
-                            *reinterpret_cast<uint4*>(const_cast<bf16*>(at(Vs + v * HEAD, first + rest / (D / 8), (rest % (D / 8)) * 8))) = make_uint4(0u, 0u, 0u, 0u);
+                            const int col = (rest % (D / 8)) * 8;  // (a whole row: the order of its chunks does not matter)
+                            *reinterpret_cast<uint4*>(Vs + row_at(first + rest / (D / 8), a.nc, v0 + v) + (col >> 6) * v_half + (col & 63)) = make_uint4(0u, 0u, 0u, 0u);
                         }
                         __syncwarp();
                     }
@@ -229,8 +252,8 @@ attn_decode_across(const __grid_constant__ CUtensorMap map_kv, const AcrossArgs 
 #pragma unroll
                             for (int k = 0; k < NK / 16; ++k) {
                                 uint32_t x[4], y[4];
-                                ldmatrix_x4(x, at(Ks, key_off + k * 16 + (lane & 15), ks * 16 + ((lane >> 4) << 3)));
-                                ldmatrix_x4(y, at(Ks, key_off + k * 16 + (lane & 15), (ks + 1) * 16 + ((lane >> 4) << 3)));
+                                ldmatrix_x4(x, Ks + k_row[k] + col_at(ks * 16 + ((lane >> 4) << 3), k_half));
+                                ldmatrix_x4(y, Ks + k_row[k] + col_at((ks + 1) * 16 + ((lane >> 4) << 3), k_half));
 #pragma unroll
                                 for (int t = 0; t < NH; ++t) {
                                     mma_bf16(s[k][t], x, q[t][0], q[t][1]);
@@ -296,7 +319,7 @@ attn_decode_across(const __grid_constant__ CUtensorMap map_kv, const AcrossArgs 
 #pragma unroll
                             for (int d = 0; d < D / 16; ++d) {
                                 uint32_t v[4];
-                                ldmatrix_x4_trans(v, at(Vs + c * HEAD, key_off + k * 16 + (lane & 7) + ((lane >> 4) << 3), d * 16 + (((lane >> 3) & 1) << 3)));
+                                ldmatrix_x4_trans(v, Vs + v_row[k] + c * v_head + col_at(d * 16 + (((lane >> 3) & 1) << 3), v_half));
 #pragma unroll
                                 for (int t = 0; t < NH; ++t) mma_bf16(o[c][d][t], v, p[k][t][0], p[k][t][1]);
                             }
@@ -362,54 +385,81 @@ struct TalkMergeArgs {
 constexpr int talk_merge_items(int n_kv, int nh) { return n_kv * AM_COLS * nh * 2; }
 constexpr int talk_merge_splits(int n_kv, int nh) { return talk_merge_items(n_kv, nh) >= AM_THREADS ? 1 : AM_THREADS / talk_merge_items(n_kv, nh); }
 
-template <int D>
-__global__ void __launch_bounds__(AM_THREADS)
+constexpr int talk_merge_smem(int n_q, int n_kv, int nh, int n_parts) {
+    const int slots = n_kv * nh * 8, splits = talk_merge_splits(n_kv, nh);
+    return (n_parts * slots + splits * slots * (AM_COLS + 1) + n_q * (n_q / n_kv)) * 4;
+}
+
+template <int D, int NH>
+__global__ void __launch_bounds__(AM_THREADS, 2)
 talk_merge_kernel(const TalkMergeArgs a) {
     extern __shared__ __align__(16) float am_smem[];
-    const int slots = a.n_kv * a.nh * 8;             // heads with the padding of every kv head
-    float* A = am_smem;                              // [splits][slots][AM_COLS + 1]
-    float* W = A + a.splits * slots * (AM_COLS + 1); // [n_parts][slots]
-    W += (4 - (a.splits * slots * (AM_COLS + 1)) % 4) % 4;
+    constexpr int wide = NH * 8;
+    const int slots = a.n_kv * wide;                 // heads with the padding of every kv head
+    float* W = am_smem;                              // [n_parts][slots]: weights of the parts
+    float* A = W + a.n_parts * slots;                // [splits][slots][AM_COLS + 1]
+    float* T = A + a.splits * slots * (AM_COLS + 1); // [n_q][per]: the mixtures of this kv head's query heads
     pdl_launch_dependents();
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int c = blockIdx.x / (D / AM_COLS), d0 = (blockIdx.x % (D / AM_COLS)) * AM_COLS, r = blockIdx.y;
     const int seq_len = a.seq_lens[r], row = a.q_start[r];
+    const int per = a.n_q / a.n_kv;
+    // the parts that hold keys: those of the first slices (as the kernel in front cut them)
+    const int tiles = seq_len > 0 ? (seq_len - 1) / a.tile_keys + 1 : 0, each = across_tiles_per_slice(tiles, a.n_slices, a.tile_keys);
+    const int parts = (tiles + each - 1) / each * (a.n_parts / a.n_slices);
+    for (int g = warp; g < a.n_q; g += AM_THREADS / 32)  // constants of the layer: before the kernel in front is complete
+        if (lane < per) T[g * per + lane] = a.table_t[g * a.n_q + c * per + lane];
     pdl_wait();
     if (seq_len <= 0) return;
-    const int per = a.n_q / a.n_kv, wide = a.nh * 8;
-    // the parts that hold keys: those of the first slices (as the kernel in front cut them)
-    const int tiles = (seq_len - 1) / a.tile_keys + 1, each = (tiles + a.n_slices - 1) / a.n_slices;
-    const int parts = (tiles + each - 1) / each * (a.n_parts / a.n_slices);
-    for (int s = warp; s < slots; s += AM_THREADS / 32) {  // a warp per head: the weights of its parts
+    float gate = 0.f;  // of this thread's first output
+    if (a.gate && tid < per * AM_COLS) gate = to_float(a.gate[row * a.gate_stride + (int64_t)(c * per + tid / AM_COLS) * D + d0 + tid % AM_COLS]);
+    // sixteen lanes per head: the weights of its parts
+    const int l16 = lane & 15;
+    for (int s = tid >> 4; s < (slots + 1) / 2 * 2; s += AM_THREADS / 16) {
         const int hr = s % wide, g = s / wide * per + hr;
-        float2 v[8];  // at most 256 parts
+        const bool on = s < slots && hr < per;
+        const float2* ml = reinterpret_cast<const float2*>(a.part_ml) + r * a.n_parts * a.n_q + g;
         float mx = -INFINITY, den = 0.f;
+        float2 v[4];
+        for (int p0 = 0; p0 < parts; p0 += 64) {
 #pragma unroll
-        for (int i = 0; i < 8; ++i) {
-            const int p = lane + 32 * i;
-            v[i] = p < parts && hr < per ? __ldcg(reinterpret_cast<const float2*>(a.part_ml) + ((int64_t)r * a.n_parts + p) * a.n_q + g)
-                                         : make_float2(-INFINITY, 0.f);
+            for (int i = 0; i < 4; ++i) {
+                const int p = p0 + l16 + 16 * i;
+                v[i] = on && p < parts ? __ldcg(ml + p * a.n_q) : make_float2(-INFINITY, 0.f);
+            }
+#pragma unroll
+            for (int i = 0; i < 4; ++i) mx = fmaxf(mx, v[i].x);
         }
 #pragma unroll
-        for (int i = 0; i < 8; ++i) mx = fmaxf(mx, v[i].x);
-        mx = warp_max(mx);
+        for (int o = 8; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+        for (int p0 = 0; p0 < parts; p0 += 64) {
+            if (parts > 64) {  // (up to 64 parts are still in registers)
 #pragma unroll
-        for (int i = 0; i < 8; ++i) {
-            v[i].x = v[i].x == -INFINITY ? 0.f : exp2f(v[i].x - mx);
-            den = fmaf(v[i].x, v[i].y, den);
+                for (int i = 0; i < 4; ++i) {
+                    const int p = p0 + l16 + 16 * i;
+                    v[i] = on && p < parts ? __ldcg(ml + p * a.n_q) : make_float2(-INFINITY, 0.f);
+                }
+            }
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                const int p = p0 + l16 + 16 * i;
+                const float e = v[i].x == -INFINITY ? 0.f : exp2f(v[i].x - mx);
+                den = fmaf(e, v[i].y, den);
+                if (s < slots && p < parts) W[p * slots + s] = e;
+            }
         }
-        den = warp_sum(den);
+#pragma unroll
+        for (int o = 8; o > 0; o >>= 1) den += __shfl_xor_sync(0xffffffffu, den, o);
         const float inv = den > 0.f ? 1.f / den : 0.f;
-#pragma unroll
-        for (int i = 0; i < 8; ++i)
-            if (lane + 32 * i < parts) W[(lane + 32 * i) * slots + s] = v[i].x * inv;
+        if (s < slots)
+            for (int p = l16; p < parts; p += 16) W[p * slots + s] *= inv;
     }
     __syncthreads();
     const int64_t head_stride = (int64_t)D * wide, part_stride = (int64_t)a.n_kv * a.n_kv * head_stride;
     const float* o = a.part_o + (int64_t)r * a.n_parts * part_stride + (int64_t)c * a.n_kv * head_stride + (int64_t)d0 * wide;
-    const int run4 = wide / 4, items = a.n_kv * AM_COLS * run4;
-    for (int i = tid; i < items * a.splits; i += AM_THREADS) {
-        const int sp = i / items, rest = i - sp * items, ka = rest / (AM_COLS * run4), at = rest - ka * (AM_COLS * run4);
+    constexpr int run4 = wide / 4, unit = AM_COLS * run4;  // float4 items of a kv head of keys
+    for (int u = tid / unit; u < a.n_kv * a.splits; u += AM_THREADS / unit) {
+        const int sp = u / a.n_kv, ka = u - sp * a.n_kv, at = tid % unit;
         const int d = at / run4, s0 = ka * wide + (at % run4) * 4;
         const float* src = o + ka * head_stride + at * 4;
         float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -427,19 +477,17 @@ talk_merge_kernel(const TalkMergeArgs a) {
     }
     __syncthreads();
     for (int i = tid; i < per * AM_COLS; i += AM_THREADS) {
-        const int hr = i / AM_COLS, d = i % AM_COLS, h = c * per + hr;
+        const int hr = i / AM_COLS, d = i % AM_COLS;
         float v = 0.f;
-        for (int ka = 0; ka < a.n_kv; ++ka) {
-#pragma unroll 4
-            for (int k = 0; k < per; ++k) {
-                const int s = ka * wide + k;
-                float x = A[s * (AM_COLS + 1) + d];
-                for (int sp = 1; sp < a.splits; ++sp) x += A[(sp * slots + s) * (AM_COLS + 1) + d];
-                v = fmaf(__ldg(a.table_t + (int64_t)(ka * per + k) * a.n_q + h), x, v);
+        for (int ka = 0; ka < a.n_kv; ++ka)
+            for (int sp = 0; sp < a.splits; ++sp) {
+                const float* x = A + (sp * slots + ka * wide) * (AM_COLS + 1) + d;
+                const float* t = T + ka * per * per + hr;
+#pragma unroll 8
+                for (int k = 0; k < per; ++k) v = fmaf(t[k * per], x[k * (AM_COLS + 1)], v);
             }
-        }
-        const int64_t col = (int64_t)h * D + d0 + d;
-        if (a.gate) v = gated<true>(v, to_float(a.gate[row * a.gate_stride + col]));
+        const int64_t col = (int64_t)(c * per + hr) * D + d0 + d;
+        if (a.gate) v = gated<true>(v, i == tid ? gate : to_float(a.gate[row * a.gate_stride + col]));
         a.out[(int64_t)row * a.n_q * D + col] = __float2bfloat16_rn(v);
     }
 }
