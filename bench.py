@@ -1721,7 +1721,7 @@ def run_compare_sazepel(args) -> int:
             us = sweep(lambda i: ops.paged_attention_decode(q, q.shape[1], out, kv_pages[i], table, starts, lens, n_req, n_q, n_kv, d, d ** -0.5, 0,
                                                             slices, stages=ops.functions.DECODE_RING_STAGES), copies)
             hbm(f"decode_attention {name} {n_req} x {tokens} (qwen2, rotation outside)", us, moved)
-            slices = ops.across_slices(n_req, n_kv, tokens, ops.sm_count(dev))
+            slices = ops.across_slices(n_req, n_q, n_kv, tokens, ops.sm_count(dev))
             us = sweep(lambda i: ops.talking_attention_decode(q, q.shape[1], kv_pages[i], table, starts, lens, n_req, n_q, n_kv, d, d ** -0.5, talk,
                                                               gate, slices), copies)
             hbm(f"decode_attention {name} {n_req} x {tokens} with talking heads (both kernels)", us, moved)

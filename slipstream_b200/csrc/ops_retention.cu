@@ -169,41 +169,53 @@ extern "C" int ss_head_norm_gate(const float* x, const void* gate, int64_t gate_
 // x[t][a][c][r][:] with g = a * G + r (common.cuh: head_pair).  Mixing the heads' weights before they meet the values
 // is the same sum in another order:
 //   out[t][h] = sigmoid(gate[t][h]) * sum_g table[h][g] x[t][g's a][h's c][g's r],      c = h / G.
-// table_t: the table transposed, float32 [g][h].  A warp takes TH_OUT heads of one kv head c of one token; a lane four
-// elements of D (a multiple of 16, padding behind the values included).
+// table_t: the table transposed, float32 [g][h].  A block takes TH_OUT heads of one kv head c of TH_ROWS tokens, with the part of
+// the table it needs in shared memory; LP lanes share a token's row of D elements (a multiple of 4, padding behind the values
+// included), four elements a lane and pass.
 #define TH_OUT 8
-template <typename T>
-__global__ void __launch_bounds__(128)
+#define TH_WARPS 8
+template <typename T, int LP>
+__global__ void __launch_bounds__(TH_WARPS * 32)
 talk_heads_kernel(const float* __restrict__ x, const float* __restrict__ table_t, const T* __restrict__ gate,
-                  int64_t gate_stride, T* __restrict__ out, int64_t units, int n_kv, int G, int D) {
+                  int64_t gate_stride, T* __restrict__ out, int n_tokens, int n_kv, int G, int D) {
     pdl_launch_dependents();
-    const int lane = threadIdx.x & 31;
-    const int64_t unit = (int64_t)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
-    pdl_wait();
-    if (unit >= units) return;
+    extern __shared__ __align__(16) float th_smem[];  // [g][TH_OUT]
     const int chunks = (G + TH_OUT - 1) / TH_OUT, H = n_kv * G;
-    const int chunk = (int)(unit % chunks);
-    const int64_t tc = unit / chunks;
-    const int c = (int)(tc % n_kv);
-    const int64_t t = tc / n_kv;
+    const int c = blockIdx.y / chunks, chunk = blockIdx.y - c * chunks;
     const int h0 = c * G + chunk * TH_OUT, n_out = min(TH_OUT, G - chunk * TH_OUT);
-    const float* xt = x + t * n_kv * H * D;
-    for (int j = lane * 4; j < D; j += 128) {
+    for (int i = threadIdx.x; i < H * TH_OUT; i += TH_WARPS * 32) {
+        const int g = i / TH_OUT, o = i % TH_OUT;
+        th_smem[i] = o < n_out ? table_t[(int64_t)g * H + h0 + o] : 0.f;
+    }
+    __syncthreads();
+    pdl_wait();
+    const int sub = threadIdx.x % LP;
+    const int t = blockIdx.x * (TH_WARPS * 32 / LP) + threadIdx.x / LP;
+    if (t >= n_tokens) return;
+    const int64_t a_stride = (int64_t)n_kv * G * D;
+    const float* xt = x + (int64_t)t * n_kv * a_stride + (int64_t)c * G * D;
+    for (int j = sub * 4; j < D; j += LP * 4) {
         float acc[TH_OUT][4];
 #pragma unroll
         for (int o = 0; o < TH_OUT; ++o) acc[o][0] = acc[o][1] = acc[o][2] = acc[o][3] = 0.f;
         for (int a = 0; a < n_kv; ++a) {
-            const float* xa = xt + (int64_t)(a * n_kv + c) * G * D + j;
-            const float* ta = table_t + (int64_t)a * G * H + h0;
-#pragma unroll 4
-            for (int r = 0; r < G; ++r) {
-                float v[4];
-                load4(xa + (int64_t)r * D, v);
+            const float* xa = xt + a * a_stride + j;
+            const float* ta = th_smem + a * G * TH_OUT;
+            for (int r0 = 0; r0 < G; r0 += 8) {
+                float v[8][4];  // eight rows in flight
 #pragma unroll
-                for (int o = 0; o < TH_OUT; ++o) {
-                    const float w = o < n_out ? __ldg(ta + (int64_t)r * H + o) : 0.f;
+                for (int r = 0; r < 8; ++r)
+                    if (r0 + r < G) load4(xa + (r0 + r) * D, v[r]);
 #pragma unroll
-                    for (int e = 0; e < 4; ++e) acc[o][e] = fmaf(w, v[e], acc[o][e]);
+                for (int r = 0; r < 8; ++r) {
+                    if (r0 + r >= G) break;
+                    float w[TH_OUT];
+                    *reinterpret_cast<float4*>(w) = *reinterpret_cast<const float4*>(ta + (r0 + r) * TH_OUT);
+                    *reinterpret_cast<float4*>(w + 4) = *reinterpret_cast<const float4*>(ta + (r0 + r) * TH_OUT + 4);
+#pragma unroll
+                    for (int o = 0; o < TH_OUT; ++o)
+#pragma unroll
+                        for (int e = 0; e < 4; ++e) acc[o][e] = fmaf(w[o], v[r][e], acc[o][e]);
                 }
             }
         }
@@ -216,9 +228,19 @@ talk_heads_kernel(const float* __restrict__ x, const float* __restrict__ table_t
 #pragma unroll
                 for (int e = 0; e < 4; ++e) acc[o][e] = gated<sizeof(T) == 2>(acc[o][e], g[e]);
             }
-            store4(out + (t * H + h0 + o) * D + j, acc[o]);
+            store4(out + ((int64_t)t * H + h0 + o) * D + j, acc[o]);
         }
     }
+}
+
+template <typename T, int LP>
+static int launch_talk_heads(const float* x, const float* table_t, const void* gate, int64_t gate_stride, void* out, int n_tokens,
+                             int n_kv, int G, int D, cudaStream_t stream) {
+    const int smem = n_kv * G * TH_OUT * 4, rows = TH_WARPS * 32 / LP;
+    if (smem > 48 * 1024) return (int)cudaErrorInvalidValue;
+    const dim3 grid((n_tokens + rows - 1) / rows, n_kv * ((G + TH_OUT - 1) / TH_OUT));
+    ss_launch(talk_heads_kernel<T, LP>, grid, dim3(TH_WARPS * 32), smem, stream, x, table_t, (const T*)gate, gate_stride, (T*)out, n_tokens, n_kv, G, D);
+    return SS_LAUNCH_CHECK();
 }
 
 extern "C" int ss_talk_heads(const float* x, const float* table_t, const void* gate, int64_t gate_stride, void* out, int n_tokens,
@@ -227,13 +249,16 @@ extern "C" int ss_talk_heads(const float* x, const float* table_t, const void* g
     const int size = dtype == SS_BF16 ? 2 : 4;
     if (n_kv < 1 || G < 1 || D < 4 || D % 4 || ((uintptr_t)x & 15) || (((uintptr_t)gate | (uintptr_t)out) & (4 * size - 1)) || gate_stride % 4)
         return (int)cudaErrorInvalidValue;
-    const int64_t units = (int64_t)n_tokens * n_kv * ((G + TH_OUT - 1) / TH_OUT);
-    const dim3 grid((unsigned)((units + 3) / 4));
-    if (dtype == SS_BF16)
-        ss_launch(talk_heads_kernel<bf16>, grid, dim3(128), 0, stream, x, table_t, (const bf16*)gate, gate_stride, (bf16*)out, units, n_kv, G, D);
-    else
-        ss_launch(talk_heads_kernel<float>, grid, dim3(128), 0, stream, x, table_t, (const float*)gate, gate_stride, (float*)out, units, n_kv, G, D);
-    return SS_LAUNCH_CHECK();
+#define TH_GO(T)                                                                                                      \
+    do {                                                                                                              \
+        if (D <= 16) return launch_talk_heads<T, 4>(x, table_t, gate, gate_stride, out, n_tokens, n_kv, G, D, stream);  \
+        if (D <= 32) return launch_talk_heads<T, 8>(x, table_t, gate, gate_stride, out, n_tokens, n_kv, G, D, stream);  \
+        if (D <= 64) return launch_talk_heads<T, 16>(x, table_t, gate, gate_stride, out, n_tokens, n_kv, G, D, stream); \
+        return launch_talk_heads<T, 32>(x, table_t, gate, gate_stride, out, n_tokens, n_kv, G, D, stream);              \
+    } while (0)
+    if (dtype == SS_BF16) TH_GO(bf16);
+    TH_GO(float);
+#undef TH_GO
 }
 
 // ---------------------------------------------------------------- two branches, each under a norm of its own

@@ -2536,9 +2536,11 @@ def across_decode_sets(head_dim: int, n_q: int, n_kv: int, page_size: int) -> tu
     return (sets, int(cols.value)) if sets else (0, 0)
 
 
-def across_slices(n_requests: int, n_kv: int, longest: int, sms: int | None = None) -> int:
-    """Into how many slices that kernel cuts the keys: a block per SM (its ring of tiles takes the SM's shared memory)."""
-    blocks = n_requests * (1 if n_kv <= 4 else (n_kv + 1) // 2)
+def across_slices(n_requests: int, n_q: int, n_kv: int, longest: int, sms: int | None = None) -> int:
+    """Into how many slices that kernel cuts the keys: a block per SM (its ring of tiles takes the SM's shared memory).  With
+    more than four kv heads several blocks share their values."""
+    per_block = n_kv if n_kv <= 4 else (4 if n_q // n_kv <= 8 else 2)
+    blocks = n_requests * -(-n_kv // per_block)
     return max(1, min((sms or sm_count()) // blocks, (longest + 31) // 32, 64))
 
 
@@ -2580,7 +2582,7 @@ def talking_attention(q: torch.Tensor, kv: torch.Tensor, block_tables: torch.Ten
     if (q.dtype == torch.bfloat16 and ctx.is_decode_only and not any(v is not None and v for v in mask.values())
             and across_decode_sets(head_dim, n_q, n_kv, kv.shape[3])[0]):
         longest = ctx.extras.get("static_max_seq_len") or ctx.max_seq_len
-        slices = across_slices(ctx.num_requests, n_kv, longest, sm_count(q.device))
+        slices = across_slices(ctx.num_requests, n_q, n_kv, longest, sm_count(q.device))
         return talking_attention_decode(q, q.shape[1], kv, block_tables, ctx.q_start, ctx.seq_lens, ctx.num_requests, n_q, n_kv, head_dim, scale,
                                         table_t, gate, slices)
     wide = torch.empty((q.shape[0], n_kv * n_q * head_dim), dtype=torch.float32, device=q.device)
