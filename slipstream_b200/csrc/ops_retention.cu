@@ -306,8 +306,9 @@ extern "C" int ss_normed_pair(const void* a, const float* wa, const void* b, con
 //
 // A block of 16 warps takes RC_COLS value columns of a head of a request and walks its tokens in chunks of RC_T:
 //   * the chunk's rows arrive in shared memory by asynchronous copies issued while the chunk in front is computed;
-//   * they are rotated and cut in two (cosines and sines of a row's offset in the chunk come from a table made once, those
-//     of the chunk's first position are formed once a chunk);
+//   * they are rotated and cut in two: a thread has one run of 8 pairs of a row of q and of k, and the cosines and sines of
+//     that row's offset in the chunk in registers, those of the chunk's first position are formed once a chunk; k_scale is
+//     left to the factors that the scores and the values meet anyway;
 //   * four warps share 16 rows: each takes 16 keys of the scores and a quarter of the state's rows, and their sums meet in
 //     shared memory;
 //   * the state stays in registers as accumulators, cut in two in shared memory once a chunk.
@@ -319,7 +320,6 @@ extern "C" int ss_normed_pair(const void* a, const float* wa, const void* b, con
 template <int D>
 struct RcSmem {
     static constexpr int S = D + 8, V = RC_COLS + 8;          // strides that spread ldmatrix over all banks
-    static constexpr int A = D / 2 + 8;                       // stride of the table of angles, for the same reason
     static constexpr int raw_qk = 0;                          // bf16 [2][RC_T][D]
     static constexpr int raw_v = raw_qk + 2 * RC_T * D * 2;   // bf16 [RC_T][RC_COLS]
     static constexpr int qk = raw_v + RC_T * RC_COLS * 2;     // bf16 [q hi, q lo, k hi, k lo][RC_T][S]
@@ -327,9 +327,9 @@ struct RcSmem {
     static constexpr int st = v + 3 * RC_T * V * 2;           // bf16 [state hi, lo][D][V]
     static constexpr int sum = st + 2 * D * V * 2;            // float [4][RC_T][V]
     static constexpr int pw = sum + 4 * RC_T * V * 4;         // float [RC_T + 4]: powers of the decay
-    static constexpr int base = pw + (RC_T + 4) * 4;          // float2 [D / 2]: the chunk's first position
-    static constexpr int turn = base + D / 2 * 8;             // float2 [RC_T][D / 2]: offsets in the chunk
-    static constexpr int bytes = turn + RC_T * A * 8;
+    static constexpr int pk = pw + (RC_T + 4) * 4;            // float [RC_T + 4]: the same times k_scale
+    static constexpr int base = pk + (RC_T + 4) * 4;          // float2 [D / 2]: the chunk's first position
+    static constexpr int bytes = base + D / 2 * 8;
 };
 
 __device__ __forceinline__ void cut_in_two(const float (&x)[8], uint4& hi, uint4& lo) {
@@ -358,7 +358,7 @@ retention_chunks_kernel(const bf16* __restrict__ proj, int64_t stride, const flo
                         const int32_t* __restrict__ slots, int heads, int dim, int vdim, int n_slots, int* err,
                         const float* __restrict__ inv_freq, int half, float k_scale) {
     using M = RcSmem<D>;
-    constexpr int S = M::S, V = M::V, A = M::A, KS = D / 16, NT = RC_COLS / 8;
+    constexpr int S = M::S, V = M::V, KS = D / 16, NT = RC_COLS / 8;
     constexpr int UT = NT / 2;  // column tiles of the state a warp holds (of 16 rows); with D = 64 half of the warps hold any
     extern __shared__ __align__(16) unsigned char smem[];
     bf16* raw = reinterpret_cast<bf16*>(smem + M::raw_qk);
@@ -375,7 +375,7 @@ retention_chunks_kernel(const bf16* __restrict__ proj, int64_t stride, const flo
     float* sums = reinterpret_cast<float*>(smem + M::sum);
     float* pw = reinterpret_cast<float*>(smem + M::pw);
     float2* base = reinterpret_cast<float2*>(smem + M::base);
-    float2* turn = reinterpret_cast<float2*>(smem + M::turn);
+    float* pk = reinterpret_cast<float*>(smem + M::pk);
 
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int col_blocks = (vdim + RC_COLS - 1) / RC_COLS;
@@ -383,13 +383,27 @@ retention_chunks_kernel(const bf16* __restrict__ proj, int64_t stride, const flo
     const float g = decay[h];
     const int half8 = half / 8;
     pdl_launch_dependents();
-    for (int i = tid; i < RC_T * half; i += RC_THREADS) {  // offsets of the rows of a chunk: constants of the layer
-        const int t = i / half, e = i - t * half;
-        float sn, cs;
-        sincosf(__fmul_rn((float)t, inv_freq[e]), &sn, &cs);
-        turn[t * A + (e & 7) * half8 + (e >> 3)] = make_float2(cs, sn);  // (as the loop below reads: runs of 8 side by side)
+    // this thread's run of pairs: elements 8 tc .. and half further of row tt of a chunk
+    static_assert(RC_T * (D / 16) <= RC_THREADS, "a thread has at most one run of pairs");
+    const bool turns = tid < RC_T * half8;
+    const int tt = turns ? tid / half8 : 0, tc = turns ? tid - tt * half8 : 0;
+    float2 off[8];
+#pragma unroll
+    for (int e = 0; e < 8; ++e) off[e] = make_float2(1.f, 0.f);
+    if (turns) {  // (constants of the layer: before the kernels in front are complete)
+#pragma unroll 1
+        for (int e = 0; e < 8; ++e) {
+            float sn, cs;
+            sincosf(__fmul_rn((float)tt, inv_freq[tc * 8 + e]), &sn, &cs);
+#pragma unroll
+            for (int k = 0; k < 8; ++k)
+                if (k == e) off[k] = make_float2(cs, sn);
+        }
     }
-    for (int i = tid; i <= RC_T; i += RC_THREADS) pw[i] = powf(g, (float)i);
+    for (int i = tid; i <= RC_T; i += RC_THREADS) {
+        pw[i] = powf(g, (float)i);
+        pk[i] = pw[i] * k_scale;
+    }
     pdl_wait();
     const int q0 = q_start[r], q_len = q_start[r + 1] - q0, seq_len = seq_lens[r];
     if (q_len <= 0 || seq_len <= 0) return;
@@ -402,18 +416,21 @@ retention_chunks_kernel(const bf16* __restrict__ proj, int64_t stride, const flo
     const int64_t k_off = (int64_t)heads * dim, v_off = 2 * k_off + (int64_t)h * vdim + c0;
 
     // a chunk's rows into shared memory, 16 bytes a copy; zeros behind the last row, the head's last element and its last column
+    constexpr int RUNS = D / 8, ROWS = RC_THREADS / RUNS;  // runs of 8 elements of a row; rows a pass over the threads covers
+    const int ft = tid / RUNS, fc = (tid % RUNS) * 8;
+    const bf16* f_src = proj + (int64_t)(q0 + ft) * stride + (int64_t)h * dim + (fc < dim ? fc : 0);
+    const int vt = tid / (RC_COLS / 8), vc = (tid % (RC_COLS / 8)) * 8;  // (the values: a quarter or half of the threads)
     auto fetch = [&](int t0) {
-        for (int i = tid; i < 2 * RC_T * (D / 8); i += RC_THREADS) {
-            const int which = i / (RC_T * (D / 8)), rest = i - which * (RC_T * (D / 8)), t = rest / (D / 8), c = (rest % (D / 8)) * 8;
-            const bool ok = t0 + t < q_len && c < dim;
-            const bf16* src = proj + (int64_t)(q0 + (ok ? t0 + t : 0)) * stride + which * k_off + (int64_t)h * dim + (ok ? c : 0);
-            cp_async16(raw + (which * RC_T + t) * D + c, src, ok);
+#pragma unroll
+        for (int w = 0; w < RC_T / ROWS; ++w) {
+            const bool ok = t0 + ft + w * ROWS < q_len && fc < dim;
+            const bf16* src = ok ? f_src + (int64_t)(t0 + w * ROWS) * stride : proj;
+            cp_async16(raw + (ft + w * ROWS) * D + fc, src, ok);
+            cp_async16(raw + (RC_T + ft + w * ROWS) * D + fc, ok ? src + k_off : proj, ok);
         }
-        for (int i = tid; i < RC_T * (RC_COLS / 8); i += RC_THREADS) {
-            const int t = i / (RC_COLS / 8), c = (i % (RC_COLS / 8)) * 8;
-            const bool ok = t0 + t < q_len && c0 + c < vdim;
-            const bf16* src = proj + (int64_t)(q0 + (ok ? t0 + t : 0)) * stride + v_off + (ok ? c : 0);
-            cp_async16(raw_v + t * RC_COLS + c, ok ? src : proj, ok);
+        if (tid < RC_T * (RC_COLS / 8)) {
+            const bool ok = t0 + vt < q_len && c0 + vc < vdim;
+            cp_async16(raw_v + vt * RC_COLS + vc, ok ? proj + (int64_t)(q0 + t0 + vt) * stride + v_off + vc : proj, ok);
         }
         cp_async_commit();
     };
@@ -445,59 +462,58 @@ retention_chunks_kernel(const bf16* __restrict__ proj, int64_t stride, const flo
         }
         cp_async_wait<0>();
         __syncthreads();  // the rows and the chunk's first angles; and the chunk in front is done with everything below
-        // rotated pairs, eight at a time
-        for (int i = tid; i < 2 * RC_T * half8; i += RC_THREADS) {
-            const int which = i / (RC_T * half8), rest = i - which * (RC_T * half8), t = rest / half8, c = (rest - t * half8) * 8;
-            const bf16* src = raw + (which * RC_T + t) * D;
-            float u[8], v[8];
-            eight(*reinterpret_cast<const uint4*>(src + c), u);
-            eight(*reinterpret_cast<const uint4*>(src + c + half), v);
-            const float f = which ? k_scale : 1.f;
+        // rotated pairs
+        if (turns) {
+            float cs[8], sn[8];
 #pragma unroll
             for (int e = 0; e < 8; ++e) {
-                const float2 a = turn[t * A + e * half8 + (c >> 3)], b = base[e * half8 + (c >> 3)];
-                const float cs = (a.x * b.x - a.y * b.y) * f, sn = (a.y * b.x + a.x * b.y) * f;
-                const float x = u[e] * cs - v[e] * sn;
-                v[e] = v[e] * cs + u[e] * sn;
-                u[e] = x;
+                const float2 b = base[e * half8 + tc];
+                cs[e] = off[e].x * b.x - off[e].y * b.y;
+                sn[e] = off[e].y * b.x + off[e].x * b.y;
             }
-            bf16* hi = which ? Kh : Qh;
-            bf16* lo = which ? Kl : Ql;
-            uint4 ph, pl;
-            cut_in_two(u, ph, pl);
-            *reinterpret_cast<uint4*>(hi + t * S + c) = ph;
-            *reinterpret_cast<uint4*>(lo + t * S + c) = pl;
-            cut_in_two(v, ph, pl);
-            *reinterpret_cast<uint4*>(hi + t * S + c + half) = ph;
-            *reinterpret_cast<uint4*>(lo + t * S + c + half) = pl;
+#pragma unroll
+            for (int which = 0; which < 2; ++which) {
+                const bf16* src = raw + (which * RC_T + tt) * D + tc * 8;
+                bf16* hi = (which ? Kh : Qh) + tt * S + tc * 8;
+                bf16* lo = (which ? Kl : Ql) + tt * S + tc * 8;
+                float u[8], v[8];
+                eight(*reinterpret_cast<const uint4*>(src), u);
+                eight(*reinterpret_cast<const uint4*>(src + half), v);
+#pragma unroll
+                for (int e = 0; e < 8; ++e) {
+                    const float x = u[e] * cs[e] - v[e] * sn[e];
+                    v[e] = v[e] * cs[e] + u[e] * sn[e];
+                    u[e] = x;
+                }
+                uint4 ph, pl;
+                cut_in_two(u, ph, pl);
+                *reinterpret_cast<uint4*>(hi) = ph;
+                *reinterpret_cast<uint4*>(lo) = pl;
+                cut_in_two(v, ph, pl);
+                *reinterpret_cast<uint4*>(hi + half) = ph;
+                *reinterpret_cast<uint4*>(lo + half) = pl;
+            }
         }
-        // elements that are not rotated (and the zeros behind the head)
+        // elements that are not rotated (and the zeros behind the head): bfloat16 as they came
         const int rest8 = D / 8 - 2 * half8;
         for (int i = tid; i < 2 * RC_T * rest8; i += RC_THREADS) {
-            const int which = i / (RC_T * rest8), rest = i - which * (RC_T * rest8), t = rest / rest8, c = 2 * half + (rest - t * rest8) * 8;
-            float u[8];
-            eight(*reinterpret_cast<const uint4*>(raw + (which * RC_T + t) * D + c), u);
-            const float f = which ? k_scale : 1.f;
-#pragma unroll
-            for (int e = 0; e < 8; ++e) u[e] *= f;
-            uint4 ph, pl;
-            cut_in_two(u, ph, pl);
-            *reinterpret_cast<uint4*>((which ? Kh : Qh) + t * S + c) = ph;
-            *reinterpret_cast<uint4*>((which ? Kl : Ql) + t * S + c) = pl;
+            const int row = i / rest8, c = 2 * half + (i - row * rest8) * 8, t = row % RC_T;
+            const bool keys = row >= RC_T;
+            *reinterpret_cast<uint4*>((keys ? Kh : Qh) + t * S + c) = *reinterpret_cast<const uint4*>(raw + row * D + c);
+            *reinterpret_cast<uint4*>((keys ? Kl : Ql) + t * S + c) = make_uint4(0u, 0u, 0u, 0u);
         }
-        for (int i = tid; i < RC_T * (RC_COLS / 8); i += RC_THREADS) {
-            const int t = i / (RC_COLS / 8), c = (i % (RC_COLS / 8)) * 8;
-            const uint4 w = *reinterpret_cast<const uint4*>(raw_v + t * RC_COLS + c);
-            *reinterpret_cast<uint4*>(Vs + t * V + c) = w;
+        if (tid < RC_T * (RC_COLS / 8)) {
+            const uint4 w = *reinterpret_cast<const uint4*>(raw_v + vt * RC_COLS + vc);
+            *reinterpret_cast<uint4*>(Vs + vt * V + vc) = w;
             float u[8];
             eight(w, u);
-            const float f = t < nb ? pw[nb - 1 - t] : 0.f;
+            const float f = vt < nb ? pk[nb - 1 - vt] : 0.f;
 #pragma unroll
             for (int e = 0; e < 8; ++e) u[e] *= f;
             uint4 ph, pl;
             cut_in_two(u, ph, pl);
-            *reinterpret_cast<uint4*>(Wh + t * V + c) = ph;
-            *reinterpret_cast<uint4*>(Wl + t * V + c) = pl;
+            *reinterpret_cast<uint4*>(Wh + vt * V + vc) = ph;
+            *reinterpret_cast<uint4*>(Wl + vt * V + vc) = pl;
         }
         if (s_nt < NT) {
 #pragma unroll
@@ -574,7 +590,7 @@ retention_chunks_kernel(const bf16* __restrict__ proj, int64_t stride, const flo
 #pragma unroll
                     for (int e = 0; e < 4; ++e) {
                         const int back = (e < 2 ? row_lo : row_hi) - (key + (e & 1));
-                        x[e] = back >= 0 ? sc[n][e] * pw[back] : 0.f;
+                        x[e] = back >= 0 ? sc[n][e] * pk[back] : 0.f;
                     }
 #pragma unroll
                     for (int e = 0; e < 2; ++e) {
