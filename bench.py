@@ -31,6 +31,10 @@ experts and a gated shared expert, one norm for both branches of a layer).
 tokens, attention whose values are the keys with a joint norm and learned sinks, norms on both sides of every branch, a
 feed-forward with the tanh form of GELU, layers that run twice with the embedding joining in between).
 
+``--compare sazepel`` does the same for the Sazepel decoder (retention with rotated queries and keys, attention whose heads
+exchange their weights behind the softmax beside a retention, each under a norm of its own, routed gated experts weighed on
+their outputs, norms with one number as their weight).
+
 ``--only decode|prefill`` runs one part and prints a short line (profiling, and measurements beside the
 headline): ``--only decode --batch 1 --prompt-len 32000 --context-len 32768`` is a decode step behind a long
 context, ``--only prefill --chunk 512 --prefix 8192 --context-len 32768`` a prompt portion behind cached tokens.
